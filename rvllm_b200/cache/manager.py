@@ -10,6 +10,10 @@ float32 tensor [slots, *shape]; a request holds one slot id for all of them, eve
 an architecture that has no such call.  A slot's records are zero when a request
 receives it (`add` clears them), so no mixer ever sees its slot's previous holder.
 
+A group may hold one row per `every` tokens instead of one per token (pooled blocks: a row
+stands for that many positions).  Its tables and its pool count rows, so both are shorter by that
+factor; every live request may begin a page of its own, so the pool has one page per request more.
+
 A request's pages are given back when it ends (`free`) and, in a group whose reach
 is bounded (a window, or chunks that do not see one another), as soon as every slot of
 the page lies behind what any future query can see (`advance`).  Released block-table entries read -1; no kernel touches them because
@@ -128,20 +132,25 @@ class CacheManager:
         self._views: List[Optional[CacheView]] = [None] * len(needs)
         call_group: Dict[int, int] = {}
         state_calls: Dict[tuple, List[int]] = {}
+        def flatten(name, need):
+            """(name, need) of every part, however deep: part j of `name` is (name, j)."""
+            if not isinstance(need, SeveralNeeds):
+                return [(name, need)]
+            return [x for j, part in enumerate(need.parts) for x in flatten((name, j), part)]
+
         flat = []
         for i, need in enumerate(needs):
-            if isinstance(need, SeveralNeeds):
-                if cache_of[i] is not None:
-                    raise CacheError(f"call {i}: a mixer of several mixers keeps its own caches")
-                flat += [((i, j), part) for j, part in enumerate(need.parts)]
-            else:
-                flat.append((i, need))
+            if isinstance(need, SeveralNeeds) and cache_of[i] is not None:
+                raise CacheError(f"call {i}: a mixer of several mixers keeps its own caches")
+            flat += flatten(i, need)
         for i, need in flat:
             if isinstance(need, PagedNeed):
                 gi = next((g for g, grp in enumerate(self.groups) if grp.need == need), None)
                 if gi is None:
                     gi = len(self.groups)
-                    self.groups.append(Group(need, [], PagePool(num_pages)))
+                    pages = num_pages if need.every == 1 else \
+                        -(-num_pages // need.every) + max_requests
+                    self.groups.append(Group(need, [], PagePool(pages)))
                 self.groups[gi].calls.append(i)
                 call_group[i] = gi
             elif isinstance(need, StateNeed):
@@ -161,7 +170,7 @@ class CacheManager:
                     self.states[i] = block[ci]
         for grp in self.groups:
             if allocate:
-                shape = (len(grp.calls), num_pages, page_size, grp.need.num_kv_heads)
+                shape = (len(grp.calls), grp.pool.num_pages, page_size, grp.need.num_kv_heads)
                 grp.k = torch.zeros(shape + (grp.need.head_dim,), dtype=dtype, device=device)
                 grp.v = torch.zeros(shape + (grp.need.value_dim,), dtype=dtype, device=device)
         def view(src, owns):
@@ -174,10 +183,15 @@ class CacheManager:
                 return CacheView("state", owns, state=self.states[src])
             return None
 
+        def several(name, need):
+            if not isinstance(need, SeveralNeeds):
+                return view(name, True)
+            return CacheView("several", True,
+                             parts=[several((name, j), part) for j, part in enumerate(need.parts)])
+
         for i, need in enumerate(needs):
             if isinstance(need, SeveralNeeds):
-                self._views[i] = CacheView("several", True,
-                                           parts=[view((i, j), True) for j in range(len(need.parts))])
+                self._views[i] = several(i, need)
                 continue
             self._views[i] = view(cache_of[i] if cache_of[i] is not None else i,
                                   cache_of[i] is None)
@@ -191,7 +205,7 @@ class CacheManager:
         """Bytes of keys and values one cached token takes over all groups."""
         size = torch.empty((), dtype=self.dtype).element_size()
         return sum(len(g.calls) * g.need.num_kv_heads * (g.need.head_dim + g.need.value_dim) * size
-                   for g in self.groups)
+                   // g.need.every for g in self.groups)
 
     # ---- requests --------------------------------------------------------------------
 
@@ -223,17 +237,33 @@ class CacheManager:
         if grp.need.chunk is not None:
             # the chunk of the next query begins here; earlier chunks are never read again
             lowest_key = max(lowest_key, computed // grp.need.chunk * grp.need.chunk)
-        return lowest_key // self.page_size
+        if grp.need.block is not None:
+            # the block that the next query's token belongs to is read once more when complete
+            lowest_key = min(lowest_key, computed // grp.need.block * grp.need.block)
+        return grp.need.rows(lowest_key) // self.page_size
+
+    def pages_for(self, grp: Group, tokens: int) -> int:
+        """Block-table entries of `grp` that cover positions [0, tokens)."""
+        return -(-grp.need.rows(tokens) // self.page_size)
+
+    def room(self, req=None) -> int:
+        """The most positions `req` (None: a new request) could cover with the free pages."""
+        rc = self.requests.get(req) if req is not None else None
+        most = 1 << 30
+        for gi, grp in enumerate(self.groups):
+            have = len(rc.tables[gi]) if rc else 0
+            rows = (have + grp.pool.available) * self.page_size
+            most = min(most, rows * grp.need.every + grp.need.every - 1)
+        return most
 
     def pages_needed(self, req, total_tokens: int) -> List[int]:
         """Pages each group would have to hand out to cover positions
         [0, total_tokens) of `req` (which may not be live yet)."""
         rc = self.requests.get(req)
-        want = -(-total_tokens // self.page_size)
         out = []
         for gi, grp in enumerate(self.groups):
             have = len(rc.tables[gi]) if rc else 0
-            out.append(max(0, want - have))
+            out.append(max(0, self.pages_for(grp, total_tokens) - have))
         return out
 
     def can_reserve(self, req, total_tokens: int) -> bool:
@@ -246,15 +276,15 @@ class CacheManager:
         rc = self.requests[req]
         if total_tokens <= rc.tokens:
             return True
-        want = -(-total_tokens // self.page_size)
-        if all(len(t) >= want for t in rc.tables):
+        want = [self.pages_for(grp, total_tokens) for grp in self.groups]
+        if all(len(t) >= w for t, w in zip(rc.tables, want)):
             rc.tokens = total_tokens                 # room left in the last page
             return True
         if not self.can_reserve(req, total_tokens):
             return False
         for gi, grp in enumerate(self.groups):
             table = rc.tables[gi]
-            while len(table) < want:
+            while len(table) < want[gi]:
                 table.append(grp.pool.alloc())
         rc.tokens = total_tokens
         return True

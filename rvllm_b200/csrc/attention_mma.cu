@@ -19,11 +19,16 @@
 // through the block table with 16-byte cp.async copies into padded shared-memory rows,
 // two stages deep; keys past the context or in released pages are zero-filled.
 //
+// With -DRV_POOLED the library has instead the two kernels for a window of tokens and pooled blocks
+// before it, with scores that may be capped (attention_pooled.cuh): the same template (flag EXT)
+// walks the tiles of the blocks' rows first, then the tokens' tiles.
+//
 // Reference counterparts: kv_gather.cu (twice), a batched SGEMM, mask_add_broadcast.cu,
 // softmax.cu, a batched SGEMM and transposes (src/cuda/model.rs:528-581).  Plain
 // reference: tests/plain_ops.py paged_attention.
 #include <cuda.h>
 
+#include "attention_pooled.cuh"
 #include "common.cuh"
 
 #ifndef RV_HD
@@ -82,12 +87,20 @@ __device__ __forceinline__ int tile_offset(int row, int chunk) {
     return SW ? row * HD + ((chunk ^ (row & 7)) << 3) : row * (HD + 8) + (chunk << 3);
 }
 
-template <int HD, bool SW = false>
+// cap * log2 e * tanh(x / cap) for a raw product s with x = s * scale: cap_arg = 2 log2 e * scale /
+// cap, cap_out = cap * log2 e.  One exponential and a fast division; its error is some 1e-7 of
+// the cap.
+__device__ __forceinline__ float capped_log2(float s, float cap_arg, float cap_out) {
+    return cap_out - 2.f * cap_out * __fdividef(1.f, 1.f + exp2f(s * cap_arg));
+}
+
+template <int HD, bool SW = false, bool EXT = false>
 __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], const bf16* kt,
                                             const bf16* vt, int tile_key0, int lane, int lo_a,
                                             int hi_a, int lo_b, int hi_b, float scale_log2,
                                             float& m_a, float& m_b, float& l_a, float& l_b,
-                                            float (&o)[HD / 8][4]) {
+                                            float (&o)[HD / 8][4], float cap_arg = 0.f,
+                                            float cap_out = 0.f) {
     constexpr int KSTEPS = HD / 16;
     // S = Q K^T for 16 rows x 64 keys
     float s[RV_BN / 8][4];
@@ -103,6 +116,13 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], co
             mma_bf16(s[2 * nb], qf[kk], b[0], b[1]);
             mma_bf16(s[2 * nb + 1], qf[kk], b[2], b[3]);
         }
+    }
+    if (EXT && cap_out > 0.f) {
+#pragma unroll
+        for (int i = 0; i < RV_BN / 8; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[i][e] = capped_log2(s[i][e], cap_arg, cap_out);
+        scale_log2 = 1.f;
     }
     // mask, scale, running maximum
     const int key0 = tile_key0 + (lane & 3) * 2;
@@ -163,14 +183,14 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], co
     }
 }
 
-template <int HD, int NWARPS, bool SPLIT>
+template <int HD, int NWARPS, bool SPLIT, bool EXT = false>
 __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(
     const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ k_cache,
     const bf16* __restrict__ v_cache, const int* __restrict__ block_table, int max_blocks,
     const int* __restrict__ q_start, const int* __restrict__ ctx_lens, bf16* __restrict__ out,
     float* __restrict__ part_o, float2* __restrict__ part_ml, int max_splits, int first_req,
     int num_heads, int num_kv_heads, int page_size, float scale_log2, int window,
-    const float* __restrict__ sinks) {
+    const float* __restrict__ sinks, const RvPooled pl) {
     rv_pdl_prologue();
     constexpr int BM = 16 * NWARPS;
     constexpr int LD = HD + 8;          // padded row: conflict-free ldmatrix for HD % 16 == 0
@@ -210,7 +230,11 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(
         key_hi = min(key_hi, split * RV_SPLIT + RV_SPLIT - 1);
         if (key_lo > key_hi) return;
     }
-    const int tile_begin = key_lo / RV_BN, tile_end = key_hi / RV_BN;
+    // EXT: tiles below zero are the pooled blocks': tile t holds rows (t + n_ptiles) * 64 on
+    const int nb_hi = EXT ? rv_seen_blocks(key_hi, window, pl.pool) : 0;     // the newest query's
+    const int n_ptiles = (nb_hi + RV_BN - 1) / RV_BN;
+    const int tile_first = key_lo / RV_BN, tile_end = key_hi / RV_BN;
+    const int tile_begin = tile_first - n_ptiles;
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int page_shift = (page_size & (page_size - 1)) == 0 ? 31 - __clz(page_size) : -1;
@@ -233,16 +257,21 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(
     auto load_tile = [&](int t, int stage) {
         bf16* kd = Ks + stage * RV_BN * LD;
         bf16* vd = Vs + stage * RV_BN * LD;
+        const bool blocks = EXT && t < tile_first;
+        const int row0 = (blocks ? t - tile_begin : t) * RV_BN, limit = blocks ? nb_hi : clen;
+        const int* tab = blocks ? pl.table + (size_t)r * pl.max_blocks : table;
+        const bf16* kc = blocks ? (const bf16*)pl.k : k_cache;
+        const bf16* vc = blocks ? (const bf16*)pl.v : v_cache;
         size_t off[ROWS];
         bool valid[ROWS];
 #pragma unroll
         for (int i = 0; i < ROWS; ++i) {
             const int c = tid + i * NWARPS * 32;
             const int row = c / CPR;
-            const int j = t * RV_BN + row;
+            const int j = row0 + row;
             int page = -1;
-            if (c < RV_BN * CPR && j < clen)
-                page = table[page_shift >= 0 ? (j >> page_shift) : (j / page_size)];
+            if (c < RV_BN * CPR && j < limit)
+                page = tab[page_shift >= 0 ? (j >> page_shift) : (j / page_size)];
             valid[i] = page >= 0;
             const int in_page = page_shift >= 0 ? (j & (page_size - 1)) : (j % page_size);
             off[i] = valid[i] ? ((size_t)page * page_size + in_page) * kv_row + (size_t)g * HD +
@@ -253,8 +282,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(
             const int c = tid + i * NWARPS * 32;
             if (c < RV_BN * CPR) {
                 const int row = c / CPR, ch = c - row * CPR;
-                cp_async_16(kd + row * LD + ch * 8, k_cache + off[i], valid[i]);
-                cp_async_16(vd + row * LD + ch * 8, v_cache + off[i], valid[i]);
+                cp_async_16(kd + row * LD + ch * 8, kc + off[i], valid[i]);
+                cp_async_16(vd + row * LD + ch * 8, vc + off[i], valid[i]);
             }
         }
     };
@@ -272,6 +301,10 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(
         lo_a = max(lo_a, key_lo); lo_b = max(lo_b, key_lo);
         hi_a = min(hi_a, key_hi); hi_b = min(hi_b, key_hi);
     }
+    const int nb_a = EXT ? rv_seen_blocks(p_a, window, pl.pool) : 0;
+    const int nb_b = EXT ? rv_seen_blocks(p_b, window, pl.pool) : 0;
+    const float cap_out = EXT ? pl.cap * 1.4426950408889634f : 0.f;
+    const float cap_arg = EXT && pl.cap > 0.f ? 2.f * scale_log2 / pl.cap : 0.f;
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
     float o[HD / 8][4];
 #pragma unroll
@@ -298,8 +331,16 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(
         const bf16* kt = Ks + stage * RV_BN * LD;
         const bf16* vt = Vs + stage * RV_BN * LD;
 
-        attend_tile<HD>(qf, kt, vt, t * RV_BN, lane, lo_a, hi_a, lo_b, hi_b, scale_log2, m_a, m_b, l_a,
-                        l_b, o);
+        if (EXT) {
+            const bool blocks = t < tile_first;
+            attend_tile<HD, false, EXT>(qf, kt, vt, (blocks ? t - tile_begin : t) * RV_BN, lane,
+                                        blocks ? 0 : lo_a, blocks ? nb_a - 1 : hi_a,
+                                        blocks ? 0 : lo_b, blocks ? nb_b - 1 : hi_b, scale_log2,
+                                        m_a, m_b, l_a, l_b, o, cap_arg, cap_out);
+        } else {
+            attend_tile<HD>(qf, kt, vt, t * RV_BN, lane, lo_a, hi_a, lo_b, hi_b, scale_log2, m_a, m_b,
+                            l_a, l_b, o);
+        }
         __syncthreads();    // every warp is done with this stage before it is refilled
     }
     l_a += __shfl_xor_sync(0xffffffffu, l_a, 1);
@@ -351,12 +392,13 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(
 // key/value head) and one split of 256 keys; its four warps take one tile of 64 keys each,
 // so all four tiles are in flight at once, and their results are combined in warp order in
 // shared memory before the split's partial result is written.
-template <int HD, int NW>
+template <int HD, int NW, bool EXT = false>
 __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
     const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ k_cache,
     const bf16* __restrict__ v_cache, const int* __restrict__ block_table, int max_blocks,
     const int* __restrict__ ctx_lens, float* __restrict__ part_o, float2* __restrict__ part_ml,
-    int max_splits, int num_heads, int num_kv_heads, int page_size, float scale_log2, int window) {
+    int max_splits, int num_heads, int num_kv_heads, int page_size, float scale_log2, int window,
+    const RvPooled pl) {
     rv_pdl_prologue();
     constexpr int LD = HD + 8;
     constexpr int CPR = HD / 8;
@@ -377,12 +419,19 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
     const int m0 = (blockIdx.x % tiles_per_head) * 16;
     const int split = blockIdx.y;
     const int p = clen - 1;
-    const int key_lo = max(window > 0 ? max(0, p - window + 1) : 0, split * SPLIT);
-    const int key_hi = min(p, split * SPLIT + SPLIT - 1);
+    // EXT: which rows this split covers (attention_pooled.cuh)
+    const int lo = window > 0 ? max(0, p - window + 1) : 0;
+    const bool blocks = EXT && split < pl.psplits;
+    const int stretch = !EXT || blocks ? split : split - pl.psplits + lo / SPLIT;
+    const int limit = blocks ? rv_seen_blocks(p, window, pl.pool) : clen;    // rows there are
+    const int key_lo = max(blocks ? 0 : lo, stretch * SPLIT);
+    const int key_hi = min(limit - 1, stretch * SPLIT + SPLIT - 1);
     if (key_lo > key_hi) return;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int page_shift = (page_size & (page_size - 1)) == 0 ? 31 - __clz(page_size) : -1;
-    const int* table = block_table + (size_t)r * max_blocks;
+    const int* table = blocks ? pl.table + (size_t)r * pl.max_blocks : block_table + (size_t)r * max_blocks;
+    const bf16* kc = blocks ? (const bf16*)pl.k : k_cache;
+    const bf16* vc = blocks ? (const bf16*)pl.v : v_cache;
     const size_t kv_row = (size_t)num_kv_heads * HD;
     const int rows = min(16, G - m0);
 
@@ -392,7 +441,7 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
         const bf16* src = q + (size_t)r * q_stride + (size_t)(g * G + m0 + (valid ? m : 0)) * HD + ch * 8;
         cp_async_16(Qs + m * LD + ch * 8, src, valid);
     }
-    const int t = split * NW + warp;   // this warp's tile
+    const int t = stretch * NW + warp;   // this warp's tile
     const bool active = t * RV_BN <= key_hi && t * RV_BN + RV_BN - 1 >= key_lo;
     bf16* kt = KV + warp * 2 * TILE;
     bf16* vt = kt + TILE;
@@ -406,7 +455,7 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
             const int row = c / CPR;
             const int j = t * RV_BN + row;
             int page = -1;
-            if (j < clen) page = table[page_shift >= 0 ? (j >> page_shift) : (j / page_size)];
+            if (j < limit) page = table[page_shift >= 0 ? (j >> page_shift) : (j / page_size)];
             valid[i] = page >= 0;
             const int in_page = page_shift >= 0 ? (j & (page_size - 1)) : (j % page_size);
             off[i] = valid[i] ? ((size_t)page * page_size + in_page) * kv_row + (size_t)g * HD +
@@ -416,8 +465,8 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
         for (int i = 0; i < ROWS; ++i) {
             const int c = lane + i * 32;
             const int row = c / CPR, ch = c - row * CPR;
-            cp_async_16(kt + row * LD + ch * 8, k_cache + off[i], valid[i]);
-            cp_async_16(vt + row * LD + ch * 8, v_cache + off[i], valid[i]);
+            cp_async_16(kt + row * LD + ch * 8, kc + off[i], valid[i]);
+            cp_async_16(vt + row * LD + ch * 8, vc + off[i], valid[i]);
         }
     }
     cp_async_commit();
@@ -437,8 +486,10 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
 #pragma unroll
         for (int kk = 0; kk < KSTEPS; ++kk)
             ldmatrix_x4(qf[kk], Qs + (lane & 15) * LD + kk * 16 + (lane >> 4) * 8);
-        attend_tile<HD>(qf, kt, vt, t * RV_BN, lane, lo_a, hi_a, lo_b, hi_b, scale_log2, m_a, m_b, l_a,
-                        l_b, o);
+        attend_tile<HD, false, EXT>(qf, kt, vt, t * RV_BN, lane, lo_a, hi_a, lo_b, hi_b, scale_log2, m_a,
+                                    m_b, l_a, l_b, o,
+                                    EXT && pl.cap > 0.f ? 2.f * scale_log2 / pl.cap : 0.f,
+                                    EXT ? pl.cap * 1.4426950408889634f : 0.f);
     }
     l_a += __shfl_xor_sync(0xffffffffu, l_a, 1);
     l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
@@ -483,7 +534,7 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
 }
 
 
-#if RV_HD == 64
+#if RV_HD == 64 && !defined(RV_POOLED)
 // ---------------------------------------------------------------------------------
 // Decode as a stream (head size 64, pages of 8, 16, 32 or 64 tokens).  One persistent block
 // per SM; each of its six warps is a pipeline of its own.  A warp takes work items --
@@ -785,13 +836,107 @@ static int fail(const char* msg) {
 #define RV_CAT(a, b) RV_CAT2(a, b)
 #define RV_SYM(name) RV_CAT(RV_CAT(name, _hd), RV_HD)
 
+#ifndef RV_POOLED
 extern "C" const char* RV_SYM(rv_attention_mma_last_error)() { return g_error; }
+#endif
 
 template <int NWARPS>
 static size_t smem_bytes() {
     return (size_t)(16 * NWARPS + 4 * RV_BN) * (RV_HD + 8) * sizeof(bf16);
 }
 
+#ifdef RV_POOLED
+extern "C" const char* RV_SYM(rv_attention_pooled_last_error)() { return g_error; }
+
+static int pooled_sizes(int num_heads, int num_kv_heads, int page_size, int window, int pool,
+                        const void* pk, const void* pv, const int* ptable) {
+    if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads || page_size <= 0 ||
+        window < 0 || pool < 0 || (pool > 0 && (window == 0 || !pk || !pv || !ptable)))
+        return fail("paged_attention_pooled: bad sizes");
+    return 0;
+}
+
+// Prefill over a window of tokens and the pooled blocks before it: requests [first_req, first_req +
+// n_reqs), the longest bringing max_q_len tokens.
+extern "C" int RV_SYM(rv_paged_attention_pooled_prefill)(
+    const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* block_table,
+    int max_blocks, const void* pk, const void* pv, const int* ptable, int pmax_blocks, int pool,
+    float cap, const int* q_start, const int* ctx_lens, void* out, int first_req, int n_reqs,
+    int max_q_len, int num_heads, int num_kv_heads, int page_size, float scale, int window,
+    const float* sinks, void* stream) {
+    if (n_reqs == 0) return 0;
+    if (max_q_len <= 0 || n_reqs < 0 ||
+        pooled_sizes(num_heads, num_kv_heads, page_size, window, pool, pk, pv, ptable))
+        return fail("paged_attention_pooled_prefill: bad sizes");
+    const int G = num_heads / num_kv_heads;
+    const long long blocks_x = ((long long)max_q_len * G + 63) / 64;
+    if (blocks_x > 0x7fffffffLL || num_kv_heads > 65535 || n_reqs > 65535)
+        return fail("paged_attention_pooled_prefill: batch too large for one launch");
+    static bool configured = false;
+    if (!configured) {
+        if (smem_bytes<4>() > 48 * 1024) {
+            cudaError_t e = cudaFuncSetAttribute(paged_attention_mma_kernel<RV_HD, 4, false, true>,
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                 (int)smem_bytes<4>());
+            if (e != cudaSuccess) return fail(cudaGetErrorString(e));
+        }
+        configured = true;
+    }
+    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, cap, 0};
+    rv_launch(paged_attention_mma_kernel<RV_HD, 4, false, true>,
+              dim3((unsigned)blocks_x, num_kv_heads, n_reqs), dim3(128), smem_bytes<4>(),
+              (cudaStream_t)stream, (const bf16*)q, q_stride, (const bf16*)k_cache,
+              (const bf16*)v_cache, block_table, max_blocks, q_start, ctx_lens, (bf16*)out,
+              (float*)nullptr, (float2*)nullptr, 0, first_req, num_heads, num_kv_heads, page_size,
+              scale * 1.4426950408889634f, window, sinks, pl);
+    cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) return fail(cudaGetErrorString(e));
+    return 0;
+}
+
+// Decode: requests [0, n_reqs) bring one token each.  Writes partial results in the layout that
+// rv_paged_attention_pooled_merge combines.
+extern "C" int RV_SYM(rv_paged_attention_pooled_decode_mma)(
+    const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* block_table,
+    int max_blocks, const void* pk, const void* pv, const int* ptable, int pmax_blocks, int pool,
+    float cap, const int* ctx_lens, void* scratch, long long scratch_bytes, int n_reqs,
+    int max_ctx_len, int num_heads, int num_kv_heads, int page_size, float scale, int window,
+    void* stream) {
+    if (n_reqs == 0) return 0;
+    if (n_reqs < 0 || pooled_sizes(num_heads, num_kv_heads, page_size, window, pool, pk, pv, ptable))
+        return fail("paged_attention_pooled_decode: bad sizes");
+    const int psplits = rv_pooled_psplits(max_ctx_len, window, pool, RV_SPLIT);
+    const int max_splits = psplits + rv_pooled_tsplits(max_ctx_len, window, RV_SPLIT);
+    const size_t slots = (size_t)n_reqs * num_heads * max_splits;
+    if ((long long)(slots * RV_HD * 4 + slots * 8) > scratch_bytes)
+        return fail("paged_attention_pooled_decode: scratch too small");
+    const int G = num_heads / num_kv_heads;
+    const int tiles_per_head = (G + 15) / 16;
+    if (n_reqs > 65535 || num_kv_heads * tiles_per_head > 65535 || max_splits > 65535)
+        return fail("paged_attention_pooled_decode: batch too large for one launch");
+    static bool configured = false;
+    const size_t smem = (size_t)(16 + 8 * RV_BN) * (RV_HD + 8) * sizeof(bf16);
+    if (!configured) {
+        if (smem > 48 * 1024) {
+            cudaError_t e = cudaFuncSetAttribute(paged_attention_decode_mma_kernel<RV_HD, 4, true>,
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (e != cudaSuccess) return fail(cudaGetErrorString(e));
+        }
+        configured = true;
+    }
+    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, cap, psplits};
+    float* part_o = (float*)scratch;
+    float2* part_ml = (float2*)((char*)scratch + slots * RV_HD * 4);
+    rv_launch(paged_attention_decode_mma_kernel<RV_HD, 4, true>,
+              dim3(num_kv_heads * tiles_per_head, max_splits, n_reqs), dim3(128), smem,
+              (cudaStream_t)stream, (const bf16*)q, q_stride, (const bf16*)k_cache,
+              (const bf16*)v_cache, block_table, max_blocks, ctx_lens, part_o, part_ml, max_splits,
+              num_heads, num_kv_heads, page_size, scale * 1.4426950408889634f, window, pl);
+    cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) return fail(cudaGetErrorString(e));
+    return 0;
+}
+#else
 // Prefill: requests [first_req, first_req + n_reqs), the longest bringing max_q_len tokens.
 extern "C" int RV_SYM(rv_paged_attention_prefill_mma)(
     const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* block_table,
@@ -833,13 +978,13 @@ extern "C" int RV_SYM(rv_paged_attention_prefill_mma)(
                   (cudaStream_t)stream, (const bf16*)q, q_stride, (const bf16*)k_cache,
                   (const bf16*)v_cache, block_table, max_blocks, q_start, ctx_lens, (bf16*)out,
                   (float*)nullptr, (float2*)nullptr, 0, first_req, num_heads, num_kv_heads, page_size,
-                  scale * 1.4426950408889634f, window, sinks);
+                  scale * 1.4426950408889634f, window, sinks, RvPooled());
     else
         rv_launch(paged_attention_mma_kernel<RV_HD, 4, false>, dim3(grid), dim3(128), smem_bytes<4>(),
                   (cudaStream_t)stream, (const bf16*)q, q_stride, (const bf16*)k_cache,
                   (const bf16*)v_cache, block_table, max_blocks, q_start, ctx_lens, (bf16*)out,
                   (float*)nullptr, (float2*)nullptr, 0, first_req, num_heads, num_kv_heads, page_size,
-                  scale * 1.4426950408889634f, window, sinks);
+                  scale * 1.4426950408889634f, window, sinks, RvPooled());
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return fail(cudaGetErrorString(e));
     return 0;
@@ -890,12 +1035,14 @@ extern "C" int RV_SYM(rv_paged_attention_decode_mma)(
         rv_launch(paged_attention_decode_mma_kernel<RV_HD, 4>, dim3(grid), dim3(128), smem4,
                   (cudaStream_t)stream, (const bf16*)q, q_stride, (const bf16*)k_cache,
                   (const bf16*)v_cache, block_table, max_blocks, ctx_lens, part_o, part_ml,
-                  max_splits, num_heads, num_kv_heads, page_size, scale * 1.4426950408889634f, window);
+                  max_splits, num_heads, num_kv_heads, page_size, scale * 1.4426950408889634f, window,
+                  RvPooled());
     else
         rv_launch(paged_attention_decode_mma_kernel<RV_HD, 2>, dim3(grid), dim3(64), smem2,
                   (cudaStream_t)stream, (const bf16*)q, q_stride, (const bf16*)k_cache,
                   (const bf16*)v_cache, block_table, max_blocks, ctx_lens, part_o, part_ml,
-                  max_splits, num_heads, num_kv_heads, page_size, scale * 1.4426950408889634f, window);
+                  max_splits, num_heads, num_kv_heads, page_size, scale * 1.4426950408889634f, window,
+                  RvPooled());
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return fail(cudaGetErrorString(e));
     return 0;
@@ -993,3 +1140,4 @@ extern "C" int RV_SYM(rv_paged_attention_decode_stream)(
     return 0;
 }
 #endif
+#endif   // RV_POOLED

@@ -22,9 +22,12 @@
 // it enters as the initial running maximum with a sum of 1, in the split form once, in the
 // merge.  Key sizes that are no multiple of 8 (bfloat16) or 4 (float32) elements take scalar
 // loads.
+// A third (template flag EXT): a window of tokens and pooled blocks before it, and capped scores
+// (attention_pooled.cuh); the plain instantiations do not carry it.
 // Reference counterparts: kv_gather.cu (twice), a batched SGEMM, mask_add_broadcast.cu,
 // softmax.cu, a batched SGEMM and transposes (src/cuda/model.rs:528-581).
 // Plain reference: tests/plain_ops.py paged_attention.
+#include "attention_pooled.cuh"
 #include "common.cuh"
 
 #define RV_ATTN_MAX_DPL 16     // head sizes up to 512: up to 16 dimensions per lane
@@ -34,6 +37,14 @@
 template <bool kFast>
 __device__ __forceinline__ float rv_exp(float x) {
     return kFast ? __expf(x) : expf(x);
+}
+
+// cap * tanh(s / cap).  kFast (the result is weighed against bfloat16 values): through one
+// exponential and a fast division, whose error is some 1e-7 of the cap.
+template <bool kFast>
+__device__ __forceinline__ float rv_cap(float s, float cap) {
+    if (!kFast) return cap * tanhf(s / cap);
+    return cap - 2.f * cap * __fdividef(1.f, 1.f + __expf(2.f * s / cap));
 }
 
 // dot product of a float32 vector in shared memory with a stored row
@@ -72,14 +83,14 @@ __device__ __forceinline__ float rv_dot_any(const float* __restrict__ q, const T
 }
 
 // ---------------------------------------------------------------------------------
-template <typename T, int DPL>
+template <typename T, int DPL, bool EXT>
 __global__ void paged_attention_warp_kernel(
     const T* __restrict__ q, int q_stride, const T* __restrict__ k_cache,
     const T* __restrict__ v_cache, const int* __restrict__ block_table, int max_blocks,
     const int* __restrict__ q_start, const int* __restrict__ ctx_lens,
     const int* __restrict__ token_req, T* __restrict__ out, int first_token, int n_tokens,
     int num_heads, int num_kv_heads, int hd, int page_size, float scale, int window, int vd,
-    const float* __restrict__ sinks) {
+    const float* __restrict__ sinks, const RvPooled pl) {
     rv_pdl_prologue();
     constexpr bool kFast = sizeof(T) == 2;
     const bool vec = hd % (16 / (int)sizeof(T)) == 0;
@@ -108,17 +119,24 @@ __global__ void paged_attention_warp_kernel(
     float m = sinks ? sinks[h] : -INFINITY, l = sinks ? 1.f : 0.f, acc[DPL];
 #pragma unroll
     for (int i = 0; i < DPL; ++i) acc[i] = 0.f;
-    const int* table = block_table + (size_t)r * max_blocks;
     const size_t row = (size_t)num_kv_heads * hd, vrow_len = (size_t)num_kv_heads * vd;
 
-    for (int base = lo & ~31; base <= p; base += 32) {
+    // EXT: the pooled blocks first, then the tokens
+    for (int part = EXT && pl.pool > 0 ? 0 : 1; part < 2; ++part) {
+    const bool blocks = EXT && part == 0;
+    const int first = blocks ? 0 : lo, last = blocks ? rv_seen_blocks(p, window, pl.pool) - 1 : p;
+    const int* table = blocks ? pl.table + (size_t)r * pl.max_blocks : block_table + (size_t)r * max_blocks;
+    const T* kc = blocks ? (const T*)pl.k : k_cache;
+    const T* vc = blocks ? (const T*)pl.v : v_cache;
+    for (int base = first & ~31; base <= last; base += 32) {
         const int j = base + lane;
-        const bool valid = j >= lo && j <= p;
+        const bool valid = j >= first && j <= last;
         int slot = 0;
         float s = -INFINITY;
         if (valid) {
             slot = table[j / page_size] * page_size + j % page_size;
-            s = rv_dot_any(qv, k_cache + (size_t)slot * row + (size_t)g * hd, hd, vec) * scale;
+            s = rv_dot_any(qv, kc + (size_t)slot * row + (size_t)g * hd, hd, vec) * scale;
+            if (EXT && pl.cap > 0.f) s = rv_cap<kFast>(s, pl.cap);
         }
         const float m_new = fmaxf(m, rv_warp_max(s));
         const float pj = valid ? rv_exp<kFast>(s - m_new) : 0.f;
@@ -127,12 +145,12 @@ __global__ void paged_attention_warp_kernel(
         m = m_new;
 #pragma unroll
         for (int i = 0; i < DPL; ++i) acc[i] *= corr;
-        const int count = min(32, p - base + 1);
+        const int count = min(32, last - base + 1);
         for (int jj = 0; jj < count; ++jj) {
             const float pk = __shfl_sync(0xffffffffu, pj, jj);
             const int sk = __shfl_sync(0xffffffffu, slot, jj);
             if (pk != 0.f) {
-                const T* vrow = v_cache + (size_t)sk * vrow_len + (size_t)g * vd;
+                const T* vrow = vc + (size_t)sk * vrow_len + (size_t)g * vd;
 #pragma unroll
                 for (int i = 0; i < DPL; ++i) {
                     const int d = lane + 32 * i;
@@ -140,6 +158,7 @@ __global__ void paged_attention_warp_kernel(
                 }
             }
         }
+    }
     }
 #pragma unroll
     for (int i = 0; i < DPL; ++i) {
@@ -151,13 +170,13 @@ __global__ void paged_attention_warp_kernel(
 // ---------------------------------------------------------------------------------
 // Decode: requests [0, n_reqs) bring one token each, token index == request index.
 // Scratch per (request, head, split): part_o[hd] (unnormalised) and part_ml = (max, sum).
-template <typename T, int DPL>
+template <typename T, int DPL, bool EXT>
 __global__ void __launch_bounds__(128) paged_attention_decode_kernel(
     const T* __restrict__ q, int q_stride, const T* __restrict__ k_cache,
     const T* __restrict__ v_cache, const int* __restrict__ block_table, int max_blocks,
     const int* __restrict__ ctx_lens, float* __restrict__ part_o, float2* __restrict__ part_ml,
     int max_splits, int num_heads, int num_kv_heads, int hd, int page_size, float scale,
-    int window, int vd) {
+    int window, int vd, const RvPooled pl) {
     rv_pdl_prologue();
     constexpr bool kFast = sizeof(T) == 2;
     constexpr int GT = RV_ATTN_GT;
@@ -174,9 +193,13 @@ __global__ void __launch_bounds__(128) paged_attention_decode_kernel(
     if (clen == 0) return;
     const int p = clen - 1;
     const int lo = window > 0 ? max(0, p - window + 1) : 0;
-    const int k0 = max(lo, split * RV_ATTN_SPLIT);
-    const int k1 = min(p, split * RV_ATTN_SPLIT + RV_ATTN_SPLIT - 1);   // inclusive
-    if (split < lo / RV_ATTN_SPLIT || k0 > k1) return;
+    // EXT: which rows this split covers (attention_pooled.cuh)
+    const bool blocks = EXT && split < pl.psplits;
+    const int stretch = !EXT || blocks ? split : split - pl.psplits + lo / RV_ATTN_SPLIT;
+    const int k0 = max(blocks ? 0 : lo, stretch * RV_ATTN_SPLIT);
+    const int k1 = min(blocks ? rv_seen_blocks(p, window, pl.pool) - 1 : p,
+                       stretch * RV_ATTN_SPLIT + RV_ATTN_SPLIT - 1);   // inclusive
+    if ((!EXT && split < lo / RV_ATTN_SPLIT) || k0 > k1) return;
 
     const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
     float* qv = smem;                                // [GT][hd]
@@ -197,12 +220,14 @@ __global__ void __launch_bounds__(128) paged_attention_decode_kernel(
 #pragma unroll
         for (int i = 0; i < DPL; ++i) acc[gi][i] = 0.f;
     }
-    const int* table = block_table + (size_t)r * max_blocks;
+    const int* table = blocks ? pl.table + (size_t)r * pl.max_blocks : block_table + (size_t)r * max_blocks;
+    const T* kc = blocks ? (const T*)pl.k : k_cache;
+    const T* vc = blocks ? (const T*)pl.v : v_cache;
     const size_t row = (size_t)num_kv_heads * hd, vrow_len = (size_t)num_kv_heads * vd;
     float* my_p = ps + w * 32 * GT;
     int* my_s = ss + w * 32;
 
-    const int split_base = split * RV_ATTN_SPLIT;
+    const int split_base = stretch * RV_ATTN_SPLIT;
     for (int base = split_base + w * 32; base <= k1; base += 4 * 32) {
         if (base + 31 < k0) continue;
         const int j = base + lane;
@@ -213,10 +238,13 @@ __global__ void __launch_bounds__(128) paged_attention_decode_kernel(
         for (int gi = 0; gi < GT; ++gi) s[gi] = -INFINITY;
         if (valid) {
             slot = table[j / page_size] * page_size + j % page_size;
-            const T* krow = k_cache + (size_t)slot * row + (size_t)g * hd;
+            const T* krow = kc + (size_t)slot * row + (size_t)g * hd;
 #pragma unroll
             for (int gi = 0; gi < GT; ++gi)
-                if (gi < gcount) s[gi] = rv_dot_any(qv + gi * hd, krow, hd, vec) * scale;
+                if (gi < gcount) {
+                    s[gi] = rv_dot_any(qv + gi * hd, krow, hd, vec) * scale;
+                    if (EXT && pl.cap > 0.f) s[gi] = rv_cap<kFast>(s[gi], pl.cap);
+                }
         }
         my_s[lane] = slot;
 #pragma unroll
@@ -237,7 +265,7 @@ __global__ void __launch_bounds__(128) paged_attention_decode_kernel(
         __syncwarp();
         const int count = min(32, k1 - base + 1);
         for (int jj = max(0, k0 - base); jj < count; ++jj) {
-            const T* vrow = v_cache + (size_t)my_s[jj] * vrow_len + (size_t)g * vd;
+            const T* vrow = vc + (size_t)my_s[jj] * vrow_len + (size_t)g * vd;
             float pk[GT];
 #pragma unroll
             for (int gi = 0; gi < GT; ++gi) pk[gi] = my_p[jj * GT + gi];
@@ -286,12 +314,13 @@ __global__ void __launch_bounds__(128) paged_attention_decode_kernel(
     }
 }
 
-template <typename T>
+template <typename T, bool EXT>
 __global__ void paged_attention_merge_kernel(const float* __restrict__ part_o,
                                              const float2* __restrict__ part_ml,
                                              const int* __restrict__ ctx_lens, T* __restrict__ out,
                                              int max_splits, int num_heads, int hd, int window,
-                                             int split_keys, const float* __restrict__ sinks) {
+                                             int split_keys, const float* __restrict__ sinks,
+                                             int psplits, int pool) {
     rv_pdl_launch_dependents();
     constexpr bool kFast = sizeof(T) == 2;
     const int r = blockIdx.y, h = blockIdx.x;
@@ -307,11 +336,14 @@ __global__ void paged_attention_merge_kernel(const float* __restrict__ part_o,
     const int lo = window > 0 ? max(0, p - window + 1) : 0;
     // A context longer than the launch's max_ctx_len has keys that no split covered: the row
     // is marked invalid (NaN) and nothing outside this head's slots is read.
-    if (clen > max_splits * split_keys) {
+    // (EXT: splits that cover blocks, then splits that cover tokens from the window's first on.)
+    const int np = EXT ? (rv_seen_blocks(p, window, pool) + split_keys - 1) / split_keys : 0;
+    const int nt = p / split_keys - lo / split_keys + 1;
+    if (EXT ? (np > psplits || nt > max_splits - psplits) : (clen > max_splits * split_keys)) {
         for (int d = threadIdx.x; d < hd; d += blockDim.x) rv_store(o + d, NAN);
         return;
     }
-    const int s0 = lo / split_keys, s1 = min(p / split_keys, max_splits - 1);
+    const int s0 = EXT ? 0 : lo / split_keys, s1 = EXT ? np + nt - 1 : min(p / split_keys, max_splits - 1);
     const size_t base = ((size_t)r * num_heads + h) * max_splits;
     // Splits are combined in order, sixteen at a time: the loads of a group are independent, so
     // a group costs one memory latency, not sixteen.
@@ -324,8 +356,9 @@ __global__ void paged_attention_merge_kernel(const float* __restrict__ part_o,
 #pragma unroll
             for (int i = 0; i < GROUP; ++i) {
                 const bool valid = sb + i <= s1;
-                ml[i] = valid ? part_ml[base + sb + i] : make_float2(-INFINITY, 0.f);
-                po[i] = valid ? part_o[(base + sb + i) * hd + d] : 0.f;
+                const int sp = EXT && sb + i >= np ? sb + i - np + psplits : sb + i;
+                ml[i] = valid ? part_ml[base + sp] : make_float2(-INFINITY, 0.f);
+                po[i] = valid ? part_o[(base + sp) * hd + d] : 0.f;
             }
             float mg = M;
 #pragma unroll
@@ -389,10 +422,10 @@ extern "C" int rv_paged_attention_warp_ex(const void* q, int dtype, int q_stride
     const size_t smem = (size_t)wpb * hd * sizeof(float);
     cudaStream_t s = (cudaStream_t)stream;
     RV_DISPATCH_DTYPE(dtype, "paged_attention",
-        RV_DISPATCH_DPL(vd, (rv_launch(paged_attention_warp_kernel<T, DPL>, dim3((int)blocks), dim3(wpb * 32), smem, s, 
+        RV_DISPATCH_DPL(vd, (rv_launch(paged_attention_warp_kernel<T, DPL, false>, dim3((int)blocks), dim3(wpb * 32), smem, s, 
             (const T*)q, q_stride, (const T*)k_cache, (const T*)v_cache, block_table, max_blocks,
             q_start, ctx_lens, token_req, (T*)out, first_token, n_tokens, num_heads, num_kv_heads,
-            hd, page_size, scale, window, vd, sinks))));
+            hd, page_size, scale, window, vd, sinks, RvPooled()))));
     RV_CHECK_LAUNCH("paged_attention");
     return 0;
 }
@@ -446,16 +479,16 @@ extern "C" int rv_paged_attention_decode_ex(const void* q, int dtype, int q_stri
                                  4 * RV_ATTN_GT * (vd + 2)) * sizeof(float);
     cudaStream_t s = (cudaStream_t)stream;
     RV_DISPATCH_DTYPE(dtype, "paged_attention_decode",
-        RV_DISPATCH_DPL(vd, (rv_launch(paged_attention_decode_kernel<T, DPL>, dim3(grid), dim3(128), smem, s, 
+        RV_DISPATCH_DPL(vd, (rv_launch(paged_attention_decode_kernel<T, DPL, false>, dim3(grid), dim3(128), smem, s, 
             (const T*)q, q_stride, (const T*)k_cache, (const T*)v_cache, block_table, max_blocks,
             ctx_lens, part_o, part_ml, max_splits, num_heads, num_kv_heads, hd, page_size, scale,
-            window, vd))));
+            window, vd, RvPooled()))));
     RV_CHECK_LAUNCH("paged_attention_decode");
     dim3 mgrid(num_heads, n_reqs);
     RV_DISPATCH_DTYPE(dtype, "paged_attention_merge",
-        (rv_launch(paged_attention_merge_kernel<T>, dim3(mgrid), dim3(merge_threads(vd)), 0, s, 
+        (rv_launch(paged_attention_merge_kernel<T, false>, dim3(mgrid), dim3(merge_threads(vd)), 0, s, 
             part_o, part_ml, ctx_lens, (T*)out, max_splits, num_heads, vd, window, RV_ATTN_SPLIT,
-            sinks)));
+            sinks, 0, 0)));
     RV_CHECK_LAUNCH("paged_attention_merge");
     return 0;
 }
@@ -490,9 +523,9 @@ extern "C" int rv_paged_attention_merge_ex(const void* scratch, const int* ctx_l
     const float2* part_ml = (const float2*)((const char*)scratch + slots * hd * 4);
     dim3 mgrid(num_heads, n_reqs);
     RV_DISPATCH_DTYPE(dtype, "paged_attention_merge",
-        (rv_launch(paged_attention_merge_kernel<T>, dim3(mgrid), dim3(merge_threads(hd)), 0, (cudaStream_t)stream, 
+        (rv_launch(paged_attention_merge_kernel<T, false>, dim3(mgrid), dim3(merge_threads(hd)), 0, (cudaStream_t)stream, 
             part_o, part_ml, ctx_lens, (T*)out, max_splits, num_heads, hd, window, split_keys,
-            sinks)));
+            sinks, 0, 0)));
     RV_CHECK_LAUNCH("paged_attention_merge");
     return 0;
 }
@@ -502,4 +535,105 @@ extern "C" int rv_paged_attention_merge(const void* scratch, const int* ctx_lens
                                         int hd, int window, int split_keys, void* stream) {
     return rv_paged_attention_merge_ex(scratch, ctx_lens, out, dtype, n_reqs, max_ctx_len,
                                        num_heads, hd, window, split_keys, nullptr, stream);
+}
+
+// ---------------------------------------------------------------------------------
+// Attention over a window of tokens and the pooled blocks before it (attention_pooled.cuh).
+// `window` 0: every token is seen; `pool` 0: no blocks (pk, pv, ptable unused); `cap` 0: scores are
+// not capped; key and value heads have the same size.
+
+// Bytes of scratch of the split form: part_o then part_ml.
+extern "C" long long rv_paged_attention_pooled_scratch_bytes(int n_reqs, int num_heads, int hd,
+                                                             int max_ctx_len, int window, int pool) {
+    const long long splits = rv_pooled_psplits(max_ctx_len, window, pool, RV_ATTN_SPLIT) +
+                             rv_pooled_tsplits(max_ctx_len, window, RV_ATTN_SPLIT);
+    return (long long)n_reqs * num_heads * splits * (hd * 4 + 8);
+}
+
+static int pooled_check(const char* name, int num_heads, int num_kv_heads, int hd, int page_size,
+                        int window, int pool, const void* pk, const void* pv, const int* ptable, int dtype) {
+    if (check_attention_sizes(name, num_heads, num_kv_heads, hd, hd, page_size, dtype)) return 1;
+    if (window < 0 || pool < 0 || (pool > 0 && (window == 0 || !pk || !pv || !ptable)))
+        RV_FAIL("%s: pooled blocks need a window, pages and a block table", name);
+    return 0;
+}
+
+// One warp per (token, query head), any number of new tokens per request.
+extern "C" int rv_paged_attention_pooled_warp(
+    const void* q, int dtype, int q_stride, const void* k_cache, const void* v_cache,
+    const int* block_table, int max_blocks, const void* pk, const void* pv, const int* ptable,
+    int pmax_blocks, int pool, float cap, const int* q_start, const int* ctx_lens,
+    const int* token_req, void* out, int first_token, int n_tokens, int num_heads, int num_kv_heads,
+    int hd, int page_size, float scale, int window, const float* sinks, void* stream) {
+    if (n_tokens == 0) return 0;
+    if (pooled_check("paged_attention_pooled", num_heads, num_kv_heads, hd, page_size, window, pool, pk,
+                     pv, ptable, dtype))
+        return 1;
+    const int wpb = 4;
+    const long long warps = (long long)n_tokens * num_heads;
+    const long long blocks = (warps + wpb - 1) / wpb;
+    if (blocks > 0x7fffffffLL) RV_FAIL("paged_attention_pooled: too many rows");
+    const size_t smem = (size_t)wpb * hd * sizeof(float);
+    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, cap, 0};
+    RV_DISPATCH_DTYPE(dtype, "paged_attention_pooled",
+        RV_DISPATCH_DPL(hd, (rv_launch(paged_attention_warp_kernel<T, DPL, true>, dim3((int)blocks),
+            dim3(wpb * 32), smem, (cudaStream_t)stream, (const T*)q, q_stride, (const T*)k_cache,
+            (const T*)v_cache, block_table, max_blocks, q_start, ctx_lens, token_req, (T*)out,
+            first_token, n_tokens, num_heads, num_kv_heads, hd, page_size, scale, window, hd, sinks, pl))));
+    RV_CHECK_LAUNCH("paged_attention_pooled");
+    return 0;
+}
+
+// The merge of split results in the layout above (this file's kernel or attention_mma.cu's).
+extern "C" int rv_paged_attention_pooled_merge(const void* scratch, const int* ctx_lens, void* out,
+                                               int dtype, int n_reqs, int max_ctx_len, int num_heads,
+                                               int hd, int window, int pool, const float* sinks,
+                                               void* stream) {
+    if (n_reqs == 0) return 0;
+    const int psplits = rv_pooled_psplits(max_ctx_len, window, pool, RV_ATTN_SPLIT);
+    const int max_splits = psplits + rv_pooled_tsplits(max_ctx_len, window, RV_ATTN_SPLIT);
+    const size_t slots = (size_t)n_reqs * num_heads * max_splits;
+    const float* part_o = (const float*)scratch;
+    const float2* part_ml = (const float2*)((const char*)scratch + slots * hd * 4);
+    RV_DISPATCH_DTYPE(dtype, "paged_attention_pooled_merge",
+        (rv_launch(paged_attention_merge_kernel<T, true>, dim3(num_heads, n_reqs), dim3(merge_threads(hd)),
+            0, (cudaStream_t)stream, part_o, part_ml, ctx_lens, (T*)out, max_splits, num_heads, hd,
+            window, RV_ATTN_SPLIT, sinks, psplits, pool)));
+    RV_CHECK_LAUNCH("paged_attention_pooled_merge");
+    return 0;
+}
+
+// Requests [0, n_reqs) bring one token each: splits, then the merge.
+extern "C" int rv_paged_attention_pooled_decode(
+    const void* q, int dtype, int q_stride, const void* k_cache, const void* v_cache,
+    const int* block_table, int max_blocks, const void* pk, const void* pv, const int* ptable,
+    int pmax_blocks, int pool, float cap, const int* ctx_lens, void* out, void* scratch,
+    long long scratch_bytes, int n_reqs, int max_ctx_len, int num_heads, int num_kv_heads, int hd,
+    int page_size, float scale, int window, const float* sinks, void* stream) {
+    if (n_reqs == 0) return 0;
+    if (pooled_check("paged_attention_pooled_decode", num_heads, num_kv_heads, hd, page_size, window,
+                     pool, pk, pv, ptable, dtype))
+        return 1;
+    const int psplits = rv_pooled_psplits(max_ctx_len, window, pool, RV_ATTN_SPLIT);
+    const int max_splits = psplits + rv_pooled_tsplits(max_ctx_len, window, RV_ATTN_SPLIT);
+    if (rv_paged_attention_pooled_scratch_bytes(n_reqs, num_heads, hd, max_ctx_len, window, pool) > scratch_bytes)
+        RV_FAIL("paged_attention_pooled_decode: scratch of %lld bytes is too small", scratch_bytes);
+    if (n_reqs > 65535 || max_splits > 65535) RV_FAIL("paged_attention_pooled_decode: batch too large");
+    const size_t slots = (size_t)n_reqs * num_heads * max_splits;
+    float* part_o = (float*)scratch;
+    float2* part_ml = (float2*)((char*)scratch + slots * hd * 4);
+    const int G = num_heads / num_kv_heads;
+    const int tiles = (G + RV_ATTN_GT - 1) / RV_ATTN_GT;
+    const size_t smem = (size_t)(RV_ATTN_GT * hd + 4 * 32 * RV_ATTN_GT + 4 * 32 +
+                                 4 * RV_ATTN_GT * (hd + 2)) * sizeof(float);
+    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, cap, psplits};
+    RV_DISPATCH_DTYPE(dtype, "paged_attention_pooled_decode",
+        RV_DISPATCH_DPL(hd, (rv_launch(paged_attention_decode_kernel<T, DPL, true>,
+            dim3(num_kv_heads * tiles, n_reqs, max_splits), dim3(128), smem, (cudaStream_t)stream,
+            (const T*)q, q_stride, (const T*)k_cache, (const T*)v_cache, block_table, max_blocks,
+            ctx_lens, part_o, part_ml, max_splits, num_heads, num_kv_heads, hd, page_size, scale,
+            window, hd, pl))));
+    RV_CHECK_LAUNCH("paged_attention_pooled_decode");
+    return rv_paged_attention_pooled_merge(scratch, ctx_lens, out, dtype, n_reqs, max_ctx_len, num_heads,
+                                           hd, window, pool, sinks, stream);
 }

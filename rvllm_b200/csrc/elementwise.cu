@@ -30,34 +30,50 @@ __device__ __forceinline__ void rv_store4(__nv_bfloat16* p, float4 v) {
 }
 
 // ---------------------------------------------------------------------------------
-// Embedding gather: out[t, :] = table[ids[t], :] (* scale), float32 out.
+// Embedding gather: out[t, :] = table[ids[t], :] (* scale) (+ pos_table[positions[t], :]),
+// float32 out.
 // Reference counterpart: embed_lookup.cu (one thread per element, float32 table).
 template <typename T>
 __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                             float* __restrict__ out, int hidden, int vocab, float scale) {
+                             float* __restrict__ out, int hidden, int vocab, float scale,
+                             const int* __restrict__ positions, const T* __restrict__ pos_table,
+                             int n_positions) {
     rv_pdl_prologue();
     const int t = blockIdx.x;
     int id = ids[t];
     id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
     const T* row = table + (size_t)id * hidden;
+    const T* prow = nullptr;
+    if (pos_table) prow = pos_table + (size_t)min(max(positions[t], 0), n_positions - 1) * hidden;
     float* o = out + (size_t)t * hidden;
-    if (hidden % 4 == 0 && ((uintptr_t)table % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
+    if (hidden % 4 == 0 && ((uintptr_t)table % 16 == 0) && ((uintptr_t)out % 16 == 0) &&
+        ((uintptr_t)pos_table % 16 == 0)) {
         for (int i = threadIdx.x; i < hidden / 4; i += blockDim.x) {
-            const float4 v = rv_load4(row + 4 * i);
-            rv_store4(o + 4 * i, make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale));
+            float4 v = rv_load4(row + 4 * i);
+            v = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+            if (prow) {
+                const float4 p = rv_load4(prow + 4 * i);
+                v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
+            }
+            rv_store4(o + 4 * i, v);
         }
         return;
     }
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = rv_load(row + i) * scale;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x)
+        o[i] = rv_load(row + i) * scale + (prow ? rv_load(prow + i) : 0.f);
 }
 
+// `pos_table` [n_positions, hidden] of the table's type and `positions` int32 [n_tokens], or null.
 extern "C" int rv_embed(const void* table, int dtype, const int* ids, float* out, int n_tokens,
-                        int hidden, int vocab, float scale, void* stream) {
+                        int hidden, int vocab, float scale, const int* positions,
+                        const void* pos_table, int n_positions, void* stream) {
     if (n_tokens == 0) return 0;
     if (n_tokens < 0 || hidden <= 0 || vocab <= 0) RV_FAIL("embed: bad sizes");
+    if (pos_table && (!positions || n_positions <= 0)) RV_FAIL("embed: a position table without positions");
     RV_DISPATCH_DTYPE(dtype, "embed",
                       (rv_launch(embed_kernel<T>, dim3(n_tokens), dim3(hidden >= 2048 ? 512 : 256), 0, (cudaStream_t)stream, 
-                          (const T*)table, ids, out, hidden, vocab, scale)));
+                          (const T*)table, ids, out, hidden, vocab, scale,
+                          positions, (const T*)pos_table, n_positions)));
     RV_CHECK_LAUNCH("embed");
     return 0;
 }

@@ -1,0 +1,703 @@
+// Linear attention with decay: per head a float32 matrix S [d, dv] that starts at zero,
+//
+//     S <- diag(a_t) S + k_t v_t^T;   o_t = S^T q_t
+//     y = o / sqrt(mean(o^2) + eps) * w * gate(g)          the mean over all heads or per head
+//
+// The decay a_t is a constant per head (log_decay [H]) or made by the token for every key channel,
+// log a = logsigmoid(z + bias) / tau.  q, k and v may pass silu; q is multiplied by q_scale.
+// Everything here is float32.
+//
+// rows [N, stride] float32: q [H d] | k [H d] | v [H dv] | g [H dv] | z [H d] (decays by tokens).
+// A request's record: [H][d][dv] float32.
+//
+// Requests [0, n_decode) bring one token each: la_token reads and writes every state element
+// once.  The others' portions are cut into chunks of 64 tokens, counted from the portion's
+// start, and a chunk is a few small matrix products instead of 64 dependent steps.  With B_i the
+// sum of the log decays of the chunk's tokens 0..i and L its last token:
+//
+//   state  block per (chunk, head, 64 x 64 tile):   KV = sum_j (k_j e^(B_L - B_j)) v_j^T
+//   scan   thread per state element: over the chunks of a request one after another, the state
+//          before the chunk replaces KV, S <- e^(B_L) S + KV; the last one is the record
+//   out    block per (chunk, head, 64 columns):
+//          o_i = sum_(j <= i) <q_i, e^(B_i - B_j) k_j> v_j + S^T (q_i e^(B_i))
+//
+// No factor is ever above 1, however strong the decays are, so nothing overflows and what underflows
+// is nothing: with decays by channel, the tokens of a chunk form eight groups of eight, a pair
+// of tokens in different groups I > J splits its factor into e^(B_i - B_(before I)) on q,
+// e^(B_(before I) - B_(end of J)) from a table, and e^(B_(end of J) - B_j) on k; a pair inside a
+// group takes the exponential of its own difference for every channel.
+//   finish  the norm, weight and gate.
+// Plain reference: tests/plain_ops.py linear_attention.
+#include "common.cuh"
+
+#define LA_C 64             // tokens a chunk
+#define LA_T 64             // columns (and rows) of a tile
+#define LA_DK 32            // key channels staged at a time in `out`
+#define LA_LD 68            // padded row of 64
+#define LA_G 8              // tokens a group
+#define LA_NG 8             // groups a chunk
+
+__device__ __forceinline__ float la_logsigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float la_act(float x, int act) { return act ? x / (1.f + expf(-x)) : x; }
+
+// Chunk `item` of the portions of requests [first_req, n_reqs): its request and its number there;
+// and how many chunks lie before the request.  Requests without a slot have none.  Whole warp.
+__device__ __forceinline__ int la_chunks(const int* q_start, const int* state_slot, int r) {
+    return state_slot[r] < 0 ? 0 : (q_start[r + 1] - q_start[r] + LA_C - 1) / LA_C;
+}
+__device__ __forceinline__ bool la_find(const int* q_start, const int* state_slot, int first_req,
+                                        int n_reqs, int item, int lane, int& r, int& before) {
+    before = 0;
+    for (int base = first_req; base < n_reqs; base += 32) {
+        const int n = base + lane < n_reqs ? la_chunks(q_start, state_slot, base + lane) : 0;
+        int incl = n;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int up = __shfl_up_sync(0xffffffffu, incl, o);
+            if (lane >= o) incl += up;
+        }
+        const unsigned hit = __ballot_sync(0xffffffffu, before + incl > item);
+        if (hit) {
+            const int l = __ffs(hit) - 1;
+            r = base + l;
+            before += __shfl_sync(0xffffffffu, incl - n, l);
+            return true;
+        }
+        before += __shfl_sync(0xffffffffu, incl, 31);
+    }
+    return false;
+}
+
+// ---- single tokens ---------------------------------------------------------------------
+// V = 4: 16-byte accesses to the state and sixteen lanes across a tile's 64 columns; V = 1: 64.
+template <int V>
+__global__ void __launch_bounds__(128) la_token_kernel(
+    const float* __restrict__ rows, int stride, const float* __restrict__ log_decay,
+    const float* __restrict__ bias, float tau, const int* __restrict__ q_start,
+    const int* __restrict__ state_slot, float* __restrict__ state, float* __restrict__ num, int H,
+    int d, int dv, int act, float q_scale) {
+    rv_pdl_launch_dependents();
+    constexpr int LANES = LA_T / V, RG = 128 / LANES;            // row groups
+    extern __shared__ float sm[];
+    float* qs = sm;                                              // [d]
+    float* ks = qs + d;
+    float* as = ks + d;
+    float* red = as + d;                                         // [RG][64]
+    const int h = blockIdx.y, r = blockIdx.z;
+    const int slot = state_slot[r];
+    const int t = q_start[r];
+    rv_pdl_wait();
+    if (slot < 0) return;
+    const float* row = rows + (size_t)t * stride;
+    const float ad = log_decay ? expf(log_decay[h]) : 0.f;
+    for (int i = threadIdx.x; i < d; i += 128) {
+        qs[i] = la_act(row[h * d + i], act) * q_scale;
+        ks[i] = la_act(row[(H + h) * d + i], act);
+        as[i] = log_decay ? ad
+                          : expf(la_logsigmoid(row[2 * H * d + 2 * H * dv + h * d + i] + bias[h * d + i]) / tau);
+    }
+    const int cl = threadIdx.x % LANES, rg = threadIdx.x / LANES;
+    const int col = blockIdx.x * LA_T + cl * V;
+    float v[V], o[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+        o[e] = 0.f;
+        v[e] = col + e < dv ? la_act(row[2 * H * d + h * dv + col + e], act) : 0.f;
+    }
+    __syncthreads();
+    float* S = state + ((size_t)slot * H + h) * d * dv;
+    if (col < dv) {
+#pragma unroll 8
+        for (int i = rg; i < d; i += RG) {
+            const float a = as[i], k = ks[i], q = qs[i];
+            float* p = S + (size_t)i * dv + col;
+            if (V == 4) {
+                float4 s = *(float4*)p;
+                s.x = fmaf(a, s.x, k * v[0]);
+                s.y = fmaf(a, s.y, k * v[1 % V]);
+                s.z = fmaf(a, s.z, k * v[2 % V]);
+                s.w = fmaf(a, s.w, k * v[3 % V]);
+                o[0] = fmaf(s.x, q, o[0]);
+                o[1 % V] = fmaf(s.y, q, o[1 % V]);
+                o[2 % V] = fmaf(s.z, q, o[2 % V]);
+                o[3 % V] = fmaf(s.w, q, o[3 % V]);
+                *(float4*)p = s;
+            } else {
+                const float s = fmaf(a, *p, k * v[0]);
+                o[0] = fmaf(s, q, o[0]);
+                *p = s;
+            }
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) red[rg * LA_T + cl * V + e] = o[e];
+    __syncthreads();
+    for (int c = threadIdx.x; c < LA_T; c += 128) {
+        if (blockIdx.x * LA_T + c >= dv) break;
+        float s = 0.f;
+#pragma unroll
+        for (int g = 0; g < RG; ++g) s += red[g * LA_T + c];
+        num[((size_t)t * H + h) * dv + blockIdx.x * LA_T + c] = s;
+    }
+}
+
+// ---- portions: every chunk's own contribution to the state ----------------------------------
+template <bool CHANNEL>
+__global__ void __launch_bounds__(256) la_state_kernel(
+    const float* __restrict__ rows, int stride, const float* __restrict__ log_decay,
+    const float* __restrict__ bias, float tau, const int* __restrict__ q_start,
+    const int* __restrict__ state_slot, int first_req, int n_reqs, float* __restrict__ kv,
+    float* __restrict__ dec, int H, int d, int dv, int act) {
+    rv_pdl_launch_dependents();
+    extern __shared__ __align__(16) float sm[];
+    float* ks = sm;                                              // [64 tokens][LD]: channels
+    float* vs = ks + LA_C * LA_LD;                               // [64 tokens][LD]: columns
+    float* lb = vs + LA_C * LA_LD;                               // [64 tokens][LD] (CHANNEL)
+    float* tot = lb + (CHANNEL ? LA_C * LA_LD : 0);              // [4][64] segments' sums
+    __shared__ int at[2];
+    const int tid = threadIdx.x, lane = tid & 31;
+    const int item = blockIdx.x, h = blockIdx.y;
+    const int tiles_v = (dv + LA_T - 1) / LA_T;
+    const int d0 = (blockIdx.z / tiles_v) * LA_T, v0 = (blockIdx.z % tiles_v) * LA_T;
+    if (tid < 32) {
+        int r = -1, before = 0;
+        const bool ok = la_find(q_start, state_slot, first_req, n_reqs, item, lane, r, before);
+        if (lane == 0) {
+            at[0] = ok ? q_start[r] + (item - before) * LA_C : -1;
+            at[1] = ok ? min(LA_C, q_start[r + 1] - at[0]) : 0;
+        }
+    }
+    __syncthreads();
+    const int t0 = at[0], L = at[1];
+    rv_pdl_wait();
+    if (t0 < 0) return;
+    const int x = tid & 63, y = tid >> 6;
+    const int dn = min(LA_T, d - d0), vn = min(LA_T, dv - v0);
+    const float* base = rows + (size_t)t0 * stride;
+    const float ld = CHANNEL ? 0.f : log_decay[h];
+    const float bz = CHANNEL && x < dn ? bias[h * d + d0 + x] : 0.f;
+    // four values of one column at a time are requested before any is worked on
+#pragma unroll 4
+    for (int j = y; j < LA_C; j += 4) {
+        const float* row = base + (size_t)j * stride;
+        const bool tj = j < L;
+        float k = tj && x < dn ? row[(H + h) * d + d0 + x] : 0.f;
+        const float v = tj && x < vn ? row[2 * H * d + h * dv + v0 + x] : 0.f;
+        k = la_act(k, act);
+        if (!CHANNEL) k *= expf(ld * (float)(L - 1 - min(j, L - 1)));
+        ks[j * LA_LD + x] = k;
+        vs[j * LA_LD + x] = la_act(v, act);
+        if (CHANNEL) {
+            const float z = tj && x < dn ? row[2 * H * d + 2 * H * dv + h * d + d0 + x] : 0.f;
+            lb[j * LA_LD + x] = tj && x < dn ? la_logsigmoid(z + bz) / tau : 0.f;
+        }
+    }
+    if (CHANNEL) {
+        __syncthreads();
+        float s = 0.f;                                           // tokens 16 y .. 16 y + 15
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+            s += lb[(16 * y + j) * LA_LD + x];
+            lb[(16 * y + j) * LA_LD + x] = s;
+        }
+        tot[y * 64 + x] = s;
+        __syncthreads();
+        float after = 0.f;                                       // the segments behind this one
+        for (int g = y + 1; g < 4; ++g) after += tot[g * 64 + x];
+#pragma unroll
+        for (int j = 0; j < 16; ++j)
+            ks[(16 * y + j) * LA_LD + x] *= expf(after + (s - lb[(16 * y + j) * LA_LD + x]));
+        if (y == 0 && v0 == 0 && x < dn)
+            dec[((size_t)item * H + h) * d + d0 + x] = expf(after + s);
+    }
+    __syncthreads();
+    const int ty = tid >> 4, tx = tid & 15;
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    const int jn = (L + 3) & ~3;                                 // zeros beyond L
+#pragma unroll 4
+    for (int j = 0; j < jn; ++j) {
+        const float4 a = *(const float4*)(ks + j * LA_LD + 4 * ty), b = *(const float4*)(vs + j * LA_LD + 4 * tx);
+        const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[i][e] = fmaf(av[i], bv[e], acc[i][e]);
+    }
+    float* o = kv + ((size_t)item * H + h) * d * dv;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int dd = 4 * ty + i;
+        if (dd >= dn) continue;
+        float* p = o + (size_t)(d0 + dd) * dv + v0 + 4 * tx;
+        if (dv % 4 == 0) {
+            if (4 * tx < vn) *(float4*)p = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                if (4 * tx + e < vn) p[e] = acc[i][e];
+        }
+    }
+}
+
+// ---- portions: the states between the chunks ---------------------------------------------------
+template <bool CHANNEL, int V>
+__global__ void __launch_bounds__(256) la_scan_kernel(
+    const float* __restrict__ log_decay, const int* __restrict__ q_start,
+    const int* __restrict__ state_slot, int first_req, float* __restrict__ kv,
+    const float* __restrict__ dec, float* __restrict__ state, int H, int d, int dv) {
+    rv_pdl_launch_dependents();
+    const int h = blockIdx.y, r = first_req + blockIdx.z;
+    const int slot = state_slot[r];
+    const int n = slot < 0 ? 0 : (q_start[r + 1] - q_start[r] + LA_C - 1) / LA_C;
+    __shared__ int first_item;
+    if (threadIdx.x < 32) {
+        int before = 0;
+        for (int b = first_req + threadIdx.x; b < r; b += 32) before += la_chunks(q_start, state_slot, b);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) before += __shfl_xor_sync(0xffffffffu, before, o);
+        if (threadIdx.x == 0) first_item = before;
+    }
+    __syncthreads();
+    const int last_len = q_start[r + 1] - q_start[r] - (n - 1) * LA_C;
+    const float ld = CHANNEL ? 0.f : log_decay[h];
+    rv_pdl_wait();
+    const long long el = ((long long)blockIdx.x * 256 + threadIdx.x) * V;
+    if (n == 0 || el >= (long long)d * dv) return;
+    const int ch = (int)(el / dv);
+    float* rec = state + ((size_t)slot * H + h) * d * dv + el;
+    float* p = kv + ((size_t)first_item * H + h) * d * dv + el;
+    const float* dp = CHANNEL ? dec + ((size_t)first_item * H + h) * d + ch : nullptr;
+    const size_t step = (size_t)H * d * dv, dstep = (size_t)H * d;
+    const float full = CHANNEL ? 0.f : expf(ld * (float)LA_C), rest = CHANNEL ? 0.f : expf(ld * (float)last_len);
+    float S[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) S[e] = 0.f;
+    if (V == 4) {
+        const float4 s = *(const float4*)rec;
+        S[0] = s.x; S[1 % V] = s.y; S[2 % V] = s.z; S[3 % V] = s.w;
+    } else {
+        S[0] = *rec;
+    }
+    constexpr int U = 4;                                         // chunks requested together
+    for (int c0 = 0; c0 < n; c0 += U) {
+        float in[U][V], a[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            if (c0 + u >= n) continue;
+            const float* s = p + (size_t)(c0 + u) * step;
+            if (V == 4) {
+                const float4 f = *(const float4*)s;
+                in[u][0] = f.x; in[u][1 % V] = f.y; in[u][2 % V] = f.z; in[u][3 % V] = f.w;
+            } else {
+                in[u][0] = *s;
+            }
+            a[u] = CHANNEL ? dp[(size_t)(c0 + u) * dstep] : (c0 + u == n - 1 ? rest : full);
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            if (c0 + u >= n) continue;
+            float* s = p + (size_t)(c0 + u) * step;
+            if (V == 4) *(float4*)s = make_float4(S[0], S[1 % V], S[2 % V], S[3 % V]);
+            else *s = S[0];
+#pragma unroll
+            for (int e = 0; e < V; ++e) S[e] = fmaf(a[u], S[e], in[u][e]);
+        }
+    }
+    if (V == 4) *(float4*)rec = make_float4(S[0], S[1 % V], S[2 % V], S[3 % V]);
+    else *rec = S[0];
+}
+
+// ---- portions: the outputs -------------------------------------------------------------------
+// A thread's share of a 64 x 64 product is rows 4 ty .. + 3 by columns 4 tx .. + 3; a warp's eight
+// rows are one group.  Operands lie with the summed index first ([c][64 tokens] and so on), so that
+// a thread reads four of its rows and four of its columns with one access each.
+template <bool CHANNEL>
+__global__ void __launch_bounds__(256) la_out_kernel(
+    const float* __restrict__ rows, int stride, const float* __restrict__ log_decay,
+    const float* __restrict__ bias, float tau, const int* __restrict__ q_start,
+    const int* __restrict__ state_slot, int first_req, int n_reqs, const float* __restrict__ kv,
+    float* __restrict__ num, int H, int d, int dv, int act, float q_scale) {
+    rv_pdl_launch_dependents();
+    extern __shared__ __align__(16) float sm[];
+    constexpr int SL = LA_DK * LA_LD;
+    float* qt = sm;                                 // [DK][LD]: q e^(B_i - B before its group)
+    float* kt = qt + SL;                            // [DK][LD]: k e^(B at its group's end - B_j)
+    float* ss = kt + SL;                            // [DK][LD]: the state's rows, 64 columns
+    float* ps = ss + SL;                            // [64 j][LD i]: scores
+    float* vs = ps + LA_C * LA_LD;                  // [64 j][LD]: values
+    float* qr = vs + LA_C * LA_LD;                  // CHANNEL: [DK][LD] q as it is
+    float* kr = qr + (CHANNEL ? SL : 0);            //          [DK][LD] k as it is
+    float* lb = kr + (CHANNEL ? SL : 0);            //          [DK][LD] B_i - B before its group
+    float* off = lb + (CHANNEL ? SL : 0);           //          [NG + 1][DK + 1] B before a group
+    float* tab = off + (CHANNEL ? (LA_NG + 1) * (LA_DK + 1) : 0);   // [NG][NG][DK + 1]
+    __shared__ int at[2];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int item = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * LA_T;
+    if (tid < 32) {
+        int r = -1, before = 0;
+        const bool ok = la_find(q_start, state_slot, first_req, n_reqs, item, lane, r, before);
+        if (lane == 0) {
+            at[0] = ok ? q_start[r] + (item - before) * LA_C : -1;
+            at[1] = ok ? min(LA_C, q_start[r + 1] - at[0]) : 0;
+        }
+    }
+    __syncthreads();
+    const int t0 = at[0], L = at[1];
+    rv_pdl_wait();
+    if (t0 < 0) return;
+    const float* base = rows + (size_t)t0 * stride;
+    const float* Sg = kv + ((size_t)item * H + h) * d * dv;
+    const int vn = min(LA_T, dv - v0);
+    const int ty = tid >> 4, tx = tid & 15;
+    const float ld = CHANNEL ? 0.f : log_decay[h];
+    // values [64 tokens][64 columns]
+    {
+        const int x = tid & 63, y = tid >> 6;
+#pragma unroll 4
+        for (int j = y; j < LA_C; j += 4)
+            vs[j * LA_LD + x] = j < L && x < vn ? la_act(base[(size_t)j * stride + 2 * H * d + h * dv + v0 + x], act) : 0.f;
+    }
+    float p[4][4], o[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) p[i][j] = o[i][j] = 0.f;
+    // CHANNEL: the pairs (i, j < i) and (i, i) inside groups, 8 x 36 of them, over the threads
+    float inner[2] = {0.f, 0.f};
+    int pi[2], pj[2];
+    if (CHANNEL) {
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int n = tid + 256 * u;            // pair n % 36 of group n / 36
+            int a = 0, b = n % 36;
+            while (b > a) b -= ++a;                 // row a has a + 1 pairs
+            pi[u] = n < 36 * LA_NG ? (n / 36) * LA_G + a : -1;
+            pj[u] = (n / 36) * LA_G + b;
+        }
+    }
+    const int I = ty >> 1;                          // the group of this thread's rows
+    const int J = tx >> 1;                          // and of its columns
+    for (int c0 = 0; c0 < d; c0 += LA_DK) {
+        const int cn = min(LA_DK, d - c0);
+        __syncthreads();                            // the slice before has been used
+        // four tokens by eight channels a warp and access: whole 32-byte pieces of the rows, and
+        // 32 different banks of the transposed slice
+        {
+            const int tl = lane & 3, cl = lane >> 2;
+#pragma unroll 4
+            for (int u = warp; u < (LA_C / 4) * (LA_DK / 8); u += 8) {
+                const int j = (u >> 2) * 4 + tl, c = (u & 3) * 8 + cl;
+                const bool in = j < L && c < cn;
+                const float* row = base + (size_t)j * stride + h * d + c0 + c;
+                const float q = in ? la_act(row[0], act) * q_scale : 0.f;
+                const float k = in ? la_act(row[(size_t)H * d], act) : 0.f;
+                if (CHANNEL) {
+                    qr[c * LA_LD + j] = q;
+                    kr[c * LA_LD + j] = k;
+                    lb[c * LA_LD + j] = in ? la_logsigmoid(row[(size_t)2 * H * d + 2 * H * dv] + bias[h * d + c0 + c]) / tau : 0.f;
+                } else {
+                    qt[c * LA_LD + j] = q;
+                    kt[c * LA_LD + j] = k;
+                }
+            }
+            const int x = tid & 63, y = tid >> 6;
+#pragma unroll 4
+            for (int c = y; c < LA_DK; c += 4)
+                ss[c * LA_LD + x] = c < cn && x < vn ? Sg[(size_t)(c0 + c) * dv + v0 + x] : 0.f;
+        }
+        if (CHANNEL) {
+            __syncthreads();
+            {
+                // sums inside the groups: thread (channel, group), then the groups' sums before
+                const int c = tid >> 3, g = tid & 7;
+                float s = 0.f, cum[LA_G];
+#pragma unroll
+                for (int j = 0; j < LA_G; ++j) {
+                    s += lb[c * LA_LD + g * LA_G + j];
+                    cum[j] = s;
+                }
+                float incl = s;
+#pragma unroll
+                for (int w = 1; w < LA_NG; w <<= 1) {
+                    const float up = __shfl_up_sync(0xffffffffu, incl, w, LA_NG);
+                    if (g >= w) incl += up;
+                }
+                // the same sums for whoever asks: B before group g is the sum of the totals before
+                off[(g + 1) * (LA_DK + 1) + c] = incl;
+                if (g == 0) off[c] = 0.f;
+#pragma unroll
+                for (int j = 0; j < LA_G; ++j) {
+                    const int e = c * LA_LD + g * LA_G + j;
+                    lb[e] = cum[j];
+                    qt[e] = qr[e] * expf(cum[j]);
+                    kt[e] = kr[e] * expf(s - cum[j]);
+                }
+            }
+            __syncthreads();
+            // tab[I][J + 1][c] = e^(B before I - B at the end of J), J < I; J = -1: the chunk's start
+            for (int n = tid; n < LA_NG * LA_NG * LA_DK; n += 256) {
+                const int c = n & (LA_DK - 1), jj = (n / LA_DK) & (LA_NG - 1), ii = n / (LA_DK * LA_NG);
+                if (jj <= ii)
+                    tab[(ii * LA_NG + jj) * (LA_DK + 1) + c] =
+                        expf(off[ii * (LA_DK + 1) + c] - off[jj * (LA_DK + 1) + c]);
+            }
+#pragma unroll
+            for (int u = 0; u < 2; ++u)
+                if (pi[u] >= 0) {
+                    float s = 0.f;
+#pragma unroll 4
+                    for (int c = 0; c < cn; ++c)
+                        s = fmaf(qr[c * LA_LD + pi[u]] * kr[c * LA_LD + pj[u]],
+                                 expf(lb[c * LA_LD + pi[u]] - lb[c * LA_LD + pj[u]]), s);
+                    inner[u] += s;
+                }
+        }
+        __syncthreads();
+        const float* tij = tab + (I * LA_NG + (J < I ? J + 1 : 0)) * (LA_DK + 1);
+        const float* ti0 = tab + I * LA_NG * (LA_DK + 1);
+#pragma unroll 4
+        for (int c = 0; c < cn; ++c) {
+            const float4 a = *(const float4*)(qt + c * LA_LD + 4 * ty), b = *(const float4*)(kt + c * LA_LD + 4 * tx),
+                         w = *(const float4*)(ss + c * LA_LD + 4 * tx);
+            const float av[4] = {a.x, a.y, a.z, a.w};
+            float bv[4] = {b.x, b.y, b.z, b.w}, wv[4] = {w.x, w.y, w.z, w.w};
+            if (CHANNEL) {
+                const float f = tij[c], f0 = ti0[c];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    bv[e] *= f;
+                    wv[e] *= f0;
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    p[i][e] = fmaf(av[i], bv[e], p[i][e]);
+                    o[i][e] = fmaf(av[i], wv[e], o[i][e]);
+                }
+        }
+    }
+    // scores to shared memory, transposed; zeros above the diagonal
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int ri = 4 * ty + i;
+        float row_f = 1.f;
+        if (!CHANNEL) row_f = expf(ld * (float)(ri + 1));
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int cj = 4 * tx + e;
+            if (CHANNEL) {
+                if (J < I) ps[cj * LA_LD + ri] = p[i][e];
+                else if (J > I) ps[cj * LA_LD + ri] = 0.f;
+                else if (cj > ri) ps[cj * LA_LD + ri] = 0.f;     // inside a group: the pairs below
+            } else {
+                ps[cj * LA_LD + ri] = cj <= ri ? p[i][e] * expf(ld * (float)(ri - cj)) : 0.f;
+                o[i][e] *= row_f;
+            }
+        }
+    }
+    if (CHANNEL) {
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+            if (pi[u] >= 0) ps[pj[u] * LA_LD + pi[u]] = inner[u];
+    }
+    __syncthreads();
+    // a warp's rows end with its group: later values have no score
+    const int jn = min((L + 3) & ~3, 8 * (I + 1));
+#pragma unroll 4
+    for (int j = 0; j < jn; ++j) {
+        const float4 a = *(const float4*)(ps + j * LA_LD + 4 * ty), b = *(const float4*)(vs + j * LA_LD + 4 * tx);
+        const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[i][e] = fmaf(av[i], bv[e], o[i][e]);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int ri = 4 * ty + i;
+        if (ri >= L) continue;
+        float* dst = num + ((size_t)(t0 + ri) * H + h) * dv + v0 + 4 * tx;
+        if (dv % 4 == 0) {
+            if (4 * tx < vn) *(float4*)dst = make_float4(o[i][0], o[i][1], o[i][2], o[i][3]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                if (4 * tx + e < vn) dst[e] = o[i][e];
+        }
+    }
+}
+
+// ---- norm, weight and gate -----------------------------------------------------------------------
+__device__ __forceinline__ float la_gate(float g, int gate) {
+    return (gate ? g : 1.f) / (1.f + expf(-g));                  // 0: sigmoid, 1: silu
+}
+
+// One norm over all heads: a block per token.
+template <typename T>
+__global__ void la_finish_all_kernel(const float* __restrict__ num, const float* __restrict__ rows,
+                                     int stride, int g_off, const float* __restrict__ norm_w, float eps,
+                                     const int* __restrict__ token_req, const int* __restrict__ state_slot,
+                                     T* __restrict__ out, int width, int gate) {
+    rv_pdl_launch_dependents();
+    __shared__ float scratch[33];
+    const int t = blockIdx.x;
+    const bool pad = state_slot[token_req[t]] < 0;
+    rv_pdl_wait();
+    T* o = out + (size_t)t * width;
+    if (pad) {
+        for (int c = threadIdx.x; c < width; c += blockDim.x) rv_store(o + c, 0.f);
+        return;
+    }
+    const float* nm = num + (size_t)t * width;
+    const float* g = rows + (size_t)t * stride + g_off;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) ss += nm[c] * nm[c];
+    const float rms = sqrtf(rv_block_sum(ss, scratch) / (float)width + eps);
+    for (int c = threadIdx.x; c < width; c += blockDim.x)
+        rv_store(o + c, nm[c] / rms * norm_w[c] * la_gate(g[c], gate));
+}
+
+// A norm per head: a warp per (token, head).
+template <typename T>
+__global__ void la_finish_head_kernel(const float* __restrict__ num, const float* __restrict__ rows,
+                                      int stride, int g_off, const float* __restrict__ norm_w, float eps,
+                                      const int* __restrict__ token_req, const int* __restrict__ state_slot,
+                                      T* __restrict__ out, int n_tokens, int H, int dv, int gate) {
+    rv_pdl_launch_dependents();
+    const long long w = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+    const int lane = threadIdx.x & 31;
+    if (w >= (long long)n_tokens * H) return;
+    const int t = (int)(w / H), h = (int)(w - (long long)t * H);
+    const bool pad = state_slot[token_req[t]] < 0;
+    rv_pdl_wait();
+    T* o = out + (size_t)t * H * dv + (size_t)h * dv;
+    if (pad) {
+        for (int c = lane; c < dv; c += 32) rv_store(o + c, 0.f);
+        return;
+    }
+    const float* nm = num + ((size_t)t * H + h) * dv;
+    const float* g = rows + (size_t)t * stride + g_off + h * dv;
+    const float* wt = norm_w + h * dv;
+    float ss = 0.f;
+    for (int c = lane; c < dv; c += 32) ss += nm[c] * nm[c];
+    const float rms = sqrtf(rv_warp_sum(ss) / (float)dv + eps);
+    for (int c = lane; c < dv; c += 32) rv_store(o + c, nm[c] / rms * wt[c] * la_gate(g[c], gate));
+}
+
+// ---------------------------------------------------------------------------------
+// The most chunks the portions of `n_tokens` tokens in `n_reqs` requests can have.
+static long long la_items(int n_tokens, int n_reqs) { return (long long)n_tokens / LA_C + n_reqs; }
+
+// Floats of scratch: num [n, H, dv]; for portions kv [items, H, d, dv] and dec [items, H, d].
+extern "C" long long rv_linear_attention_scratch(int n_tokens, int n_decode, int n_reqs, int H, int d,
+                                                 int dv) {
+    long long f = ((long long)n_tokens * H * dv + 3) & ~3LL;
+    if (n_reqs > n_decode && n_tokens > n_decode)
+        f += la_items(n_tokens - n_decode, n_reqs - n_decode) * H * ((long long)d * dv + d);
+    return f;
+}
+
+// log_decay [H] or null; then bias [H d] and z at the end of the rows.  act: 1 silu; norm_head: 0 all
+// heads together, 1 per head; gate: 0 sigmoid, 1 silu; norm_w [H dv].  Requests [0, n_decode) bring
+// one token each (token r is request r's).
+extern "C" int rv_linear_attention(const float* rows, int stride, const float* log_decay,
+                                   const float* bias, float tau, const float* norm_w, float* state,
+                                   const int* token_req, const int* q_start, const int* state_slot,
+                                   float* scratch, void* out, int out_dtype, int n_tokens, int n_decode,
+                                   int n_reqs, int H, int d, int dv, int act, float q_scale,
+                                   int norm_head, int gate, float eps, void* stream) {
+    if (n_tokens == 0 || n_reqs == 0) return 0;
+    if (n_tokens < 0 || n_decode < 0 || n_decode > n_reqs || n_decode > n_tokens || H < 1 || d < 1 || dv < 1)
+        RV_FAIL("linear_attention: bad sizes");
+    if (!log_decay && (!bias || !(tau > 0.f))) RV_FAIL("linear_attention: neither a decay nor a bias and tau");
+    if (stride < 2 * H * d + 2 * H * dv + (log_decay ? 0 : H * d)) RV_FAIL("linear_attention: rows are too short");
+    if (n_reqs > 65535 || H > 65535 || d > 2048 || dv > 65535) RV_FAIL("linear_attention: too many requests or heads");
+    if (((uintptr_t)scratch | (uintptr_t)state) & 15) RV_FAIL("linear_attention: scratch and records must be 16-byte aligned");
+    cudaStream_t s = (cudaStream_t)stream;
+    const int tiles_d = (d + LA_T - 1) / LA_T, tiles_v = (dv + LA_T - 1) / LA_T;
+    float* num = scratch;
+    const bool v4 = dv % 4 == 0;
+    if (n_decode > 0) {
+        const size_t smem = (size_t)(3 * d + (v4 ? 8 : 2) * LA_T) * sizeof(float);
+        const dim3 grid(tiles_v, H, n_decode);
+        if (v4)
+            rv_launch(la_token_kernel<4>, grid, dim3(128), smem, s, rows, stride, log_decay, bias, tau,
+                      q_start, state_slot, state, num, H, d, dv, act, q_scale);
+        else
+            rv_launch(la_token_kernel<1>, grid, dim3(128), smem, s, rows, stride, log_decay, bias, tau,
+                      q_start, state_slot, state, num, H, d, dv, act, q_scale);
+        RV_CHECK_LAUNCH("linear_attention_token");
+    }
+    if (n_tokens > n_decode && n_reqs > n_decode) {
+        const long long items = la_items(n_tokens - n_decode, n_reqs - n_decode);
+        float* kv = scratch + (((size_t)n_tokens * H * dv + 3) & ~(size_t)3);
+        float* dec = kv + (size_t)items * H * d * dv;
+        if (tiles_d * tiles_v > 65535 || items > 0x7fffffffLL) RV_FAIL("linear_attention: heads are too large");
+        const bool ch = log_decay == nullptr;
+        const size_t sm1 = (size_t)((ch ? 3 : 2) * LA_C * LA_LD + 4 * 64) * sizeof(float);
+        const size_t sm3 = (size_t)((ch ? 6 : 3) * LA_DK * LA_LD + 2 * LA_C * LA_LD +
+                                    (ch ? (LA_NG + 1 + LA_NG * LA_NG) * (LA_DK + 1) : 0)) * sizeof(float);
+        static bool configured = false;
+        if (!configured) {
+            const int big = 128 * 1024;
+            if (cudaFuncSetAttribute(la_state_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, big) != cudaSuccess ||
+                cudaFuncSetAttribute(la_state_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big) != cudaSuccess ||
+                cudaFuncSetAttribute(la_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, big) != cudaSuccess ||
+                cudaFuncSetAttribute(la_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big) != cudaSuccess)
+                RV_FAIL("linear_attention: %d bytes of shared memory are not to be had", big);
+            configured = true;
+        }
+        const int first = n_decode, np = n_reqs - n_decode;
+        const dim3 g1((unsigned)items, H, tiles_d * tiles_v), g3((unsigned)items, H, tiles_v);
+        const long long el = (long long)d * dv;
+        const dim3 g2((unsigned)((el + 256 * (v4 ? 4 : 1) - 1) / (256 * (v4 ? 4 : 1))), H, np);
+        if (ch) {
+            rv_launch(la_state_kernel<true>, g1, dim3(256), sm1, s, rows, stride, log_decay, bias, tau, q_start,
+                      state_slot, first, n_reqs, kv, dec, H, d, dv, act);
+            if (v4)
+                rv_launch(la_scan_kernel<true, 4>, g2, dim3(256), 0, s, log_decay, q_start, state_slot, first,
+                          kv, dec, state, H, d, dv);
+            else
+                rv_launch(la_scan_kernel<true, 1>, g2, dim3(256), 0, s, log_decay, q_start, state_slot, first,
+                          kv, dec, state, H, d, dv);
+            rv_launch(la_out_kernel<true>, g3, dim3(256), sm3, s, rows, stride, log_decay, bias, tau, q_start,
+                      state_slot, first, n_reqs, (const float*)kv, num, H, d, dv, act, q_scale);
+        } else {
+            rv_launch(la_state_kernel<false>, g1, dim3(256), sm1, s, rows, stride, log_decay, bias, tau, q_start,
+                      state_slot, first, n_reqs, kv, dec, H, d, dv, act);
+            if (v4)
+                rv_launch(la_scan_kernel<false, 4>, g2, dim3(256), 0, s, log_decay, q_start, state_slot, first,
+                          kv, dec, state, H, d, dv);
+            else
+                rv_launch(la_scan_kernel<false, 1>, g2, dim3(256), 0, s, log_decay, q_start, state_slot, first,
+                          kv, dec, state, H, d, dv);
+            rv_launch(la_out_kernel<false>, g3, dim3(256), sm3, s, rows, stride, log_decay, bias, tau, q_start,
+                      state_slot, first, n_reqs, (const float*)kv, num, H, d, dv, act, q_scale);
+        }
+        RV_CHECK_LAUNCH("linear_attention");
+    }
+    const int g_off = 2 * H * d + H * dv;
+    if (norm_head) {
+        const long long blocks = ((long long)n_tokens * H + 3) / 4;
+        if (blocks > 0x7fffffffLL) RV_FAIL("linear_attention: too many tokens");
+        RV_DISPATCH_DTYPE(out_dtype, "linear_attention",
+                          (rv_launch(la_finish_head_kernel<T>, dim3((int)blocks), dim3(128), 0, s,
+                                     (const float*)num, rows, stride, g_off, norm_w, eps, token_req,
+                                     state_slot, (T*)out, n_tokens, H, dv, gate)));
+    } else {
+        const int width = H * dv;
+        const int threads = width >= 1024 ? 256 : 128;
+        RV_DISPATCH_DTYPE(out_dtype, "linear_attention",
+                          (rv_launch(la_finish_all_kernel<T>, dim3(n_tokens), dim3(threads), 0, s,
+                                     (const float*)num, rows, stride, g_off, norm_w, eps, token_req,
+                                     state_slot, (T*)out, width, gate)));
+    }
+    RV_CHECK_LAUNCH("linear_attention_finish");
+    return 0;
+}

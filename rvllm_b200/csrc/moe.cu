@@ -9,7 +9,8 @@
 //                  largest allowed s are chosen (ties: the lower index first, for groups too);
 //                  weights = chosen s / (their sum + weight_eps).  One warp per token.
 //                  Options: score_mode 1 makes s the softmax of the logits over all experts
-//                  instead of their sigmoids; renorm 0 leaves the chosen s undivided; every
+//                  instead of their sigmoids; score_mode 2 compares the logits themselves and
+//                  weighs with the softmax over the chosen ones; renorm 0 leaves the chosen s undivided; every
 //                  weight is multiplied by route_scale.  `choice_bias` float32 [E], if given,
 //                  is added to s wherever experts (and groups) are compared; the weights are
 //                  made from s without it.
@@ -75,7 +76,7 @@ __device__ __forceinline__ void moe_select_warp(float* sc, float* gs, int E, int
         }
         tot = rv_warp_sum(tot);
         for (int e = lane; e < E; e += 32) sc[e] = sc[e] / tot;
-    } else {
+    } else if (score_mode == 0) {
         for (int e = lane; e < E; e += 32) sc[e] = 1.f / (1.f + expf(-sc[e]));
     }
     if (choice_bias) {                               // compare s + bias, weigh with s
@@ -137,13 +138,17 @@ __device__ __forceinline__ void moe_select_warp(float* sc, float* gs, int E, int
             if (gs[e / size] != INFINITY) sc[e] = -3.0e38f;      // below every score
         __syncwarp();
     }
-    float sum = 0.f, mine = 0.f;
+    float sum = 0.f, mine = 0.f, first = 0.f;
     int mine_id = 0;
     for (int k = 0; k < top; ++k) {
         float v;
         int i;
         moe_warp_argmax(sc, 0, E, lane, v, i);
         if (choice_bias) v = orig[i];
+        if (score_mode == 2) {                       // relative to the first chosen logit
+            if (k == 0) first = v;
+            v = expf(v - first);
+        }
         sum += v;
         if (lane == (k & 31) && k < 32) {
             mine = v;

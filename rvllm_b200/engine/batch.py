@@ -40,6 +40,8 @@ class GroupContext:
     max_blocks: int
     page_size: int
     window: Optional[int]
+    every: int = 1                  # tokens a row stands for; > 1: the slot mapping names a slot for
+                                    # the tokens that complete a row and -1 for all others
 
 
 @dataclass
@@ -153,7 +155,7 @@ class BatchBuilder:
         n_groups = len(cache.groups)
         max_blocks = []
         for gi in range(n_groups):
-            mb = max([-(-c // ps) for c in ctx] + [1])
+            mb = max([cache.pages_for(cache.groups[gi], c) for c in ctx] + [1])
             max_blocks.append(max(mb, pad_blocks))
 
         # layout, in int32 words
@@ -219,14 +221,25 @@ class BatchBuilder:
                 k += 1
         for gi in range(n_groups):
             mb = max_blocks[gi]
+            every = cache.groups[gi].need.every
             table = view(f"table{gi}").reshape(R, mb)
             table[:] = -1
             slots = view(f"slot{gi}")
             slots[:] = -1
             for r, a, rc, s, q, c in zip(req_of, first, rcs, starts, q_lens, ctx):
                 t = rc.tables[gi].view()
-                nb = -(-c // ps)
+                nb = cache.pages_for(cache.groups[gi], c)
                 table[r, :nb] = t[:nb]
+                if every > 1:
+                    # rows completed by this step: row k by the token at (k + 1) * every - 1
+                    k0, k1 = s // every, c // every
+                    if k1 - k0 == 1:
+                        slots[a + k1 * every - 1 - s] = int(t[k0 // ps]) * ps + k0 % ps
+                    elif k1 > k0:
+                        k = np.arange(k0, k1)
+                        slots[a + (k + 1) * every - 1 - s] = \
+                            t[k // ps].astype(np.int64) * ps + k % ps
+                    continue
                 if q == 1:
                     page = int(t[s // ps])
                     if page < 0:
@@ -254,7 +267,7 @@ class BatchBuilder:
             groups.append(GroupContext(
                 block_table=dview(f"table{gi}").view(R, max_blocks[gi]),
                 slot_mapping=dview(f"slot{gi}"), max_blocks=max_blocks[gi],
-                page_size=ps, window=grp.need.window))
+                page_size=ps, window=grp.need.window, every=grp.need.every))
         ctx_all = [0] * R
         for r, c in zip(req_of, ctx):
             ctx_all[r] = c

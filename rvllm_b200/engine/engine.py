@@ -143,13 +143,12 @@ class Engine:
             if len(seq.generated) + 1 >= seq.max_tokens:      # ends by length after this step
                 return False
         # pages for one more token each, without preempting anybody
-        ps = sch.cfg.block_size
         cache = self.runner.cache
         need = [0] * len(cache.groups)
         for e in plan:
             rc = cache.requests[e.seq.request.id]
-            want = -(-(e.start + e.count + 1) // ps)
             for gi, table in enumerate(rc.tables):
+                want = cache.pages_for(cache.groups[gi], e.start + e.count + 1)
                 if len(table) < want:
                     need[gi] += want - len(table)
         return all(n <= g.pool.available for n, g in zip(need, cache.groups))

@@ -249,13 +249,8 @@ class Scheduler:
 
     def _tokens_that_fit(self, seq: Sequence_, fresh: bool = False) -> int:
         """How many more tokens of `seq` the free pages can take."""
-        ps = self.cfg.block_size
-        free_pages = min(g.pool.available for g in self.cache.groups) if self.cache.groups \
-            else 1 << 30
-        have = 0 if fresh else self.cache.requests[seq.request.id].tokens
-        reserved_pages = -(-have // ps)
-        room = (reserved_pages + free_pages) * ps - seq.computed
-        return max(0, room)
+        room = self.cache.room(None if fresh else seq.request.id)
+        return max(0, room - seq.computed)
 
     # ---- after the step --------------------------------------------------------------
 

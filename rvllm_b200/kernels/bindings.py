@@ -52,6 +52,8 @@ class CudaOps:
         self.lib.rv_gemm_tiled_bytes.restype = c_longlong
         self.lib.rv_gated_delta_scratch.restype = c_longlong
         self.lib.rv_mlstm_scratch.restype = c_longlong
+        self.lib.rv_linear_attention_scratch.restype = c_longlong
+        self.lib.rv_paged_attention_pooled_scratch_bytes.restype = c_longlong
         self.lib.rv_paged_attention_mixed_scratch_bytes.restype = c_longlong
         self._scratch = {}
         self._retired = []
@@ -127,14 +129,24 @@ class CudaOps:
 
     # ---- embedding -------------------------------------------------------------------
 
-    def embed(self, table, ids, out, scale=None):
+    def embed(self, table, ids, out, scale=None, positions=None, position_table=None):
+        """`position_table` [positions, hidden] (the table's type): row positions[t] is added to
+        token t's (scaled) row."""
         self._need(table, "embedding table")
         self._need(ids, "token ids", torch.int32)
         self._need(out, "embedding output", torch.float32)
         n, hidden = out.shape
+        rows = 0
+        if position_table is not None:
+            self._need(position_table, "position table", table.dtype)
+            self._need(positions, "positions", torch.int32)
+            rows = position_table.shape[0]
+            if position_table.shape[1] != hidden:
+                raise KernelError("embed: the position table has another width")
         self._check(self.lib.rv_embed(_ptr(table), _code(table.dtype), _ptr(ids), _ptr(out),
                                       c_int(n), c_int(hidden), c_int(table.shape[0]),
-                                      c_float(1.0 if scale is None else scale), self._stream()),
+                                      c_float(1.0 if scale is None else scale), _ptr(positions),
+                                      _ptr(position_table), c_int(rows), self._stream()),
                     "embed")
 
     # ---- residual add + RMSNorm ------------------------------------------------------
@@ -169,6 +181,51 @@ class CudaOps:
             _ptr(resid), _ptr(delta), _code(delta.dtype) if delta is not None else _F32,
             _ptr(weight), _ptr(out), _code(out.dtype), _ptr(rows), c_int(n), c_int(hidden),
             c_float(eps), _ptr(delta_scale), _ptr(add), self._stream()), "add_rmsnorm")
+
+    def add_rmsnorm_shift(self, resid, new_resid, delta, weight, eps, out, ctx, shift, state,
+                          delta_scale=None, add=None, add_rows=None):
+        """x = resid + delta (* delta_scale) + add_rows + add -> `new_resid`; h = x / rms(x) * weight;
+        `out` = h + (h of the token before - h) * shift.  The h before a request's first row is
+        its record in `state` float32 [slots, hidden], which then receives the h of its last row.
+        `shift` None: `out` = h, and `new_resid` may be `resid`."""
+        for t, what in ((resid, "residual stream"), (new_resid, "residual stream"),
+                        (weight, "norm weight"), (delta_scale, "scale of the pending rows"),
+                        (add, "added vector"), (add_rows, "added rows"), (shift, "token shift"),
+                        (state, "last rows")):
+            if t is not None:
+                self._need(t, what, torch.float32)
+        self._need(out, "norm output")
+        n, hidden = out.shape
+        if delta is not None:
+            self._need(delta, "pending sub-layer output")
+        for t in (resid, new_resid, delta, add_rows):
+            if t is not None and t.shape != (n, hidden):
+                raise KernelError("add_rmsnorm_shift: the rows differ in shape")
+        for t in (weight, delta_scale, add, shift):
+            if t is not None and t.shape != (hidden,):
+                raise KernelError("add_rmsnorm_shift: widths disagree")
+        if shift is not None and (state is None or state.shape[1] != hidden):
+            raise KernelError("add_rmsnorm_shift: a shift needs the last rows' records")
+        self._check(self.lib.rv_add_rmsnorm_shift(
+            _ptr(resid), _ptr(new_resid), _ptr(delta),
+            _code(delta.dtype) if delta is not None else _F32, _ptr(delta_scale), _ptr(add),
+            _ptr(add_rows), _ptr(weight), c_float(eps), _ptr(out), _code(out.dtype), _ptr(shift),
+            _ptr(state), _ptr(ctx.token_req), _ptr(ctx.q_start), _ptr(ctx.state_slot), c_int(n),
+            c_int(hidden), self._stream()), "add_rmsnorm_shift")
+
+    def normed_sum(self, a, wa, sa, b, wb, sb, eps, out):
+        """out = sa * rmsnorm(a; wa) + sb * rmsnorm(b; wb), float32 arithmetic."""
+        self._need(a, "first summand")
+        self._need(b, "second summand", a.dtype)
+        self._need(out, "sum", a.dtype)
+        self._need(wa, "norm weight", torch.float32)
+        self._need(wb, "norm weight", torch.float32)
+        n, hidden = out.shape
+        if a.shape != out.shape or b.shape != out.shape or wa.shape != (hidden,) or wb.shape != (hidden,):
+            raise KernelError("normed_sum: shapes disagree")
+        self._check(self.lib.rv_normed_sum(
+            _ptr(a), _ptr(wa), c_float(sa), _ptr(b), _ptr(wb), c_float(sb), c_float(eps), _ptr(out),
+            _code(out.dtype), c_int(n), c_int(hidden), self._stream()), "normed_sum")
 
     # ---- matrix product (library) -------------------------------------------------------
 
@@ -737,7 +794,10 @@ class CudaOps:
     # ---- partial rotation + cache write ------------------------------------------------
 
     def rope_partial_write(self, rows, num_heads, num_kv_heads, head_dim, v_head_dim, freq,
-                           positions, slot_mapping, k_cache, v_cache):
+                           positions, slot_mapping, k_cache, v_cache, amplitude=1.0,
+                           values_are_keys=False):
+        """`amplitude` multiplies cosine and sine; `values_are_keys`: the rows have no value
+        columns, a token's value is its key before the rotation."""
         self._need(rows, "q|k|v rows")
         if k_cache is not None:
             self._need(k_cache, "key pages", rows.dtype)
@@ -751,7 +811,126 @@ class CudaOps:
             _ptr(rows), _code(rows.dtype), c_int(rows.shape[1]), c_int(rows.shape[0]),
             c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(v_head_dim), _ptr(inv),
             c_int(dims), _ptr(positions), _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache),
-            self._stream()), "rope_partial_write")
+            c_float(amplitude), c_int(1 if values_are_keys else 0), self._stream()),
+            "rope_partial_write")
+
+    # ---- pooled blocks: their rows; attention over a window and the blocks before it --------
+
+    def pool_rows(self, k_cache, v_cache, group, ctx, pool, slots, k_out, v_out):
+        """For every token t with slots[t] >= 0, the last of a block of `pool` tokens: the means of
+        the block's cached keys and values (read through `group`'s block table) -> row
+        slots[t] of `k_out` and `v_out`."""
+        self._need(k_cache, "key pages")
+        self._need(slots, "slots of completed blocks", torch.int32)
+        for t, what in ((v_cache, "value pages"), (k_out, "block keys"), (v_out, "block values")):
+            self._need(t, what, k_cache.dtype)
+            if t.shape[-2:] != k_cache.shape[-2:]:
+                raise KernelError("pool_rows: the pages differ in shape")
+        self._check(self.lib.rv_pool_rows(
+            _ptr(k_cache), _ptr(v_cache), _code(k_cache.dtype), _ptr(group.block_table),
+            c_int(group.max_blocks), c_int(group.page_size), _ptr(ctx.token_req), _ptr(ctx.positions),
+            _ptr(slots), c_int(pool), _ptr(k_out), _ptr(v_out), c_int(ctx.n_tokens),
+            c_int(k_cache.shape[-2] * k_cache.shape[-1]), self._stream()), "pool_rows")
+
+    def attention_pooled_scratch_bytes(self, n_reqs, num_heads, head_dim, max_ctx_len, window,
+                                       pool) -> int:
+        return int(self.lib.rv_paged_attention_pooled_scratch_bytes(
+            c_int(n_reqs), c_int(num_heads), c_int(head_dim), c_int(max_ctx_len),
+            c_int(window or 0), c_int(pool or 0)))
+
+    def _pooled_lib(self, head_dim: int):
+        """The tensor-core pooled attention library for this head size, built at first use."""
+        key = ("pooled", head_dim)
+        lib = self._attn_libs.get(key)
+        if lib is None:
+            path = build_variant("attention_mma.cu", {"RV_HD": head_dim, "RV_POOLED": 1},
+                                 f"attnpool_hd{head_dim}", verbose=self._verbose_build)
+            try:
+                lib = ctypes.CDLL(path)
+            except OSError as e:
+                raise KernelError(f"cannot load the kernel library {path}: {e}") from None
+            getattr(lib, f"rv_attention_pooled_last_error_hd{head_dim}").restype = ctypes.c_char_p
+            self._attn_libs[key] = lib
+        return lib
+
+    def paged_attention_pooled(self, rows, num_heads, num_kv_heads, head_dim, k_cache, v_cache, ctx,
+                               group, pooled, scale, softcap, window, sinks, out):
+        """Attention over the last `window` tokens (None: all) and the pooled blocks before them:
+        `pooled` = (block keys, block values, their group, tokens a block) or None.  `softcap`: scores
+        become c tanh(score / c); `sinks` float32 [heads]: one more term in the denominator.
+        Single tokens go to a split kernel and its merge, portions to one launch; bfloat16 heads
+        whose size is a multiple of 16 up to 128 take the tensor cores."""
+        self._need(rows, "query rows")
+        self._need(out, "attention output", rows.dtype)
+        self._need(k_cache, "key pages", rows.dtype)
+        self._need(v_cache, "value pages", rows.dtype)
+        H, G, d = num_heads, num_kv_heads, head_dim
+        if out.shape[1] != H * d or rows.shape[1] < H * d:
+            raise KernelError("paged_attention_pooled: row widths and head sizes disagree")
+        if sinks is not None:
+            self._need(sinks, "sinks", torch.float32)
+            if sinks.shape[0] != H:
+                raise KernelError("paged_attention_pooled: one sink per query head")
+        pk = pv = ptable = None
+        pmax = pool = 0
+        if pooled is not None:
+            pk, pv, pgroup, pool = pooled
+            self._need(pk, "block keys", rows.dtype)
+            self._need(pv, "block values", rows.dtype)
+            if window is None or pgroup.page_size != group.page_size:
+                raise KernelError("paged_attention_pooled: blocks lie before a window, in pages of "
+                                  "the tokens' size")
+            ptable, pmax = pgroup.block_table, pgroup.max_blocks
+        mma = (self._mma_ok(rows.dtype, d) and rows.shape[1] % 8 == 0 and rows.data_ptr() % 16 == 0
+               and k_cache.data_ptr() % 16 == 0 and v_cache.data_ptr() % 16 == 0)
+        code, nd = _code(rows.dtype), ctx.n_decode
+        pages = (_ptr(k_cache), _ptr(v_cache), _ptr(group.block_table), c_int(group.max_blocks),
+                 _ptr(pk), _ptr(pv), _ptr(ptable), c_int(pmax), c_int(pool),
+                 c_float(softcap or 0.0))
+        heads = (c_int(H), c_int(G))
+        win = c_int(window or 0)
+        lib = tag = None
+        if mma and (self.decode_attention == "mma" or self.prefill_attention != "simt"):
+            lib, tag = self._pooled_lib(d), f"hd{d}"
+
+        def check_mma(rc, what):
+            self.launches += 1
+            if rc != 0:
+                msg = getattr(lib, f"rv_attention_pooled_last_error_{tag}")().decode()
+                raise KernelError(f"{what}: {msg}")
+
+        if nd > 0:
+            need = self.attention_pooled_scratch_bytes(nd, H, d, ctx.max_ctx_len, window, pool)
+            scratch = self._scratch_buffer(need, rows.device)
+            if lib is not None and self.decode_attention == "mma":
+                check_mma(getattr(lib, f"rv_paged_attention_pooled_decode_mma_{tag}")(
+                    _ptr(rows), c_int(rows.shape[1]), *pages, _ptr(ctx.ctx_lens), _ptr(scratch),
+                    c_longlong(scratch.numel()), c_int(nd), c_int(ctx.max_ctx_len), *heads,
+                    c_int(group.page_size), c_float(scale), win, self._stream()),
+                    "paged_attention_pooled_decode")
+                self._check(self.lib.rv_paged_attention_pooled_merge(
+                    _ptr(scratch), _ptr(ctx.ctx_lens), _ptr(out), code, c_int(nd),
+                    c_int(ctx.max_ctx_len), c_int(H), c_int(d), win, c_int(pool), _ptr(sinks),
+                    self._stream()), "paged_attention_pooled_merge")
+            else:
+                self._check(self.lib.rv_paged_attention_pooled_decode(
+                    _ptr(rows), code, c_int(rows.shape[1]), *pages, _ptr(ctx.ctx_lens), _ptr(out),
+                    _ptr(scratch), c_longlong(scratch.numel()), c_int(nd), c_int(ctx.max_ctx_len),
+                    *heads, c_int(d), c_int(group.page_size), c_float(scale), win, _ptr(sinks),
+                    self._stream()), "paged_attention_pooled_decode")
+                self.launches += 1
+        if ctx.n_tokens > nd and lib is not None and self.prefill_attention != "simt":
+            check_mma(getattr(lib, f"rv_paged_attention_pooled_prefill_{tag}")(
+                _ptr(rows), c_int(rows.shape[1]), *pages, _ptr(ctx.q_start), _ptr(ctx.ctx_lens),
+                _ptr(out), c_int(nd), c_int(ctx.n_reqs - nd), c_int(ctx.max_q_len), *heads,
+                c_int(group.page_size), c_float(scale), win, _ptr(sinks), self._stream()),
+                "paged_attention_pooled_prefill")
+        elif ctx.n_tokens > nd:
+            self._check(self.lib.rv_paged_attention_pooled_warp(
+                _ptr(rows), code, c_int(rows.shape[1]), *pages, _ptr(ctx.q_start),
+                _ptr(ctx.ctx_lens), _ptr(ctx.token_req), _ptr(out), c_int(nd),
+                c_int(ctx.n_tokens - nd), *heads, c_int(d), c_int(group.page_size), c_float(scale),
+                win, _ptr(sinks), self._stream()), "paged_attention_pooled")
 
     # ---- attention with mixed heads ------------------------------------------------------
 
@@ -950,7 +1129,7 @@ class CudaOps:
 
     # ---- mixture of experts ---------------------------------------------------------------
 
-    SCORE_MODES = {"sigmoid": 0, "softmax": 1}
+    SCORE_MODES = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}
     EXPERT_ACTIVATIONS = {"swiglu": 0, "glu_clamp": 1, "relu2": 2}
 
     def _choice_bias(self, choice_bias, experts):
@@ -962,7 +1141,8 @@ class CudaOps:
 
     def moe_select(self, logits, groups, keep, group_top, weight_eps, ids, weights,
                    score="sigmoid", renormalize=True, route_scale=1.0, choice_bias=None):
-        """`score`: how logits become scores ("sigmoid", or "softmax" over all experts);
+        """`score`: how logits become scores ("sigmoid", "softmax" over all experts, or
+        "softmax_chosen": the logits are compared, the chosen ones' softmax are the weights);
         `renormalize` false: the chosen scores are not divided by their sum; every weight is
         multiplied by `route_scale`; `choice_bias` float32 [experts] is added to the scores
         where experts are compared, not where they are weighed."""
@@ -1247,6 +1427,40 @@ class CudaOps:
             _ptr(scratch), _ptr(out), _code(out.dtype), c_int(n), c_int(ctx.n_reqs), c_int(heads),
             c_int(dim), c_int(vdim), c_float(cap), c_float(eps), self._stream()), "mlstm")
         self.launches += 2
+
+    # ---- linear attention with decay -----------------------------------------------------------
+
+    def linear_attention(self, rows, log_decay, decay_bias, tau, norm_w, state, ctx, out, heads, dim,
+                         vdim, activation, q_scale, norm, gate, eps):
+        """Linear attention over the step's tokens; see csrc/linear_attention.cu for the layout of
+        `rows` (q | k | v | g (| z), float32) and of the record [heads, dim, vdim].  `log_decay`
+        float32 [heads], or None: decays by token and channel from z, `decay_bias` and `tau`."""
+        for t, what in ((rows, "projection rows"), (log_decay, "decays"),
+                        (decay_bias, "decay bias"), (norm_w, "output norm weight"),
+                        (state, "state records")):
+            if t is not None:
+                self._need(t, what, torch.float32)
+        self._need(out, "mixer output")
+        n = rows.shape[0]
+        if state.shape[1] != heads * dim * vdim or out.shape != (n, heads * vdim) or \
+                norm_w.shape != (heads * vdim,):
+            raise KernelError("linear_attention: the record, the weight or the output has another size")
+        if (log_decay is None) != (decay_bias is not None) or \
+                (log_decay is not None and log_decay.shape != (heads,)) or \
+                (decay_bias is not None and decay_bias.shape != (heads * dim,)):
+            raise KernelError("linear_attention: a decay per head, or a bias per head and channel")
+        need = self.lib.rv_linear_attention_scratch(
+            c_int(n), c_int(ctx.n_decode), c_int(ctx.n_reqs), c_int(heads), c_int(dim), c_int(vdim))
+        scratch = torch.empty((need,), dtype=torch.float32, device=rows.device)
+        self._check(self.lib.rv_linear_attention(
+            _ptr(rows), c_int(rows.shape[1]), _ptr(log_decay), _ptr(decay_bias), c_float(tau),
+            _ptr(norm_w), _ptr(state), _ptr(ctx.token_req), _ptr(ctx.q_start), _ptr(ctx.state_slot),
+            _ptr(scratch), _ptr(out), _code(out.dtype), c_int(n), c_int(ctx.n_decode),
+            c_int(ctx.n_reqs), c_int(heads), c_int(dim), c_int(vdim),
+            c_int({None: 0, "silu": 1}[activation]), c_float(q_scale),
+            c_int({"all": 0, "head": 1}[norm]), c_int({"sigmoid": 0, "silu": 1}[gate]), c_float(eps),
+            self._stream()), "linear_attention")
+        self.launches += (ctx.n_decode > 0) + 3 * (n > ctx.n_decode)
 
     def softcap(self, logits, cap):
         self._need(logits, "logits", torch.float32)

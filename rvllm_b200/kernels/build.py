@@ -157,7 +157,7 @@ def build_variant(source: str, defines: dict, tag: str, verbose: bool = True) ->
         lock = _variant_locks.setdefault(tag, threading.Lock())
     with lock:
         h = hashlib.sha256()
-        for name in (source, "common.cuh"):
+        for name in [source] + sorted(f for f in os.listdir(CSRC) if f.endswith(".cuh")):
             with open(os.path.join(CSRC, name), "rb") as f:
                 h.update(f.read())
         flags = [f"-D{k}={v}" for k, v in sorted(defines.items())]

@@ -30,13 +30,18 @@ class PagedNeed:
     (counted from position 0) are.  Both tell the cache manager which pages it may take
     back early; neither changes the layout.  `v_head_dim`: size of a value head when it is
     not the key size.  `values` false: one row per token is all there is (a latent row that
-    keys and values are both made from); no value pages exist."""
+    keys and values are both made from); no value pages exist.  `every` > 1: one row per `every`
+    tokens (made from them when the last of them is written) instead of one per token.  `block`:
+    the rows of the newest incomplete block of `block` positions are read once more when it
+    completes, so their pages stay until then whatever the window says."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     chunk: Optional[int] = None
     v_head_dim: Optional[int] = None
     values: bool = True
+    every: int = 1
+    block: Optional[int] = None
 
     @property
     def value_dim(self) -> int:
@@ -46,13 +51,18 @@ class PagedNeed:
 
     def layout(self):
         """What two calls must agree on to share pages."""
-        return (self.num_kv_heads, self.head_dim, self.value_dim)
+        return (self.num_kv_heads, self.head_dim, self.value_dim, self.every)
+
+    def rows(self, tokens: int) -> int:
+        """Rows that the first `tokens` positions of a request have."""
+        return tokens // self.every
 
 
 @dataclass(frozen=True)
 class SeveralNeeds:
     """What a mixer made of several mixers has to remember: one need (or None) per branch, in
-    the branches' order.  The call's cache view then has `parts`, one view (or None) each."""
+    the branches' order.  The call's cache view then has `parts`, one view (or None) each.  A part
+    may itself be several."""
     parts: Tuple[object, ...]
 
 
@@ -157,6 +167,10 @@ class PositionEncoding:
 class Arrangement:
     """How a block wires norm, mixer and feed-forward around the residual stream.
 
+    `cache_need(spec)` is what one call of the block has to remember: the mixer's need unless
+    the arrangement itself keeps something between steps.  `fresh_stream`: the block's first norm
+    leaves the residual rows it is given as they are and goes on with new ones.
+
     forward(stream, ctx, cache) -> stream, where `stream` is a `Stream`: the float32
     residual plus the last sub-layer's output that is still to be added (so that the
     addition can be fused into the next norm).
@@ -166,6 +180,12 @@ class Arrangement:
     def params(spec, owns_cache: bool = True) -> Dict[str, ParamDecl]:
         """Full tensor names -> declarations for one block."""
         raise NotImplementedError
+
+    fresh_stream = False
+
+    @staticmethod
+    def cache_need(spec):
+        return mixer_class(spec.mixer.kind).cache_need(spec.mixer)
 
     def __init__(self, spec, tensors, ops, dtype):
         raise NotImplementedError
@@ -185,6 +205,7 @@ class Stream:
                                             # channel by channel, as it is added
     pending_add: Optional[object] = None    # float32 [hidden]: one vector that every row of the
                                             # stream still has to receive
+    pending_rows: Optional[object] = None   # float32 [N, hidden]: rows still to be added as well
 
 
 _MIXERS: Dict[str, type] = {}

@@ -8,12 +8,14 @@ added by the next norm's kernel, together with the norm it still has to pass thr
 the block has one after the sub-layer.  A block without a feed-forward is its first half.
 A block may scale each sub-layer's output channel by channel before the addition (a learned
 vector per sub-layer and one factor for the whole model); the scale travels with the pending
-rows and is applied by the same kernel.
+rows and is applied by the same kernel.  A block with a token shift gives its mixer rows that are
+moved towards the row of the token before, channel by channel; each call remembers the last
+normed row of every request in a state record beside the mixer's own cache.
 """
 from __future__ import annotations
 
-from .base import (Arrangement, Stream, feed_forward_class, mixer_class, norm_class,
-                   register_arrangement)
+from .base import (Arrangement, SeveralNeeds, StateNeed, Stream, feed_forward_class, mixer_class,
+                   norm_class, register_arrangement)
 import torch
 
 from .spec import BlockSpec, ParamDecl
@@ -53,6 +55,8 @@ def stream_options(stream: Stream) -> dict:
         options["delta_scale"] = stream.pending_scale
     if stream.pending_add is not None:
         options["add"] = stream.pending_add
+    if stream.pending_rows is not None:
+        options["add_rows"] = stream.pending_rows
     return options
 
 
@@ -94,7 +98,16 @@ class PreNormBlock(Arrangement):
             if place not in ("mixer", "ffn") or (place == "ffn" and spec.feed_forward is None):
                 raise ValueError(f"a pre_norm block has no sub-layer {place!r} to scale")
             out[name] = ParamDecl((spec.mixer.hidden,), "norm")
+        if spec.token_shift is not None:
+            out[spec.token_shift] = ParamDecl((spec.mixer.hidden,), "normal", mean=0.5, std=0.2)
         return out
+
+    @staticmethod
+    def cache_need(spec: BlockSpec):
+        need = mixer_class(spec.mixer.kind).cache_need(spec.mixer)
+        if spec.token_shift is None:
+            return need
+        return SeveralNeeds((need, StateNeed((spec.mixer.hidden,))))
 
     def __init__(self, spec: BlockSpec, tensors, ops, dtype):
         self._check(spec)
@@ -126,18 +139,32 @@ class PreNormBlock(Arrangement):
             return (tensors[name].to(torch.float32) * float(spec.residual_scale)).contiguous()
 
         self.mixer_scale, self.ffn_scale = scale("mixer"), scale("ffn")
+        self.shift = None
+        if spec.token_shift is not None:
+            if not hasattr(self.mixer_norm, "add_norm_shift"):
+                raise ValueError(f"a {spec.norms['mixer'][0].kind} norm has no token shift")
+            self.shift = tensors[spec.token_shift].to(torch.float32).contiguous()
+            self.fresh_stream = True
 
     def forward(self, stream: Stream, ctx, cache) -> Stream:
-        normed = self.mixer_norm.add_norm(stream.resid, stream.pending, ctx,
-                                          delta_norm=stream.pending_norm, **stream_options(stream))
+        resid = stream.resid
+        if self.shift is None:
+            normed = self.mixer_norm.add_norm(resid, stream.pending, ctx,
+                                              delta_norm=stream.pending_norm,
+                                              **stream_options(stream))
+        else:
+            cache, last = cache.parts
+            resid, normed = self.mixer_norm.add_norm_shift(
+                resid, stream.pending, ctx, self.shift, last.state,
+                delta_norm=stream.pending_norm, **stream_options(stream))
         mixed = self.mixer.forward(normed, ctx, cache)
         if self.feed_forward is None:
-            return Stream(stream.resid, mixed, self.post_mixer, pending_scale=self.mixer_scale)
+            return Stream(resid, mixed, self.post_mixer, pending_scale=self.mixer_scale)
         options = {} if self.mixer_scale is None else {"delta_scale": self.mixer_scale}
-        normed2 = self.ffn_norm.add_norm(stream.resid, mixed, ctx, delta_norm=self.post_mixer,
+        normed2 = self.ffn_norm.add_norm(resid, mixed, ctx, delta_norm=self.post_mixer,
                                          **options)
         out = self.feed_forward.forward(normed2, ctx)
-        return Stream(stream.resid, out, self.post_ffn, pending_scale=self.ffn_scale)
+        return Stream(resid, out, self.post_ffn, pending_scale=self.ffn_scale)
 
 
 register_arrangement("pre_norm", PreNormBlock)

@@ -161,9 +161,10 @@ class MoE(FeedForward):
     where the experts' weighted sum starts; experts without a gate, down_e(max(up_e x, 0)^2)
     (`activation` "relu2": no "gate" tensors, the stack is [experts, ffn, hidden]); a learned
     number per expert that is added to the scores where experts are compared and nowhere else
-    (`choice_bias`, tensor "correction").
+    (`choice_bias`, tensor "correction"); logits that are compared as they are and weighed by the
+    softmax over the chosen ones (score "softmax_chosen").
     """
-    SCORES = ("sigmoid", "softmax")
+    SCORES = ("sigmoid", "softmax", "softmax_chosen")
     ACTIVATIONS = ("swiglu", "glu_clamp", "relu2")
 
     @staticmethod

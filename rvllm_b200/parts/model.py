@@ -35,6 +35,8 @@ def param_decls(spec: ModelSpec) -> Dict[str, ParamDecl]:
     out.update(norm_params(spec.final_norm, spec.final_norm_name))
     if spec.embedding_norm is not None:
         out.update(norm_params(*spec.embedding_norm))
+    if spec.position_embedding is not None:
+        out[spec.position_embedding] = ParamDecl((spec.max_position, spec.hidden), "embedding")
     for name, rows in added_rows(spec).items():
         out[name] = ParamDecl((rows, spec.hidden), "bias")
     if spec.head_name is not None:
@@ -81,6 +83,9 @@ def validate_order(spec: ModelSpec) -> None:
             if any(isinstance(spec.layers[c.layer].mixer, ParallelSpec) for c in (call, src)):
                 raise ValueError(f"run order entry {pos}: a mixer of several mixers keeps "
                                  f"caches of its own")
+            if any(spec.layers[c.layer].token_shift is not None for c in (call, src)):
+                raise ValueError(f"run order entry {pos}: a block with a token shift keeps a "
+                                 f"state of its own")
             a = mixer_class(spec.layers[call.layer].mixer.kind).cache_need(
                 spec.layers[call.layer].mixer)
             b = mixer_class(spec.layers[src.layer].mixer.kind).cache_need(
@@ -109,6 +114,12 @@ class Model:
             if not hasattr(self.embedding_norm, "norm_f32"):
                 raise ValueError(f"a {spec.embedding_norm[0].kind} norm cannot normalise the "
                                  f"embedding rows in float32")
+        self.positions = tensors[spec.position_embedding].contiguous() \
+            if spec.position_embedding is not None else None
+        self.adds_start = any(call.add_start for call in spec.order)
+        if self.adds_start and (spec.streams >= 1 or spec.order[0].add_start):
+            raise ValueError("the first layer's input is added again after the first call, to a "
+                             "plain residual")
         self.added = {name: tensors[name].to(torch.float32).contiguous()
                       for name in added_rows(spec)}
         used = {call.layer for call in spec.order}
@@ -122,8 +133,8 @@ class Model:
         window or chunk): the owner's pages are then kept for as long as the request lives."""
         needs = []
         for call in self.spec.order:
-            m = self.spec.layers[call.layer].mixer
-            need = mixer_class(m.kind).cache_need(m)
+            block = self.spec.layers[call.layer]
+            need = arrangement_class(block.arrangement).cache_need(block)
             if call.cache_of is None:
                 needs.append(need)
                 continue
@@ -138,13 +149,20 @@ class Model:
         """Run the step's tokens; float32 logits [len(ctx.logit_rows), vocab]."""
         n = ctx.n_tokens
         resid = torch.empty((n, self.spec.hidden), dtype=torch.float32, device=self.device)
-        self.ops.embed(self.embedding, ctx.token_ids, resid, self.spec.embedding_scale)
+        options = {} if self.positions is None else \
+            {"positions": ctx.positions, "position_table": self.positions}
+        self.ops.embed(self.embedding, ctx.token_ids, resid, self.spec.embedding_scale, **options)
         if self.embedding_norm is not None:
             resid = self.embedding_norm.norm_f32(resid)
+        start = resid
+        if self.adds_start and not self.blocks[self.spec.order[0].layer].fresh_stream:
+            resid = resid.clone()          # the first block updates its rows in place
         stream = Stream(resid, None)
         for call, cache in zip(self.spec.order, caches):
             if call.add is not None:
                 stream.pending_add = self.added[call.add[0]][call.add[1]]
+            if call.add_start:
+                stream.pending_rows = start
             stream = self.blocks[call.layer].forward(stream, ctx, cache)
         if ctx.logit_rows.shape[0] == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32,

@@ -27,10 +27,17 @@ class RMSNorm(Norm):
         # bfloat16 file without loss.
         self.weight = tensors["weight"].to(torch.float32).contiguous()
 
-    def add_norm(self, resid, delta, ctx, rows=None, delta_norm=None, delta_scale=None, add=None):
+    def add_norm(self, resid, delta, ctx, rows=None, delta_norm=None, delta_scale=None, add=None,
+                 add_rows=None):
         """`delta_scale` float32 [size] multiplies the pending rows before they are added, `add`
-        float32 [size] is added to every row of the stream; both in the same kernel."""
+        float32 [size] is added to every row of the stream, `add_rows` float32 [N, size] row by
+        row; all in the same kernel."""
         delta = self._normed_delta(delta, delta_norm, ctx)
+        if add_rows is not None:
+            if rows is not None:
+                raise ValueError("rmsnorm: rows are added to the whole stream only")
+            return self.add_norm_shift(resid, delta, ctx, None, None, delta_scale=delta_scale,
+                                       add=add, add_rows=add_rows)[1]
         n = resid.shape[0] if rows is None else rows.shape[0]
         out = self.ops.new_rows(n, self.spec.size, self.dtype, resid.device)
         if delta_scale is None and add is None:
@@ -39,6 +46,20 @@ class RMSNorm(Norm):
             self.ops.add_rmsnorm(resid, delta, self.weight, self.spec.eps, out, rows,
                                  delta_scale=delta_scale if delta is not None else None, add=add)
         return out
+
+    def add_norm_shift(self, resid, delta, ctx, shift, state, delta_norm=None, delta_scale=None,
+                       add=None, add_rows=None):
+        """(the stream's new rows, the normalised rows h moved towards the token before them:
+        h_p + (h_(p-1) - h_p) * shift).  `state` float32 [slots, size] holds every request's last
+        h; with `shift` the rows of `resid` stay as they are (a row is read by its neighbour's
+        work as well), without it they are updated in place."""
+        delta = self._normed_delta(delta, delta_norm, ctx)
+        out = self.ops.new_rows(resid.shape[0], self.spec.size, self.dtype, resid.device)
+        new = torch.empty_like(resid) if shift is not None else resid
+        self.ops.add_rmsnorm_shift(resid, new, delta, self.weight, self.spec.eps, out, ctx, shift,
+                                   state, delta_scale=delta_scale if delta is not None else None,
+                                   add=add, add_rows=add_rows)
+        return new, out
 
     def norm_f32(self, x):
         """The normalised float32 rows of float32 `x`: rows that go on as the residual stream."""

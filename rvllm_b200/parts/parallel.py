@@ -3,14 +3,18 @@ keeps a cache of its own kind (pages, a state record, nothing), and the mixer's 
 
     y = sum_j scale_j * branch_j(x)
 
+or, with a norm on every branch's output, y = sum_j scale_j * rmsnorm_j(branch_j(x)).
+
 Any registered mixer can be a branch; a branch's tensors lie under its prefix below the
 mixer's own.  The sum of two branches is one elementwise kernel in float32 arithmetic; more
 branches are added one at a time.
 """
 from __future__ import annotations
 
+import torch
+
 from .base import Mixer, SeveralNeeds, mixer_class, register_mixer
-from .spec import ParallelSpec
+from .spec import ParallelSpec, ParamDecl
 
 
 class Parallel(Mixer):
@@ -21,6 +25,9 @@ class Parallel(Mixer):
             raise ValueError("parallel: one factor and one prefix per branch, at least one branch")
         if len(set(spec.prefixes)) != n:
             raise ValueError("parallel: two branches share a prefix")
+        if spec.out_norm is not None and (n != 2 or len(spec.out_norm_names) != n):
+            raise ValueError("parallel: norms on the outputs are for two branches, with a weight's "
+                             "name for each")
         for b in spec.branches:
             if b.hidden != spec.hidden:
                 raise ValueError("parallel: a branch has another width than the mixer")
@@ -32,6 +39,9 @@ class Parallel(Mixer):
         for b, prefix in zip(spec.branches, spec.prefixes):
             for k, d in mixer_class(b.kind).params(b, True).items():
                 out[prefix + k] = d
+        if spec.out_norm is not None:
+            for prefix, name in zip(spec.prefixes, spec.out_norm_names):
+                out[prefix + name] = ParamDecl((spec.hidden,), "norm")
         return out
 
     @staticmethod
@@ -52,12 +62,21 @@ class Parallel(Mixer):
         for b, prefix in zip(spec.branches, spec.prefixes):
             sub = {k[len(prefix):]: v for k, v in tensors.items() if k.startswith(prefix)}
             self.branches.append(mixer_class(b.kind)(b, sub, ops, dtype))
+        self.out_weights = None
+        if spec.out_norm is not None:
+            self.out_weights = [tensors[prefix + name].to(torch.float32).contiguous()
+                                for prefix, name in zip(spec.prefixes, spec.out_norm_names)]
 
     def forward(self, normed, ctx, cache):
         if cache is None or cache.parts is None or len(cache.parts) != len(self.branches):
             raise ValueError("parallel: the call's cache has no part per branch")
         outs = [b.forward(normed, ctx, part) for b, part in zip(self.branches, cache.parts)]
         scales = self.spec.scales
+        if self.out_weights is not None:
+            total = self.ops.new_rows(normed.shape[0], self.spec.hidden, self.dtype, normed.device)
+            self.ops.normed_sum(outs[0], self.out_weights[0], scales[0], outs[1],
+                                self.out_weights[1], scales[1], self.spec.out_norm.eps, total)
+            return total
         if len(outs) == 1:
             outs.append(outs[0])
             scales = (scales[0], 0.0)

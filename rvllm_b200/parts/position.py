@@ -9,6 +9,8 @@ call (src/model.rs:487-492).
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 from .base import PositionEncoding, register_position
@@ -42,18 +44,36 @@ class PartialRope(PositionEncoding):
     """The rotate-half rotation on the first `rot_dims` dimensions of a head only: dimension
     i turns with i + rot_dims/2 by the angle pos * theta^(-2i/rot_dims); the others pass.
     There is no table over positions: the kernels form the angle (float32) from the position
-    and `frequencies()`, so no longest context has to be known."""
+    and `frequencies()`, so no longest context has to be known.  With `yarn` (see `PositionSpec`)
+    slow pairs turn `factor` times slower, and `amplitude` multiplies cosine and sine."""
 
     def __init__(self, spec: PositionSpec, device):
         dims = spec.rot_dims or spec.head_dim
+        self.amplitude = 1.0
         if dims % 2 or dims > spec.head_dim or dims < 0:
             raise ValueError(f"rope_partial needs an even number of turning dimensions within "
                              f"the head's {spec.head_dim}, got {dims}")
         self.spec = spec
         self.rot_dims = dims
         i = torch.arange(dims // 2, dtype=torch.float64)
-        self.inv_freq = torch.pow(torch.tensor(spec.theta, dtype=torch.float64),
-                                  -2.0 * i / max(dims, 1)).to(torch.float32).to(device).contiguous()
+        f = torch.pow(torch.tensor(spec.theta, dtype=torch.float64), -2.0 * i / max(dims, 1))
+        if spec.yarn is not None:
+            factor, original, fast, slow = spec.yarn
+            if not (factor > 0 and original > 0 and fast > 0 and slow > 0 and spec.theta > 1):
+                raise ValueError("rope_partial: the scaling needs positive numbers and a base "
+                                 "above 1")
+
+            def dim(turns):
+                """The dimension that makes this many turns over the original length."""
+                return dims * math.log(original / (2.0 * math.pi * turns)) / \
+                    (2.0 * math.log(spec.theta))
+
+            lo = max(math.floor(dim(fast)), 0)
+            hi = min(math.ceil(dim(slow)), dims - 1)
+            ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+            f = f / factor * ramp + f * (1.0 - ramp)
+            self.amplitude = 0.1 * math.log(factor) + 1.0
+        self.inv_freq = f.to(torch.float32).to(device).contiguous()
 
     def rotation_table(self):
         return None

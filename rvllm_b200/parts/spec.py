@@ -53,13 +53,20 @@ class PositionSpec:
     `scaling` = (factor, low, high, original) stretches its long wavelengths: with wavelength
     l = 2 pi / f a frequency stays when l < original / high, becomes f / factor when
     l > original / low, and in between is (1 - s) f / factor + s f with
-    s = (original / l - low) / (high - low)."""
+    s = (original / l - low) / (high - low).
+    `yarn` = (factor, original, fast, slow) (kind "rope_partial"; "YaRN: Efficient Context Window
+    Extension of Large Language Models", Peng et al.): with
+    dim(t) = n ln(original / (2 pi t)) / (2 ln theta) for n turning dimensions, lo =
+    max(floor(dim(fast)), 0) and hi = min(ceil(dim(slow)), n - 1), frequency f_i becomes
+    r_i f_i / factor + (1 - r_i) f_i with r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), and
+    cosine and sine are multiplied by 0.1 ln(factor) + 1."""
     kind: str
     head_dim: int = 0
     theta: float = 0.0
     max_position: int = 0
     rot_dims: int = 0
     scaling: Optional[Tuple[float, float, float, int]] = None
+    yarn: Optional[Tuple[float, float, float, float]] = None
 
 
 @dataclass(frozen=True)
@@ -156,6 +163,53 @@ class MixedAttentionSpec(AttentionSpec):
 
 
 @dataclass(frozen=True)
+class PooledAttentionSpec(AttentionSpec):
+    """Grouped-query attention over a window of tokens and, before the window, pooled blocks.
+
+    pool             tokens per block P (None: no blocks).  The query at position i sees, besides
+                     the tokens of its window, block b (positions bP .. bP + P - 1) once
+                     bP + P - 1 <= i - window; its key and value are the means of the block's
+                     cached keys and values.  A token that has left the window and whose
+                     block is not seen yet is not seen.  One softmax over both.
+    softcap          c: scores become c tanh(score / c) after the scale
+    values_are_keys  a token's value is its key before the rotation (no "v" tensor)
+    `sinks` (tensor "sink" [heads]) as in the base class; the position kind is "rope_partial" or
+    "none".
+    """
+    pool: Optional[int] = None
+    softcap: Optional[float] = None
+    values_are_keys: bool = False
+
+
+@dataclass(frozen=True)
+class LinearAttentionSpec(MixerSpec):
+    """A linear attention with decay: per head S <- diag(a) S + k v^T, o = S^T q.
+
+    decay        a constant a per head; or None: one decay per token and key channel,
+                 a = sigmoid(z)^(1 / decay_tau) with z = W_a2 (W_a1 x) + bias of rank
+                 `decay_rank` (tensors "a1", "a2", "a2.b")
+    activation   "silu" on the three projections q, k and v, or None
+    q_scale      factor on q
+    norm         the read-out's RMS norm: "all" over the concatenated heads (weight
+                 [heads * v_head_dim]) or "head" over each head with one shared weight
+                 [v_head_dim]
+    gate         "sigmoid" or "silu" of W_g x multiplies the normed read-out
+    """
+    num_heads: int = 0
+    head_dim: int = 0
+    v_head_dim: int = 0
+    decay: Optional[Tuple[float, ...]] = None
+    decay_rank: int = 0
+    decay_tau: float = 1.0
+    activation: Optional[str] = None
+    q_scale: float = 1.0
+    norm: str = "all"
+    gate: str = "sigmoid"
+    norm_eps: float = 1e-6
+    names: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
+
+
+@dataclass(frozen=True)
 class MinGRUSpec(MixerSpec):
     """A gated recurrence whose gates read only the current token; `width` channels."""
     width: int = 0
@@ -199,10 +253,14 @@ class MLSTMSpec(MixerSpec):
 class ParallelSpec(MixerSpec):
     """Several mixers side by side that read the same input; the result is the sum of their
     outputs, each times its factor.  `prefixes[j]` is where branch j's tensors lie below the
-    mixer's own prefix.  Every branch keeps a cache of its own."""
+    mixer's own prefix.  Every branch keeps a cache of its own.  With `out_norm` every branch's
+    output passes an RMS norm of its own over the width before the sum; `out_norm_names[j]` is the
+    weight's name below branch j's prefix."""
     branches: Tuple[MixerSpec, ...] = ()
     scales: Tuple[float, ...] = ()
     prefixes: Tuple[str, ...] = ()
+    out_norm: Optional[NormSpec] = None
+    out_norm_names: Tuple[str, ...] = ()
 
 
 @dataclass(frozen=True)
@@ -258,7 +316,9 @@ class MoESpec(FeedForwardSpec):
     that every token passes as well and whose output is added (tensors under "shared.");
     `activation` "relu2": experts without a gate, down_e(max(up_e x, 0)^2); `choice_bias`: a
     learned number per expert (tensor "correction" [experts]) is added to the scores where
-    experts are compared, while the weights are made from the scores without it."""
+    experts are compared, while the weights are made from the scores without it; score
+    "softmax_chosen": the logits themselves are compared and the weights are the softmax over the
+    chosen logits alone."""
     ffn_dim: int = 0
     experts: int = 0
     top: int = 0
@@ -299,6 +359,10 @@ class BlockSpec:
     "hyper_pre_norm" keeps `streams` >= 1 copies of the residual (hyper-connections); `hyper` maps
     the places "mixer" and "ffn" to the prefix of that sub-layer's three tensors (".in" [S],
     ".out" [S], ".mix" [S, S]).
+
+    `token_shift` names a tensor [hidden] ("pre_norm" blocks): the mixer reads
+    h_p + (h_(p-1) - h_p) * shift, h the normed rows and h_(-1) = 0; every call keeps its last
+    normed row.
     """
     arrangement: str
     mixer: MixerSpec
@@ -310,6 +374,7 @@ class BlockSpec:
     hyper: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
     layer_scale: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
     residual_scale: float = 1.0
+    token_shift: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -318,10 +383,11 @@ class LayerCall:
     index (in the order list) of an earlier call whose cache this call reads instead of
     owning one.  `add` = (tensor name, row): that row of a tensor [rows, hidden] is added to the
     residual stream right before the call (what a repeated stretch of layers adds at the start
-    of each pass)."""
+    of each pass); `add_start`: so are the rows the first layer read."""
     layer: int
     cache_of: Optional[int] = None
     add: Optional[Tuple[str, int]] = None
+    add_start: bool = False
 
 
 @dataclass(frozen=True)
@@ -345,3 +411,5 @@ class ModelSpec:
     eos_token_id: Optional[int] = None
     embedding_norm: Optional[Tuple[NormSpec, object]] = None   # (norm, tensor name): the
                                                 # embedding rows pass it before the first layer
+    position_embedding: Optional[str] = None    # tensor [max_position, hidden]: row p is added to
+                                                # the (scaled) embedding row of position p

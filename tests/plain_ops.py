@@ -24,9 +24,12 @@ class PlainOps:
     name = "plain"
 
     # ---- embedding -------------------------------------------------------------------
-    def embed(self, table, ids, out, scale=None):
+    def embed(self, table, ids, out, scale=None, positions=None, position_table=None):
         x = _f(table[ids.long()])
-        out.copy_(x if scale is None else x * scale)
+        x = x if scale is None else x * scale
+        if positions is not None:
+            x = x + _f(position_table[positions.long()])
+        out.copy_(x)
 
     # ---- residual add + RMSNorm ------------------------------------------------------
     def add_rmsnorm(self, resid, delta, weight, eps, out, rows=None, delta_scale=None, add=None):
@@ -48,6 +51,37 @@ class PlainOps:
                 x = x + _f(add)
         rms = (x.pow(2).mean(dim=-1, keepdim=True) + eps).sqrt()
         out.copy_((x / rms * _f(weight)).to(out.dtype))
+
+    def add_rmsnorm_shift(self, resid, new_resid, delta, weight, eps, out, ctx, shift, state,
+                          delta_scale=None, add=None, add_rows=None):
+        x = resid.clone()
+        if delta is not None:
+            x = x + (_f(delta) * _f(delta_scale) if delta_scale is not None else _f(delta))
+        if add_rows is not None:
+            x = x + add_rows
+        if add is not None:
+            x = x + _f(add)
+        new_resid.copy_(x)
+        h = x / (x.pow(2).mean(dim=-1, keepdim=True) + eps).sqrt() * _f(weight)
+        if shift is not None:
+            q_start, slots = ctx.q_start.tolist(), ctx.state_slot.tolist()
+            moved = h.clone()
+            for r in range(ctx.n_reqs):
+                a, b = q_start[r], q_start[r + 1]
+                if a == b:
+                    continue
+                first = state[slots[r]] if slots[r] >= 0 else torch.zeros_like(h[a])
+                before = torch.cat([first[None], h[a:b - 1]])
+                moved[a:b] = h[a:b] + (before - h[a:b]) * _f(shift)
+                if slots[r] >= 0:
+                    state[slots[r]] = h[b - 1]
+            h = moved
+        out.copy_(h.to(out.dtype))
+
+    def normed_sum(self, a, wa, sa, b, wb, sb, eps, out):
+        def rms(x):
+            return x / (x.pow(2).mean(dim=-1, keepdim=True) + eps).sqrt()
+        out.copy_((sa * rms(_f(a)) * _f(wa) + sb * rms(_f(b)) * _f(wb)).to(out.dtype))
 
     # ---- matrix product --------------------------------------------------------------
     def linear(self, x, w, bias=None, out_dtype=None):
@@ -220,7 +254,8 @@ class PlainOps:
 
     # ---- partial rotation + cache write ------------------------------------------------
     def rope_partial_write(self, rows, num_heads, num_kv_heads, head_dim, v_head_dim, freq,
-                           positions, slot_mapping, k_cache, v_cache):
+                           positions, slot_mapping, k_cache, v_cache, amplitude=1.0,
+                           values_are_keys=False):
         n = rows.shape[0]
         H, G, d, dv = num_heads, num_kv_heads, head_dim, v_head_dim
 
@@ -230,21 +265,107 @@ class PlainOps:
             inv, dims = freq
             half = dims // 2
             a = positions.to(torch.float32)[:, None] * inv[None, :]
-            cos, sin = torch.cos(a)[:, None, :], torch.sin(a)[:, None, :]
+            cos, sin = torch.cos(a)[:, None, :] * amplitude, torch.sin(a)[:, None, :] * amplitude
             u, v = x[..., :half], x[..., half:dims]
             return torch.cat([u * cos - v * sin, v * cos + u * sin, x[..., dims:]], dim=-1)
 
         q = turn(_f(rows[:, :H * d]).reshape(n, H, d))
-        rows[:, :H * d] = q.reshape(n, H * d).to(rows.dtype)
+        rows[:, :H * d] = q.reshape(n, H * d).to(rows.dtype).clone()
         if G:
             k = turn(_f(rows[:, H * d:(H + G) * d]).reshape(n, G, d))
-            v = rows[:, (H + G) * d:(H + G) * d + G * dv].reshape(n, G, dv)
+            v_off = H * d if values_are_keys else (H + G) * d
+            v = rows[:, v_off:v_off + G * dv].reshape(n, G, dv)
             kc, vc = k_cache.view(-1, G, d), v_cache.view(-1, G, dv)
             for t in range(n):
                 s = int(slot_mapping[t])
                 if s >= 0:
                     kc[s] = k[t].to(kc.dtype)
                     vc[s] = v[t].to(vc.dtype)
+
+    # ---- pooled blocks: their rows, and attention over a window and the blocks before it ----
+    def pool_rows(self, k_cache, v_cache, group, ctx, pool, slots, k_out, v_out):
+        G, d = k_cache.shape[-2:]
+        ps = group.page_size
+        treq, pos = ctx.token_req.tolist(), ctx.positions.tolist()
+        for t, s in enumerate(slots.tolist()):
+            if s < 0:
+                continue
+            table = group.block_table[treq[t]].tolist()
+            idx = torch.tensor([table[j // ps] * ps + j % ps
+                                for j in range(pos[t] - pool + 1, pos[t] + 1)])
+            for src, dst in ((k_cache, k_out), (v_cache, v_out)):
+                mean = _f(src.view(-1, G, d)[idx]).mean(dim=0)
+                dst.view(-1, G, d)[s] = mean.to(dst.dtype)
+
+    def paged_attention_pooled(self, rows, num_heads, num_kv_heads, head_dim, k_cache, v_cache, ctx,
+                               group, pooled, scale, softcap, window, sinks, out):
+        H, G, d = num_heads, num_kv_heads, head_dim
+        ps = group.page_size
+        q_start, ctx_lens = ctx.q_start.tolist(), ctx.ctx_lens.tolist()
+        for r in range(ctx.n_reqs):
+            clen = ctx_lens[r]
+            a, b = q_start[r], q_start[r + 1]
+            if clen == 0:
+                out[a:b] = 0
+                continue
+            table = group.block_table[r].tolist()
+            for t in range(a, b):
+                p = clen - (b - a) + (t - a)
+                lo = 0 if window is None else max(0, p - window + 1)
+                idx = torch.tensor([table[j // ps] * ps + j % ps for j in range(lo, p + 1)])
+                k, v = _f(k_cache.view(-1, G, d)[idx]), _f(v_cache.view(-1, G, d)[idx])
+                if pooled is not None:
+                    pk, pv, pgroup, pool = pooled
+                    nb = max(0, p - window + 1) // pool
+                    ptab = pgroup.block_table[r].tolist()
+                    pidx = torch.tensor([ptab[j // ps] * ps + j % ps for j in range(nb)],
+                                        dtype=torch.long)
+                    k = torch.cat([_f(pk.view(-1, G, d)[pidx]), k])
+                    v = torch.cat([_f(pv.view(-1, G, d)[pidx]), v])
+                q = _f(rows[t, :H * d]).reshape(H, d)
+                for h in range(H):
+                    s = (k[:, h // (H // G)] @ q[h]) * scale
+                    if softcap is not None:
+                        s = softcap * torch.tanh(s / softcap)
+                    if sinks is not None:
+                        s = torch.cat([s, _f(sinks[h:h + 1])])
+                    w = torch.softmax(s, dim=0)[:k.shape[0]]
+                    out[t, h * d:(h + 1) * d] = (w @ v[:, h // (H // G)]).to(out.dtype)
+
+    # ---- linear attention with decay ---------------------------------------------------------
+    def linear_attention(self, rows, log_decay, decay_bias, tau, norm_w, state, ctx, out, heads, dim,
+                         vdim, activation, q_scale, norm, gate, eps):
+        H, d, dv = heads, dim, vdim
+        q_start, slots = ctx.q_start.tolist(), ctx.state_slot.tolist()
+        p = _f(rows)
+        act = torch.nn.functional.silu if activation == "silu" else (lambda x: x)
+        o_k, o_v = H * d, 2 * H * d
+        o_g = o_v + H * dv
+        o_z = o_g + H * dv
+        out.zero_()
+        for r in range(ctx.n_reqs):
+            a, b = q_start[r], q_start[r + 1]
+            if slots[r] < 0 or a == b:
+                continue
+            S = state[slots[r]].reshape(H, d, dv).clone()
+            for t in range(a, b):
+                q = act(p[t, :o_k]).reshape(H, d) * q_scale
+                k = act(p[t, o_k:o_v]).reshape(H, d)
+                v = act(p[t, o_v:o_g]).reshape(H, dv)
+                if log_decay is None:
+                    z = p[t, o_z:o_z + H * d] + _f(decay_bias)
+                    keep = torch.exp(torch.nn.functional.logsigmoid(z) / tau).reshape(H, d)
+                else:
+                    keep = torch.exp(_f(log_decay))[:, None].expand(H, d)
+                S = keep[:, :, None] * S + k[:, :, None] * v[:, None, :]
+                o = torch.einsum("hdv,hd->hv", S, q)
+                if norm == "all":
+                    o = o.reshape(-1)
+                o = o / (o.pow(2).mean(dim=-1, keepdim=True) + eps).sqrt()
+                g = p[t, o_g:o_g + H * dv]
+                g = torch.sigmoid(g) if gate == "sigmoid" else torch.nn.functional.silu(g)
+                out[t] = (o.reshape(-1) * _f(norm_w) * g).to(out.dtype)
+            state[slots[r]] = S.reshape(-1)
 
     # ---- attention with mixed heads over the pages ---------------------------------------
     def paged_attention_mixed(self, rows, gate_off, num_heads, num_kv_heads, head_dim, v_head_dim,
@@ -336,8 +457,9 @@ class PlainOps:
         top = ids.shape[1]
         size = E // groups
         for t in range(n):
-            s = torch.sigmoid(_f(logits[t])) if score == "sigmoid" else \
-                torch.softmax(_f(logits[t]), dim=0)
+            s = _f(logits[t])
+            if score != "softmax_chosen":
+                s = torch.sigmoid(s) if score == "sigmoid" else torch.softmax(s, dim=0)
             allowed = s.clone() if choice_bias is None else s + _f(choice_bias)
             if groups > 1:
                 gs = allowed.reshape(groups, size).sort(dim=1, descending=True).values[:, :group_top].sum(1)
@@ -347,7 +469,10 @@ class PlainOps:
                         allowed[g * size:(g + 1) * size] = -3.0e38
             chosen = torch.sort(allowed, descending=True, stable=True).indices[:top]
             ids[t] = chosen.to(torch.int32)
-            w = s[chosen] / (s[chosen].sum() + weight_eps) if renormalize else s[chosen]
+            if score == "softmax_chosen":
+                w = torch.softmax(s[chosen], dim=0)
+            else:
+                w = s[chosen] / (s[chosen].sum() + weight_eps) if renormalize else s[chosen]
             weights[t] = w * route_scale
 
     def moe_route(self, x, router, groups, keep, group_top, weight_eps, ids, weights, **options):
