@@ -231,14 +231,14 @@ class BatchBuilder:
                 nb = cache.pages_for(cache.groups[gi], c)
                 table[r, :nb] = t[:nb]
                 if every > 1:
-                    # rows completed by this step: row k by the token at (k + 1) * every - 1
+                    # rows completed by this step: row i by the token at (i + 1) * every - 1
                     k0, k1 = s // every, c // every
                     if k1 - k0 == 1:
                         slots[a + k1 * every - 1 - s] = int(t[k0 // ps]) * ps + k0 % ps
                     elif k1 > k0:
-                        k = np.arange(k0, k1)
-                        slots[a + (k + 1) * every - 1 - s] = \
-                            t[k // ps].astype(np.int64) * ps + k % ps
+                        done = np.arange(k0, k1)
+                        slots[a + (done + 1) * every - 1 - s] = \
+                            t[done // ps].astype(np.int64) * ps + done % ps
                     continue
                 if q == 1:
                     page = int(t[s // ps])
