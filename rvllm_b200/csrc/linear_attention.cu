@@ -618,11 +618,11 @@ extern "C" int rv_linear_attention(const float* rows, int stride, const float* l
     if (!log_decay && (!bias || !(tau > 0.f))) RV_FAIL("linear_attention: neither a decay nor a bias and tau");
     if (stride < 2 * H * d + 2 * H * dv + (log_decay ? 0 : H * d)) RV_FAIL("linear_attention: rows are too short");
     if (n_reqs > 65535 || H > 65535 || d > 2048 || dv > 65535) RV_FAIL("linear_attention: too many requests or heads");
-    if (((uintptr_t)scratch | (uintptr_t)state) & 15) RV_FAIL("linear_attention: scratch and records must be 16-byte aligned");
+    if ((uintptr_t)scratch & 15) RV_FAIL("linear_attention: the scratch must be 16-byte aligned");
     cudaStream_t s = (cudaStream_t)stream;
     const int tiles_d = (d + LA_T - 1) / LA_T, tiles_v = (dv + LA_T - 1) / LA_T;
     float* num = scratch;
-    const bool v4 = dv % 4 == 0;
+    const bool v4 = dv % 4 == 0 && ((uintptr_t)state & 15) == 0;
     if (n_decode > 0) {
         const size_t smem = (size_t)(3 * d + (v4 ? 8 : 2) * LA_T) * sizeof(float);
         const dim3 grid(tiles_v, H, n_decode);

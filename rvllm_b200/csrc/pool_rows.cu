@@ -23,8 +23,10 @@ __global__ void pool_rows_kernel(const T* __restrict__ k_cache, const T* __restr
         const T* src = i < width ? k_cache + i : v_cache + (i - width);
         float sum = 0.f;
 #pragma unroll 8
-        for (int j = p1 - pool + 1; j <= p1; ++j)
-            sum += rv_load(src + ((size_t)table[j / page_size] * page_size + j % page_size) * width);
+        for (int j = max(0, p1 - pool + 1); j <= p1; ++j) {
+            const int page = table[j / page_size];
+            if (page >= 0) sum += rv_load(src + ((size_t)page * page_size + j % page_size) * width);
+        }
         rv_store((i < width ? k_out + i : v_out + (i - width)) + (size_t)slot * width, sum / (float)pool);
     }
 }
