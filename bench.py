@@ -961,6 +961,39 @@ def mevuvik_config(sz):
             "loop": {"start": 2, "stop": 4, "times": 2}, "layers": layers}
 
 
+FEKIZEN_SIZES = {
+    # linear attention with constant decays and (window-and-blocks attention beside a linear
+    # attention with decays by channel) in turn; six layers of which the middle two run twice:
+    # eight layer runs, as Mevuvik's.  Both linear attentions have the heads and sizes of Mevuvik's
+    # matrix memory.  The fields Mevuvik reads are here too, so that it runs beside at equal sizes.
+    "w1024": {"width": 1024, "layers": 8, "heads": 16, "kv": 4, "dim": 64, "rank": 128, "rot": 16,
+              "q_rank": 256, "mem_heads": 8, "mem_dim": 64, "mem_vdim": 128, "window": 512, "pool": 16,
+              "experts": 16, "top": 4, "groups": (4, 2), "ff": 1024, "vocab": 32768},
+    "w2048": {"width": 2048, "layers": 8, "heads": 32, "kv": 8, "dim": 64, "rank": 128, "rot": 16,
+              "q_rank": 512, "mem_heads": 16, "mem_dim": 64, "mem_vdim": 128, "window": 512, "pool": 16,
+              "experts": 16, "top": 4, "groups": (4, 2), "ff": 2048, "vocab": 32768},
+}
+
+
+def fekizen_config(sz):
+    mlp = {"kind": "moe", "expert": {"ff": sz["ff"]},
+           "router": {"experts": sz["experts"], "top": sz["top"]}, "shared": {"ff": sz["ff"]}}
+    H, d, dv = sz["mem_heads"], sz["mem_dim"], sz["mem_vdim"]
+    lightning = {"heads": H, "dim": d, "vdim": dv,
+                 "decay": [1.0 - 2.0 ** (-1.0 - 9.0 * h / max(1, H - 1)) for h in range(H)]}
+    par = {"left": {"heads": sz["heads"], "kv_heads": sz["kv"], "dim": sz["dim"], "vdim": sz["dim"],
+                    "scale": sz["dim"] ** -0.5, "softcap": 50.0,
+                    "mask": {"size": sz["window"], "pool": sz["pool"]},
+                    "rot": {"base": 10000.0, "dims": sz["dim"],
+                            "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}},
+           "right": {"heads": H, "dim": d, "vdim": dv, "tau": 16.0, "rank": 16}}
+    layers = [{"type": "lightning", "mixer": lightning, "mlp": mlp} if i % 2 == 0 else
+              {"type": "parallel", "mixer": par, "mlp": mlp} for i in range(sz["layers"] - 2)]
+    return {"architecture": "Fekizen", "vocab": sz["vocab"], "width": sz["width"], "max_positions": 8192,
+            "norm": {"eps": 1e-5}, "embedding": {"scale": sz["width"] ** 0.5},
+            "loop": {"start": 2, "stop": 4, "times": 2}, "layers": layers}
+
+
 def lfm2_all_attention(sz):
     """LFM2 with the same width and layer count, attention in every layer with the same head
     counts and sizes, and a SwiGLU as wide as the experts a token uses together."""
@@ -991,7 +1024,9 @@ class OpTimer:
              "short_conv", "mingru_scan", "swiglu", "xielu", "qk_unit_write", "latent_norm_write",
              "heads_product", "sigmoid_gate", "moe_select", "moe_route", "moe_experts", "softcap",
              "hyper_norm", "qkv_full_norm_rope_write", "gated_delta", "glu_clamp", "relu2",
-             "weighted_sum", "latent_prepare", "rope_heads", "head_gate", "mlstm")
+             "weighted_sum", "latent_prepare", "rope_heads", "head_gate", "mlstm",
+             "add_rmsnorm_shift", "normed_sum", "pool_rows", "paged_attention_pooled",
+             "linear_attention")
 
     def __init__(self, torch, ops):
         self.torch, self.ops, self.events, self.saved = torch, ops, [], {}
@@ -1028,8 +1063,8 @@ class OpTimer:
 
 
 def run_designs(args, which="retorax"):
-    """Retorax (`--only retorax`) or Bizenex (`--only bizenex`) beside LFM2, Mevuvik (`--only mevuvik`) beside Bizenex, or Vifanex
-    (`--only vifanex`) beside Bizenex, at equal sizes:
+    """Retorax (`--only retorax`) or Bizenex (`--only bizenex`) beside LFM2, Mevuvik (`--only mevuvik`) or Vifanex
+    (`--only vifanex`) beside Bizenex, or Fekizen (`--only fekizen`) beside Mevuvik, at equal sizes:
     prompt and single-token throughput, and the device time of every kernel of one prompt step
     and one single-token step with its share of the roofline.  One JSON line."""
     import torch
@@ -1045,7 +1080,7 @@ def run_designs(args, which="retorax"):
     sampler = ClockSampler()
     sampler.start()
     sizes = {"retorax": RETORAX_SIZES, "bizenex": BIZENEX_SIZES, "vifanex": VIFANEX_SIZES,
-             "mevuvik": MEVUVIK_SIZES}[which]
+             "mevuvik": MEVUVIK_SIZES, "fekizen": FEKIZEN_SIZES}[which]
     for size_name, sz in sizes.items():
         if args.design_size not in ("all", size_name):
             continue
@@ -1054,6 +1089,8 @@ def run_designs(args, which="retorax"):
             pair = (("retorax", retorax_config(sz)), ("lfm2", lfm2_like(sz)))
         elif which == "bizenex":
             pair = (("bizenex", bizenex_config(sz)), ("lfm2", lfm2_all_attention(sz)))
+        elif which == "fekizen":
+            pair = (("fekizen", fekizen_config(sz)), ("mevuvik", mevuvik_config(sz)))
         elif which == "mevuvik":
             pair = (("mevuvik", mevuvik_config(sz)), ("bizenex", bizenex_config(sz)))
         else:
@@ -1129,7 +1166,8 @@ def run_designs(args, which="retorax"):
             torch.cuda.empty_cache()
         entry["rooflines"] = {"retorax": design_rooflines, "bizenex": bizenex_rooflines,
                               "vifanex": vifanex_rooflines,
-                              "mevuvik": mevuvik_rooflines}[which](sz, entry, pk, T, CTX)
+                              "mevuvik": mevuvik_rooflines,
+                              "fekizen": fekizen_rooflines}[which](sz, entry, pk, T, CTX)
         out[size_name] = entry
     out["clocks"] = sampler.stop()
     print(json.dumps(out))
@@ -1371,6 +1409,90 @@ def mevuvik_rooflines(sz, entry, pk, T, CTX):
     return rows
 
 
+def fekizen_rooflines(sz, entry, pk, T, CTX):
+    """Per kernel pair (Fekizen's kernel, Mevuvik's like kernel): device time of all calls in the
+    prompt step and in a single-token step of batch 64, and the time the roofline allows: bytes /
+    measured copy rate for the elementwise kernels and for single tokens, tensor FLOPs / measured
+    GEMM rate for attention and the experts' products, and for the linear attentions and the
+    matrix memory the float32 FLOPs of the recurrence (5 a state element a token: decay, write,
+    read-out) on the CUDA cores at their nominal rate."""
+    W, F, H, G, D, R = sz["width"], sz["ff"], sz["heads"], sz["kv"], sz["dim"], sz["rank"]
+    top, rot, Rq = sz["top"], sz["rot"], sz["q_rank"]
+    Hm, Dm, Vm = sz["mem_heads"], sz["mem_dim"], sz["mem_vdim"]
+    win, pool = sz["window"], sz["pool"]
+    runs = sz["layers"]
+    half = runs // 2                                 # parallel runs of both designs, and the others
+    hbm, tens, fp32 = pk["hbm_gbs"] * 1e3, pk["bf16_tflops"] * 1e6, FP32_TFLOPS_NOMINAL * 1e6
+    pairs = T * (T + 1) // 2
+    seen = sum(min(i + 1, win) + max(0, i - win + 1) // pool for i in range(T))
+    state = Hm * Dm * Vm
+    la_cols, ml_cols = 2 * Hm * Dm + 2 * Hm * Vm, 2 * Hm * Dm + 2 * Hm * Vm + 2 * Hm
+    la = runs * T * 5.0 * state / fp32
+    ideal = {
+        # stream read and written, pending rows read, normed rows written
+        "add_rmsnorm_shift": runs * T * W * (4 + 4 + 2 + 2) / hbm,
+        "add_rmsnorm": (runs + 1) * T * W * (4 + 4 + 2 + 2) / hbm,
+        "add_rmsnorm_mevuvik": (2 * runs + 2) * T * W * (4 + 4 + 2 + 2) / hbm,
+        # queries turned in place, keys read once, keys and values written
+        "rope_partial_write": half * T * (2 * H * D + 3 * G * D) * 2 / hbm,
+        "latent_prepare": half * T * (Rq + R) * 4 / hbm,
+        "pool_rows": half * T * 2 * G * D * 2 * (1.0 + 1.0 / pool) / hbm,
+        "qk_unit_write": half * T * ((H + 2 * G) * D * 2 + 2 * G * D * 2) / hbm,
+        "paged_attention_pooled": half * seen * 4.0 * H * D / tens,
+        "paged_attention": (half * pairs * 4.0 * H * R + half * pairs * 4.0 * H * D) / tens,
+        "normed_sum": half * T * W * 6 / hbm,
+        "weighted_sum": half * T * W * 6 / hbm,
+        "swiglu": runs * T * F * 6 / hbm,
+        "relu2": T * top * F * 4 / hbm,
+        "moe_route": runs * T * (W * 2 + top * 8) / hbm,
+        "moe_route_mevuvik": (runs - 1) * T * (W * 2 + top * 8) / hbm,
+        "moe_experts": runs * T * top * 6.0 * F * W / tens,
+        "moe_experts_mevuvik": (runs - 1) * T * top * 4.0 * F * W / tens,
+        "linear_attention": max(la, T * (runs * (la_cols * 4 + Hm * Vm * 2) + half * Hm * Dm * 4) / hbm),
+        "mlstm": half * max(T * Hm * 5.0 * Dm * (Vm + 1) / fp32, T * (ml_cols * 4 + Hm * Vm * 2) / hbm),
+    }
+    like = (("add_rmsnorm_shift", "add_rmsnorm", "add_rmsnorm_mevuvik"),
+            ("add_rmsnorm", "add_rmsnorm", "add_rmsnorm_mevuvik"),
+            ("rope_partial_write", "latent_prepare", "latent_prepare"),
+            ("pool_rows", "qk_unit_write", "qk_unit_write"),
+            ("paged_attention_pooled", "paged_attention", "paged_attention"),
+            ("normed_sum", "weighted_sum", "weighted_sum"),
+            ("swiglu", "relu2", "relu2"),
+            ("moe_route", "moe_route", "moe_route_mevuvik"),
+            ("moe_experts", "moe_experts", "moe_experts_mevuvik"),
+            ("linear_attention", "mlstm", "mlstm"))
+    # single tokens at batch 64: every request's records and visible rows are read (records written)
+    B = 64
+    dec = {
+        "linear_attention": runs * B * 2.0 * state * 4 / hbm,
+        "mlstm": half * B * 2.0 * Hm * Dm * (Vm + 1) * 4 / hbm,
+        "paged_attention_pooled": half * B * (win + (CTX - win) // pool) * 2 * G * D * 2 / hbm,
+        "paged_attention": half * B * CTX * (R * 2 + 2 * G * D * 2) / hbm,
+    }
+
+    def table(ours, theirs, pairs_, bound):
+        rows = {}
+        for mine, other, other_ideal in pairs_:
+            a, b = ours.get(mine), theirs.get(other)
+            if not a or mine not in bound:
+                continue
+            rows[mine] = {"us": a["us"], "calls": a["calls"], "roofline_us": round(bound[mine], 1),
+                          "times_roofline": round(a["us"] / bound[mine], 2)}
+            if b:
+                rows[mine].update({"like": other, "like_us": b["us"], "like_calls": b["calls"],
+                                   "like_roofline_us": round(bound[other_ideal], 1),
+                                   "like_times_roofline": round(b["us"] / bound[other_ideal], 2)})
+        return rows
+
+    key = "prefill_2048_kernels_us"
+    out = table(entry["fekizen"][key], entry["mevuvik"][key], like, ideal)
+    key = "decode_b64_kernels_us"
+    out["decode_b64"] = table(entry["fekizen"][key], entry["mevuvik"][key],
+                              (("linear_attention", "mlstm", "mlstm"),
+                               ("paged_attention_pooled", "paged_attention", "paged_attention")), dec)
+    return out
+
+
 def run_reference(args):
     print(json.dumps({
         "impl": "reference",
@@ -1388,14 +1510,14 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--size", default="1.2b", choices=sorted(SIZES),
                     help="layer sizes: LFM2-1.2B (the default and the headline), 700M or 350M")
-    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "kernels", "breakdown", "workload", "further", "retorax", "bizenex", "vifanex", "mevuvik"],
+    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "kernels", "breakdown", "workload", "further", "retorax", "bizenex", "vifanex", "mevuvik", "fekizen"],
                     help="run one part only (for profiling); the JSON line then lacks the rest")
     ap.add_argument("--workloads", default="both", choices=["both", "none"] + sorted(WORKLOADS),
                     help="scheduler workloads to add to the line (default: both)")
     ap.add_argument("--workload", default="350m-mixed", choices=sorted(WORKLOADS),
                     help="with --only workload: which one")
     ap.add_argument("--design-size", default="all", choices=["all"] + sorted(set(RETORAX_SIZES) | set(VIFANEX_SIZES)),
-                    help="with --only retorax, bizenex, vifanex or mevuvik: which of the sizes")
+                    help="with --only retorax, bizenex, vifanex, mevuvik or fekizen: which of the sizes")
     ap.add_argument("--kernel", default="all",
                     help="with --only kernels: attn_decode, attn_prefill, gemm, gemm:NxK, elementwise, copy_rate or all")
     ap.add_argument("--kernel-batch", type=int, default=64)
@@ -1426,6 +1548,8 @@ def main():
         return run_designs(args, "vifanex")
     if args.only == "mevuvik":
         return run_designs(args, "mevuvik")
+    if args.only == "fekizen":
+        return run_designs(args, "fekizen")
     if args.only == "workload":
         print(json.dumps({"only": "workload", args.workload: run_workload(args.workload)}))
         return 0

@@ -5,10 +5,11 @@
 //
 // The decay a_t is a constant per head (log_decay [H]) or made by the token for every key channel,
 // log a = logsigmoid(z + bias) / tau.  q, k and v may pass silu; q is multiplied by q_scale.
-// Everything here is float32.
 //
-// rows [N, stride] float32: q [H d] | k [H d] | v [H dv] | g [H dv] | z [H d] (decays by tokens).
-// A request's record: [H][d][dv] float32.
+// rows [N, stride] of the compute type: q [H d] | k [H d] | v [H dv] | g [H dv]; z [N, H d] float32.
+// A request's record: [H][d][dv] float32.  Everything after the projections is float32, but that an
+// activated q, k or v of bfloat16 rows is rounded to bfloat16 again, in every path alike, so
+// that the tensor cores can take it (below).
 //
 // Requests [0, n_decode) bring one token each: la_token reads and writes every state element
 // once.  The others' portions are cut into chunks of 64 tokens, counted from the portion's
@@ -27,18 +28,35 @@
 // e^(B_(before I) - B_(end of J)) from a table, and e^(B_(end of J) - B_j) on k; a pair inside a
 // group takes the exponential of its own difference for every channel.
 //   finish  the norm, weight and gate.
+//
+// bfloat16 rows with d and dv in multiples of 16 (d up to 128) take the tensor-core forms of `state`
+// and `out`.  Their float32 operands (the state, the scores, everything multiplied by a decay) go
+// through the bfloat16 product without being rounded: x = x1 + x2 + x3, each part the
+// bfloat16 nearest to what is left, holds all 24 bits, so x times a bfloat16 is three exact
+// products added in float32, and a product of two such sums is the six of its nine products that
+// reach a float32's last bits.  There a chunk's pairs take q_i e^(B_i) and k_j e^(-B_j), as long
+// as no channel's B_L lies below -40 (then no factor leaves float32's range by far); a chunk with a
+// stronger decay takes the exponential of every pair's own difference instead.
 // Plain reference: tests/plain_ops.py linear_attention.
 #include "common.cuh"
+#include "mma_bf16.cuh"
 
 #define LA_C 64             // tokens a chunk
 #define LA_T 64             // columns (and rows) of a tile
 #define LA_DK 32            // key channels staged at a time in `out`
 #define LA_LD 68            // padded row of 64
 #define LA_G 8              // tokens a group
+#define LA_SCAN_THREADS 64
 #define LA_NG 8             // groups a chunk
 
 __device__ __forceinline__ float la_logsigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float la_act(float x, int act) { return act ? x / (1.f + expf(-x)) : x; }
+__device__ __forceinline__ float la_silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+// a projection as the recurrence reads it
+__device__ __forceinline__ float la_in(const float* p, int act) { return act ? *p / (1.f + expf(-*p)) : *p; }
+__device__ __forceinline__ float la_in(const bf16* p, int act) {
+    const float x = __bfloat162float(*p);
+    return act ? __bfloat162float(__float2bfloat16_rn(la_silu(x))) : x;
+}
 
 // Chunk `item` of the portions of requests [first_req, n_reqs): its request and its number there;
 // and how many chunks lie before the request.  Requests without a slot have none.  Whole warp.
@@ -70,9 +88,9 @@ __device__ __forceinline__ bool la_find(const int* q_start, const int* state_slo
 
 // ---- single tokens ---------------------------------------------------------------------
 // V = 4: 16-byte accesses to the state and sixteen lanes across a tile's 64 columns; V = 1: 64.
-template <int V>
+template <typename T, int V>
 __global__ void __launch_bounds__(128) la_token_kernel(
-    const float* __restrict__ rows, int stride, const float* __restrict__ log_decay,
+    const T* __restrict__ rows, int stride, const float* __restrict__ z, const float* __restrict__ log_decay,
     const float* __restrict__ bias, float tau, const int* __restrict__ q_start,
     const int* __restrict__ state_slot, float* __restrict__ state, float* __restrict__ num, int H,
     int d, int dv, int act, float q_scale) {
@@ -88,13 +106,12 @@ __global__ void __launch_bounds__(128) la_token_kernel(
     const int t = q_start[r];
     rv_pdl_wait();
     if (slot < 0) return;
-    const float* row = rows + (size_t)t * stride;
+    const T* row = rows + (size_t)t * stride;
     const float ad = log_decay ? expf(log_decay[h]) : 0.f;
     for (int i = threadIdx.x; i < d; i += 128) {
-        qs[i] = la_act(row[h * d + i], act) * q_scale;
-        ks[i] = la_act(row[(H + h) * d + i], act);
-        as[i] = log_decay ? ad
-                          : expf(la_logsigmoid(row[2 * H * d + 2 * H * dv + h * d + i] + bias[h * d + i]) / tau);
+        qs[i] = la_in(row + h * d + i, act);
+        ks[i] = la_in(row + (H + h) * d + i, act);
+        as[i] = log_decay ? ad : expf(la_logsigmoid(z[(size_t)t * H * d + h * d + i] + bias[h * d + i]) / tau);
     }
     const int cl = threadIdx.x % LANES, rg = threadIdx.x / LANES;
     const int col = blockIdx.x * LA_T + cl * V;
@@ -102,7 +119,7 @@ __global__ void __launch_bounds__(128) la_token_kernel(
 #pragma unroll
     for (int e = 0; e < V; ++e) {
         o[e] = 0.f;
-        v[e] = col + e < dv ? la_act(row[2 * H * d + h * dv + col + e], act) : 0.f;
+        v[e] = col + e < dv ? la_in(row + 2 * H * d + h * dv + col + e, act) : 0.f;
     }
     __syncthreads();
     float* S = state + ((size_t)slot * H + h) * d * dv;
@@ -137,14 +154,14 @@ __global__ void __launch_bounds__(128) la_token_kernel(
         float s = 0.f;
 #pragma unroll
         for (int g = 0; g < RG; ++g) s += red[g * LA_T + c];
-        num[((size_t)t * H + h) * dv + blockIdx.x * LA_T + c] = s;
+        num[((size_t)t * H + h) * dv + blockIdx.x * LA_T + c] = s * q_scale;
     }
 }
 
 // ---- portions: every chunk's own contribution to the state ----------------------------------
-template <bool CHANNEL>
+template <typename T, bool CHANNEL>
 __global__ void __launch_bounds__(256) la_state_kernel(
-    const float* __restrict__ rows, int stride, const float* __restrict__ log_decay,
+    const T* __restrict__ rows, int stride, const float* __restrict__ zr, const float* __restrict__ log_decay,
     const float* __restrict__ bias, float tau, const int* __restrict__ q_start,
     const int* __restrict__ state_slot, int first_req, int n_reqs, float* __restrict__ kv,
     float* __restrict__ dec, int H, int d, int dv, int act) {
@@ -173,22 +190,21 @@ __global__ void __launch_bounds__(256) la_state_kernel(
     if (t0 < 0) return;
     const int x = tid & 63, y = tid >> 6;
     const int dn = min(LA_T, d - d0), vn = min(LA_T, dv - v0);
-    const float* base = rows + (size_t)t0 * stride;
+    const T* base = rows + (size_t)t0 * stride;
     const float ld = CHANNEL ? 0.f : log_decay[h];
     const float bz = CHANNEL && x < dn ? bias[h * d + d0 + x] : 0.f;
     // four values of one column at a time are requested before any is worked on
 #pragma unroll 4
     for (int j = y; j < LA_C; j += 4) {
-        const float* row = base + (size_t)j * stride;
+        const T* row = base + (size_t)j * stride;
         const bool tj = j < L;
-        float k = tj && x < dn ? row[(H + h) * d + d0 + x] : 0.f;
-        const float v = tj && x < vn ? row[2 * H * d + h * dv + v0 + x] : 0.f;
-        k = la_act(k, act);
+        float k = tj && x < dn ? la_in(row + (H + h) * d + d0 + x, act) : 0.f;
+        const float v = tj && x < vn ? la_in(row + 2 * H * d + h * dv + v0 + x, act) : 0.f;
         if (!CHANNEL) k *= expf(ld * (float)(L - 1 - min(j, L - 1)));
         ks[j * LA_LD + x] = k;
-        vs[j * LA_LD + x] = la_act(v, act);
+        vs[j * LA_LD + x] = v;
         if (CHANNEL) {
-            const float z = tj && x < dn ? row[2 * H * d + 2 * H * dv + h * d + d0 + x] : 0.f;
+            const float z = tj && x < dn ? zr[(size_t)(t0 + j) * H * d + h * d + d0 + x] : 0.f;
             lb[j * LA_LD + x] = tj && x < dn ? la_logsigmoid(z + bz) / tau : 0.f;
         }
     }
@@ -245,7 +261,7 @@ __global__ void __launch_bounds__(256) la_state_kernel(
 
 // ---- portions: the states between the chunks ---------------------------------------------------
 template <bool CHANNEL, int V>
-__global__ void __launch_bounds__(256) la_scan_kernel(
+__global__ void __launch_bounds__(LA_SCAN_THREADS) la_scan_kernel(
     const float* __restrict__ log_decay, const int* __restrict__ q_start,
     const int* __restrict__ state_slot, int first_req, float* __restrict__ kv,
     const float* __restrict__ dec, float* __restrict__ state, int H, int d, int dv) {
@@ -265,7 +281,7 @@ __global__ void __launch_bounds__(256) la_scan_kernel(
     const int last_len = q_start[r + 1] - q_start[r] - (n - 1) * LA_C;
     const float ld = CHANNEL ? 0.f : log_decay[h];
     rv_pdl_wait();
-    const long long el = ((long long)blockIdx.x * 256 + threadIdx.x) * V;
+    const long long el = ((long long)blockIdx.x * LA_SCAN_THREADS + threadIdx.x) * V;
     if (n == 0 || el >= (long long)d * dv) return;
     const int ch = (int)(el / dv);
     float* rec = state + ((size_t)slot * H + h) * d * dv + el;
@@ -282,7 +298,7 @@ __global__ void __launch_bounds__(256) la_scan_kernel(
     } else {
         S[0] = *rec;
     }
-    constexpr int U = 4;                                         // chunks requested together
+    constexpr int U = 8;                                         // chunks requested together
     for (int c0 = 0; c0 < n; c0 += U) {
         float in[U][V], a[U];
 #pragma unroll
@@ -315,9 +331,9 @@ __global__ void __launch_bounds__(256) la_scan_kernel(
 // A thread's share of a 64 x 64 product is rows 4 ty .. + 3 by columns 4 tx .. + 3; a warp's eight
 // rows are one group.  Operands lie with the summed index first ([c][64 tokens] and so on), so that
 // a thread reads four of its rows and four of its columns with one access each.
-template <bool CHANNEL>
+template <typename T, bool CHANNEL>
 __global__ void __launch_bounds__(256) la_out_kernel(
-    const float* __restrict__ rows, int stride, const float* __restrict__ log_decay,
+    const T* __restrict__ rows, int stride, const float* __restrict__ zr, const float* __restrict__ log_decay,
     const float* __restrict__ bias, float tau, const int* __restrict__ q_start,
     const int* __restrict__ state_slot, int first_req, int n_reqs, const float* __restrict__ kv,
     float* __restrict__ num, int H, int d, int dv, int act, float q_scale) {
@@ -349,7 +365,7 @@ __global__ void __launch_bounds__(256) la_out_kernel(
     const int t0 = at[0], L = at[1];
     rv_pdl_wait();
     if (t0 < 0) return;
-    const float* base = rows + (size_t)t0 * stride;
+    const T* base = rows + (size_t)t0 * stride;
     const float* Sg = kv + ((size_t)item * H + h) * d * dv;
     const int vn = min(LA_T, dv - v0);
     const int ty = tid >> 4, tx = tid & 15;
@@ -359,7 +375,7 @@ __global__ void __launch_bounds__(256) la_out_kernel(
         const int x = tid & 63, y = tid >> 6;
 #pragma unroll 4
         for (int j = y; j < LA_C; j += 4)
-            vs[j * LA_LD + x] = j < L && x < vn ? la_act(base[(size_t)j * stride + 2 * H * d + h * dv + v0 + x], act) : 0.f;
+            vs[j * LA_LD + x] = j < L && x < vn ? la_in(base + (size_t)j * stride + 2 * H * d + h * dv + v0 + x, act) : 0.f;
     }
     float p[4][4], o[4][4];
 #pragma unroll
@@ -392,13 +408,13 @@ __global__ void __launch_bounds__(256) la_out_kernel(
             for (int u = warp; u < (LA_C / 4) * (LA_DK / 8); u += 8) {
                 const int j = (u >> 2) * 4 + tl, c = (u & 3) * 8 + cl;
                 const bool in = j < L && c < cn;
-                const float* row = base + (size_t)j * stride + h * d + c0 + c;
-                const float q = in ? la_act(row[0], act) * q_scale : 0.f;
-                const float k = in ? la_act(row[(size_t)H * d], act) : 0.f;
+                const T* row = base + (size_t)j * stride + h * d + c0 + c;
+                const float q = in ? la_in(row, act) : 0.f;
+                const float k = in ? la_in(row + (size_t)H * d, act) : 0.f;
                 if (CHANNEL) {
                     qr[c * LA_LD + j] = q;
                     kr[c * LA_LD + j] = k;
-                    lb[c * LA_LD + j] = in ? la_logsigmoid(row[(size_t)2 * H * d + 2 * H * dv] + bias[h * d + c0 + c]) / tau : 0.f;
+                    lb[c * LA_LD + j] = in ? la_logsigmoid(zr[(size_t)(t0 + j) * H * d + h * d + c0 + c] + bias[h * d + c0 + c]) / tau : 0.f;
                 } else {
                     qt[c * LA_LD + j] = q;
                     kt[c * LA_LD + j] = k;
@@ -522,6 +538,8 @@ __global__ void __launch_bounds__(256) la_out_kernel(
     for (int i = 0; i < 4; ++i) {
         const int ri = 4 * ty + i;
         if (ri >= L) continue;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[i][e] *= q_scale;
         float* dst = num + ((size_t)(t0 + ri) * H + h) * dv + v0 + 4 * tx;
         if (dv % 4 == 0) {
             if (4 * tx < vn) *(float4*)dst = make_float4(o[i][0], o[i][1], o[i][2], o[i][3]);
@@ -538,9 +556,48 @@ __device__ __forceinline__ float la_gate(float g, int gate) {
     return (gate ? g : 1.f) / (1.f + expf(-g));                  // 0: sigmoid, 1: silu
 }
 
+// Four neighbouring values (16- and 8-byte accesses) or one.
+template <typename T, int V>
+__device__ __forceinline__ void la_load(const T* p, float (&x)[V]) {
+    if (V == 4 && sizeof(T) == 4) {
+        const float4 f = *(const float4*)p;
+        x[0] = f.x; x[1 % V] = f.y; x[2 % V] = f.z; x[3 % V] = f.w;
+    } else if (V == 4) {
+        const uint2 u = *(const uint2*)p;
+        const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&u.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&u.y);
+        x[0] = a.x; x[1 % V] = a.y; x[2 % V] = b.x; x[3 % V] = b.y;
+    } else {
+        x[0] = rv_load(p);
+    }
+}
+template <typename T, int V>
+__device__ __forceinline__ void la_store(T* p, const float (&x)[V]) {
+    if (V == 4 && sizeof(T) == 4) {
+        *(float4*)p = make_float4(x[0], x[1 % V], x[2 % V], x[3 % V]);
+    } else if (V == 4) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(x[0], x[1 % V]), b = __floats2bfloat162_rn(x[2 % V], x[3 % V]);
+        uint2 u;
+        u.x = *(const unsigned*)&a;
+        u.y = *(const unsigned*)&b;
+        *(uint2*)p = u;
+    } else {
+        rv_store(p, x[0]);
+    }
+}
+template <typename T, int V>
+__device__ __forceinline__ void la_finish_at(const float* nm, const T* g, const float* w, T* o, int c, float rms, int gate) {
+    float x[V], y[V], z[V];
+    la_load<float, V>(nm + c, x);
+    la_load<T, V>(g + c, y);
+    la_load<float, V>(w + c, z);
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[e] = x[e] / rms * z[e] * la_gate(y[e], gate);
+    la_store<T, V>(o + c, x);
+}
+
 // One norm over all heads: a block per token.
-template <typename T>
-__global__ void la_finish_all_kernel(const float* __restrict__ num, const float* __restrict__ rows,
+template <typename T, int V>
+__global__ void la_finish_all_kernel(const float* __restrict__ num, const T* __restrict__ rows,
                                      int stride, int g_off, const float* __restrict__ norm_w, float eps,
                                      const int* __restrict__ token_req, const int* __restrict__ state_slot,
                                      T* __restrict__ out, int width, int gate) {
@@ -555,17 +612,21 @@ __global__ void la_finish_all_kernel(const float* __restrict__ num, const float*
         return;
     }
     const float* nm = num + (size_t)t * width;
-    const float* g = rows + (size_t)t * stride + g_off;
     float ss = 0.f;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) ss += nm[c] * nm[c];
+    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+        float x[V];
+        la_load<float, V>(nm + c, x);
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss += x[e] * x[e];
+    }
     const float rms = sqrtf(rv_block_sum(ss, scratch) / (float)width + eps);
-    for (int c = threadIdx.x; c < width; c += blockDim.x)
-        rv_store(o + c, nm[c] / rms * norm_w[c] * la_gate(g[c], gate));
+    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V)
+        la_finish_at<T, V>(nm, rows + (size_t)t * stride + g_off, norm_w, o, c, rms, gate);
 }
 
 // A norm per head: a warp per (token, head).
-template <typename T>
-__global__ void la_finish_head_kernel(const float* __restrict__ num, const float* __restrict__ rows,
+template <typename T, int V>
+__global__ void la_finish_head_kernel(const float* __restrict__ num, const T* __restrict__ rows,
                                       int stride, int g_off, const float* __restrict__ norm_w, float eps,
                                       const int* __restrict__ token_req, const int* __restrict__ state_slot,
                                       T* __restrict__ out, int n_tokens, int H, int dv, int gate) {
@@ -582,13 +643,19 @@ __global__ void la_finish_head_kernel(const float* __restrict__ num, const float
         return;
     }
     const float* nm = num + ((size_t)t * H + h) * dv;
-    const float* g = rows + (size_t)t * stride + g_off + h * dv;
-    const float* wt = norm_w + h * dv;
     float ss = 0.f;
-    for (int c = lane; c < dv; c += 32) ss += nm[c] * nm[c];
+    for (int c = lane * V; c < dv; c += 32 * V) {
+        float x[V];
+        la_load<float, V>(nm + c, x);
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss += x[e] * x[e];
+    }
     const float rms = sqrtf(rv_warp_sum(ss) / (float)dv + eps);
-    for (int c = lane; c < dv; c += 32) rv_store(o + c, nm[c] / rms * wt[c] * la_gate(g[c], gate));
+    for (int c = lane * V; c < dv; c += 32 * V)
+        la_finish_at<T, V>(nm, rows + (size_t)t * stride + g_off + h * dv, norm_w + h * dv, o, c, rms, gate);
 }
+
+#include "linear_attention_mma.cuh"
 
 // ---------------------------------------------------------------------------------
 // The most chunks the portions of `n_tokens` tokens in `n_reqs` requests can have.
@@ -603,101 +670,165 @@ extern "C" long long rv_linear_attention_scratch(int n_tokens, int n_decode, int
     return f;
 }
 
-// log_decay [H] or null; then bias [H d] and z at the end of the rows.  act: 1 silu; norm_head: 0 all
+struct LaArgs {
+    const float *z, *log_decay, *bias, *norm_w;
+    float *state, *scratch;
+    const int *token_req, *q_start, *state_slot;
+    float tau, q_scale, eps;
+    int stride, n_tokens, n_decode, n_reqs, H, d, dv, act, norm_head, gate, tensor;
+};
+
+#define LA_SMEM(kernel, bytes)                                                                       \
+    {                                                                                                \
+        static size_t have = 48 * 1024;                                                              \
+        if ((bytes) > have) {                                                                        \
+            if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,            \
+                                     (int)(bytes)) != cudaSuccess)                                   \
+                RV_FAIL("linear_attention: %zu bytes of shared memory are not to be had", (size_t)(bytes)); \
+            have = (bytes);                                                                          \
+        }                                                                                            \
+    }
+
+// The tensor-core forms exist for bfloat16 rows.
+template <bool CH>
+static int la_tensor_launch(const float* rows, const LaArgs& a, int what, dim3 grid, float* kv, float* dec,
+                            float* num, cudaStream_t s) {
+    (void)rows; (void)a; (void)what; (void)grid; (void)kv; (void)dec; (void)num; (void)s;
+    RV_FAIL("linear_attention: float32 rows on the tensor cores");
+}
+template <bool CH>
+static int la_tensor_launch(const bf16* rows, const LaArgs& a, int what, dim3 grid, float* kv, float* dec,
+                            float* num, cudaStream_t s) {
+    if (what == 0) {
+        const size_t smem = lm_state_smem(CH);
+        LA_SMEM(la_state_mma_kernel<CH>, smem)
+        rv_launch(la_state_mma_kernel<CH>, grid, dim3(128), smem, s, rows, a.stride, a.z, a.log_decay, a.bias,
+                  a.tau, a.q_start, a.state_slot, a.n_decode, a.n_reqs, kv, dec, a.H, a.d, a.dv, a.act);
+    } else {
+        const size_t smem = lm_out_smem(CH, a.d);
+        LA_SMEM(la_out_mma_kernel<CH>, smem)
+        rv_launch(la_out_mma_kernel<CH>, grid, dim3(128), smem, s, rows, a.stride, a.z, a.log_decay, a.bias,
+                  a.tau, a.q_start, a.state_slot, a.n_decode, a.n_reqs, (const float*)kv, num, a.H, a.d, a.dv,
+                  a.act, a.q_scale);
+    }
+    return 0;
+}
+
+template <typename T, bool CH>
+static int la_portions(const T* rows, const LaArgs& a, float* num, float* kv, float* dec, unsigned items,
+                       cudaStream_t s) {
+    const int tiles_d = (a.d + LA_T - 1) / LA_T, tiles_v = (a.dv + LA_T - 1) / LA_T;
+    const dim3 g1(items, a.H, tiles_d * tiles_v), g3(items, a.H, tiles_v);
+    if (a.tensor) {
+        if (la_tensor_launch<CH>(rows, a, 0, g1, kv, dec, num, s)) return 1;
+    } else {
+        const size_t smem = (size_t)((CH ? 3 : 2) * LA_C * LA_LD + 4 * 64) * sizeof(float);
+        auto kernel = la_state_kernel<T, CH>;
+        LA_SMEM(kernel, smem)
+        rv_launch(kernel, g1, dim3(256), smem, s, rows, a.stride, a.z, a.log_decay, a.bias, a.tau, a.q_start,
+                  a.state_slot, a.n_decode, a.n_reqs, kv, dec, a.H, a.d, a.dv, a.act);
+    }
+    RV_CHECK_LAUNCH("linear_attention_state");
+    const bool v4 = a.dv % 4 == 0 && ((uintptr_t)a.state & 15) == 0;
+    const long long per = LA_SCAN_THREADS * (v4 ? 4 : 1);
+    const dim3 g2((unsigned)(((long long)a.d * a.dv + per - 1) / per), a.H, a.n_reqs - a.n_decode);
+    if (v4)
+        rv_launch(la_scan_kernel<CH, 4>, g2, dim3(LA_SCAN_THREADS), 0, s, a.log_decay, a.q_start, a.state_slot,
+                  a.n_decode, kv, dec, a.state, a.H, a.d, a.dv);
+    else
+        rv_launch(la_scan_kernel<CH, 1>, g2, dim3(LA_SCAN_THREADS), 0, s, a.log_decay, a.q_start, a.state_slot,
+                  a.n_decode, kv, dec, a.state, a.H, a.d, a.dv);
+    RV_CHECK_LAUNCH("linear_attention_scan");
+    if (a.tensor) {
+        if (la_tensor_launch<CH>(rows, a, 1, g3, kv, dec, num, s)) return 1;
+    } else {
+        const size_t smem = (size_t)((CH ? 6 : 3) * LA_DK * LA_LD + 2 * LA_C * LA_LD +
+                                     (CH ? (LA_NG + 1 + LA_NG * LA_NG) * (LA_DK + 1) : 0)) * sizeof(float);
+        auto kernel = la_out_kernel<T, CH>;
+        LA_SMEM(kernel, smem)
+        rv_launch(kernel, g3, dim3(256), smem, s, rows, a.stride, a.z, a.log_decay, a.bias, a.tau, a.q_start,
+                  a.state_slot, a.n_decode, a.n_reqs, (const float*)kv, num, a.H, a.d, a.dv, a.act, a.q_scale);
+    }
+    RV_CHECK_LAUNCH("linear_attention_out");
+    return 0;
+}
+
+template <typename T>
+static int la_run(const T* rows, const LaArgs& a, T* out, cudaStream_t s) {
+    float* num = a.scratch;
+    if (a.n_decode > 0) {
+        const bool v4 = a.dv % 4 == 0 && ((uintptr_t)a.state & 15) == 0;
+        const size_t smem = (size_t)(3 * a.d + (v4 ? 8 : 2) * LA_T) * sizeof(float);
+        const dim3 grid((a.dv + LA_T - 1) / LA_T, a.H, a.n_decode);
+        if (v4)
+            rv_launch(la_token_kernel<T, 4>, grid, dim3(128), smem, s, rows, a.stride, a.z, a.log_decay, a.bias,
+                      a.tau, a.q_start, a.state_slot, a.state, num, a.H, a.d, a.dv, a.act, a.q_scale);
+        else
+            rv_launch(la_token_kernel<T, 1>, grid, dim3(128), smem, s, rows, a.stride, a.z, a.log_decay, a.bias,
+                      a.tau, a.q_start, a.state_slot, a.state, num, a.H, a.d, a.dv, a.act, a.q_scale);
+        RV_CHECK_LAUNCH("linear_attention_token");
+    }
+    if (a.n_tokens > a.n_decode && a.n_reqs > a.n_decode) {
+        const long long items = la_items(a.n_tokens - a.n_decode, a.n_reqs - a.n_decode);
+        float* kv = a.scratch + (((size_t)a.n_tokens * a.H * a.dv + 3) & ~(size_t)3);
+        float* dec = kv + (size_t)items * a.H * a.d * a.dv;
+        if (items > 0x7fffffffLL) RV_FAIL("linear_attention: too many tokens");
+        if (a.log_decay ? la_portions<T, false>(rows, a, num, kv, dec, (unsigned)items, s)
+                        : la_portions<T, true>(rows, a, num, kv, dec, (unsigned)items, s))
+            return 1;
+    }
+    const int g_off = 2 * a.H * a.d + a.H * a.dv;
+    // four values an access: every row, head, weight and gate begins on such a boundary
+    const bool vec = a.dv % 4 == 0 && g_off % 4 == 0 && a.stride % 4 == 0 &&
+                     (((uintptr_t)rows | (uintptr_t)out | (uintptr_t)a.norm_w) & 15) == 0;
+    if (a.norm_head) {
+        const long long blocks = ((long long)a.n_tokens * a.H + 3) / 4;
+        if (blocks > 0x7fffffffLL) RV_FAIL("linear_attention: too many tokens");
+        if (vec)
+            rv_launch(la_finish_head_kernel<T, 4>, dim3((int)blocks), dim3(128), 0, s, (const float*)num, rows,
+                      a.stride, g_off, a.norm_w, a.eps, a.token_req, a.state_slot, out, a.n_tokens, a.H, a.dv, a.gate);
+        else
+            rv_launch(la_finish_head_kernel<T, 1>, dim3((int)blocks), dim3(128), 0, s, (const float*)num, rows,
+                      a.stride, g_off, a.norm_w, a.eps, a.token_req, a.state_slot, out, a.n_tokens, a.H, a.dv, a.gate);
+    } else {
+        const int width = a.H * a.dv;
+        const dim3 threads(width >= 1024 ? 256 : 128);
+        if (vec)
+            rv_launch(la_finish_all_kernel<T, 4>, dim3(a.n_tokens), threads, 0, s, (const float*)num, rows,
+                      a.stride, g_off, a.norm_w, a.eps, a.token_req, a.state_slot, out, width, a.gate);
+        else
+            rv_launch(la_finish_all_kernel<T, 1>, dim3(a.n_tokens), threads, 0, s, (const float*)num, rows,
+                      a.stride, g_off, a.norm_w, a.eps, a.token_req, a.state_slot, out, width, a.gate);
+    }
+    RV_CHECK_LAUNCH("linear_attention_finish");
+    return 0;
+}
+
+// log_decay [H]; or null, then z float32 [n, H d], bias [H d] and tau.  act: 1 silu; norm_head: 0 all
 // heads together, 1 per head; gate: 0 sigmoid, 1 silu; norm_w [H dv].  Requests [0, n_decode) bring
-// one token each (token r is request r's).
-extern "C" int rv_linear_attention(const float* rows, int stride, const float* log_decay,
-                                   const float* bias, float tau, const float* norm_w, float* state,
-                                   const int* token_req, const int* q_start, const int* state_slot,
-                                   float* scratch, void* out, int out_dtype, int n_tokens, int n_decode,
-                                   int n_reqs, int H, int d, int dv, int act, float q_scale,
-                                   int norm_head, int gate, float eps, void* stream) {
+// one token each (token r is request r's).  `tensor`: whether portions may take the tensor-core
+// forms (where their sizes allow).  rows and out have the type `dtype`.
+extern "C" int rv_linear_attention(const void* rows, int dtype, int stride, const float* z,
+                                   const float* log_decay, const float* bias, float tau,
+                                   const float* norm_w, float* state, const int* token_req,
+                                   const int* q_start, const int* state_slot, float* scratch, void* out,
+                                   int n_tokens, int n_decode, int n_reqs, int H, int d, int dv, int act,
+                                   float q_scale, int norm_head, int gate, float eps, int tensor,
+                                   void* stream) {
     if (n_tokens == 0 || n_reqs == 0) return 0;
     if (n_tokens < 0 || n_decode < 0 || n_decode > n_reqs || n_decode > n_tokens || H < 1 || d < 1 || dv < 1)
         RV_FAIL("linear_attention: bad sizes");
-    if (!log_decay && (!bias || !(tau > 0.f))) RV_FAIL("linear_attention: neither a decay nor a bias and tau");
-    if (stride < 2 * H * d + 2 * H * dv + (log_decay ? 0 : H * d)) RV_FAIL("linear_attention: rows are too short");
-    if (n_reqs > 65535 || H > 65535 || d > 2048 || dv > 65535) RV_FAIL("linear_attention: too many requests or heads");
-    if ((uintptr_t)scratch & 15) RV_FAIL("linear_attention: the scratch must be 16-byte aligned");
-    cudaStream_t s = (cudaStream_t)stream;
+    if (!log_decay && (!z || !bias || !(tau > 0.f))) RV_FAIL("linear_attention: neither a decay nor z, a bias and tau");
+    if (stride < 2 * H * d + 2 * H * dv) RV_FAIL("linear_attention: rows are too short");
     const int tiles_d = (d + LA_T - 1) / LA_T, tiles_v = (dv + LA_T - 1) / LA_T;
-    float* num = scratch;
-    const bool v4 = dv % 4 == 0 && ((uintptr_t)state & 15) == 0;
-    if (n_decode > 0) {
-        const size_t smem = (size_t)(3 * d + (v4 ? 8 : 2) * LA_T) * sizeof(float);
-        const dim3 grid(tiles_v, H, n_decode);
-        if (v4)
-            rv_launch(la_token_kernel<4>, grid, dim3(128), smem, s, rows, stride, log_decay, bias, tau,
-                      q_start, state_slot, state, num, H, d, dv, act, q_scale);
-        else
-            rv_launch(la_token_kernel<1>, grid, dim3(128), smem, s, rows, stride, log_decay, bias, tau,
-                      q_start, state_slot, state, num, H, d, dv, act, q_scale);
-        RV_CHECK_LAUNCH("linear_attention_token");
-    }
-    if (n_tokens > n_decode && n_reqs > n_decode) {
-        const long long items = la_items(n_tokens - n_decode, n_reqs - n_decode);
-        float* kv = scratch + (((size_t)n_tokens * H * dv + 3) & ~(size_t)3);
-        float* dec = kv + (size_t)items * H * d * dv;
-        if (tiles_d * tiles_v > 65535 || items > 0x7fffffffLL) RV_FAIL("linear_attention: heads are too large");
-        const bool ch = log_decay == nullptr;
-        const size_t sm1 = (size_t)((ch ? 3 : 2) * LA_C * LA_LD + 4 * 64) * sizeof(float);
-        const size_t sm3 = (size_t)((ch ? 6 : 3) * LA_DK * LA_LD + 2 * LA_C * LA_LD +
-                                    (ch ? (LA_NG + 1 + LA_NG * LA_NG) * (LA_DK + 1) : 0)) * sizeof(float);
-        static bool configured = false;
-        if (!configured) {
-            const int big = 128 * 1024;
-            if (cudaFuncSetAttribute(la_state_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, big) != cudaSuccess ||
-                cudaFuncSetAttribute(la_state_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big) != cudaSuccess ||
-                cudaFuncSetAttribute(la_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, big) != cudaSuccess ||
-                cudaFuncSetAttribute(la_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big) != cudaSuccess)
-                RV_FAIL("linear_attention: %d bytes of shared memory are not to be had", big);
-            configured = true;
-        }
-        const int first = n_decode, np = n_reqs - n_decode;
-        const dim3 g1((unsigned)items, H, tiles_d * tiles_v), g3((unsigned)items, H, tiles_v);
-        const long long el = (long long)d * dv;
-        const dim3 g2((unsigned)((el + 256 * (v4 ? 4 : 1) - 1) / (256 * (v4 ? 4 : 1))), H, np);
-        if (ch) {
-            rv_launch(la_state_kernel<true>, g1, dim3(256), sm1, s, rows, stride, log_decay, bias, tau, q_start,
-                      state_slot, first, n_reqs, kv, dec, H, d, dv, act);
-            if (v4)
-                rv_launch(la_scan_kernel<true, 4>, g2, dim3(256), 0, s, log_decay, q_start, state_slot, first,
-                          kv, dec, state, H, d, dv);
-            else
-                rv_launch(la_scan_kernel<true, 1>, g2, dim3(256), 0, s, log_decay, q_start, state_slot, first,
-                          kv, dec, state, H, d, dv);
-            rv_launch(la_out_kernel<true>, g3, dim3(256), sm3, s, rows, stride, log_decay, bias, tau, q_start,
-                      state_slot, first, n_reqs, (const float*)kv, num, H, d, dv, act, q_scale);
-        } else {
-            rv_launch(la_state_kernel<false>, g1, dim3(256), sm1, s, rows, stride, log_decay, bias, tau, q_start,
-                      state_slot, first, n_reqs, kv, dec, H, d, dv, act);
-            if (v4)
-                rv_launch(la_scan_kernel<false, 4>, g2, dim3(256), 0, s, log_decay, q_start, state_slot, first,
-                          kv, dec, state, H, d, dv);
-            else
-                rv_launch(la_scan_kernel<false, 1>, g2, dim3(256), 0, s, log_decay, q_start, state_slot, first,
-                          kv, dec, state, H, d, dv);
-            rv_launch(la_out_kernel<false>, g3, dim3(256), sm3, s, rows, stride, log_decay, bias, tau, q_start,
-                      state_slot, first, n_reqs, (const float*)kv, num, H, d, dv, act, q_scale);
-        }
-        RV_CHECK_LAUNCH("linear_attention");
-    }
-    const int g_off = 2 * H * d + H * dv;
-    if (norm_head) {
-        const long long blocks = ((long long)n_tokens * H + 3) / 4;
-        if (blocks > 0x7fffffffLL) RV_FAIL("linear_attention: too many tokens");
-        RV_DISPATCH_DTYPE(out_dtype, "linear_attention",
-                          (rv_launch(la_finish_head_kernel<T>, dim3((int)blocks), dim3(128), 0, s,
-                                     (const float*)num, rows, stride, g_off, norm_w, eps, token_req,
-                                     state_slot, (T*)out, n_tokens, H, dv, gate)));
-    } else {
-        const int width = H * dv;
-        const int threads = width >= 1024 ? 256 : 128;
-        RV_DISPATCH_DTYPE(out_dtype, "linear_attention",
-                          (rv_launch(la_finish_all_kernel<T>, dim3(n_tokens), dim3(threads), 0, s,
-                                     (const float*)num, rows, stride, g_off, norm_w, eps, token_req,
-                                     state_slot, (T*)out, width, gate)));
-    }
-    RV_CHECK_LAUNCH("linear_attention_finish");
+    if (n_reqs > 65535 || H > 65535 || d > 2048 || dv > 65535 || tiles_d * tiles_v > 65535)
+        RV_FAIL("linear_attention: too many requests or heads, or heads that are too large");
+    if ((uintptr_t)scratch & 15) RV_FAIL("linear_attention: the scratch must be 16-byte aligned");
+    tensor = tensor && dtype == RV_DTYPE_BF16 && d % 16 == 0 && dv % 16 == 0 && d <= 128 && stride % 8 == 0 &&
+             ((uintptr_t)rows & 15) == 0;
+    const LaArgs a = {z, log_decay, bias, norm_w, state, scratch, token_req, q_start, state_slot, tau, q_scale, eps,
+                      stride, n_tokens, n_decode, n_reqs, H, d, dv, act, norm_head, gate, tensor};
+    RV_DISPATCH_DTYPE(dtype, "linear_attention",
+                      return la_run<T>((const T*)rows, a, (T*)out, (cudaStream_t)stream));
     return 0;
 }

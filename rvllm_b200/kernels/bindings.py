@@ -95,6 +95,9 @@ class CudaOps:
         # grouped from `moe_grouped_min` (token, expert) pairs on
         self.moe_mode = os.environ.get("RVLLM_MOE", "auto")
         self.moe_grouped_min = int(os.environ.get("RVLLM_MOE_GROUPED_MIN", "16"))
+        # portions of bfloat16 linear attention: "tensor" = tensor-core kernels where the sizes allow
+        # (head sizes in multiples of 16, keys up to 128), "simt" = float32 arithmetic
+        self.linear_attention_mode = os.environ.get("RVLLM_LINEAR_ATTENTION", "tensor")
         # float32 products must be float32: no TF32, no reduced-precision accumulation
         torch.backends.cuda.matmul.allow_tf32 = False
         torch.backends.cudnn.allow_tf32 = False
@@ -1430,18 +1433,22 @@ class CudaOps:
 
     # ---- linear attention with decay -----------------------------------------------------------
 
-    def linear_attention(self, rows, log_decay, decay_bias, tau, norm_w, state, ctx, out, heads, dim,
-                         vdim, activation, q_scale, norm, gate, eps):
+    def linear_attention(self, rows, z, log_decay, decay_bias, tau, norm_w, state, ctx, out, heads,
+                         dim, vdim, activation, q_scale, norm, gate, eps):
         """Linear attention over the step's tokens; see csrc/linear_attention.cu for the layout of
-        `rows` (q | k | v | g (| z), float32) and of the record [heads, dim, vdim].  `log_decay`
-        float32 [heads], or None: decays by token and channel from z, `decay_bias` and `tau`."""
-        for t, what in ((rows, "projection rows"), (log_decay, "decays"),
+        `rows` (q | k | v | g) and of the record [heads, dim, vdim].  `log_decay` float32 [heads], or
+        None: decays by token and channel from `z` float32 [n, heads * dim], `decay_bias` and
+        `tau`."""
+        for t, what in ((z, "decay rows"), (log_decay, "decays"),
                         (decay_bias, "decay bias"), (norm_w, "output norm weight"),
                         (state, "state records")):
             if t is not None:
                 self._need(t, what, torch.float32)
-        self._need(out, "mixer output")
+        self._need(rows, "projection rows")
+        self._need(out, "mixer output", rows.dtype)
         n = rows.shape[0]
+        if log_decay is None and (z is None or z.shape != (n, heads * dim)):
+            raise KernelError("linear_attention: decays by channel need a value per token and channel")
         if state.shape[1] != heads * dim * vdim or out.shape != (n, heads * vdim) or \
                 norm_w.shape != (heads * vdim,):
             raise KernelError("linear_attention: the record, the weight or the output has another size")
@@ -1453,13 +1460,15 @@ class CudaOps:
             c_int(n), c_int(ctx.n_decode), c_int(ctx.n_reqs), c_int(heads), c_int(dim), c_int(vdim))
         scratch = torch.empty((need,), dtype=torch.float32, device=rows.device)
         self._check(self.lib.rv_linear_attention(
-            _ptr(rows), c_int(rows.shape[1]), _ptr(log_decay), _ptr(decay_bias), c_float(tau),
-            _ptr(norm_w), _ptr(state), _ptr(ctx.token_req), _ptr(ctx.q_start), _ptr(ctx.state_slot),
-            _ptr(scratch), _ptr(out), _code(out.dtype), c_int(n), c_int(ctx.n_decode),
+            _ptr(rows), _code(rows.dtype), c_int(rows.shape[1]), _ptr(z), _ptr(log_decay),
+            _ptr(decay_bias), c_float(tau), _ptr(norm_w), _ptr(state), _ptr(ctx.token_req),
+            _ptr(ctx.q_start), _ptr(ctx.state_slot), _ptr(scratch), _ptr(out), c_int(n),
+            c_int(ctx.n_decode),
             c_int(ctx.n_reqs), c_int(heads), c_int(dim), c_int(vdim),
             c_int({None: 0, "silu": 1}[activation]), c_float(q_scale),
             c_int({"all": 0, "head": 1}[norm]), c_int({"sigmoid": 0, "silu": 1}[gate]), c_float(eps),
-            self._stream()), "linear_attention")
+            c_int(1 if self.linear_attention_mode == "tensor" else 0), self._stream()),
+            "linear_attention")
         self.launches += (ctx.n_decode > 0) + 3 * (n > ctx.n_decode)
 
     def softcap(self, logits, cap):

@@ -12,12 +12,12 @@ together or per head, and is multiplied by a gate before the output product:
 
 S starts at zero and is the request's record in a state slot: float32 whatever the compute type.
 
-W_q | W_k | W_v | W_g and, for decays made by tokens, W_z are one matrix whose product stays
-float32, so that everything that enters the recurrence is 32-bit.  W_z = W_a2 W_a1 is formed once
-when the weights are loaded: the rank of the two factors saves parameters in the file, but as a
-product of its own it would cost two more launches a layer for a few columns.  Activations,
-decays, recurrence, norm and gate are `ops.linear_attention`, for any mixture of prompt portions
-and single tokens.
+W_q | W_k | W_v | W_g are one matrix, whose product has the compute type.  z = W_z x of decays made
+by tokens is another product whose result stays float32 (decays are 32-bit throughout).  W_z =
+W_a2 W_a1 is formed once when the weights are loaded: the rank of the two factors saves
+parameters in the file, but each is a product of a few columns or a few terms, and two of them
+take longer than the one.  Activations, decays, recurrence, norm and gate are
+`ops.linear_attention`, for any mixture of prompt portions and single tokens.
 """
 from __future__ import annotations
 
@@ -81,10 +81,10 @@ class LinearAttention(Mixer):
         n = self._names(spec)
         q = tensors[n["q"]]
         parts = [tensors[n[k]].to(q.dtype) for k in ("q", "k", "v", "g")]
-        self.log_decay = self.decay_bias = None
+        self.log_decay = self.decay_bias = self.w_z = None
         if spec.decay is None:
             wide = torch.float64
-            parts.append((tensors[n["a2"]].to(wide) @ tensors[n["a1"]].to(wide)).to(q.dtype))
+            self.w_z = (tensors[n["a2"]].to(wide) @ tensors[n["a1"]].to(wide)).to(q.dtype).contiguous()
             self.decay_bias = tensors[n["a2.b"]].to(torch.float32).contiguous()
         else:
             # a decay of 0 forgets everything: e^-1e4 is 0 in float32, without an infinity whose
@@ -102,10 +102,11 @@ class LinearAttention(Mixer):
         if cache is None or not cache.owns:
             raise ValueError("linear_attention: a recurrent state cannot be shared between calls")
         s = self.spec
-        rows = self.ops.linear(normed, self.w_in, out_dtype=torch.float32)
+        rows = self.ops.linear(normed, self.w_in, out_dtype=self.dtype)
+        z = self.ops.linear(normed, self.w_z, out_dtype=torch.float32) if self.w_z is not None else None
         y = self.ops.new_rows(normed.shape[0], s.num_heads * s.v_head_dim, self.dtype,
                               normed.device)
-        self.ops.linear_attention(rows, self.log_decay, self.decay_bias, s.decay_tau, self.norm,
+        self.ops.linear_attention(rows, z, self.log_decay, self.decay_bias, s.decay_tau, self.norm,
                                   cache.state, ctx, y, s.num_heads, s.head_dim, s.v_head_dim,
                                   s.activation, s.q_scale, s.norm, s.gate, s.norm_eps)
         return self.ops.linear(y, self.w_out, out_dtype=self.dtype)

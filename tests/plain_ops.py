@@ -333,15 +333,15 @@ class PlainOps:
                     out[t, h * d:(h + 1) * d] = (w @ v[:, h // (H // G)]).to(out.dtype)
 
     # ---- linear attention with decay ---------------------------------------------------------
-    def linear_attention(self, rows, log_decay, decay_bias, tau, norm_w, state, ctx, out, heads, dim,
+    def linear_attention(self, rows, z_rows, log_decay, decay_bias, tau, norm_w, state, ctx, out, heads, dim,
                          vdim, activation, q_scale, norm, gate, eps):
         H, d, dv = heads, dim, vdim
         q_start, slots = ctx.q_start.tolist(), ctx.state_slot.tolist()
         p = _f(rows)
-        act = torch.nn.functional.silu if activation == "silu" else (lambda x: x)
+        act = (lambda x: _f(torch.nn.functional.silu(x).to(rows.dtype))) if activation == "silu" \
+            else (lambda x: x)
         o_k, o_v = H * d, 2 * H * d
         o_g = o_v + H * dv
-        o_z = o_g + H * dv
         out.zero_()
         for r in range(ctx.n_reqs):
             a, b = q_start[r], q_start[r + 1]
@@ -353,7 +353,7 @@ class PlainOps:
                 k = act(p[t, o_k:o_v]).reshape(H, d)
                 v = act(p[t, o_v:o_g]).reshape(H, dv)
                 if log_decay is None:
-                    z = p[t, o_z:o_z + H * d] + _f(decay_bias)
+                    z = z_rows[t] + _f(decay_bias)
                     keep = torch.exp(torch.nn.functional.logsigmoid(z) / tau).reshape(H, d)
                 else:
                     keep = torch.exp(_f(log_decay))[:, None].expand(H, d)

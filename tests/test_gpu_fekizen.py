@@ -340,20 +340,21 @@ def test_many_blocks_and_windows_beyond_a_split(ops, dtype, sizes):
 # ---- linear attention ----------------------------------------------------------------------------------
 
 def _memory(gen, H, d, dv, constant, silu, head_norm, silu_gate, n):
-    cols = 2 * H * d + 2 * H * dv + (0 if constant else H * d)
     m = SimpleNamespace(H=H, d=d, dv=dv, silu=silu, head=head_norm, gate=silu_gate, tau=3.0, eps=1e-5,
                         q_scale=0.7)
-    m.rows = rnd(gen, torch.float32, n, cols).numpy()
+    m.rows = rnd(gen, torch.bfloat16, n, 2 * H * d + 2 * H * dv).numpy()     # both types hold these
+    m.z = None if constant else rnd(gen, torch.float32, n, H * d).numpy()
     m.log_decay = np.log(np.linspace(0.3, 0.999, H)) if constant else None
     m.bias = None if constant else rnd(gen, torch.float32, H * d).numpy()
     m.norm = 1.0 + 0.1 * rnd(gen, torch.float32, H * dv).numpy()
     return m
 
 
-def _memory_plain(m, rows, state=None):
+def _memory_plain(m, rows=None, state=None):
+    rows, z = m.rows if rows is None else rows, m.z
     H, d, dv, T = m.H, m.d, m.dv, rows.shape[0]
     f = plain.silu if m.silu else (lambda x: x)
-    q, k, v, g, z = np.split(rows, np.cumsum([H * d, H * d, H * dv, H * dv]), axis=1)
+    q, k, v, g = np.split(rows, np.cumsum([H * d, H * d, H * dv]), axis=1)
     if m.log_decay is None:
         a = np.exp(plain.log_sigmoid(z + m.bias) / m.tau).reshape(T, H, d)
     else:
@@ -363,10 +364,10 @@ def _memory_plain(m, rows, state=None):
     return o * m.norm * (plain.silu(g) if m.gate else plain.sigmoid(g)), S
 
 
-def _memory_run(ops, m, rows, state, ctx, dtype):
+def _memory_run(ops, m, rows, z, state, ctx, dtype):
     f = lambda x: None if x is None else dev(torch.from_numpy(np.asarray(x)).float())
     out = torch.full((rows.shape[0], m.H * m.dv), float("nan"), device="cuda", dtype=dtype)
-    ops.linear_attention(f(rows), f(m.log_decay), f(m.bias), m.tau, f(m.norm), state, ctx, out, m.H, m.d, m.dv,
+    ops.linear_attention(f(rows).to(dtype), f(z), f(m.log_decay), f(m.bias), m.tau, f(m.norm), state, ctx, out, m.H, m.d, m.dv,
                          "silu" if m.silu else None, m.q_scale, "head" if m.head else "all",
                          "silu" if m.gate else "sigmoid", m.eps)
     return out
@@ -387,7 +388,7 @@ def test_linear_attention_kernel(ops, dtype, constant, sizes):
     base = ms["a"]
     for m in ms.values():
         m.bias, m.norm = base.bias, base.norm
-    want = {r: _memory_plain(m, m.rows) for r, m in ms.items()}
+    want = {r: _memory_plain(m) for r, m in ms.items()}
     state = torch.zeros(6, H * d * dv, device="cuda")
     state[4].fill_(3.0)                                      # never touched
     slot = {"a": 5, "b": 0, "c": 2}
@@ -400,9 +401,10 @@ def test_linear_attention_kernel(ops, dtype, constant, sizes):
         # empty requests and filling requests without a slot, as padded steps have
         layout = single + [(None, 1)] + parts[len(single):] + [(None, 0), (None, 70)]
         ctx, starts = step_context([(n, slot[r] if r else -1) for r, n in layout])
-        rows = np.concatenate([ms[r].rows[done[r]:done[r] + n] if r else np.full((n, base.rows.shape[1]), 1e3)
-                               for r, n in layout])
-        out = _memory_run(ops, base, rows, state, ctx, dtype)
+        rows, z = (None if x == "z" and constant else np.concatenate(
+            [getattr(ms[r], x)[done[r]:done[r] + n] if r else np.full((n, getattr(base, x).shape[1]), 1e3)
+             for r, n in layout]) for x in ("rows", "z"))
+        out = _memory_run(ops, base, rows, z, state, ctx, dtype)
         for (r, n), a in zip(layout, starts):
             if r:
                 got[r].append(out[a:a + n].cpu())
@@ -412,28 +414,32 @@ def test_linear_attention_kernel(ops, dtype, constant, sizes):
     for r in lengths:
         close(torch.cat(got[r]), want[r][0], dtype, bound=3e-5 if dtype == torch.float32 else None)
         S = want[r][1]
-        close(state[slot[r]], S.reshape(-1), torch.float32, bound=3e-5, scale=max(1.0, float(np.abs(S).max())))
+        # (activated keys and values of bfloat16 rows are rounded once more)
+        loose = dtype == torch.bfloat16 and flags[0]
+        close(state[slot[r]], S.reshape(-1), torch.float32, bound=1e-2 if loose else 3e-5, scale=max(1.0, float(np.abs(S).max())))
     assert float((state[4] - 3.0).abs().max()) == 0 and float(state[1].abs().max()) == 0
 
 
-def test_decays_from_nothing_to_one(ops):
+@pytest.mark.parametrize("dtype,sizes", [(torch.float32, (3, 40, 24)), (torch.bfloat16, (3, 48, 32)),
+                                         (torch.bfloat16, (2, 128, 80)), (torch.bfloat16, (2, 20, 12))])
+def test_decays_from_nothing_to_one(ops, dtype, sizes):
     """Decays that forget everything at once, beside decays that forget nothing, over many chunks: no
     infinity, no lost token.  Constant decays of 0 and 1, and decays by channel whose exponents
     reach some thousands within a chunk."""
     gen = torch.Generator().manual_seed(5)
-    H, d, dv, n = 3, 40, 24, 400
+    (H, d, dv), n = sizes, 400
     for constant in (True, False):
-        m = _memory(gen, H, d, dv, constant, True, False, False, n)
+        m = _memory(gen, H, d, dv, constant, False, False, False, n)
         if constant:
-            m.log_decay = np.array([-1e4, 0.0, np.log(0.5)])
+            m.log_decay = np.array([-1e4, 0.0, np.log(0.5)])[:H]
         else:
             m.tau = 0.5
-            z = m.rows[:, -H * d:].reshape(n, H, d)
+            z = m.z.reshape(n, H, d)
             z[:, :, ::3] = -150.0                            # forgets all
             z[:, :, 1::3] = 60.0                             # forgets nothing
             z[::50, :, 2::3] = -40.0                         # now and then
-        want, S = _memory_plain(m, m.rows)
-        for cut in ([n], [64, 1, 2, 130] * 3, [1] * 30 + [n - 30]):
+        want, S = _memory_plain(m)
+        for cut in ([n], [64, 1, 2, 130] * 2 + [6], [1] * 30 + [n - 30]):
             state = torch.zeros(1, H * d * dv, device="cuda")
             outs, at = [], 0
             for c in cut:
@@ -441,24 +447,26 @@ def test_decays_from_nothing_to_one(ops):
                 if c <= 0:
                     break
                 ctx, _ = step_context([(c, 0)])
-                outs.append(_memory_run(ops, m, m.rows[at:at + c], state, ctx, torch.float32).cpu())
+                outs.append(_memory_run(ops, m, m.rows[at:at + c], None if m.z is None else m.z[at:at + c], state, ctx, dtype).cpu())
                 at += c
             got = torch.cat(outs)
-            close(got, want[:at], torch.float32, bound=1e-4)
-            if at == n:
-                close(state[0], S.reshape(-1), torch.float32, bound=1e-4)
+            assert at == n
+            close(got, want, dtype, bound=1e-4 if dtype == torch.float32 else None)
+            close(state[0], S.reshape(-1), torch.float32, bound=1e-4)
 
 
-def test_an_early_token_among_hundreds_is_not_lost(ops):
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_an_early_token_among_hundreds_is_not_lost(ops, dtype):
     """One early token's key and value are large and every decay is near one: it is seen by a query of
     each later chunk, in portions and in single tokens."""
     gen = torch.Generator().manual_seed(6)
-    H, d, dv, n = 2, 16, 8, 330
+    H, d, dv, n = 2, 16, 16, 330
     m = _memory(gen, H, d, dv, True, False, True, True, n)
     m.log_decay = np.log(np.array([0.9999, 0.999]))
     m.rows[:, H * d:2 * H * d + H * dv] *= 0.01
     m.rows[3, H * d:2 * H * d + H * dv] *= 3000.0
-    want, _ = _memory_plain(m, m.rows)
+    m.rows = torch.from_numpy(m.rows).to(torch.bfloat16).double().numpy()
+    want, _ = _memory_plain(m)
     without = m.rows.copy()
     without[3, H * d:2 * H * d] = 0.0
     assert np.abs(_memory_plain(m, without)[0][-1] - want[-1]).max() > 0.1     # to the last query
@@ -466,9 +474,9 @@ def test_an_early_token_among_hundreds_is_not_lost(ops):
         state, outs, at = torch.zeros(1, H * d * dv, device="cuda"), [], 0
         for c in cut:
             ctx, _ = step_context([(c, 0)])
-            outs.append(_memory_run(ops, m, m.rows[at:at + c], state, ctx, torch.float32).cpu())
+            outs.append(_memory_run(ops, m, m.rows[at:at + c], None if m.z is None else m.z[at:at + c], state, ctx, dtype).cpu())
             at += c
-        close(torch.cat(outs), want, torch.float32, bound=3e-5)
+        close(torch.cat(outs), want, dtype, bound=3e-5 if dtype == torch.float32 else None)
 
 
 # ---- router -----------------------------------------------------------------------------------------
