@@ -1025,7 +1025,7 @@ class OpTimer:
              "heads_product", "sigmoid_gate", "moe_select", "moe_route", "moe_experts", "softcap",
              "hyper_norm", "qkv_full_norm_rope_write", "gated_delta", "glu_clamp", "relu2",
              "weighted_sum", "latent_prepare", "rope_heads", "head_gate", "mlstm",
-             "add_rmsnorm_shift", "normed_sum", "pool_rows", "paged_attention_pooled",
+             "add_rmsnorm_shift", "normed_sum", "rope_pool_write", "paged_attention_pooled",
              "linear_attention")
 
     def __init__(self, torch, ops):
@@ -1433,10 +1433,9 @@ def fekizen_rooflines(sz, entry, pk, T, CTX):
         "add_rmsnorm_shift": runs * T * W * (4 + 4 + 2 + 2) / hbm,
         "add_rmsnorm": (runs + 1) * T * W * (4 + 4 + 2 + 2) / hbm,
         "add_rmsnorm_mevuvik": (2 * runs + 2) * T * W * (4 + 4 + 2 + 2) / hbm,
-        # queries turned in place, keys read once, keys and values written
-        "rope_partial_write": half * T * (2 * H * D + 3 * G * D) * 2 / hbm,
+        # queries turned in place, keys read once, keys, values and blocks' rows written
+        "rope_pool_write": half * T * (2 * H * D + G * D * (3.0 + 2.0 / pool)) * 2 / hbm,
         "latent_prepare": half * T * (Rq + R) * 4 / hbm,
-        "pool_rows": half * T * 2 * G * D * 2 * (1.0 + 1.0 / pool) / hbm,
         "qk_unit_write": half * T * ((H + 2 * G) * D * 2 + 2 * G * D * 2) / hbm,
         "paged_attention_pooled": half * seen * 4.0 * H * D / tens,
         "paged_attention": (half * pairs * 4.0 * H * R + half * pairs * 4.0 * H * D) / tens,
@@ -1453,8 +1452,7 @@ def fekizen_rooflines(sz, entry, pk, T, CTX):
     }
     like = (("add_rmsnorm_shift", "add_rmsnorm", "add_rmsnorm_mevuvik"),
             ("add_rmsnorm", "add_rmsnorm", "add_rmsnorm_mevuvik"),
-            ("rope_partial_write", "latent_prepare", "latent_prepare"),
-            ("pool_rows", "qk_unit_write", "qk_unit_write"),
+            ("rope_pool_write", "latent_prepare", "latent_prepare"),
             ("paged_attention_pooled", "paged_attention", "paged_attention"),
             ("normed_sum", "weighted_sum", "weighted_sum"),
             ("swiglu", "relu2", "relu2"),

@@ -56,9 +56,19 @@ __device__ __forceinline__ int tile_offset(int row, int chunk) {
 // cap * log2 e * tanh(x / cap) for a raw product s with x = s * scale: cap_arg = 2 log2 e * scale /
 // cap, cap_out = cap * log2 e.  One exponential and a fast division; its error is some 1e-7 of
 // the cap.
-__device__ __forceinline__ float capped_log2(float s, float cap_arg, float cap_out) {
-    return cap_out - 2.f * cap_out * __fdividef(1.f, 1.f + exp2f(s * cap_arg));
+__device__ __forceinline__ float fast_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
+__device__ __forceinline__ float capped_log2(float s, float cap_arg, float cap_out) {
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + fast_exp2(s * cap_arg)));
+    return fmaf(-2.f * cap_out, r, cap_out);
+}
+// 2^x where the plain instantiations use the library's form
+template <bool EXT>
+__device__ __forceinline__ float tile_exp2(float x) { return EXT ? fast_exp2(x) : exp2f(x); }
 
 template <int HD, bool SW = false, bool EXT = false>
 __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], const bf16* kt,
@@ -83,25 +93,52 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], co
             mma_bf16(s[2 * nb + 1], qf[kk], b[2], b[3]);
         }
     }
-    if (EXT && cap_out > 0.f) {
+    // EXT: caps and scales first; a tile whose keys all count for all of the warp's rows has no mask
+    bool whole = false;
+    if (EXT) {
+        if (cap_out > 0.f) {
 #pragma unroll
-        for (int i = 0; i < RV_BN / 8; ++i)
+            for (int i = 0; i < RV_BN / 8; ++i)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) s[i][e] = capped_log2(s[i][e], cap_arg, cap_out);
-        scale_log2 = 1.f;
+                for (int e = 0; e < 4; ++e) s[i][e] = capped_log2(s[i][e], cap_arg, cap_out);
+        } else {
+#pragma unroll
+            for (int i = 0; i < RV_BN / 8; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[i][e] *= scale_log2;
+        }
+        whole = __all_sync(0xffffffffu, max(lo_a, lo_b) <= tile_key0 && min(hi_a, hi_b) >= tile_key0 + RV_BN - 1);
     }
     // mask, scale, running maximum
     const int key0 = tile_key0 + (lane & 3) * 2;
     float mx_a = -INFINITY, mx_b = -INFINITY;
+    if (EXT) {
+        if (!whole) {
 #pragma unroll
-    for (int i = 0; i < RV_BN / 8; ++i) {
+            for (int i = 0; i < RV_BN / 8; ++i)
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const int key = key0 + i * 8 + e;
-            s[i][e] = (key >= lo_a && key <= hi_a) ? s[i][e] * scale_log2 : -INFINITY;
-            s[i][2 + e] = (key >= lo_b && key <= hi_b) ? s[i][2 + e] * scale_log2 : -INFINITY;
-            mx_a = fmaxf(mx_a, s[i][e]);
-            mx_b = fmaxf(mx_b, s[i][2 + e]);
+                for (int e = 0; e < 2; ++e) {
+                    const int key = key0 + i * 8 + e;
+                    if (!(key >= lo_a && key <= hi_a)) s[i][e] = -INFINITY;
+                    if (!(key >= lo_b && key <= hi_b)) s[i][2 + e] = -INFINITY;
+                }
+        }
+#pragma unroll
+        for (int i = 0; i < RV_BN / 8; ++i) {
+            mx_a = fmaxf(mx_a, fmaxf(s[i][0], s[i][1]));
+            mx_b = fmaxf(mx_b, fmaxf(s[i][2], s[i][3]));
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < RV_BN / 8; ++i) {
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int key = key0 + i * 8 + e;
+                s[i][e] = (key >= lo_a && key <= hi_a) ? s[i][e] * scale_log2 : -INFINITY;
+                s[i][2 + e] = (key >= lo_b && key <= hi_b) ? s[i][2 + e] * scale_log2 : -INFINITY;
+                mx_a = fmaxf(mx_a, s[i][e]);
+                mx_b = fmaxf(mx_b, s[i][2 + e]);
+            }
         }
     }
     mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1));
@@ -110,7 +147,7 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], co
     mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
     const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b);
     const float off_a = mn_a == -INFINITY ? 0.f : mn_a, off_b = mn_b == -INFINITY ? 0.f : mn_b;
-    const float corr_a = exp2f(m_a - off_a), corr_b = exp2f(m_b - off_b);   // m = -inf -> 0
+    const float corr_a = tile_exp2<EXT>(m_a - off_a), corr_b = tile_exp2<EXT>(m_b - off_b);   // m = -inf -> 0
     m_a = mn_a;
     m_b = mn_b;
     l_a *= corr_a;
@@ -125,8 +162,8 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], co
     unsigned pa[RV_BN / 16][4];
 #pragma unroll
     for (int i = 0; i < RV_BN / 8; ++i) {
-        const float e0 = exp2f(s[i][0] - off_a), e1 = exp2f(s[i][1] - off_a);
-        const float e2 = exp2f(s[i][2] - off_b), e3 = exp2f(s[i][3] - off_b);
+        const float e0 = tile_exp2<EXT>(s[i][0] - off_a), e1 = tile_exp2<EXT>(s[i][1] - off_a);
+        const float e2 = tile_exp2<EXT>(s[i][2] - off_b), e3 = tile_exp2<EXT>(s[i][3] - off_b);
         const __nv_bfloat162 ra = __floats2bfloat162_rn(e0, e1);
         const __nv_bfloat162 rb = __floats2bfloat162_rn(e2, e3);
         const float2 fa = __bfloat1622float2(ra), fb = __bfloat1622float2(rb);
@@ -150,7 +187,7 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], co
 }
 
 template <int HD, int NWARPS, bool SPLIT, bool EXT = false>
-__global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(
+__global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_attention_mma_kernel(
     const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ k_cache,
     const bf16* __restrict__ v_cache, const int* __restrict__ block_table, int max_blocks,
     const int* __restrict__ q_start, const int* __restrict__ ctx_lens, bf16* __restrict__ out,

@@ -819,21 +819,33 @@ class CudaOps:
 
     # ---- pooled blocks: their rows; attention over a window and the blocks before it --------
 
-    def pool_rows(self, k_cache, v_cache, group, ctx, pool, slots, k_out, v_out):
-        """For every token t with slots[t] >= 0, the last of a block of `pool` tokens: the means of
-        the block's cached keys and values (read through `group`'s block table) -> row
-        slots[t] of `k_out` and `v_out`."""
-        self._need(k_cache, "key pages")
+    def rope_pool_write(self, rows, num_heads, num_kv_heads, head_dim, freq, ctx, group, k_cache,
+                        v_cache, pool, slots, k_blocks, v_blocks, amplitude=1.0,
+                        values_are_keys=False):
+        """`rope_partial_write` for keys and values of one size, and the rows of the pooled blocks
+        that the step completes: for every token t with slots[t] >= 0, the last of a block of `pool`
+        tokens, the means of the block's cached keys and values go to row slots[t] of
+        `k_blocks` and `v_blocks`."""
+        self._need(rows, "q|k|v rows")
         self._need(slots, "slots of completed blocks", torch.int32)
-        for t, what in ((v_cache, "value pages"), (k_out, "block keys"), (v_out, "block values")):
-            self._need(t, what, k_cache.dtype)
-            if t.shape[-2:] != k_cache.shape[-2:]:
-                raise KernelError("pool_rows: the pages differ in shape")
-        self._check(self.lib.rv_pool_rows(
-            _ptr(k_cache), _ptr(v_cache), _code(k_cache.dtype), _ptr(group.block_table),
-            c_int(group.max_blocks), c_int(group.page_size), _ptr(ctx.token_req), _ptr(ctx.positions),
-            _ptr(slots), c_int(pool), _ptr(k_out), _ptr(v_out), c_int(ctx.n_tokens),
-            c_int(k_cache.shape[-2] * k_cache.shape[-1]), self._stream()), "pool_rows")
+        for t, what in ((k_cache, "key pages"), (v_cache, "value pages"), (k_blocks, "block keys"),
+                        (v_blocks, "block values")):
+            self._need(t, what, rows.dtype)
+            if t.shape[-2:] != (num_kv_heads, head_dim):
+                raise KernelError("rope_pool_write: the pages and the head sizes disagree")
+        inv, dims = freq if freq is not None else (None, 0)
+        if inv is not None:
+            self._need(inv, "rotation frequencies", torch.float32)
+            if inv.shape[0] != dims // 2:
+                raise KernelError("rope_pool_write: one frequency per pair of turning dimensions")
+        self._check(self.lib.rv_rope_pool_write(
+            _ptr(rows), _code(rows.dtype), c_int(rows.shape[1]), c_int(rows.shape[0]),
+            c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), _ptr(inv), c_int(dims),
+            c_float(amplitude), c_int(1 if values_are_keys else 0), _ptr(ctx.positions),
+            _ptr(ctx.token_req), _ptr(ctx.q_start), _ptr(group.slot_mapping),
+            _ptr(group.block_table), c_int(group.max_blocks), c_int(group.page_size), c_int(pool),
+            _ptr(slots), _ptr(k_cache), _ptr(v_cache), _ptr(k_blocks), _ptr(v_blocks),
+            self._stream()), "rope_pool_write")
 
     def attention_pooled_scratch_bytes(self, n_reqs, num_heads, head_dim, max_ctx_len, window,
                                        pool) -> int:

@@ -10,11 +10,11 @@ before the rotation.
 Two page groups serve a call: the tokens' keys and values, whose pages are given back once they
 lie before the window *and* before the newest incomplete block, and one row per block, which is
 kept as long as the request lives.  A block's row is formed in the step that brings the block's
-last token, always from the cached rows of its tokens (`ops.pool_rows`), so it does not
-depend on how the block's tokens were cut into steps.
+last token, always from its tokens' rows as the cache holds them, so it does not depend on how
+the block's tokens were cut into steps.
 
-q and k (and v, when it has a projection) are one product; rotation and the cache write are one
-kernel.
+q and k (and v, when it has a projection) are one product; rotation, the cache write and the
+blocks' rows are one kernel (`ops.rope_pool_write`).
 """
 from __future__ import annotations
 
@@ -100,14 +100,15 @@ class PooledAttention(Mixer):
         freq, amplitude = None, 1.0
         if s.position.kind == "rope_partial":
             freq, amplitude = self.position.frequencies(), self.position.amplitude
-        self.ops.rope_partial_write(rows, H, G, d, d, freq, ctx.positions, group.slot_mapping,
-                                    tokens.k, tokens.v, amplitude=amplitude,
-                                    values_are_keys=s.values_are_keys)
+        options = dict(amplitude=amplitude, values_are_keys=s.values_are_keys)
         pooled = None
-        if blocks is not None:
+        if blocks is None:
+            self.ops.rope_partial_write(rows, H, G, d, d, freq, ctx.positions, group.slot_mapping,
+                                        tokens.k, tokens.v, **options)
+        else:
             bgroup = ctx.groups[blocks.group]
-            self.ops.pool_rows(tokens.k, tokens.v, group, ctx, s.pool, bgroup.slot_mapping,
-                               blocks.k, blocks.v)
+            self.ops.rope_pool_write(rows, H, G, d, freq, ctx, group, tokens.k, tokens.v, s.pool,
+                                     bgroup.slot_mapping, blocks.k, blocks.v, **options)
             pooled = (blocks.k, blocks.v, bgroup, s.pool)
         out = self.ops.new_rows(normed.shape[0], H * d, self.dtype, normed.device)
         self.ops.paged_attention_pooled(rows, H, G, d, tokens.k, tokens.v, ctx, group, pooled,

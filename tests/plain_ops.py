@@ -283,7 +283,10 @@ class PlainOps:
                     vc[s] = v[t].to(vc.dtype)
 
     # ---- pooled blocks: their rows, and attention over a window and the blocks before it ----
-    def pool_rows(self, k_cache, v_cache, group, ctx, pool, slots, k_out, v_out):
+    def rope_pool_write(self, rows, num_heads, num_kv_heads, head_dim, freq, ctx, group, k_cache,
+                        v_cache, pool, slots, k_out, v_out, **options):
+        self.rope_partial_write(rows, num_heads, num_kv_heads, head_dim, head_dim, freq,
+                                ctx.positions, group.slot_mapping, k_cache, v_cache, **options)
         G, d = k_cache.shape[-2:]
         ps = group.page_size
         treq, pos = ctx.token_req.tolist(), ctx.positions.tolist()

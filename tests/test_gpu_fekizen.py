@@ -172,25 +172,76 @@ def test_rotation_with_amplitude_and_values_that_are_keys(ops, dtype, sizes):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-def test_rows_of_blocks_are_means_of_the_cached_rows(ops, dtype):
-    g = torch.Generator().manual_seed(8)
-    G, d, page, pool = 3, 10, 4, 7
-    k, v = rnd(g, dtype, 12, page, G, d), rnd(g, dtype, 12, page, G, d)
-    table = torch.tensor([[5, 0, 9, 2, 7, 10], [1, 11, 3, -1, -1, -1]], dtype=torch.int32)
-    # request 0 brings positions 12..20 (blocks 1 = 7..13 and 2 = 14..20 complete), request 1 position 6
-    pos = [6] + list(range(12, 21))
-    slots = [4] + [7 if p == 13 else (2 if p == 20 else -1) for p in range(12, 21)]
-    ctx = SimpleNamespace(token_req=i32([1] + [0] * 9), positions=i32(pos), n_tokens=10)
-    group = SimpleNamespace(block_table=dev(table), max_blocks=6, page_size=page)
-    ko = torch.full((5, 2, G, d), 9.0, device="cuda", dtype=dtype)
-    vo = torch.full((5, 2, G, d), 9.0, device="cuda", dtype=dtype)
-    ops.pool_rows(dev(k, dtype), dev(v, dtype), group, ctx, pool, i32(slots), ko, vo)
-    for r, b, s in ((0, 1, 7), (0, 2, 2), (1, 0, 4)):
-        at = [(int(table[r, j // page]), j % page) for j in range(b * pool, b * pool + pool)]
-        close(ko.reshape(10, G, d)[s], sum(k[a, o] for a, o in at) / pool, dtype)
-        close(vo.reshape(10, G, d)[s], sum(v[a, o] for a, o in at) / pool, dtype)
-    rest = [s for s in range(10) if s not in (7, 2, 4)]
-    assert float((ko.reshape(10, G, d)[rest] - 9.0).abs().max()) == 0
+@pytest.mark.parametrize("sizes", [(6, 3, 10, 6, 7), (8, 2, 64, 64, 16), (5, 5, 16, 0, 1), (4, 1, 80, 16, 40)])
+@pytest.mark.parametrize("v_is_k", [True, False])
+def test_rows_of_blocks_are_means_of_the_cached_rows(ops, dtype, sizes, v_is_k):
+    """Three requests in portions of every kind against pool borders: queries, cached rows and the
+    blocks' rows, which are the means of the rows as they are cached, whatever the cut."""
+    H, G, d, dims, pool = sizes
+    page, n_req = 4, 3
+    lengths = (95, 41, pool)
+    rot = fk._rot(dims, 300.0, (4.0, 64, 8.0, 1.0)) if dims else None
+    freq, amp = None, 1.0
+    if dims:
+        f, amp = plain.yarn_frequencies(rot)
+        freq = (dev(torch.from_numpy(f).float()), dims)
+    g = torch.Generator().manual_seed(d)
+    rows = [rnd(g, dtype, n, (H + G * (1 if v_is_k else 2)) * d) for n in lengths]
+    rng = random.Random(pool)
+    ids = rng.sample(range(60), 60)
+    table = torch.tensor([ids[20 * r:20 * r + 24] if r < 2 else ids[40:60] + [-1] * 4 for r in range(3)],
+                         dtype=torch.int32)
+    table[0] = torch.tensor(ids[:24]); table[1] = torch.tensor(ids[24:48]); table[2, :12] = torch.tensor(ids[48:60])
+    pids = rng.sample(range(140), 140)                       # rows of blocks, anywhere
+    k = torch.full((60, page, G, d), 9.0, device="cuda", dtype=dtype)
+    v = torch.full_like(k, 9.0)
+    kb = torch.full((35, 4, G, d), 9.0, device="cuda", dtype=dtype)
+    vb = torch.full_like(kb, 9.0)
+    done = [0, 0, 0]
+    cuts = [[1, 1, 39, 2, 3, 49], [2, 30, 1, 1, 7], [pool]]
+    qs = [[], [], []]
+    for step in range(6):
+        parts = [(r, cuts[r][step]) for r in range(n_req) if step < len(cuts[r])]
+        parts.sort(key=lambda x: x[1] != 1)
+        layout = [(m, 0) for _, m in parts] + [(3, -1)]      # a filling request writes nothing
+        ctx, starts = step_context(layout)
+        pos, slots, done_slots, x = [], [], [], []
+        for r, m in parts:
+            for p in range(done[r], done[r] + m):
+                pos.append(p)
+                slots.append(int(table[r, p // page]) * page + p % page)
+                done_slots.append(pids[r * 45 + p // pool] if (p + 1) % pool == 0 and p // pool < 45 else -1)
+            x.append(rows[r][done[r]:done[r] + m])
+        ctx.positions = i32(pos + [0] * 3)
+        tabs = torch.cat([table[[r for r, _ in parts]], torch.full((1, 24), -1, dtype=torch.int32)])
+        group = SimpleNamespace(block_table=dev(tabs), max_blocks=24, page_size=page,
+                                slot_mapping=i32(slots + [-1] * 3))
+        xs = dev(torch.cat(x + [torch.full((3, rows[0].shape[1]), 50.0, dtype=torch.float64)]), dtype)
+        ops.rope_pool_write(xs, H, G, d, freq, ctx, group, k, v, pool, i32(done_slots + [-1] * 3), kb, vb,
+                            amplitude=amp, values_are_keys=v_is_k)
+        for (r, m), a in zip(parts, starts):
+            qs[r].append(xs[a:a + m, :H * d].cpu())
+            done[r] += m
+    written, wrows = set(), set()
+    for r, n in enumerate(lengths[:2] + (pool,)):
+        n = done[r]
+        q = rows[r][:n, :H * d].reshape(n, H, d).numpy()
+        kk = rows[r][:n, H * d:(H + G) * d].reshape(n, G, d).numpy()
+        vv = kk if v_is_k else rows[r][:n, (H + G) * d:].reshape(n, G, d).numpy()
+        close(torch.cat(qs[r]), np.stack([plain.rotate(q[t], t, rot) for t in range(n)]), dtype, bound=5e-5)
+        at = [int(table[r, p // page]) * page + p % page for p in range(n)]
+        written |= set(at)
+        ck, cv = k.reshape(-1, G, d)[at].cpu().double(), v.reshape(-1, G, d)[at].cpu().double()
+        close(ck, np.stack([plain.rotate(kk[t], t, rot) for t in range(n)]), dtype, bound=5e-5)
+        assert float((cv - torch.from_numpy(vv)).abs().max()) == 0
+        for b in range(min(n // pool, 45)):
+            s = pids[r * 45 + b]
+            wrows.add(s)
+            close(kb.reshape(-1, G, d)[s], ck[b * pool:(b + 1) * pool].mean(0), dtype, scale=1.0)
+            close(vb.reshape(-1, G, d)[s], cv[b * pool:(b + 1) * pool].mean(0), dtype, scale=1.0)
+    for t, used in ((k, written), (v, written), (kb, wrows), (vb, wrows)):
+        rest = [s for s in range(t.shape[0] * t.shape[1]) if s not in used]
+        assert float((t.reshape(-1, G, d)[rest] - 9.0).abs().max()) == 0
 
 
 # ---- attention over a window and the blocks before it ------------------------------------------------------
