@@ -30,7 +30,7 @@
 //   finish  the norm, weight and gate.
 //
 // bfloat16 rows with d and dv in multiples of 16 (d up to 128) take the tensor-core forms of `state`
-// and `out`.  Their float32 operands (the state, the scores, everything multiplied by a decay) go
+// and `out` (with decays by channel, after a kernel that leaves the sums B where z was).  Their float32 operands (the state, the scores, everything multiplied by a decay) go
 // through the bfloat16 product without being rounded: x = x1 + x2 + x3, each part the
 // bfloat16 nearest to what is left, holds all 24 bits, so x times a bfloat16 is three exact
 // products added in float32, and a product of two such sums is the six of its nine products that
@@ -671,7 +671,8 @@ extern "C" long long rv_linear_attention_scratch(int n_tokens, int n_decode, int
 }
 
 struct LaArgs {
-    const float *z, *log_decay, *bias, *norm_w;
+    float* z;
+    const float *log_decay, *bias, *norm_w;
     float *state, *scratch;
     const int *token_req, *q_start, *state_slot;
     float tau, q_scale, eps;
@@ -700,15 +701,15 @@ template <bool CH>
 static int la_tensor_launch(const bf16* rows, const LaArgs& a, int what, dim3 grid, float* kv, float* dec,
                             float* num, cudaStream_t s) {
     if (what == 0) {
-        const size_t smem = lm_state_smem(CH);
+        const size_t smem = lm_state_smem();
         LA_SMEM(la_state_mma_kernel<CH>, smem)
-        rv_launch(la_state_mma_kernel<CH>, grid, dim3(128), smem, s, rows, a.stride, a.z, a.log_decay, a.bias,
-                  a.tau, a.q_start, a.state_slot, a.n_decode, a.n_reqs, kv, dec, a.H, a.d, a.dv, a.act);
+        rv_launch(la_state_mma_kernel<CH>, grid, dim3(128), smem, s, rows, a.stride, (const float*)a.z,
+                  a.log_decay, a.q_start, a.state_slot, a.n_decode, a.n_reqs, kv, dec, a.H, a.d, a.dv, a.act);
     } else {
         const size_t smem = lm_out_smem(CH, a.d);
         LA_SMEM(la_out_mma_kernel<CH>, smem)
-        rv_launch(la_out_mma_kernel<CH>, grid, dim3(128), smem, s, rows, a.stride, a.z, a.log_decay, a.bias,
-                  a.tau, a.q_start, a.state_slot, a.n_decode, a.n_reqs, (const float*)kv, num, a.H, a.d, a.dv,
+        rv_launch(la_out_mma_kernel<CH>, grid, dim3(128), smem, s, rows, a.stride, (const float*)a.z,
+                  a.log_decay, a.q_start, a.state_slot, a.n_decode, a.n_reqs, (const float*)kv, num, a.H, a.d, a.dv,
                   a.act, a.q_scale);
     }
     return 0;
@@ -720,6 +721,12 @@ static int la_portions(const T* rows, const LaArgs& a, float* num, float* kv, fl
     const int tiles_d = (a.d + LA_T - 1) / LA_T, tiles_v = (a.dv + LA_T - 1) / LA_T;
     const dim3 g1(items, a.H, tiles_d * tiles_v), g3(items, a.H, tiles_v);
     if (a.tensor) {
+        if (CH) {
+            const int width = a.H * a.d;
+            rv_launch(la_decay_kernel, dim3(items, (width + 31) / 32), dim3(256), 0, s, a.z, a.bias,
+                      1.4426950408889634f / a.tau, a.q_start, a.state_slot, a.n_decode, a.n_reqs, width);
+            RV_CHECK_LAUNCH("linear_attention_decay");
+        }
         if (la_tensor_launch<CH>(rows, a, 0, g1, kv, dec, num, s)) return 1;
     } else {
         const size_t smem = (size_t)((CH ? 3 : 2) * LA_C * LA_LD + 4 * 64) * sizeof(float);
@@ -804,11 +811,12 @@ static int la_run(const T* rows, const LaArgs& a, T* out, cudaStream_t s) {
     return 0;
 }
 
-// log_decay [H]; or null, then z float32 [n, H d], bias [H d] and tau.  act: 1 silu; norm_head: 0 all
+// log_decay [H]; or null, then z float32 [n, H d] (used up: the tensor-core forms leave sums of log
+// decays there), bias [H d] and tau.  act: 1 silu; norm_head: 0 all
 // heads together, 1 per head; gate: 0 sigmoid, 1 silu; norm_w [H dv].  Requests [0, n_decode) bring
 // one token each (token r is request r's).  `tensor`: whether portions may take the tensor-core
 // forms (where their sizes allow).  rows and out have the type `dtype`.
-extern "C" int rv_linear_attention(const void* rows, int dtype, int stride, const float* z,
+extern "C" int rv_linear_attention(const void* rows, int dtype, int stride, float* z,
                                    const float* log_decay, const float* bias, float tau,
                                    const float* norm_w, float* state, const int* token_req,
                                    const int* q_start, const int* state_slot, float* scratch, void* out,
@@ -825,7 +833,7 @@ extern "C" int rv_linear_attention(const void* rows, int dtype, int stride, cons
         RV_FAIL("linear_attention: too many requests or heads, or heads that are too large");
     if ((uintptr_t)scratch & 15) RV_FAIL("linear_attention: the scratch must be 16-byte aligned");
     tensor = tensor && dtype == RV_DTYPE_BF16 && d % 16 == 0 && dv % 16 == 0 && d <= 128 && stride % 8 == 0 &&
-             ((uintptr_t)rows & 15) == 0;
+             (((uintptr_t)rows | (uintptr_t)z) & 15) == 0;
     const LaArgs a = {z, log_decay, bias, norm_w, state, scratch, token_req, q_start, state_slot, tau, q_scale, eps,
                       stride, n_tokens, n_decode, n_reqs, H, d, dv, act, norm_head, gate, tensor};
     RV_DISPATCH_DTYPE(dtype, "linear_attention",

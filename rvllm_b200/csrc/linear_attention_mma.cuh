@@ -47,49 +47,66 @@ __device__ __forceinline__ void lm_locate(const int* q_start, const int* state_s
     }
     __syncthreads();
 }
-// Sums of log decays over the tokens of a chunk, in place: lb [64 tokens][ldb], `n` channels.  128
-// threads: a channel's tokens in `segs` stretches (segs * n <= 128), then the stretches before.
-__device__ __forceinline__ void lm_cumsum(float* lb, int ldb, int n, float* tot /* [128] */) {
-    const int segs = n <= 16 ? 8 : n <= 32 ? 4 : n <= 64 ? 2 : 1;
-    const int len = LA_C / segs;
-    const int c = threadIdx.x % n, g = threadIdx.x / n;
-    const bool mine = g < segs;
-    if (mine) {
-        float s = 0.f;
-        for (int j = g * len; j < (g + 1) * len; j += 8) {
-            float v[8];
-#pragma unroll
-            for (int u = 0; u < 8; ++u) v[u] = lb[(j + u) * ldb + c];
-#pragma unroll
-            for (int u = 0; u < 8; ++u) {
-                s += v[u];
-                lb[(j + u) * ldb + c] = s;
-            }
+__device__ __forceinline__ float lm_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// z -> B: what the tokens of a chunk up to and with this one keep of a channel, as a power of two
+// (sums of log2 a), in place, so that neither of the kernels below repeats it for its tiles.  A
+// warp has eight tokens of 32 channels.
+#define LM_STRONG -57.7f    // -40 log2 e
+__global__ void __launch_bounds__(256) la_decay_kernel(float* __restrict__ z, const float* __restrict__ bias,
+                                                       float scale, const int* __restrict__ q_start,
+                                                       const int* __restrict__ state_slot, int first_req,
+                                                       int n_reqs, int width) {
+    rv_pdl_launch_dependents();
+    __shared__ float tot[8][32];
+    __shared__ int at[2];
+    const int lane = threadIdx.x & 31, g = threadIdx.x >> 5, c = blockIdx.y * 32 + lane;
+    if (threadIdx.x < 32) {
+        int r = -1, before = 0;
+        const bool ok = la_find(q_start, state_slot, first_req, n_reqs, blockIdx.x, lane, r, before);
+        if (lane == 0) {
+            at[0] = ok ? q_start[r] + ((int)blockIdx.x - before) * LA_C : -1;
+            at[1] = ok ? min(LA_C, q_start[r + 1] - at[0]) : 0;
         }
-        tot[g * n + c] = s;
     }
     __syncthreads();
-    if (mine && g > 0) {
-        float before = 0.f;
-        for (int i = 0; i < g; ++i) before += tot[i * n + c];
-#pragma unroll 8
-        for (int j = g * len; j < (g + 1) * len; ++j) lb[j * ldb + c] += before;
+    const int t0 = at[0], L = at[1];
+    const float b = c < width ? bias[c] : 0.f;
+    rv_pdl_wait();
+    if (t0 < 0) return;
+    float v[8], s = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+        v[j] = 8 * g + j < L && c < width ? z[(size_t)(t0 + 8 * g + j) * width + c] : 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+        s += la_logsigmoid(v[j] + b) * scale;
+        v[j] = s;
     }
+    tot[g][lane] = s;
     __syncthreads();
+    float before = 0.f;
+    for (int i = 0; i < g; ++i) before += tot[i][lane];
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+        if (8 * g + j < L && c < width) z[(size_t)(t0 + 8 * g + j) * width + c] = before + v[j];
 }
 
 // KV = sum_j (k_j e^(B_L - B_j)) v_j^T for 64 channels by 64 columns: a warp has 16 channels.
 template <bool CHANNEL>
 __global__ void __launch_bounds__(128) la_state_mma_kernel(
-    const bf16* __restrict__ rows, int stride, const float* __restrict__ zr,
-    const float* __restrict__ log_decay, const float* __restrict__ bias, float tau,
+    const bf16* __restrict__ rows, int stride, const float* __restrict__ zb,
+    const float* __restrict__ log_decay,
     const int* __restrict__ q_start, const int* __restrict__ state_slot, int first_req, int n_reqs,
     float* __restrict__ kv, float* __restrict__ dec, int H, int d, int dv, int act) {
     rv_pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char smraw[];
     bf16* ks = (bf16*)smraw;                            // [3][64 tokens][LM_LD]
     bf16* vs = ks + 3 * LA_C * LM_LD;                   // [64 tokens][LM_LD]
-    float* lb = (float*)(vs + LA_C * LM_LD);            // CHANNEL: [64][65], then [128]
     __shared__ int at[2];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int item = blockIdx.x, h = blockIdx.y;
@@ -112,15 +129,15 @@ __global__ void __launch_bounds__(128) la_state_mma_kernel(
         kreg[u] = lm_in8(row + (H + h) * d + d0 + 8 * ch, j < L && 8 * ch < dn, act);
         vreg[u] = lm_in8(row + 2 * H * d + h * dv + v0 + 8 * ch, j < L && 8 * ch < vn, act);
     }
+    float bl[8];                                        // CHANNEL: B of the chunk's last token
     if (CHANNEL) {
-        const int c = tid & 63;
-        const float b = c < dn ? bias[h * d + d0 + c] : 0.f;
-#pragma unroll 8
-        for (int j = tid >> 6; j < LA_C; j += 2)
-            lb[j * 65 + c] = j < L && c < dn ? la_logsigmoid(zr[(size_t)(t0 + j) * H * d + h * d + d0 + c] + b) / tau : 0.f;
-        __syncthreads();
-        lm_cumsum(lb, 65, 64, lb + 64 * 65);
-        if (v0 == 0 && tid < dn) dec[((size_t)item * H + h) * d + d0 + tid] = expf(lb[63 * 65 + tid]);
+        const float* p = zb + (size_t)(t0 + L - 1) * H * d + h * d + d0;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) bl[e] = 8 * ch < dn ? p[8 * ch + e] : 0.f;
+        if (v0 == 0 && jr == 0 && 8 * ch < dn)
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+                dec[((size_t)item * H + h) * d + d0 + 8 * ch + e] = lm_exp2(bl[e]);
     }
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
@@ -128,16 +145,23 @@ __global__ void __launch_bounds__(128) la_state_mma_kernel(
         *(uint4*)(vs + j * LM_LD + 8 * ch) = vreg[u];
         const unsigned in[4] = {kreg[u].x, kreg[u].y, kreg[u].z, kreg[u].w};
         unsigned o[3][4];
-        float f = 0.f;
+        float f = 0.f, bj[8];
         if (!CHANNEL) f = expf(ld * (float)(L - 1 - min(j, L - 1)));
+        if (CHANNEL) {
+            const float* p = zb + (size_t)(t0 + min(j, L - 1)) * H * d + h * d + d0 + 8 * ch;
+#pragma unroll
+            for (int e = 0; e < 8; e += 4) {
+                const float4 x = 8 * ch < dn ? *(const float4*)(p + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+                bj[e] = x.x; bj[e + 1] = x.y; bj[e + 2] = x.z; bj[e + 3] = x.w;
+            }
+        }
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const float2 k2 = lm_pair(in[e]);
             float fx = f, fy = f;
             if (CHANNEL) {
-                const int c = 8 * ch + 2 * e;
-                fx = expf(lb[63 * 65 + c] - lb[j * 65 + c]);
-                fy = expf(lb[63 * 65 + c + 1] - lb[j * 65 + c + 1]);
+                fx = lm_exp2(bl[2 * e] - bj[2 * e]);
+                fy = lm_exp2(bl[2 * e + 1] - bj[2 * e + 1]);
             }
             lm_split(k2.x * fx, k2.y * fy, o[0][e], o[1][e], o[2][e]);
         }
@@ -178,12 +202,13 @@ __global__ void __launch_bounds__(128) la_state_mma_kernel(
     }
 }
 
+// (B in powers of two here: zb is what la_decay left.)
 // o = (scores, masked) V + (q e^(B_i)) S for the chunk's 64 tokens by 64 columns: a warp has 16
 // tokens.  CHANNEL: B is kept whole (bs), q e^(B_i) is formed in fragments, k e^(-B_j) in shared memory.
 template <bool CHANNEL>
 __global__ void __launch_bounds__(128) la_out_mma_kernel(
-    const bf16* __restrict__ rows, int stride, const float* __restrict__ zr,
-    const float* __restrict__ log_decay, const float* __restrict__ bias, float tau,
+    const bf16* __restrict__ rows, int stride, const float* __restrict__ zb,
+    const float* __restrict__ log_decay,
     const int* __restrict__ q_start, const int* __restrict__ state_slot, int first_req, int n_reqs,
     const float* __restrict__ kv, float* __restrict__ num, int H, int d, int dv, int act, float q_scale) {
     rv_pdl_launch_dependents();
@@ -193,7 +218,7 @@ __global__ void __launch_bounds__(128) la_out_mma_kernel(
     bf16* vs = ss + 3 * d * LM_LD;                      // [64][LM_LD]
     bf16* qs = vs + LA_C * LM_LD;                       // [64][LQ]
     bf16* ks = qs + LA_C * LQ;                          // [1 or 3][64][LQ]
-    float* bs = (float*)(ks + (CHANNEL ? 3 : 1) * LA_C * LQ);   // CHANNEL: [64][LB], then [128]
+    float* bs = (float*)(ks + (CHANNEL ? 3 : 1) * LA_C * LQ);   // CHANNEL: [64][LB]
     __shared__ float pw[LA_C + 1];                      // constant decay: its powers
     __shared__ int at[2];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -239,14 +264,17 @@ __global__ void __launch_bounds__(128) la_out_mma_kernel(
     }
     bool strong = false;
     if (CHANNEL) {
-#pragma unroll 8
-        for (int n = tid; n < LA_C * d; n += 128) {
-            const int j = n / d, c = n - j * d;
-            bs[j * LB + c] = j < L ? la_logsigmoid(zr[(size_t)(t0 + j) * H * d + h * d + c] + bias[h * d + c]) / tau : 0.f;
+        const int cpr = d >> 2;
+        bool low = false;
+#pragma unroll 4
+        for (int n = tid; n < LA_C * cpr; n += 128) {
+            const int j = n / cpr, c = (n - j * cpr) * 4;
+            const float4 x = *(const float4*)(zb + (size_t)(t0 + min(j, L - 1)) * H * d + h * d + c);
+            *(float2*)(bs + j * LB + c) = make_float2(x.x, x.y);
+            *(float2*)(bs + j * LB + c + 2) = make_float2(x.z, x.w);
+            low |= fminf(fminf(x.x, x.y), fminf(x.z, x.w)) < LM_STRONG;
         }
-        __syncthreads();
-        lm_cumsum(bs, LB, d, bs + LA_C * LB);
-        strong = __syncthreads_or(tid < d && bs[(LA_C - 1) * LB + tid] < -40.f);
+        strong = __syncthreads_or(low);
         if (!strong) {
 #pragma unroll 2
             for (int n = tid; n < LA_C * (d >> 1); n += 128) {
@@ -254,7 +282,7 @@ __global__ void __launch_bounds__(128) la_out_mma_kernel(
                 unsigned* k0 = (unsigned*)(ks + j * LQ + c);
                 const float2 k2 = lm_pair(*k0), b2 = *(const float2*)(bs + j * LB + c);
                 unsigned p[3];
-                lm_split(k2.x * expf(-b2.x), k2.y * expf(-b2.y), p[0], p[1], p[2]);
+                lm_split(k2.x * lm_exp2(-b2.x), k2.y * lm_exp2(-b2.y), p[0], p[1], p[2]);
                 k0[0] = p[0];
                 *(unsigned*)(ks + LA_C * LQ + j * LQ + c) = p[1];
                 *(unsigned*)(ks + 2 * LA_C * LQ + j * LQ + c) = p[2];
@@ -277,7 +305,7 @@ __global__ void __launch_bounds__(128) la_out_mma_kernel(
             for (int e = 0; e < 4; ++e) {
                 const float2 q2 = lm_pair(a[0][e]);
                 const float2 b2 = *(const float2*)(bs + ((e & 1) ? row_b : row_a) * LB + kk * 16 + (e >> 1) * 8 + (lane & 3) * 2);
-                lm_split(q2.x * expf(b2.x), q2.y * expf(b2.y), a[0][e], a[CHANNEL ? 1 : 0][e], a[CHANNEL ? 2 : 0][e]);
+                lm_split(q2.x * lm_exp2(b2.x), q2.y * lm_exp2(b2.y), a[0][e], a[CHANNEL ? 1 : 0][e], a[CHANNEL ? 2 : 0][e]);
             }
         }
         // scores: keys up to the warp's own tokens
@@ -327,7 +355,7 @@ __global__ void __launch_bounds__(128) la_out_mma_kernel(
                 if (j <= r)
                     for (int c = 0; c < d; ++c)
                         s = fmaf(__bfloat162float(qs[r * LQ + c]) * __bfloat162float(ks[j * LQ + c]),
-                                 expf(bs[r * LB + c] - bs[j * LB + c]), s);
+                                 lm_exp2(bs[r * LB + c] - bs[j * LB + c]), s);
                 p[i][e] = s;
             }
         }
@@ -376,10 +404,10 @@ __global__ void __launch_bounds__(128) la_out_mma_kernel(
     }
 }
 
-static inline size_t lm_state_smem(bool channel) {
-    return (size_t)4 * LA_C * LM_LD * 2 + (channel ? (size_t)(LA_C * 65 + 128) * 4 : 0);
+static inline size_t lm_state_smem() {
+    return (size_t)4 * LA_C * LM_LD * 2;
 }
 static inline size_t lm_out_smem(bool channel, int d) {
     return (size_t)(3 * d + LA_C) * LM_LD * 2 + (size_t)(channel ? 4 : 2) * LA_C * (d + 8) * 2 +
-           (channel ? (size_t)(LA_C * (d + 2) + 128) * 4 : 0);
+           (channel ? (size_t)LA_C * (d + 2) * 4 : 0);
 }
