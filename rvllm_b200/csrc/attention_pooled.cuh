@@ -3,7 +3,7 @@
 // kernels (attention_mma.cu).
 //
 // The query at position p sees the tokens j with p - window < j <= p and the pooled blocks
-// b < rv_seen_blocks(p): those of `pool` tokens that lie wholly before the window.  A block's key
+// b < rv_seen_blocks(p): stretches of `pool` tokens that have left the window whole.  A block's key
 // and value are rows of page tensors of their own with a block table of their own.  Scores may be
 // capped, cap * tanh(score / cap).
 //

@@ -585,13 +585,13 @@ __device__ __forceinline__ void la_store(T* p, const float (&x)[V]) {
     }
 }
 template <typename T, int V>
-__device__ __forceinline__ void la_finish_at(const float* nm, const T* g, const float* w, T* o, int c, float rms, int gate) {
+__device__ __forceinline__ void la_finish_at(const float* nm, const T* g, const float* w, T* o, int c, float inv, int gate) {
     float x[V], y[V], z[V];
     la_load<float, V>(nm + c, x);
     la_load<T, V>(g + c, y);
     la_load<float, V>(w + c, z);
 #pragma unroll
-    for (int e = 0; e < V; ++e) x[e] = x[e] / rms * z[e] * la_gate(y[e], gate);
+    for (int e = 0; e < V; ++e) x[e] = x[e] * inv * z[e] * la_gate(y[e], gate);
     la_store<T, V>(o + c, x);
 }
 
@@ -619,9 +619,9 @@ __global__ void la_finish_all_kernel(const float* __restrict__ num, const T* __r
 #pragma unroll
         for (int e = 0; e < V; ++e) ss += x[e] * x[e];
     }
-    const float rms = sqrtf(rv_block_sum(ss, scratch) / (float)width + eps);
+    const float inv = 1.f / sqrtf(rv_block_sum(ss, scratch) / (float)width + eps);
     for (int c = threadIdx.x * V; c < width; c += blockDim.x * V)
-        la_finish_at<T, V>(nm, rows + (size_t)t * stride + g_off, norm_w, o, c, rms, gate);
+        la_finish_at<T, V>(nm, rows + (size_t)t * stride + g_off, norm_w, o, c, inv, gate);
 }
 
 // A norm per head: a warp per (token, head).
@@ -650,9 +650,9 @@ __global__ void la_finish_head_kernel(const float* __restrict__ num, const T* __
 #pragma unroll
         for (int e = 0; e < V; ++e) ss += x[e] * x[e];
     }
-    const float rms = sqrtf(rv_warp_sum(ss) / (float)dv + eps);
+    const float inv = 1.f / sqrtf(rv_warp_sum(ss) / (float)dv + eps);
     for (int c = lane * V; c < dv; c += 32 * V)
-        la_finish_at<T, V>(nm, rows + (size_t)t * stride + g_off + h * dv, norm_w + h * dv, o, c, rms, gate);
+        la_finish_at<T, V>(nm, rows + (size_t)t * stride + g_off + h * dv, norm_w + h * dv, o, c, inv, gate);
 }
 
 #include "linear_attention_mma.cuh"

@@ -43,7 +43,6 @@ template <> struct NsVec<4> {
     __device__ __forceinline__ void zero() { v = make_float4(0.f, 0.f, 0.f, 0.f); }
     __device__ __forceinline__ void add(const NsVec& o) { v.x += o.v.x; v.y += o.v.y; v.z += o.v.z; v.w += o.v.w; }
     __device__ __forceinline__ void mul(const NsVec& o) { v.x *= o.v.x; v.y *= o.v.y; v.z *= o.v.z; v.w *= o.v.w; }
-    __device__ __forceinline__ void div(float s) { v.x /= s; v.y /= s; v.z /= s; v.w /= s; }
     __device__ __forceinline__ void scale(float s) { v.x *= s; v.y *= s; v.z *= s; v.w *= s; }
     __device__ __forceinline__ float sq() const { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
     // this + (before - this) * m
@@ -61,7 +60,6 @@ template <> struct NsVec<1> {
     __device__ __forceinline__ void zero() { v = 0.f; }
     __device__ __forceinline__ void add(const NsVec& o) { v += o.v; }
     __device__ __forceinline__ void mul(const NsVec& o) { v *= o.v; }
-    __device__ __forceinline__ void div(float s) { v /= s; }
     __device__ __forceinline__ void scale(float s) { v *= s; }
     __device__ __forceinline__ float sq() const { return v * v; }
     __device__ __forceinline__ NsVec towards(const NsVec& before, const NsVec& m) const {
@@ -179,14 +177,14 @@ __global__ void add_rmsnorm_shift_kernel(
     for (int k = 0; k <= ROWS; ++k) {
         const bool there = k == 0 ? inside[0] : t0 + k - 1 < n_rows;
         if (!there) continue;
-        const float rms = sqrtf(ss[k] / (float)hidden + eps);
+        const float inv = 1.f / sqrtf(ss[k] / (float)hidden + eps);
 #pragma unroll
         for (int c = 0; c < CHUNKS; ++c) {
             const int i = (tid + c * nt) * V;
             if (i >= hidden) continue;
             if (k > 0 && resid_out != resid) x[k][c].store(resid_out + (size_t)(t0 + k - 1) * hidden + i);
             else if (k > 0 && (delta || rows_add || add)) x[k][c].store(resid_out + (size_t)(t0 + k - 1) * hidden + i);
-            x[k][c].div(rms);
+            x[k][c].scale(inv);
             x[k][c].mul(w[c]);                                  // h
         }
     }
@@ -227,12 +225,12 @@ __global__ void add_rmsnorm_shift_kernel(
         NsVec<V> z[CHUNKS];
         float s1[1] = {load_row(last, z)};
         ns_block_sums<1>(s1, scratch);
-        const float rms = sqrtf(s1[0] / (float)hidden + eps);
+        const float inv = 1.f / sqrtf(s1[0] / (float)hidden + eps);
 #pragma unroll
         for (int c = 0; c < CHUNKS; ++c) {
             const int i = (tid + c * nt) * V;
             if (i < hidden) {
-                z[c].div(rms);
+                z[c].scale(inv);
                 z[c].mul(w[c]);
                 z[c].store(rec + i);
             }

@@ -10,8 +10,8 @@ out through one norm over all heads and a sigmoid gate; or half the sum of two m
 each normed over the model's width: a grouped-query attention whose values are its unrotated
 keys (YaRN-scaled rotation, capped scores, a learned sink, a window of tokens and before it one
 mean key and value per block), and a linear attention with a decay per key channel, read out
-through a norm per head and a silu gate.  The feed-forward is a mixture of experts weighed by the
-softmax over the chosen logits, plus a shared expert.  Layers [start, stop) may run several times
+through a norm per head and a silu gate.  The feed-forward is a mixture of gated experts whose
+weights come from the chosen experts' logits only, with one more expert for all tokens.  Layers [start, stop) may run several times
 with the same weights: every pass has caches of its own, begins by adding its row of `loop.step`
 to the stream and, from the second on, the embedding rows once more.  The head is a matrix of
 its own.

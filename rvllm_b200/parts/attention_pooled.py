@@ -1,11 +1,12 @@
 """Grouped-query attention over a window of tokens and the pooled blocks before it
 (`PooledAttentionSpec`).
 
-The query at position i sees the tokens j with i - window < j <= i and, for each block of `pool`
-tokens that lies wholly before the window, one key and one value: the means of the block's
-cached keys and values.  Tokens and blocks share one softmax, whose denominator may hold one more
-term exp(sink_h); scores may be capped, c tanh(s / c).  Values may be the keys as projected,
-before the rotation.
+A query weighs two kinds of rows in the same softmax.  Its own position and the window - 1 before
+it are single tokens.  What is older is there as means: every `pool` consecutive positions (0 to
+pool - 1, and so on) give one key and one value, the means of what the pages hold for them, and a
+query at i takes the first max(0, i - window + 1) // pool of these.  So between the newest mean it
+takes and its window up to pool - 1 positions are hidden from it.  Options: a further term
+exp(sink_h) in the denominator; capped scores, c tanh(s / c); keys that serve, unrotated, as values.
 
 Two page groups serve a call: the tokens' keys and values, whose pages are given back once they
 lie before the window *and* before the newest incomplete block, and one row per block, which is

@@ -55,11 +55,10 @@ class PositionSpec:
     l > original / low, and in between is (1 - s) f / factor + s f with
     s = (original / l - low) / (high - low).
     `yarn` = (factor, original, fast, slow) (kind "rope_partial"; "YaRN: Efficient Context Window
-    Extension of Large Language Models", Peng et al.): with
-    dim(t) = n ln(original / (2 pi t)) / (2 ln theta) for n turning dimensions, lo =
-    max(floor(dim(fast)), 0) and hi = min(ceil(dim(slow)), n - 1), frequency f_i becomes
-    r_i f_i / factor + (1 - r_i) f_i with r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), and
-    cosine and sine are multiplied by 0.1 ln(factor) + 1."""
+    Extension of Large Language Models", Peng et al.): pairs that make more than `fast` turns over
+    `original` positions keep their frequency, those of fewer than `slow` turns are slowed down
+    by `factor`, and in between the share of the slowed one grows linearly with the pair's
+    index (`PartialRope` has the bounds); cosine and sine grow by 1 + ln(factor) / 10."""
     kind: str
     head_dim: int = 0
     theta: float = 0.0
@@ -166,11 +165,10 @@ class MixedAttentionSpec(AttentionSpec):
 class PooledAttentionSpec(AttentionSpec):
     """Grouped-query attention over a window of tokens and, before the window, pooled blocks.
 
-    pool             tokens per block P (None: no blocks).  The query at position i sees, besides
-                     the tokens of its window, block b (positions bP .. bP + P - 1) once
-                     bP + P - 1 <= i - window; its key and value are the means of the block's
-                     cached keys and values.  A token that has left the window and whose
-                     block is not seen yet is not seen.  One softmax over both.
+    pool             tokens per block P (None: no blocks).  A query at i takes its window's tokens
+                     and the means (of keys and of values, as cached) of the first
+                     max(0, i - window + 1) // P blocks; the fewer than P positions between
+                     the two are hidden from it until their block is full and old enough
     softcap          c: scores become c tanh(score / c) after the scale
     values_are_keys  a token's value is its key before the rotation (no "v" tensor)
     `sinks` (tensor "sink" [heads]) as in the base class; the position kind is "rope_partial" or
@@ -317,8 +315,8 @@ class MoESpec(FeedForwardSpec):
     `activation` "relu2": experts without a gate, down_e(max(up_e x, 0)^2); `choice_bias`: a
     learned number per expert (tensor "correction" [experts]) is added to the scores where
     experts are compared, while the weights are made from the scores without it; score
-    "softmax_chosen": the logits themselves are compared and the weights are the softmax over the
-    chosen logits alone."""
+    "softmax_chosen": the logits themselves are compared, and the chosen ones, exponentiated and
+    divided by their own sum, are the weights."""
     ffn_dim: int = 0
     experts: int = 0
     top: int = 0

@@ -3,8 +3,8 @@ plainest form.  It shares no code with the package: the tests compare the engine
 
 A model is a dict `cfg` (the nested config.json of the design) and a dict of float64 arrays
 by tensor name.  `forward(cfg, w, tokens)` gives the logits of every position of one
-sequence; `forward(..., layers_out=[])` also collects the residual stream after every layer
-run (a layer inside the repeated stretch counts once per pass).
+sequence; `forward(..., layers_out=[])` also collects the stream as every layer's run leaves it
+(a layer of the repeated stretch once for every pass).
 
     start:   e = N(scale * embed[token] + pos[p]) * g_embed;  x = e
     layer:   h = N(x) * g1;  h_p <- h_p + (h_(p-1) - h_p) * shift  (h_(-1) = 0)
@@ -96,8 +96,8 @@ def attend(q, keys, values, scale, cap, sink):
 
 
 def pooled_window_attention(h, m, t):
-    """Grouped heads whose values are the unrotated keys; a window of tokens and, before it, one
-    mean key and value for each block of tokens that lies wholly before the window."""
+    """Grouped heads whose values are the unrotated keys; a window of single tokens, and older
+    tokens as the mean keys and values of full blocks."""
     H, G, d = m["heads"], m["kv_heads"], m["dim"]
     size, P = m["mask"]["size"], m["mask"]["pool"]
     T = h.shape[0]

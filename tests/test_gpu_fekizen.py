@@ -364,9 +364,9 @@ def test_pooled_attention_every_visible_key(ops, dtype, sizes, window, pool, cap
 @pytest.mark.parametrize("dtype,sizes", [SHAPES[0], SHAPES[2], SHAPES[4]])
 @pytest.mark.parametrize("decoded", [True, False])
 def test_one_key_stands_out_at_every_edge(ops, dtype, sizes, decoded):
-    """For one query the key just inside the window, the last outside it, a token that has left the
-    window and whose block is not seen yet, the first and last token of the newest seen block and
-    of the oldest one, page borders: each made the one whose score stands out."""
+    """For one query the window's oldest key and the one before it, a position hidden between the
+    window and the newest mean, the ends of the newest mean's block, of the one after it and of the
+    oldest, page borders: each made the one whose score stands out."""
     window, pool, page, n = 40, 8, 16, 200
     P = n - 1                                                # the last query
     nb = plain.seen_blocks(P, window, pool)
