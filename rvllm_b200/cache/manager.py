@@ -17,7 +17,8 @@ factor; every live request may begin a page of its own, so the pool has one page
 A request's pages are given back when it ends (`free`) and, in a group whose reach
 is bounded (a window, or chunks that do not see one another), as soon as every slot of
 the page lies behind what any future query can see (`advance`).  Released block-table entries read -1; no kernel touches them because
-the window bound excludes their positions.
+the window bound excludes their positions.  Where a window keeps its first positions visible, their
+pages stay as long as the request lives.
 
 In the reference the same duties are split between `KvStorage` (per-layer K and V
 tensors [num_blocks, block_size, kv_heads, head_dim], src/kv_storage.rs:7, 92-98),
@@ -303,7 +304,9 @@ class CacheManager:
         freed = 0
         for gi, grp in enumerate(self.groups):
             first = min(self._first_needed_page(grp, computed), len(rc.tables[gi]))
-            for p in range(rc.first_live[gi], first):
+            # the pages of positions that stay visible for good are never given back before the end
+            kept = -(-grp.need.rows(grp.need.keep_first) // self.page_size)
+            for p in range(max(rc.first_live[gi], kept), first):
                 grp.pool.free(rc.tables[gi][p])
                 rc.tables[gi][p] = -1
                 freed += 1

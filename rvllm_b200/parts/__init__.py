@@ -2,7 +2,8 @@
 encodings and their arrangement in a block.  Importing the package registers the
 built-in kinds."""
 from . import (attention, attention_latent, attention_mixed, attention_pooled, block, feed_forward, gated_delta,  # noqa: F401
-               hyper, linear_attention, mingru, mlstm, norm, parallel, position, short_conv)
+               hyper, linear_attention, mingru, mlstm, norm, parallel, position, short_conv,
+               state_space)
 from .base import (Arrangement, FeedForward, Mixer, Norm, PagedNeed, PositionEncoding,
                    SeveralNeeds, StateNeed, Stream, arrangement_class, feed_forward_class, mixer_class,
                    norm_class, position_class, register_arrangement,
@@ -12,4 +13,4 @@ from .spec import (AttentionSpec, BlockSpec, FeedForwardSpec, LayerCall, MixerSp
                    ModelSpec, NormSpec, ParamDecl, PositionSpec, ShortConvSpec, SwiGLUSpec,
                    DenseSpec, MinGRUSpec, MixedAttentionSpec, LatentAttentionSpec, MoESpec,
                    GatedDeltaSpec, GluClampSpec, MLSTMSpec, ParallelSpec,
-                   LinearAttentionSpec, PooledAttentionSpec)
+                   LinearAttentionSpec, PooledAttentionSpec, StateSpaceSpec)

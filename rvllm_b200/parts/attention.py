@@ -31,11 +31,18 @@ product; W_g's rows ride at the end of the q|k|v product and `ops.head_gate` app
 A third form (`_prepared`), chosen by any of: biases on the q, k and v projections (`bias`); a
 norm over the whole query projection and one over the whole key projection, before the split
 into heads (`qk_norm` of kind "rms_full"); a rotation of neighbouring dimensions (position
-kind "rope_pairs"); value mixing (`value_mix`): the first such call of a step keeps its values
+kind "rope_pairs") or of the first dimensions of a head by halves ("rope_partial"); value mixing (`value_mix`): the first such call of a step keeps its values
 ("source"), every later one caches v <- (1 - l) v + l v_source with its learned scalar l.  The
 q|k|v product stays float32 and one kernel (`ops.qkv_full_norm_rope_write`) adds the biases,
 normalises, rotates, mixes and writes the cache.  A sink, a window and a value size of its own
 go with it.
+
+With a window, the first `keep_first` positions can stay visible for good: the query at p sees j iff
+j <= p and (p - j < window or j < keep_first), and the kept tokens keep their positions.  Before
+its window a query then sees min(keep_first, max(0, p - window + 1)) more rows of the same pages,
+which is what the attention over a window and older rows (`ops.paged_attention_pooled`) computes,
+with rows of one token; the cache manager keeps those pages.  `out_bias`: a bias on the output
+product.
 """
 from __future__ import annotations
 
@@ -55,7 +62,8 @@ class Attention(Mixer):
                 ("q_proj", "k_proj", "v_proj", "out_proj", "q_norm", "k_norm", "sink")} | \
             {"head_gate": n.get("head_gate", "g")} | \
             {k: n.get(k, d) for k, d in (("q_bias", "q_proj.bias"), ("k_bias", "k_proj.bias"),
-                                         ("v_bias", "v_proj.bias"), ("vmix", "vmix"))}
+                                         ("v_bias", "v_proj.bias"), ("vmix", "vmix"),
+                                         ("out_bias", "out_proj.bias"))}
 
     @staticmethod
     def params(spec: AttentionSpec, owns_cache: bool = True):
@@ -77,6 +85,10 @@ class Attention(Mixer):
             if owns_cache:
                 p[n["k_bias"]] = ParamDecl((kd,), "bias")
                 p[n["v_bias"]] = ParamDecl((spec.num_kv_heads * dv,), "bias")
+        if spec.out_bias:
+            p[n["out_bias"]] = ParamDecl((spec.hidden,), "bias")
+        if spec.keep_first and (spec.keep_first < 0 or not spec.window):
+            raise ValueError("attention: first tokens are kept before a window")
         if spec.value_mix is not None:
             if spec.value_mix not in ("source", "mix"):
                 raise ValueError(f"attention: value_mix is 'source' or 'mix', "
@@ -98,7 +110,8 @@ class Attention(Mixer):
     @staticmethod
     def _prepared(spec) -> bool:
         """Whether the layer takes the form served by `ops.qkv_full_norm_rope_write`."""
-        return spec.bias or spec.value_mix is not None or spec.position.kind == "rope_pairs" \
+        return spec.bias or spec.value_mix is not None \
+            or spec.position.kind in ("rope_pairs", "rope_partial") \
             or (spec.qk_norm is not None and spec.qk_norm.kind == "rms_full")
 
     @staticmethod
@@ -112,10 +125,16 @@ class Attention(Mixer):
     def cache_need(spec: AttentionSpec):
         dv = spec.v_head_dim or spec.head_dim
         return PagedNeed(spec.num_kv_heads, spec.head_dim, spec.window,
-                         v_head_dim=dv if dv != spec.head_dim else None)
+                         v_head_dim=dv if dv != spec.head_dim else None,
+                         keep_first=spec.keep_first)
 
     @staticmethod
     def workspace_bytes(spec: AttentionSpec, ops, max_requests: int, max_context: int) -> int:
+        if spec.keep_first:
+            sizer = getattr(ops, "attention_pooled_scratch_bytes", None)
+            return 0 if sizer is None else sizer(
+                max_requests, spec.num_heads, spec.v_head_dim or spec.head_dim, max_context,
+                spec.window, 1, spec.keep_first)
         sizer = getattr(ops, "attention_scratch_bytes", None)
         if sizer is None:
             return 0
@@ -154,6 +173,7 @@ class Attention(Mixer):
         self.w_q = self.w_qkv[:spec.num_heads * spec.head_dim] if not spec.head_gate else \
             fused([q])
         self.w_out = tensors[n["out_proj"]].contiguous()
+        self.b_out = tensors[n["out_bias"]].to(torch.float32).contiguous() if spec.out_bias else None
         self.q_norm = self.k_norm = None
         self.v_dim = spec.v_head_dim or spec.head_dim
         self.sinks = None
@@ -197,10 +217,21 @@ class Attention(Mixer):
             self.position.rotation_table(), ctx.positions, group.slot_mapping,
             cache.k if owns else None, cache.v if owns else None, out_dtype=self.dtype)
         out = self.ops.new_rows(normed.shape[0], s.num_heads * s.head_dim, self.dtype, normed.device)
-        self.ops.paged_attention(qkv, s.num_heads, s.num_kv_heads, s.head_dim,
+        self._attend(qkv, cache, ctx, group, out)
+        return self.ops.linear(out, self.w_out, bias=self.b_out, out_dtype=self.dtype)
+
+    def _attend(self, rows, cache, ctx, group, out):
+        s = self.spec
+        if s.keep_first:
+            self.ops.paged_attention_pooled(
+                rows, s.num_heads, s.num_kv_heads, s.head_dim, cache.k, cache.v, ctx, group,
+                (cache.k, cache.v, group, 1), self.scale, None, s.window, self.sinks, out,
+                v_head_dim=self.v_dim, most_blocks=s.keep_first)
+            return
+        options = {} if self.v_dim == s.head_dim else {"v_head_dim": self.v_dim}
+        self.ops.paged_attention(rows, s.num_heads, s.num_kv_heads, s.head_dim,
                                  cache.k, cache.v, ctx, group, self.scale, s.window, out,
-                                 sinks=self.sinks)
-        return self.ops.linear(out, self.w_out, out_dtype=self.dtype)
+                                 sinks=self.sinks, **options)
 
     def _forward_options(self, normed, ctx, cache, group):
         s = self.spec
@@ -216,14 +247,11 @@ class Attention(Mixer):
                                cache.k if owns else None, cache.v if owns else None)
         out = self.ops.new_rows(normed.shape[0], s.num_heads * self.v_dim, self.dtype,
                                 normed.device)
-        self.ops.paged_attention(rows, s.num_heads, s.num_kv_heads, s.head_dim,
-                                 cache.k, cache.v, ctx, group, self.scale, s.window, out,
-                                 sinks=self.sinks, v_head_dim=self.v_dim)
+        self._attend(rows, cache, ctx, group, out)
         if s.head_gate:
             self.ops.head_gate(out, s.num_heads, self.v_dim, rows,
                                s.num_heads * s.head_dim + kv * (s.head_dim + self.v_dim))
-        return self.ops.linear(out, self.w_out, out_dtype=self.dtype)
-
+        return self.ops.linear(out, self.w_out, bias=self.b_out, out_dtype=self.dtype)
 
     CARRY_VALUES = "attention.source_values"
 
@@ -234,8 +262,9 @@ class Attention(Mixer):
                                        spec.qk_norm.kind not in ("rms_full",)):
             raise ValueError("attention: biases, a whole-projection norm, a pairwise rotation "
                              "and value mixing go with no other q/k norm and no temperature")
-        if spec.position.kind not in ("rope_pairs", "none"):
-            raise ValueError("attention: this form turns neighbouring dimensions or none")
+        if spec.position.kind not in ("rope_pairs", "rope_partial", "none"):
+            raise ValueError("attention: this form turns neighbouring dimensions, a head's first "
+                             "dimensions by halves, or none")
 
     def _forward_prepared(self, normed, ctx, cache, group):
         s = self.spec
@@ -255,15 +284,19 @@ class Attention(Mixer):
                 raise ValueError("attention: values are mixed with those of an earlier call of "
                                  "the step, and none of this shape ran")
         freq, rot_dims = (None, 0) if s.position.kind == "none" else self.position.frequencies()
+        options = {}
+        if s.position.kind == "rope_partial":
+            options = dict(pairs=False, amplitude=self.position.amplitude)
+        elif s.position.kind == "rope_pairs" and self.position.amplitude != 1.0:
+            options = dict(amplitude=self.position.amplitude)
         self.ops.qkv_full_norm_rope_write(
             rows, self.bias, s.num_heads, s.num_kv_heads, s.head_dim, self.v_dim, self.q_norm,
             self.k_norm, s.qk_norm.eps if s.qk_norm is not None else 0.0, freq, rot_dims,
-            ctx.positions, group.slot_mapping, q, cache.k, cache.v, first_in, first_out, self.vmix)
+            ctx.positions, group.slot_mapping, q, cache.k, cache.v, first_in, first_out, self.vmix,
+            **options)
         out = self.ops.new_rows(n, s.num_heads * self.v_dim, self.dtype, normed.device)
-        self.ops.paged_attention(q, s.num_heads, s.num_kv_heads, s.head_dim, cache.k, cache.v,
-                                 ctx, group, self.scale, s.window, out, sinks=self.sinks,
-                                 v_head_dim=self.v_dim)
-        return self.ops.linear(out, self.w_out, out_dtype=self.dtype)
+        self._attend(q, cache, ctx, group, out)
+        return self.ops.linear(out, self.w_out, bias=self.b_out, out_dtype=self.dtype)
 
 
 register_mixer("attention", Attention)

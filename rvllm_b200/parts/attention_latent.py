@@ -31,7 +31,10 @@ query carried into that space is [W_uk[h]^T q_h[:d] | turn_p(q_h[d:])]: one per-
 with the matrix [[W_uk[h], 0], [0, 1]].  Attention is the same paged attention with one shared
 head of size kv_rank + rot_dim whose values are its keys; the turned part of its result meets
 zero rows of the matrix that carries it out ([W_uv[h]^T; 0]), so nothing but sizes changed.
-W_dq and W_dkv are one product; the two norms, the turn of the key part and the cache write
+The turned part turns by halves or pair by pair (`rot_pairs`), with plain or YaRN-scaled frequencies
+(`rot_yarn`, whose amplitude multiplies queries' and keys' turned parts).  `window`: a query sees
+only the last so many positions, and the cache manager takes the older rows' pages back.  W_dq and
+W_dkv are one product; the two norms, the turn of the key part and the cache write
 are one kernel (`ops.latent_prepare`), the turn of the queries another (`ops.rope_heads`).
 """
 from __future__ import annotations
@@ -79,7 +82,7 @@ class LatentAttention(Mixer):
 
     @staticmethod
     def cache_need(spec: LatentAttentionSpec):
-        return PagedNeed(1, spec.kv_rank + spec.rot_dim, values=False)
+        return PagedNeed(1, spec.kv_rank + spec.rot_dim, spec.window, values=False)
 
     @staticmethod
     def workspace_bytes(spec: LatentAttentionSpec, ops, max_requests: int, max_context: int) -> int:
@@ -109,6 +112,7 @@ class LatentAttention(Mixer):
         self.w_uq = tensors[n["uq"]].contiguous() if qr else None
         w_uk = tensors[n["uk"]].reshape(H, d, R)
         w_uv_t = tensors[n["uv"]].reshape(H, dv, R).transpose(1, 2)
+        self.turn = {}
         if rot:
             # [[W_uk, 0], [0, 1]] carries [q plain | q turned] into [latent | turned] space, and
             # [W_uv^T; 0] drops the turned part of what comes back
@@ -118,9 +122,16 @@ class LatentAttention(Mixer):
             uv = torch.zeros((H, R + rot, dv), dtype=w_uk.dtype, device=w_uk.device)
             uv[:, :R] = w_uv_t
             w_uk, w_uv_t = uk, uv
-            self.freq = position_class("rope_partial")(
-                PositionSpec("rope_partial", head_dim=rot, theta=spec.rot_theta, rot_dims=rot),
-                q.device).frequencies()[0]
+            kind = "rope_pairs" if spec.rot_pairs else "rope_partial"
+            position = position_class(kind)(
+                PositionSpec(kind, head_dim=rot, theta=spec.rot_theta, rot_dims=rot,
+                             yarn=spec.rot_yarn), q.device)
+            self.freq = position.frequencies()[0]
+            # what the kernels that turn are told beyond the frequencies (nothing at the defaults)
+            if spec.rot_pairs:
+                self.turn["pairs"] = True
+            if position.amplitude != 1.0:
+                self.turn["amplitude"] = position.amplitude
         self.w_uk = w_uk.contiguous()                  # [H, d + rot, R + rot]
         self.w_uv_t = w_uv_t.contiguous()              # [H, R + rot, dv]
         self.w_out = tensors[n["o"]].contiguous()
@@ -149,19 +160,19 @@ class LatentAttention(Mixer):
         if owns:
             self.ops.latent_prepare(rows, 0, qr, self.q_norm, cq, kv_off, R, rot,
                                     self.latent_norm, s.norm_eps, self.freq if rot else None,
-                                    ctx.positions, group.slot_mapping, cache.k)
+                                    ctx.positions, group.slot_mapping, cache.k, **self.turn)
         elif qr:
             cq = self.ops.new_rows(n, qr, self.dtype, normed.device)
             self.ops.add_rmsnorm(None, rows[:, :qr].contiguous(), self.q_norm, s.norm_eps, cq, None)
         q = self.ops.linear(cq, self.w_uq, out_dtype=self.dtype) if qr else rows
         if rot:
-            self.ops.rope_heads(q, H, d + rot, d, rot, self.freq, ctx.positions)
+            self.ops.rope_heads(q, H, d + rot, d, rot, self.freq, ctx.positions, **self.turn)
         # queries into the space of the page slots: [n, H, d + rot] x [H, d + rot, R + rot]
         q_lat = self.ops.new_rows(n, H * (R + rot), self.dtype, normed.device)
         self.ops.heads_product(q, 0, H, d + rot, self.w_uk, q_lat)
         mixed = self.ops.new_rows(n, H * (R + rot), self.dtype, normed.device)
         self.ops.paged_attention(q_lat, H, 1, R + rot, cache.k, cache.k, ctx, group, self.scale,
-                                 None, mixed, sinks=self.sinks)
+                                 s.window, mixed, sinks=self.sinks)
         out = self.ops.new_rows(n, H * dv, self.dtype, normed.device)
         self.ops.heads_product(mixed, 0, H, R + rot, self.w_uv_t, out,
                                gate_rows=rows if s.out_gate else None, gate_off=gate_off)
@@ -186,7 +197,7 @@ class LatentAttention(Mixer):
         q_lat = self.ops.new_rows(n, H * R, self.dtype, normed.device)
         self.ops.heads_product(rows, 0, H, d, self.w_uk, q_lat)
         mixed = self.ops.new_rows(n, H * R, self.dtype, normed.device)
-        self.ops.paged_attention(q_lat, H, 1, R, cache.k, cache.k, ctx, group, self.scale, None,
+        self.ops.paged_attention(q_lat, H, 1, R, cache.k, cache.k, ctx, group, self.scale, s.window,
                                  mixed, sinks=self.sinks)
         # and out of it: [n, H, R] x [H, R, dv] -> [n, H, dv]
         out = self.ops.new_rows(n, H * dv, self.dtype, normed.device)

@@ -33,7 +33,8 @@ class PagedNeed:
     keys and values are both made from); no value pages exist.  `every` > 1: one row per `every`
     tokens (made from them when the last of them is written) instead of one per token.  `block`:
     the rows of the newest incomplete block of `block` positions are read once more when it
-    completes, so their pages stay until then whatever the window says."""
+    completes, so their pages stay until then whatever the window says.  `keep_first`: the first so
+    many positions stay visible whatever the window says, and so do their pages."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
@@ -42,6 +43,7 @@ class PagedNeed:
     values: bool = True
     every: int = 1
     block: Optional[int] = None
+    keep_first: int = 0
 
     @property
     def value_dim(self) -> int:
@@ -147,6 +149,10 @@ class Norm:
     def norm(self, x, ctx):
         """The normalised rows of `x` (compute dtype), with no residual stream involved:
         what a norm placed after a sub-layer applies to its output."""
+        raise NotImplementedError
+
+    def scale_output(self, factor: float) -> None:
+        """From now on the normalised rows come out times `factor` (the weights take it in)."""
         raise NotImplementedError
 
 

@@ -162,7 +162,9 @@ class MoE(FeedForward):
     (`activation` "relu2": no "gate" tensors, the stack is [experts, ffn, hidden]); a learned
     number per expert that is added to the scores where experts are compared and nowhere else
     (`choice_bias`, tensor "correction"); logits that are compared as they are and weighed by the
-    softmax over the chosen ones (score "softmax_chosen").
+    softmax over the chosen ones (score "softmax_chosen"); `identity` further router outputs whose
+    output, when chosen, is the token's own row times the weight: they take part in scores, groups
+    and choice like experts, and the kernels that add up a token's experts read the row itself.
     """
     SCORES = ("sigmoid", "softmax", "softmax_chosen")
     ACTIVATIONS = ("swiglu", "glu_clamp", "relu2")
@@ -183,23 +185,24 @@ class MoE(FeedForward):
         if spec.activation not in MoE.ACTIVATIONS:
             raise ValueError(f"unknown expert activation {spec.activation!r} "
                              f"(known: {MoE.ACTIVATIONS})")
-        if spec.experts < 1 or not 1 <= spec.top <= spec.experts:
-            raise ValueError(f"a mixture of {spec.experts} experts cannot use {spec.top} a token")
-        if spec.groups < 1 or spec.experts % spec.groups or not 1 <= spec.keep <= spec.groups:
-            raise ValueError(f"{spec.experts} experts do not form {spec.groups} equal groups "
+        outputs = spec.outputs
+        if spec.experts < 1 or spec.identity < 0 or not 1 <= spec.top <= outputs:
+            raise ValueError(f"a mixture of {outputs} experts cannot use {spec.top} a token")
+        if spec.groups < 1 or outputs % spec.groups or not 1 <= spec.keep <= spec.groups:
+            raise ValueError(f"{outputs} experts do not form {spec.groups} equal groups "
                              f"of which {spec.keep} are kept")
-        if spec.keep * (spec.experts // spec.groups) < spec.top:
-            raise ValueError(f"{spec.keep} groups of {spec.experts // spec.groups} experts "
+        if spec.keep * (outputs // spec.groups) < spec.top:
+            raise ValueError(f"{spec.keep} groups of {outputs // spec.groups} experts "
                              f"cannot give {spec.top} experts")
 
     @staticmethod
     def params(spec: MoESpec):
         MoE._check(spec)
         n = MoE._names(spec)
-        p = {n["router"]: ParamDecl((spec.experts, spec.hidden), "normal", mean=0.0,
+        p = {n["router"]: ParamDecl((spec.outputs, spec.hidden), "normal", mean=0.0,
                                     std=spec.hidden ** -0.5)}
         if spec.choice_bias:
-            p[n["correction"]] = ParamDecl((spec.experts,), "normal", mean=0.0, std=0.1)
+            p[n["correction"]] = ParamDecl((spec.outputs,), "normal", mean=0.0, std=0.1)
         for e in range(spec.experts):
             if spec.activation != "relu2":
                 p[n[(e, "gate")]] = ParamDecl((spec.ffn_dim, spec.hidden), "linear")
@@ -258,6 +261,8 @@ class MoE(FeedForward):
             extra = dict(activation=s.activation, limit=s.limit, alpha=s.alpha)
         if self.shared is not None:
             extra["addend"] = self.shared.forward(normed, ctx).contiguous()
+        if s.identity:
+            extra["identity"] = s.identity
         self.ops.moe_experts(normed, ids, weights, self.gate_up, self.down, out, **extra)
         return out
 

@@ -108,6 +108,8 @@ class Model:
         self.head = (tensors[spec.head_name].contiguous() if spec.head_name is not None
                      else self.embedding)
         self.final_norm = build_norm(spec.final_norm, spec.final_norm_name, tensors, ops, dtype)
+        if spec.logit_scale != 1.0:
+            self.final_norm.scale_output(spec.logit_scale)     # the head's input carries the factor
         self.embedding_norm = None
         if spec.embedding_norm is not None:
             self.embedding_norm = build_norm(*spec.embedding_norm, tensors, ops, dtype)
@@ -141,8 +143,10 @@ class Model:
             needs.append(None)
             own = needs[call.cache_of]
             if isinstance(own, PagedNeed) and isinstance(need, PagedNeed) and \
-                    (own.window, own.chunk) != (need.window, need.chunk):
-                needs[call.cache_of] = dataclasses.replace(own, window=None, chunk=None)
+                    (own.window, own.chunk, own.keep_first) != \
+                    (need.window, need.chunk, need.keep_first):
+                needs[call.cache_of] = dataclasses.replace(own, window=None, chunk=None,
+                                                           keep_first=0)
         return needs
 
     def forward(self, ctx, caches) -> torch.Tensor:

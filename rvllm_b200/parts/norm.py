@@ -61,6 +61,9 @@ class RMSNorm(Norm):
                                    add=add, add_rows=add_rows)
         return new, out
 
+    def scale_output(self, factor: float) -> None:
+        self.weight = (self.weight * factor).contiguous()
+
     def norm_f32(self, x):
         """The normalised float32 rows of float32 `x`: rows that go on as the residual stream."""
         out = torch.empty_like(x)
@@ -108,7 +111,12 @@ class LayerNorm(Norm):
         self.ops = ops
         self.dtype = dtype
         self.weight = tensors["weight"].to(torch.float32).contiguous()
-        self.bias = tensors["bias"].to(torch.float32).contiguous()
+        self.bias = tensors["bias"].to(torch.float32).contiguous() if "bias" in tensors else None
+
+    def scale_output(self, factor: float) -> None:
+        self.weight = (self.weight * factor).contiguous()
+        if self.bias is not None:
+            self.bias = (self.bias * factor).contiguous()
 
     def add_norm(self, resid, delta, ctx, rows=None, delta_norm=None):
         n = resid.shape[0] if rows is None else rows.shape[0]
@@ -128,6 +136,15 @@ class LayerNorm(Norm):
         return out
 
 
+class WeightLayerNorm(LayerNorm):
+    """LayerNorm without a bias."""
+
+    @staticmethod
+    def params(spec: NormSpec):
+        return {"weight": ParamDecl((spec.size,), "norm")}
+
+
+register_norm("layernorm_weight", WeightLayerNorm)
 register_norm("rmsnorm", RMSNorm)
 register_norm("rmsnorm_scalar", ScalarRMSNorm)
 register_norm("layernorm", LayerNorm)

@@ -19,6 +19,26 @@ from .spec import PositionSpec
 _TABLES = {}
 
 
+def yarn_frequencies(f, dims: int, theta: float, yarn):
+    """(frequencies, amplitude) of a rotation of `dims` dimensions with frequencies `f` (float64
+    [dims/2]) stretched as `PositionSpec.yarn` says: with dim(t) = dims ln(original / (2 pi t)) /
+    (2 ln theta), the dimension that makes t turns over the original length, pair i's share of the
+    slowed frequency grows from 0 at floor(dim(fast)) to 1 at ceil(dim(slow)), both bounded to
+    [0, dims - 1]."""
+    factor, original, fast, slow = yarn
+    if not (factor > 0 and original > 0 and fast > 0 and slow > 0 and theta > 1):
+        raise ValueError("rotation: the scaling needs positive numbers and a base above 1")
+
+    def dim(turns):
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+
+    lo = max(math.floor(dim(fast)), 0)
+    hi = min(math.ceil(dim(slow)), dims - 1)
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return f / factor * ramp + f * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
 class Rope(PositionEncoding):
     def __init__(self, spec: PositionSpec, device):
         if spec.head_dim % 2:
@@ -58,21 +78,7 @@ class PartialRope(PositionEncoding):
         i = torch.arange(dims // 2, dtype=torch.float64)
         f = torch.pow(torch.tensor(spec.theta, dtype=torch.float64), -2.0 * i / max(dims, 1))
         if spec.yarn is not None:
-            factor, original, fast, slow = spec.yarn
-            if not (factor > 0 and original > 0 and fast > 0 and slow > 0 and spec.theta > 1):
-                raise ValueError("rope_partial: the scaling needs positive numbers and a base "
-                                 "above 1")
-
-            def dim(turns):
-                """The dimension that makes this many turns over the original length."""
-                return dims * math.log(original / (2.0 * math.pi * turns)) / \
-                    (2.0 * math.log(spec.theta))
-
-            lo = max(math.floor(dim(fast)), 0)
-            hi = min(math.ceil(dim(slow)), dims - 1)
-            ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
-            f = f / factor * ramp + f * (1.0 - ramp)
-            self.amplitude = 0.1 * math.log(factor) + 1.0
+            f, self.amplitude = yarn_frequencies(f, dims, spec.theta, spec.yarn)
         self.inv_freq = f.to(torch.float32).to(device).contiguous()
 
     def rotation_table(self):
@@ -87,7 +93,7 @@ class PairRope(PositionEncoding):
     """A rotation of neighbouring dimensions: in each head the pair (2i, 2i + 1), i < rot_dims/2,
     at position p turns by p * f_i with f_i = theta^(-2i/rot_dims); the dimensions from rot_dims
     on pass.  With `scaling` = (factor, low, high, original) long wavelengths are stretched
-    (see `PositionSpec`).  As with `PartialRope` the kernels form the angle in float32 from
+    (see `PositionSpec`); with `yarn` as `PartialRope`'s are.  As with `PartialRope` the kernels form the angle in float32 from
     the position and `frequencies()`, so no longest context has to be known."""
 
     def __init__(self, spec: PositionSpec, device):
@@ -109,6 +115,11 @@ class PairRope(PositionEncoding):
             between = (1.0 - s) * f / factor + s * f
             f = torch.where(wavelength < original / high, f,
                             torch.where(wavelength > original / low, f / factor, between))
+        self.amplitude = 1.0
+        if spec.yarn is not None:
+            if spec.scaling is not None:
+                raise ValueError("rope_pairs: one kind of scaling at a time")
+            f, self.amplitude = yarn_frequencies(f, dims, spec.theta, spec.yarn)
         self.inv_freq = f.to(torch.float32).to(device).contiguous()
 
     def rotation_table(self):

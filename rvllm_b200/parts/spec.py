@@ -54,11 +54,11 @@ class PositionSpec:
     l = 2 pi / f a frequency stays when l < original / high, becomes f / factor when
     l > original / low, and in between is (1 - s) f / factor + s f with
     s = (original / l - low) / (high - low).
-    `yarn` = (factor, original, fast, slow) (kind "rope_partial"; "YaRN: Efficient Context Window
+    `yarn` = (factor, original, fast, slow) (both partial kinds; "YaRN: Efficient Context Window
     Extension of Large Language Models", Peng et al.): pairs that make more than `fast` turns over
     `original` positions keep their frequency, those of fewer than `slow` turns are slowed down
     by `factor`, and in between the share of the slowed one grows linearly with the pair's
-    index (`PartialRope` has the bounds); cosine and sine grow by 1 + ln(factor) / 10."""
+    index (`yarn_frequencies` has the bounds); cosine and sine grow by 1 + ln(factor) / 10."""
     kind: str
     head_dim: int = 0
     theta: float = 0.0
@@ -103,6 +103,9 @@ class AttentionSpec(MixerSpec):
     head_gate: bool = False                     # head j's result is multiplied by
                                                 # sigmoid(W_g x)_j, one number per head (tensor
                                                 # "g" [heads, hidden]), before the output product
+    keep_first: int = 0                         # with a window: the first so many positions stay
+                                                # visible for good, at their true positions
+    out_bias: bool = False                      # the output projection has a bias
 
 
 @dataclass(frozen=True)
@@ -124,6 +127,10 @@ class LatentAttentionSpec(MixerSpec):
                 turned by the position (rotate-half over the whole part, frequencies
                 rot_theta^(-2i/rot_dim)); the turned key part is shared by all heads, cached
                 beside the latent row, and the score is the sum of both parts' products
+    rot_pairs   the turned part turns neighbouring dimensions (2i, 2i + 1) together instead
+    rot_yarn    (factor, original, fast, slow): the frequencies are scaled as `PositionSpec.yarn`
+                says, and the turned parts of queries and keys grow with its amplitude
+    window      a query sees its own position and the window - 1 before it (None: all)
     """
     num_heads: int = 0
     head_dim: int = 0
@@ -137,6 +144,9 @@ class LatentAttentionSpec(MixerSpec):
     q_rank: int = 0
     rot_dim: int = 0
     rot_theta: float = 10000.0
+    rot_pairs: bool = False
+    rot_yarn: Optional[Tuple[float, float, float, float]] = None
+    window: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -216,11 +226,18 @@ class MinGRUSpec(MixerSpec):
 
 @dataclass(frozen=True)
 class GatedDeltaSpec(MixerSpec):
-    """The gated delta rule with one decay per key channel.  `num_kv_heads` query/key heads of
-    size `head_dim`, `num_heads` value heads of size `v_head_dim`; q, k and v pass a causal
-    convolution of `taps` taps and silu; the decay and the output gate are products of rank
-    `decay_rank` and `gate_rank`; `unit_eps` sits under the root of the unit norms of q and
-    k, `norm_eps` under that of the output norm."""
+    """The gated delta rule.  `num_kv_heads` query/key heads of size `head_dim`, `num_heads` value
+    heads of size `v_head_dim`; q, k and v pass a causal convolution of `taps` taps and silu;
+    `unit_eps` sits under the root of the unit norms of q and k, `norm_eps` under that of the
+    output norm.
+
+    decay       "channel": one decay per token and key channel, a product of rank `decay_rank`
+                (tensors "a1", "a2"); "head": one per token and value head (tensor "a" [heads,
+                hidden], "dt_bias" [heads])
+    gate_rank   > 0: the output gate is a product of that rank (tensors "g1", "g2"); 0: of full
+                rank (tensor "g" [heads * v_head_dim, hidden])
+    gate        "sigmoid" or "silu" of it multiplies the normed read-out
+    Either both the decay per channel and the gate are low-rank products or neither is."""
     num_heads: int = 0
     num_kv_heads: int = 0
     head_dim: int = 0
@@ -230,6 +247,25 @@ class GatedDeltaSpec(MixerSpec):
     gate_rank: int = 0
     norm_eps: float = 1e-6
     unit_eps: float = 1e-6
+    names: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
+    decay: str = "channel"
+    gate: str = "sigmoid"
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec(MixerSpec):
+    """A selective state space with one decay per token and head (the Mamba-2 form).  `num_heads`
+    heads of size `v_head_dim`; a state of `state` rows per head; heads share their input and
+    output vectors B and C in `groups` equal groups of neighbours; x, B and C pass a causal
+    convolution of `taps` taps with a bias and silu; the read-out is gated with silu and then
+    RMS-normed in `norm_groups` equal parts of a row, `norm_eps` under each root."""
+    num_heads: int = 0
+    v_head_dim: int = 0
+    state: int = 0
+    groups: int = 1
+    taps: int = 0
+    norm_groups: int = 1
+    norm_eps: float = 1e-6
     names: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
 
 
@@ -316,7 +352,9 @@ class MoESpec(FeedForwardSpec):
     learned number per expert (tensor "correction" [experts]) is added to the scores where
     experts are compared, while the weights are made from the scores without it; score
     "softmax_chosen": the logits themselves are compared, and the chosen ones, exponentiated and
-    divided by their own sum, are the weights."""
+    divided by their own sum, are the weights; `identity`: so many further router outputs, after
+    the experts', stand for experts whose output is the token itself and that have no tensors
+    (scores, correction and groups range over the experts and these together)."""
     ffn_dim: int = 0
     experts: int = 0
     top: int = 0
@@ -333,6 +371,12 @@ class MoESpec(FeedForwardSpec):
     shared: Optional[FeedForwardSpec] = None
     names: Mapping[str, str] = field(default_factory=dict, hash=False, compare=False)
     choice_bias: bool = False
+    identity: int = 0
+
+    @property
+    def outputs(self) -> int:
+        """Rows of the router."""
+        return self.experts + self.identity
 
 
 @dataclass(frozen=True)
@@ -411,3 +455,4 @@ class ModelSpec:
                                                 # embedding rows pass it before the first layer
     position_embedding: Optional[str] = None    # tensor [max_position, hidden]: row p is added to
                                                 # the (scaled) embedding row of position p
+    logit_scale: float = 1.0                    # factor on the logits (before the cap)

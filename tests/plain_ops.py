@@ -207,7 +207,8 @@ class PlainOps:
         def ln(x, w, b, e):
             mu = x.mean(dim=-1, keepdim=True)
             var = (x - mu).pow(2).mean(dim=-1, keepdim=True)
-            return (x - mu) / (var + e).sqrt() * _f(w) + _f(b)
+            y = (x - mu) / (var + e).sqrt() * _f(w)
+            return y if b is None else y + _f(b)
 
         d = None if delta is None else _f(delta)
         if d is not None and delta_weight is not None:
@@ -301,8 +302,10 @@ class PlainOps:
                 dst.view(-1, G, d)[s] = mean.to(dst.dtype)
 
     def paged_attention_pooled(self, rows, num_heads, num_kv_heads, head_dim, k_cache, v_cache, ctx,
-                               group, pooled, scale, softcap, window, sinks, out):
+                               group, pooled, scale, softcap, window, sinks, out,
+                               v_head_dim=None, most_blocks=0):
         H, G, d = num_heads, num_kv_heads, head_dim
+        dv = v_head_dim or d
         ps = group.page_size
         q_start, ctx_lens = ctx.q_start.tolist(), ctx.ctx_lens.tolist()
         for r in range(ctx.n_reqs):
@@ -316,15 +319,16 @@ class PlainOps:
                 p = clen - (b - a) + (t - a)
                 lo = 0 if window is None else max(0, p - window + 1)
                 idx = torch.tensor([table[j // ps] * ps + j % ps for j in range(lo, p + 1)])
-                k, v = _f(k_cache.view(-1, G, d)[idx]), _f(v_cache.view(-1, G, d)[idx])
+                k, v = _f(k_cache.view(-1, G, d)[idx]), _f(v_cache.view(-1, G, dv)[idx])
                 if pooled is not None:
                     pk, pv, pgroup, pool = pooled
                     nb = max(0, p - window + 1) // pool
+                    nb = min(nb, most_blocks) if most_blocks else nb
                     ptab = pgroup.block_table[r].tolist()
                     pidx = torch.tensor([ptab[j // ps] * ps + j % ps for j in range(nb)],
                                         dtype=torch.long)
                     k = torch.cat([_f(pk.view(-1, G, d)[pidx]), k])
-                    v = torch.cat([_f(pv.view(-1, G, d)[pidx]), v])
+                    v = torch.cat([_f(pv.view(-1, G, dv)[pidx]), v])
                 q = _f(rows[t, :H * d]).reshape(H, d)
                 for h in range(H):
                     s = (k[:, h // (H // G)] @ q[h]) * scale
@@ -333,7 +337,7 @@ class PlainOps:
                     if sinks is not None:
                         s = torch.cat([s, _f(sinks[h:h + 1])])
                     w = torch.softmax(s, dim=0)[:k.shape[0]]
-                    out[t, h * d:(h + 1) * d] = (w @ v[:, h // (H // G)]).to(out.dtype)
+                    out[t, h * dv:(h + 1) * dv] = (w @ v[:, h // (H // G)]).to(out.dtype)
 
     # ---- linear attention with decay ---------------------------------------------------------
     def linear_attention(self, rows, z_rows, log_decay, decay_bias, tau, norm_w, state, ctx, out, heads, dim,
@@ -483,7 +487,7 @@ class PlainOps:
                         **options)
 
     def moe_experts(self, x, ids, weights, gate_up, down, out, activation="swiglu", limit=0.0,
-                    alpha=1.0, addend=None):
+                    alpha=1.0, addend=None, identity=0):
         n, top = ids.shape
         F = down.shape[2]
         y = torch.zeros((n, out.shape[1]), dtype=torch.float32)
@@ -492,6 +496,9 @@ class PlainOps:
         for t in range(n):
             for k in range(top):
                 e = int(ids[t, k])
+                if e >= down.shape[0]:                       # an identity expert
+                    y[t] += float(weights[t, k]) * _f(x[t])
+                    continue
                 gu = _f(gate_up[e]) @ _f(x[t])               # gate and up rows alternate
                 if activation == "relu2":                    # no gate: the up rows alone
                     act = gu.clamp(min=0).pow(2).to(x.dtype)
@@ -515,24 +522,29 @@ class PlainOps:
 
     # ---- latent rows with a query latent and a turned key part ---------------------------
     @staticmethod
-    def _turn(x, positions, freq):
-        """x [n, ..., rot]: dimension i with i + rot/2 by the angle position * freq[i]."""
+    def _turn(x, positions, freq, pairs=False, amplitude=1.0):
+        """x [n, ..., rot]: dimension i with i + rot/2 (`pairs`: 2i with 2i + 1) by the angle
+        position * freq[i]; cosine and sine times `amplitude`."""
         half = x.shape[-1] // 2
         ang = positions.to(torch.float32)[:, None] * _f(freq)[None, :]
         shape = (x.shape[0],) + (1,) * (x.dim() - 2) + (half,)
-        cos, sin = torch.cos(ang).reshape(shape), torch.sin(ang).reshape(shape)
+        cos, sin = (amplitude * f(ang).reshape(shape) for f in (torch.cos, torch.sin))
+        if pairs:
+            u, v = x[..., 0::2], x[..., 1::2]
+            return torch.stack([u * cos - v * sin, v * cos + u * sin], dim=-1).reshape(x.shape)
         u, v = x[..., :half], x[..., half:]
         return torch.cat([u * cos - v * sin, v * cos + u * sin], dim=-1)
 
     def latent_prepare(self, rows, q_off, q_rank, q_weight, cq, kv_off, rank, rot, kv_weight, eps,
-                       freq, positions, slot_mapping, cache):
+                       freq, positions, slot_mapping, cache, **turn):
         def norm(x, w):
             return x / (x.pow(2).mean(dim=-1, keepdim=True) + eps).sqrt() * _f(w)
         if q_rank:
             cq.copy_(norm(_f(rows[:, q_off:q_off + q_rank]), q_weight).to(cq.dtype))
         c = norm(_f(rows[:, kv_off:kv_off + rank]), kv_weight)
         if rot:
-            turned = self._turn(_f(rows[:, kv_off + rank:kv_off + rank + rot]), positions, freq)
+            turned = self._turn(_f(rows[:, kv_off + rank:kv_off + rank + rot]), positions, freq,
+                                **turn)
             c = torch.cat([c, turned], dim=-1)
         pages = cache.view(-1, rank + rot)
         for t in range(rows.shape[0]):
@@ -540,12 +552,12 @@ class PlainOps:
             if s >= 0:
                 pages[s] = c[t].to(pages.dtype)
 
-    def rope_heads(self, x, heads, size, off, rot, freq, positions):
+    def rope_heads(self, x, heads, size, off, rot, freq, positions, **turn):
         if not rot:
             return
         n = x.shape[0]
         v = x[:, :heads * size].reshape(n, heads, size)
-        turned = self._turn(_f(v[..., off:off + rot]), positions, freq)
+        turned = self._turn(_f(v[..., off:off + rot]), positions, freq, **turn)
         v[..., off:off + rot] = turned.to(x.dtype)
         x[:, :heads * size] = v.reshape(n, heads * size)
 
@@ -614,7 +626,7 @@ class PlainOps:
     def qkv_full_norm_rope_write(self, rows, bias, num_heads, num_kv_heads, head_dim, v_head_dim,
                                  q_weight, k_weight, eps, freq, rot_dims, positions, slot_mapping,
                                  q_out, k_cache, v_cache, v_first_in=None, v_first_out=None,
-                                 lam=None):
+                                 lam=None, pairs=True, amplitude=1.0):
         n = rows.shape[0]
         Q, K = num_heads * head_dim, num_kv_heads * head_dim
         x = _f(rows) if bias is None else _f(rows) + _f(bias)
@@ -628,11 +640,8 @@ class PlainOps:
         def turn(t, heads):
             t = t.reshape(n, heads, head_dim).clone()
             if rot_dims:
-                ang = positions.to(torch.float32)[:, None] * _f(freq)[None, :]
-                c, s = ang.cos()[:, None, :], ang.sin()[:, None, :]
-                a, b = t[..., 0:rot_dims:2].clone(), t[..., 1:rot_dims:2].clone()
-                t[..., 0:rot_dims:2] = a * c - b * s
-                t[..., 1:rot_dims:2] = b * c + a * s
+                t[..., :rot_dims] = self._turn(t[..., :rot_dims].clone(), positions, freq, pairs,
+                                               amplitude)
             return t.reshape(n, heads * head_dim)
 
         q = turn(norm(q, q_weight), num_heads)
@@ -655,8 +664,9 @@ class PlainOps:
         return (taps - 1) * (2 * kv_heads * dim + heads * vdim) + heads * dim * vdim
 
     def gated_delta(self, proj, lowrank, filt, a_log, dt_bias, norm_w, state, ctx, out, heads,
-                    kv_heads, dim, vdim, taps, unit_eps, eps):
+                    kv_heads, dim, vdim, taps, unit_eps, eps, head_decay=False, gate="sigmoid"):
         H, G, d, dv = heads, kv_heads, dim, vdim
+        ND = H if head_decay else H * d
         C = 2 * G * d + H * dv
         q_start = ctx.q_start.tolist()
         slots = ctx.state_slot.tolist()
@@ -683,18 +693,54 @@ class PlainOps:
                 k = k / (k.pow(2).sum(-1, keepdim=True) + unit_eps).sqrt()
                 beta = torch.sigmoid(p[t, C:C + H])
                 decay = torch.exp(-torch.exp(_f(a_log))[:, None] * torch.nn.functional.softplus(
-                    low[t, :H * d] + _f(dt_bias)).reshape(H, d))
-                gate = torch.sigmoid(low[t, H * d:H * d + H * dv]).reshape(H, dv)
+                    low[t, :ND] + _f(dt_bias)).reshape(H, ND // H)).expand(H, d)
+                z = low[t, ND:ND + H * dv]
+                gates = (torch.sigmoid(z) if gate == "sigmoid"
+                         else torch.nn.functional.silu(z)).reshape(H, dv)
                 for h in range(H):
                     kh, qh = k[h // (H // G)], q[h // (H // G)]
                     S[h] = decay[h][:, None] * S[h]
                     u = beta[h] * (v[h] - S[h].t() @ kh)
                     S[h] = S[h] + torch.outer(kh, u)
                     o = S[h].t() @ qh
-                    o = o / (o.pow(2).mean() + eps).sqrt() * _f(norm_w) * gate[h]
+                    o = o / (o.pow(2).mean() + eps).sqrt() * _f(norm_w) * gates[h]
                     out[t, h * dv:(h + 1) * dv] = o.to(out.dtype)
             rec[:(taps - 1) * C] = rows[n:].reshape(-1)
             rec[(taps - 1) * C:] = S.reshape(-1)
+
+    # ---- state space: one decay per token and head -------------------------------------
+    def state_space(self, proj, filt, conv_bias, dt_bias, a_log, skip, norm_w, conv_state, state,
+                    ctx, out, heads, vdim, d_state, groups, taps, norm_groups, eps):
+        H, dv, N, G = heads, vdim, d_state, groups
+        inner, C = H * dv, H * dv + 2 * G * N
+        q_start, slots = ctx.q_start.tolist(), ctx.state_slot.tolist()
+        p = _f(proj)
+        out.zero_()
+        for r in range(ctx.n_reqs):
+            a, b = q_start[r], q_start[r + 1]
+            if slots[r] < 0 or a == b:
+                continue
+            x = p[a:b, inner:inner + C]
+            rows = x if taps == 1 else torch.cat([conv_state[slots[r]], x])
+            n = b - a
+            act = _f(conv_bias) + sum(rows[j:j + n] * _f(filt)[:, j] for j in range(taps))
+            act = _f(torch.nn.functional.silu(act).to(out.dtype))
+            S = state[slots[r]].reshape(H, N, dv).clone()
+            for i in range(n):
+                xs = act[i, :inner].reshape(H, dv)
+                B = act[i, inner:inner + G * N].reshape(G, N).repeat_interleave(H // G, 0)
+                Cq = act[i, inner + G * N:].reshape(G, N).repeat_interleave(H // G, 0)
+                dt = torch.nn.functional.softplus(p[a + i, inner + C:] + _f(dt_bias), threshold=60.0)
+                keep = torch.exp(-torch.exp(_f(a_log)) * dt)
+                S = keep[:, None, None] * S + (dt[:, None] * B)[:, :, None] * xs[:, None, :]
+                y = torch.einsum("hnv,hn->hv", S, Cq) + _f(skip)[:, None] * xs
+                y = y.reshape(inner) * torch.nn.functional.silu(p[a + i, :inner])
+                y = y.reshape(norm_groups, -1)
+                y = y / (y.pow(2).mean(dim=-1, keepdim=True) + eps).sqrt()
+                out[a + i] = (y.reshape(inner) * _f(norm_w)).to(out.dtype)
+            state[slots[r]] = S.reshape(-1)
+            if taps > 1:
+                conv_state[slots[r]] = rows[n:]
 
     # ---- clamped gated activation ----------------------------------------------------
     def glu_clamp(self, gate_up, bias, out, limit, alpha):
