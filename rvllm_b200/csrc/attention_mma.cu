@@ -234,7 +234,7 @@ __global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_at
         if (key_lo > key_hi) return;
     }
     // EXT: tiles below zero are the pooled blocks': tile t holds rows (t + n_ptiles) * 64 on
-    const int nb_hi = EXT ? rv_seen_blocks(key_hi, window, pl.pool) : 0;     // the newest query's
+    const int nb_hi = EXT ? rv_seen_blocks(key_hi, window, pl.pool, pl.most) : 0;     // the newest query's
     const int n_ptiles = (nb_hi + RV_BN - 1) / RV_BN;
     const int tile_first = key_lo / RV_BN, tile_end = key_hi / RV_BN;
     const int tile_begin = tile_first - n_ptiles;
@@ -304,8 +304,8 @@ __global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_at
         lo_a = max(lo_a, key_lo); lo_b = max(lo_b, key_lo);
         hi_a = min(hi_a, key_hi); hi_b = min(hi_b, key_hi);
     }
-    const int nb_a = EXT ? rv_seen_blocks(p_a, window, pl.pool) : 0;
-    const int nb_b = EXT ? rv_seen_blocks(p_b, window, pl.pool) : 0;
+    const int nb_a = EXT ? rv_seen_blocks(p_a, window, pl.pool, pl.most) : 0;
+    const int nb_b = EXT ? rv_seen_blocks(p_b, window, pl.pool, pl.most) : 0;
     const float cap_out = EXT ? pl.cap * 1.4426950408889634f : 0.f;
     const float cap_arg = EXT && pl.cap > 0.f ? 2.f * scale_log2 / pl.cap : 0.f;
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
@@ -426,7 +426,7 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
     const int lo = window > 0 ? max(0, p - window + 1) : 0;
     const bool blocks = EXT && split < pl.psplits;
     const int stretch = !EXT || blocks ? split : split - pl.psplits + lo / SPLIT;
-    const int limit = blocks ? rv_seen_blocks(p, window, pl.pool) : clen;    // rows there are
+    const int limit = blocks ? rv_seen_blocks(p, window, pl.pool, pl.most) : clen;    // rows there are
     const int key_lo = max(blocks ? 0 : lo, stretch * SPLIT);
     const int key_hi = min(limit - 1, stretch * SPLIT + SPLIT - 1);
     if (key_lo > key_hi) return;
@@ -864,7 +864,7 @@ static int pooled_sizes(int num_heads, int num_kv_heads, int page_size, int wind
 extern "C" int RV_SYM(rv_paged_attention_pooled_prefill)(
     const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* block_table,
     int max_blocks, const void* pk, const void* pv, const int* ptable, int pmax_blocks, int pool,
-    float cap, const int* q_start, const int* ctx_lens, void* out, int first_req, int n_reqs,
+    int most, float cap, const int* q_start, const int* ctx_lens, void* out, int first_req, int n_reqs,
     int max_q_len, int num_heads, int num_kv_heads, int page_size, float scale, int window,
     const float* sinks, void* stream) {
     if (n_reqs == 0) return 0;
@@ -885,7 +885,7 @@ extern "C" int RV_SYM(rv_paged_attention_pooled_prefill)(
         }
         configured = true;
     }
-    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, cap, 0};
+    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, most, cap, 0};
     rv_launch(paged_attention_mma_kernel<RV_HD, 4, false, true>,
               dim3((unsigned)blocks_x, num_kv_heads, n_reqs), dim3(128), smem_bytes<4>(),
               (cudaStream_t)stream, (const bf16*)q, q_stride, (const bf16*)k_cache,
@@ -902,13 +902,13 @@ extern "C" int RV_SYM(rv_paged_attention_pooled_prefill)(
 extern "C" int RV_SYM(rv_paged_attention_pooled_decode_mma)(
     const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* block_table,
     int max_blocks, const void* pk, const void* pv, const int* ptable, int pmax_blocks, int pool,
-    float cap, const int* ctx_lens, void* scratch, long long scratch_bytes, int n_reqs,
+    int most, float cap, const int* ctx_lens, void* scratch, long long scratch_bytes, int n_reqs,
     int max_ctx_len, int num_heads, int num_kv_heads, int page_size, float scale, int window,
     void* stream) {
     if (n_reqs == 0) return 0;
     if (n_reqs < 0 || pooled_sizes(num_heads, num_kv_heads, page_size, window, pool, pk, pv, ptable))
         return fail("paged_attention_pooled_decode: bad sizes");
-    const int psplits = rv_pooled_psplits(max_ctx_len, window, pool, RV_SPLIT);
+    const int psplits = rv_pooled_psplits(max_ctx_len, window, pool, most, RV_SPLIT);
     const int max_splits = psplits + rv_pooled_tsplits(max_ctx_len, window, RV_SPLIT);
     const size_t slots = (size_t)n_reqs * num_heads * max_splits;
     if ((long long)(slots * RV_HD * 4 + slots * 8) > scratch_bytes)
@@ -927,7 +927,7 @@ extern "C" int RV_SYM(rv_paged_attention_pooled_decode_mma)(
         }
         configured = true;
     }
-    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, cap, psplits};
+    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, most, cap, psplits};
     float* part_o = (float*)scratch;
     float2* part_ml = (float2*)((char*)scratch + slots * RV_HD * 4);
     rv_launch(paged_attention_decode_mma_kernel<RV_HD, 4, true>,

@@ -124,7 +124,7 @@ __global__ void paged_attention_warp_kernel(
     // EXT: the pooled blocks first, then the tokens
     for (int part = EXT && pl.pool > 0 ? 0 : 1; part < 2; ++part) {
     const bool blocks = EXT && part == 0;
-    const int first = blocks ? 0 : lo, last = blocks ? rv_seen_blocks(p, window, pl.pool) - 1 : p;
+    const int first = blocks ? 0 : lo, last = blocks ? rv_seen_blocks(p, window, pl.pool, pl.most) - 1 : p;
     const int* table = blocks ? pl.table + (size_t)r * pl.max_blocks : block_table + (size_t)r * max_blocks;
     const T* kc = blocks ? (const T*)pl.k : k_cache;
     const T* vc = blocks ? (const T*)pl.v : v_cache;
@@ -197,7 +197,7 @@ __global__ void __launch_bounds__(128) paged_attention_decode_kernel(
     const bool blocks = EXT && split < pl.psplits;
     const int stretch = !EXT || blocks ? split : split - pl.psplits + lo / RV_ATTN_SPLIT;
     const int k0 = max(blocks ? 0 : lo, stretch * RV_ATTN_SPLIT);
-    const int k1 = min(blocks ? rv_seen_blocks(p, window, pl.pool) - 1 : p,
+    const int k1 = min(blocks ? rv_seen_blocks(p, window, pl.pool, pl.most) - 1 : p,
                        stretch * RV_ATTN_SPLIT + RV_ATTN_SPLIT - 1);   // inclusive
     if ((!EXT && split < lo / RV_ATTN_SPLIT) || k0 > k1) return;
 
@@ -320,7 +320,7 @@ __global__ void paged_attention_merge_kernel(const float* __restrict__ part_o,
                                              const int* __restrict__ ctx_lens, T* __restrict__ out,
                                              int max_splits, int num_heads, int hd, int window,
                                              int split_keys, const float* __restrict__ sinks,
-                                             int psplits, int pool) {
+                                             int psplits, int pool, int most) {
     rv_pdl_launch_dependents();
     constexpr bool kFast = sizeof(T) == 2;
     const int r = blockIdx.y, h = blockIdx.x;
@@ -337,7 +337,7 @@ __global__ void paged_attention_merge_kernel(const float* __restrict__ part_o,
     // A context longer than the launch's max_ctx_len has keys that no split covered: the row
     // is marked invalid (NaN) and nothing outside this head's slots is read.
     // (EXT: splits that cover blocks, then splits that cover tokens from the window's first on.)
-    const int np = EXT ? (rv_seen_blocks(p, window, pool) + split_keys - 1) / split_keys : 0;
+    const int np = EXT ? (rv_seen_blocks(p, window, pool, most) + split_keys - 1) / split_keys : 0;
     const int nt = p / split_keys - lo / split_keys + 1;
     if (EXT ? (np > psplits || nt > max_splits - psplits) : (clen > max_splits * split_keys)) {
         for (int d = threadIdx.x; d < hd; d += blockDim.x) rv_store(o + d, NAN);
@@ -442,12 +442,16 @@ extern "C" int rv_paged_attention_warp(const void* q, int dtype, int q_stride, c
                                       nullptr, stream);
 }
 
+// Bytes of part_o for so many (request, head, split) triples, before part_ml's pairs of floats: a
+// multiple of 8 (an odd value size times an odd count is not).
+static size_t part_bytes(size_t slots, int vd) { return (slots * vd * 4 + 7) & ~(size_t)7; }
+
 // Bytes of scratch rv_paged_attention_decode needs: part_o then part_ml (`hd`: the value size).
 extern "C" long long rv_paged_attention_decode_scratch_bytes(int n_reqs, int num_heads, int hd,
                                                              int max_ctx_len) {
     const long long splits = (max_ctx_len + RV_ATTN_SPLIT - 1) / RV_ATTN_SPLIT;
     const long long slots = (long long)n_reqs * num_heads * (splits > 0 ? splits : 1);
-    return slots * hd * 4 + slots * 8;
+    return (long long)part_bytes(slots, hd) + slots * 8;
 }
 
 static int merge_threads(int hd) { return hd < 32 ? 32 : (hd > 128 ? 128 : ((hd + 31) / 32) * 32); }
@@ -471,7 +475,7 @@ extern "C" int rv_paged_attention_decode_ex(const void* q, int dtype, int q_stri
     if (n_reqs > 65535 || max_splits > 65535) RV_FAIL("paged_attention_decode: batch too large");
     const size_t slots = (size_t)n_reqs * num_heads * max_splits;
     float* part_o = (float*)scratch;
-    float2* part_ml = (float2*)((char*)scratch + slots * vd * 4);
+    float2* part_ml = (float2*)((char*)scratch + part_bytes(slots, vd));
     const int G = num_heads / num_kv_heads;
     const int tiles = (G + RV_ATTN_GT - 1) / RV_ATTN_GT;
     dim3 grid(num_kv_heads * tiles, n_reqs, max_splits);
@@ -488,7 +492,7 @@ extern "C" int rv_paged_attention_decode_ex(const void* q, int dtype, int q_stri
     RV_DISPATCH_DTYPE(dtype, "paged_attention_merge",
         (rv_launch(paged_attention_merge_kernel<T, false>, dim3(mgrid), dim3(merge_threads(vd)), 0, s, 
             part_o, part_ml, ctx_lens, (T*)out, max_splits, num_heads, vd, window, RV_ATTN_SPLIT,
-            sinks, 0, 0)));
+            sinks, 0, 0, 0)));
     RV_CHECK_LAUNCH("paged_attention_merge");
     return 0;
 }
@@ -520,12 +524,12 @@ extern "C" int rv_paged_attention_merge_ex(const void* scratch, const int* ctx_l
         RV_FAIL("paged_attention_merge: bad sizes");
     const size_t slots = (size_t)n_reqs * num_heads * max_splits;
     const float* part_o = (const float*)scratch;
-    const float2* part_ml = (const float2*)((const char*)scratch + slots * hd * 4);
+    const float2* part_ml = (const float2*)((const char*)scratch + part_bytes(slots, hd));
     dim3 mgrid(num_heads, n_reqs);
     RV_DISPATCH_DTYPE(dtype, "paged_attention_merge",
         (rv_launch(paged_attention_merge_kernel<T, false>, dim3(mgrid), dim3(merge_threads(hd)), 0, (cudaStream_t)stream, 
             part_o, part_ml, ctx_lens, (T*)out, max_splits, num_heads, hd, window, split_keys,
-            sinks, 0, 0)));
+            sinks, 0, 0, 0)));
     RV_CHECK_LAUNCH("paged_attention_merge");
     return 0;
 }
@@ -539,21 +543,24 @@ extern "C" int rv_paged_attention_merge(const void* scratch, const int* ctx_lens
 
 // ---------------------------------------------------------------------------------
 // Attention over a window of tokens and the pooled blocks before it (attention_pooled.cuh).
-// `window` 0: every token is seen; `pool` 0: no blocks (pk, pv, ptable unused); `cap` 0: scores are
-// not capped; key and value heads have the same size.
+// `window` 0: every token is seen; `pool` 0: no blocks (pk, pv, ptable unused); `most` 0: no bound on
+// the blocks seen; `cap` 0: scores are not capped; `vd`: the size of a value head.
 
 // Bytes of scratch of the split form: part_o then part_ml.
-extern "C" long long rv_paged_attention_pooled_scratch_bytes(int n_reqs, int num_heads, int hd,
-                                                             int max_ctx_len, int window, int pool) {
-    const long long splits = rv_pooled_psplits(max_ctx_len, window, pool, RV_ATTN_SPLIT) +
+extern "C" long long rv_paged_attention_pooled_scratch_bytes(int n_reqs, int num_heads, int vd,
+                                                             int max_ctx_len, int window, int pool,
+                                                             int most) {
+    const long long splits = rv_pooled_psplits(max_ctx_len, window, pool, most, RV_ATTN_SPLIT) +
                              rv_pooled_tsplits(max_ctx_len, window, RV_ATTN_SPLIT);
-    return (long long)n_reqs * num_heads * splits * (hd * 4 + 8);
+    const long long slots = (long long)n_reqs * num_heads * splits;
+    return (long long)part_bytes(slots, vd) + slots * 8;
 }
 
-static int pooled_check(const char* name, int num_heads, int num_kv_heads, int hd, int page_size,
-                        int window, int pool, const void* pk, const void* pv, const int* ptable, int dtype) {
-    if (check_attention_sizes(name, num_heads, num_kv_heads, hd, hd, page_size, dtype)) return 1;
-    if (window < 0 || pool < 0 || (pool > 0 && (window == 0 || !pk || !pv || !ptable)))
+static int pooled_check(const char* name, int num_heads, int num_kv_heads, int hd, int vd, int page_size,
+                        int window, int pool, int most, const void* pk, const void* pv, const int* ptable,
+                        int dtype) {
+    if (check_attention_sizes(name, num_heads, num_kv_heads, hd, vd, page_size, dtype)) return 1;
+    if (window < 0 || pool < 0 || most < 0 || (pool > 0 && (window == 0 || !pk || !pv || !ptable)))
         RV_FAIL("%s: pooled blocks need a window, pages and a block table", name);
     return 0;
 }
@@ -562,24 +569,24 @@ static int pooled_check(const char* name, int num_heads, int num_kv_heads, int h
 extern "C" int rv_paged_attention_pooled_warp(
     const void* q, int dtype, int q_stride, const void* k_cache, const void* v_cache,
     const int* block_table, int max_blocks, const void* pk, const void* pv, const int* ptable,
-    int pmax_blocks, int pool, float cap, const int* q_start, const int* ctx_lens,
+    int pmax_blocks, int pool, int most, float cap, const int* q_start, const int* ctx_lens,
     const int* token_req, void* out, int first_token, int n_tokens, int num_heads, int num_kv_heads,
-    int hd, int page_size, float scale, int window, const float* sinks, void* stream) {
+    int hd, int page_size, float scale, int window, int vd, const float* sinks, void* stream) {
     if (n_tokens == 0) return 0;
-    if (pooled_check("paged_attention_pooled", num_heads, num_kv_heads, hd, page_size, window, pool, pk,
-                     pv, ptable, dtype))
+    if (pooled_check("paged_attention_pooled", num_heads, num_kv_heads, hd, vd, page_size, window, pool,
+                     most, pk, pv, ptable, dtype))
         return 1;
     const int wpb = 4;
     const long long warps = (long long)n_tokens * num_heads;
     const long long blocks = (warps + wpb - 1) / wpb;
     if (blocks > 0x7fffffffLL) RV_FAIL("paged_attention_pooled: too many rows");
     const size_t smem = (size_t)wpb * hd * sizeof(float);
-    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, cap, 0};
+    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, most, cap, 0};
     RV_DISPATCH_DTYPE(dtype, "paged_attention_pooled",
-        RV_DISPATCH_DPL(hd, (rv_launch(paged_attention_warp_kernel<T, DPL, true>, dim3((int)blocks),
+        RV_DISPATCH_DPL(vd, (rv_launch(paged_attention_warp_kernel<T, DPL, true>, dim3((int)blocks),
             dim3(wpb * 32), smem, (cudaStream_t)stream, (const T*)q, q_stride, (const T*)k_cache,
             (const T*)v_cache, block_table, max_blocks, q_start, ctx_lens, token_req, (T*)out,
-            first_token, n_tokens, num_heads, num_kv_heads, hd, page_size, scale, window, hd, sinks, pl))));
+            first_token, n_tokens, num_heads, num_kv_heads, hd, page_size, scale, window, vd, sinks, pl))));
     RV_CHECK_LAUNCH("paged_attention_pooled");
     return 0;
 }
@@ -587,18 +594,18 @@ extern "C" int rv_paged_attention_pooled_warp(
 // The merge of split results in the layout above (this file's kernel or attention_mma.cu's).
 extern "C" int rv_paged_attention_pooled_merge(const void* scratch, const int* ctx_lens, void* out,
                                                int dtype, int n_reqs, int max_ctx_len, int num_heads,
-                                               int hd, int window, int pool, const float* sinks,
-                                               void* stream) {
+                                               int hd, int window, int pool, int most,
+                                               const float* sinks, void* stream) {
     if (n_reqs == 0) return 0;
-    const int psplits = rv_pooled_psplits(max_ctx_len, window, pool, RV_ATTN_SPLIT);
+    const int psplits = rv_pooled_psplits(max_ctx_len, window, pool, most, RV_ATTN_SPLIT);
     const int max_splits = psplits + rv_pooled_tsplits(max_ctx_len, window, RV_ATTN_SPLIT);
     const size_t slots = (size_t)n_reqs * num_heads * max_splits;
     const float* part_o = (const float*)scratch;
-    const float2* part_ml = (const float2*)((const char*)scratch + slots * hd * 4);
+    const float2* part_ml = (const float2*)((const char*)scratch + part_bytes(slots, hd));
     RV_DISPATCH_DTYPE(dtype, "paged_attention_pooled_merge",
         (rv_launch(paged_attention_merge_kernel<T, true>, dim3(num_heads, n_reqs), dim3(merge_threads(hd)),
             0, (cudaStream_t)stream, part_o, part_ml, ctx_lens, (T*)out, max_splits, num_heads, hd,
-            window, RV_ATTN_SPLIT, sinks, psplits, pool)));
+            window, RV_ATTN_SPLIT, sinks, psplits, pool, most)));
     RV_CHECK_LAUNCH("paged_attention_pooled_merge");
     return 0;
 }
@@ -607,33 +614,34 @@ extern "C" int rv_paged_attention_pooled_merge(const void* scratch, const int* c
 extern "C" int rv_paged_attention_pooled_decode(
     const void* q, int dtype, int q_stride, const void* k_cache, const void* v_cache,
     const int* block_table, int max_blocks, const void* pk, const void* pv, const int* ptable,
-    int pmax_blocks, int pool, float cap, const int* ctx_lens, void* out, void* scratch,
+    int pmax_blocks, int pool, int most, float cap, const int* ctx_lens, void* out, void* scratch,
     long long scratch_bytes, int n_reqs, int max_ctx_len, int num_heads, int num_kv_heads, int hd,
-    int page_size, float scale, int window, const float* sinks, void* stream) {
+    int page_size, float scale, int window, int vd, const float* sinks, void* stream) {
     if (n_reqs == 0) return 0;
-    if (pooled_check("paged_attention_pooled_decode", num_heads, num_kv_heads, hd, page_size, window,
-                     pool, pk, pv, ptable, dtype))
+    if (pooled_check("paged_attention_pooled_decode", num_heads, num_kv_heads, hd, vd, page_size, window,
+                     pool, most, pk, pv, ptable, dtype))
         return 1;
-    const int psplits = rv_pooled_psplits(max_ctx_len, window, pool, RV_ATTN_SPLIT);
+    const int psplits = rv_pooled_psplits(max_ctx_len, window, pool, most, RV_ATTN_SPLIT);
     const int max_splits = psplits + rv_pooled_tsplits(max_ctx_len, window, RV_ATTN_SPLIT);
-    if (rv_paged_attention_pooled_scratch_bytes(n_reqs, num_heads, hd, max_ctx_len, window, pool) > scratch_bytes)
+    if (rv_paged_attention_pooled_scratch_bytes(n_reqs, num_heads, vd, max_ctx_len, window, pool, most) >
+        scratch_bytes)
         RV_FAIL("paged_attention_pooled_decode: scratch of %lld bytes is too small", scratch_bytes);
     if (n_reqs > 65535 || max_splits > 65535) RV_FAIL("paged_attention_pooled_decode: batch too large");
     const size_t slots = (size_t)n_reqs * num_heads * max_splits;
     float* part_o = (float*)scratch;
-    float2* part_ml = (float2*)((char*)scratch + slots * hd * 4);
+    float2* part_ml = (float2*)((char*)scratch + part_bytes(slots, vd));
     const int G = num_heads / num_kv_heads;
     const int tiles = (G + RV_ATTN_GT - 1) / RV_ATTN_GT;
     const size_t smem = (size_t)(RV_ATTN_GT * hd + 4 * 32 * RV_ATTN_GT + 4 * 32 +
-                                 4 * RV_ATTN_GT * (hd + 2)) * sizeof(float);
-    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, cap, psplits};
+                                 4 * RV_ATTN_GT * (vd + 2)) * sizeof(float);
+    const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, most, cap, psplits};
     RV_DISPATCH_DTYPE(dtype, "paged_attention_pooled_decode",
-        RV_DISPATCH_DPL(hd, (rv_launch(paged_attention_decode_kernel<T, DPL, true>,
+        RV_DISPATCH_DPL(vd, (rv_launch(paged_attention_decode_kernel<T, DPL, true>,
             dim3(num_kv_heads * tiles, n_reqs, max_splits), dim3(128), smem, (cudaStream_t)stream,
             (const T*)q, q_stride, (const T*)k_cache, (const T*)v_cache, block_table, max_blocks,
             ctx_lens, part_o, part_ml, max_splits, num_heads, num_kv_heads, hd, page_size, scale,
-            window, hd, pl))));
+            window, vd, pl))));
     RV_CHECK_LAUNCH("paged_attention_pooled_decode");
     return rv_paged_attention_pooled_merge(scratch, ctx_lens, out, dtype, n_reqs, max_ctx_len, num_heads,
-                                           hd, window, pool, sinks, stream);
+                                           vd, window, pool, most, sinks, stream);
 }

@@ -1,4 +1,4 @@
-// The gated delta rule with one decay per key channel, over any mixture of prompt portions and
+// The gated delta rule with one decay per key channel or per value head, over any mixture of prompt portions and
 // single tokens.  Per request a float32 record holds the last taps-1 inputs of the short
 // convolutions, [taps-1, C] oldest first with C = 2 G d + H dv channels (q | k | v), and then
 // the state S, stored [H, dv, d]: the d rows of a column lie side by side, because a thread owns
@@ -11,7 +11,8 @@
 //     token's; the inputs before a request's first token of the step come from its record)
 //     and then silu; q and k become unit vectors per head, x / sqrt(sum x^2 + unit_eps), q also
 //     times d^(-1/2); beta = sigmoid(proj beta); decay g = exp(-exp(A_log[h]) * softplus(a +
-//     dt_bias)) with a = lowrank[n, h d + i].  Output prep [N, PW] float32, every part a
+//     dt_bias)) with a = lowrank[n, h d + i] (one decay per head: a = lowrank[n, h], dt_bias [H],
+//     the same g for all rows).  Output prep [N, PW] float32, every part a
 //     multiple of four floats so that it can be copied 16 bytes at a time:
 //     q [G, dp] | k [G, dp] | g [H, dp] | v [H dv] | beta [H] | q.k [G], where dp >= d is the
 //     number of state rows the scan's threads hold together; rows d .. dp-1 carry q = k = 0,
@@ -42,8 +43,8 @@
 //     rows meanwhile, and writes them back with the write added.  Small blocks, so that many
 //     fit a multiprocessor: the step is bound by reading and writing every state once.
 //   gdr_finish  (one block per token, and one per request)
-//     y = o / sqrt(mean_j o^2 + eps) * norm[j] * sigmoid(gate[n, h dv + j]), gate being the
-//     columns lowrank[n, H d + ...]; and the request's convolution inputs move on (the last
+//     y = o / sqrt(mean_j o^2 + eps) * norm[j] * sigmoid(gate[n, h dv + j]) (or silu), gate being
+//     the columns of lowrank behind the decays'; and the request's convolution inputs move on (the last
 //     taps-1 of old record | this step's rows).
 // All arithmetic is float32; y is the compute type.  Plain reference: tests/plain_ops.py
 // gated_delta.
@@ -62,8 +63,8 @@ __global__ void gdr_prepare_kernel(const float* __restrict__ proj, int P,
                                    const int* __restrict__ q_start,
                                    const int* __restrict__ state_slot, float* __restrict__ prep,
                                    int PW, int H, int G, int d, int dp, int dv, int taps,
-                                   float unit_eps) {
-    extern __shared__ float act[];                 // [C]
+                                   float unit_eps, int head_decay) {
+    extern __shared__ float act[];                 // [C], then [H] decays per head
     const int n = blockIdx.x;
     const int r = token_req[n];
     const int slot = state_slot[r];
@@ -82,6 +83,9 @@ __global__ void gdr_prepare_kernel(const float* __restrict__ proj, int P,
         }
         act[c] = acc * gd_sigmoid(acc);
     }
+    if (head_decay)
+        for (int h = threadIdx.x; h < H; h += blockDim.x)
+            act[C + h] = expf(-expf(a_log[h]) * gd_softplus(lowrank[(size_t)n * LW + h] + dt_bias[h]));
     __syncthreads();
     float* out = prep + (size_t)n * PW;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
@@ -111,7 +115,9 @@ __global__ void gdr_prepare_kernel(const float* __restrict__ proj, int P,
     for (int e = threadIdx.x; e < H * dp; e += blockDim.x) {
         const int h = e / dp, i = e - h * dp;
         float g = 1.f;
-        if (i < d) {
+        if (i < d && head_decay) {
+            g = act[C + h];
+        } else if (i < d) {
             const float a = lowrank[(size_t)n * LW + h * d + i] + dt_bias[h * d + i];
             g = expf(-expf(a_log[h]) * gd_softplus(a));
         }
@@ -490,7 +496,8 @@ __global__ void gdr_finish_kernel(const float* __restrict__ o_in, const float* _
                                   long long rec, const int* __restrict__ token_req,
                                   const int* __restrict__ q_start,
                                   const int* __restrict__ state_slot, TO* __restrict__ y,
-                                  int n_tokens, int H, int G, int d, int dv, int taps, float eps) {
+                                  int n_tokens, int H, int G, int d, int dv, int taps, float eps,
+                                  int gate_off, int silu_gate) {
     rv_pdl_launch_dependents();
     const int C = 2 * G * d + H * dv;
     if ((int)blockIdx.x >= n_tokens) {
@@ -521,7 +528,8 @@ __global__ void gdr_finish_kernel(const float* __restrict__ o_in, const float* _
         ss = rv_warp_sum(ss);
         const float inv = 1.f / sqrtf(ss / (float)dv + eps);
         for (int j = lane; j < dv; j += 32) {
-            const float gate = gd_sigmoid(lowrank[(size_t)n * LW + H * d + h * dv + j]);
+            const float z = lowrank[(size_t)n * LW + gate_off + h * dv + j];
+            const float gate = silu_gate ? z * gd_sigmoid(z) : gd_sigmoid(z);
             rv_store(y + (size_t)n * H * dv + h * dv + j, o[j] * inv * norm_w[j] * gate);
         }
     }
@@ -593,20 +601,23 @@ static void gd_launch_scan(const float* prep, int PW, float* state, long long re
               state, rec, q_start, state_slot, o, H, G, d, dv, taps, col_blocks, chunk);
 }
 
-// proj [N, P] float32 (P >= C + H); lowrank [N, LW] float32 (LW >= H d + H dv: the decays'
-// pre-activations, then the output gates'); filt [C, taps]; a_log [H]; dt_bias [H d]; norm_w
+// proj [N, P] float32 (P >= C + H); lowrank [N, LW] float32 (H d, with head_decay H, of the decays'
+// pre-activations, then H dv of the output gates'; LW is the stride of its rows, which may lie
+// inside proj's); filt [C, taps]; a_log [H]; dt_bias [H d] or [H]; norm_w
 // [dv]; state [slots, record]; scratch: rv_gated_delta_scratch floats; y [N, H dv].
 extern "C" int rv_gated_delta(const float* proj, int P, const float* lowrank, int LW,
                               const float* filt, const float* a_log, const float* dt_bias,
                               const float* norm_w, float* state, const int* token_req,
                               const int* q_start, const int* state_slot, float* scratch, void* y,
                               int out_dtype, int n_tokens, int n_reqs, int H, int G, int d, int dv,
-                              int taps, float unit_eps, float eps, void* stream) {
+                              int taps, float unit_eps, float eps, int head_decay, int silu_gate,
+                              void* stream) {
     if (n_tokens == 0 || n_reqs == 0) return 0;
     if (n_tokens < 0 || n_reqs < 0 || H < 1 || G < 1 || H % G || d < 1 || dv < 1 || taps < 1)
         RV_FAIL("gated_delta: bad sizes");
     const int C = 2 * G * d + H * dv;
-    if (P < C + H || LW < H * d + H * dv) RV_FAIL("gated_delta: rows are too narrow");
+    const int n_decays = head_decay ? H : H * d;
+    if (P < C + H || LW < n_decays + H * dv) RV_FAIL("gated_delta: rows are too narrow");
     int R = 0, TP = 0;
     if (!gd_shape(d, &R, &TP))
         RV_FAIL("gated_delta: key heads of %d are not supported (at most 1024)", d);
@@ -614,7 +625,7 @@ extern "C" int rv_gated_delta(const float* proj, int P, const float* lowrank, in
     const int dp = R * TP;
     const int PW = (2 * G + H) * dp + gd_pad4(H * dv) + gd_pad4(H) + gd_pad4(G);
     const long long rec = rv_gated_delta_record(H, G, d, dv, taps);
-    const size_t smem1 = (size_t)C * sizeof(float);
+    const size_t smem1 = (size_t)(C + (head_decay ? H : 0)) * sizeof(float);
     if (smem1 > 200 * 1024) RV_FAIL("gated_delta: %d channels do not fit shared memory", C);
     float* prep = scratch;
     float* o = scratch + (size_t)n_tokens * PW;
@@ -623,7 +634,7 @@ extern "C" int rv_gated_delta(const float* proj, int P, const float* lowrank, in
         cudaFuncSetAttribute(gdr_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
     rv_launch(gdr_prepare_kernel, dim3(n_tokens), dim3(256), smem1, s, proj, P, lowrank, LW, filt, a_log,
               dt_bias, (const float*)state, rec, token_req, q_start, state_slot, prep, PW, H, G, d, dp, dv,
-              taps, unit_eps);
+              taps, unit_eps, head_decay);
     RV_CHECK_LAUNCH("gated_delta prepare");
     // the staging buffers are sized for the longest portion the step can have if every request
     // brings a token; the size changes only how often the scan's blocks meet, not what they compute
@@ -647,7 +658,7 @@ extern "C" int rv_gated_delta(const float* proj, int P, const float* lowrank, in
     RV_DISPATCH_DTYPE(out_dtype, "gated_delta", {
         rv_launch(gdr_finish_kernel<T>, dim3(n_tokens + n_reqs), dim3(128), 0, s, (const float*)o, proj, P,
                   lowrank, LW, norm_w, state, rec, token_req, q_start, state_slot, (T*)y, n_tokens, H, G, d,
-                  dv, taps, eps);
+                  dv, taps, eps, n_decays, silu_gate);
     });
     RV_CHECK_LAUNCH("gated_delta finish");
     return 0;

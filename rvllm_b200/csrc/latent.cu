@@ -13,7 +13,8 @@
 //                       [N, q_rank]; columns [kv_off, kv_off + rank) are RMS-normed into the first
 //                       `rank` values of the token's page slot; the `rot` columns after them are
 //                       turned by the token's position (dimension i with i + rot/2, angle
-//                       position * freq[i], float32) into the slot's last `rot` values.
+//                       position * freq[i], float32) into the slot's last `rot` values.  `pairs`:
+//                       dimension 2i with 2i + 1 instead; `amplitude` multiplies cosine and sine.
 //   rope_heads          x [N, heads * size] in place: in every head the `rot` values from `off` on
 //                       are turned the same way.
 //   head_gate           x[n, h * size + c] <- x[n, h * size + c] * sigmoid(rows[n, gate_off + h]):
@@ -131,7 +132,8 @@ __global__ void latent_prepare_kernel(const T* __restrict__ rows, int row_stride
                                       const float* __restrict__ kv_weight, float eps,
                                       const float* __restrict__ freq,
                                       const int* __restrict__ positions,
-                                      const int* __restrict__ slot_mapping, T* __restrict__ cache) {
+                                      const int* __restrict__ slot_mapping, T* __restrict__ cache,
+                                      int pairs, float amplitude) {
     rv_pdl_launch_dependents();
     const long long warp = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
     const int lane = threadIdx.x & 31;
@@ -169,16 +171,20 @@ __global__ void latent_prepare_kernel(const T* __restrict__ rows, int row_stride
     for (int i = lane; i < half; i += 32) {
         float sn, cs;
         sincosf(pos * freq[i], &sn, &cs);
-        const float u = rv_load(src + rank + i), v = rv_load(src + rank + half + i);
-        rv_store(dst + rank + i, u * cs - v * sn);
-        rv_store(dst + rank + half + i, v * cs + u * sn);
+        sn *= amplitude;
+        cs *= amplitude;
+        const int iu = rank + (pairs ? 2 * i : i), iv = rank + (pairs ? 2 * i + 1 : half + i);
+        const float u = rv_load(src + iu), v = rv_load(src + iv);
+        rv_store(dst + iu, u * cs - v * sn);
+        rv_store(dst + iv, v * cs + u * sn);
     }
 }
 
 template <typename T>
 __global__ void rope_heads_kernel(T* __restrict__ x, int row_stride, int heads, int size, int off,
                                   int half, const float* __restrict__ freq,
-                                  const int* __restrict__ positions, long long total) {
+                                  const int* __restrict__ positions, long long total, int pairs,
+                                  float amplitude) {
     rv_pdl_launch_dependents();
     const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= total) return;
@@ -190,10 +196,13 @@ __global__ void rope_heads_kernel(T* __restrict__ x, int row_stride, int heads, 
     rv_pdl_wait();
     float sn, cs;
     sincosf(ang, &sn, &cs);
+    sn *= amplitude;
+    cs *= amplitude;
     T* p = x + t * row_stride + (size_t)h * size + off;
-    const float u = rv_load(p + i), v = rv_load(p + half + i);
-    rv_store(p + i, u * cs - v * sn);
-    rv_store(p + half + i, v * cs + u * sn);
+    const int iu = pairs ? 2 * i : i, iv = pairs ? 2 * i + 1 : half + i;
+    const float u = rv_load(p + iu), v = rv_load(p + iv);
+    rv_store(p + iu, u * cs - v * sn);
+    rv_store(p + iv, v * cs + u * sn);
 }
 
 template <typename T>
@@ -212,7 +221,7 @@ extern "C" int rv_latent_prepare(const void* rows, int dtype, int row_stride, in
                                  int q_rank, const float* q_weight, void* cq, int kv_off, int rank,
                                  int rot, const float* kv_weight, float eps, const float* freq,
                                  const int* positions, const int* slot_mapping, void* cache,
-                                 void* stream) {
+                                 int pairs, float amplitude, void* stream) {
     if (n_tokens == 0) return 0;
     if (n_tokens < 0 || rank <= 0 || rot < 0 || rot % 2 || q_rank < 0 || q_off < 0 || kv_off < 0 ||
         row_stride < kv_off + rank + rot || row_stride < q_off + q_rank)
@@ -225,14 +234,14 @@ extern "C" int rv_latent_prepare(const void* rows, int dtype, int row_stride, in
                       (rv_launch(latent_prepare_kernel<T>, dim3((int)blocks), dim3(128), 0,
                                  (cudaStream_t)stream, (const T*)rows, row_stride, n_tokens, q_off,
                                  q_rank, q_weight, (T*)cq, kv_off, rank, rot, kv_weight, eps, freq,
-                                 positions, slot_mapping, (T*)cache)));
+                                 positions, slot_mapping, (T*)cache, pairs, amplitude)));
     RV_CHECK_LAUNCH("latent_prepare");
     return 0;
 }
 
 extern "C" int rv_rope_heads(void* x, int dtype, int row_stride, int n_tokens, int heads, int size,
-                             int off, int rot, const float* freq, const int* positions,
-                             void* stream) {
+                             int off, int rot, const float* freq, const int* positions, int pairs,
+                             float amplitude, void* stream) {
     if (n_tokens == 0 || rot == 0) return 0;
     if (n_tokens < 0 || heads <= 0 || size <= 0 || off < 0 || rot < 0 || rot % 2 || off + rot > size ||
         row_stride < heads * size)
@@ -244,7 +253,7 @@ extern "C" int rv_rope_heads(void* x, int dtype, int row_stride, int n_tokens, i
     RV_DISPATCH_DTYPE(dtype, "rope_heads",
                       (rv_launch(rope_heads_kernel<T>, dim3((int)blocks), dim3(256), 0,
                                  (cudaStream_t)stream, (T*)x, row_stride, heads, size, off, rot / 2,
-                                 freq, positions, total)));
+                                 freq, positions, total, pairs, amplitude)));
     RV_CHECK_LAUNCH("rope_heads");
     return 0;
 }

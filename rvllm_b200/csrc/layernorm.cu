@@ -1,4 +1,4 @@
-// Layer norm with weight and bias, alone or fused with the addition into the float32 residual
+// Layer norm with weight and (optional: null for none) bias, alone or fused with the addition into the float32 residual
 // stream, and with a second layer norm applied to the rows that are being added:
 //   d   = delta                         or  LN(delta; dw, db, deps)   (a norm after a sub-layer)
 //   x   = resid + d  (written back to the stream unless `rows` selects rows)
@@ -79,7 +79,7 @@ __global__ void add_layernorm_kernel(float* __restrict__ resid, const TD* __rest
             }
             const float sd = sqrtf(rv_block_sum(q, scratch) / (float)hidden + deps);
             for (int i = threadIdx.x; i < hidden; i += blockDim.x)
-                row[i] = (row[i] - mean) / sd * dw[i] + db[i];
+                row[i] = (row[i] - mean) / sd * dw[i] + (db ? db[i] : 0.f);
         }
     }
     float s = 0.f;
@@ -99,7 +99,7 @@ __global__ void add_layernorm_kernel(float* __restrict__ resid, const TD* __rest
     const float sd = sqrtf(rv_block_sum(q, scratch) / (float)hidden + eps);
     TO* o = out + (size_t)m * hidden;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x)
-        rv_store(o + i, (row[i] - mean) / sd * w[i] + b[i]);
+        rv_store(o + i, (row[i] - mean) / sd * w[i] + (b ? b[i] : 0.f));
 }
 
 // Widths that are multiples of 4 up to 8192: a thread keeps CHUNKS groups of four values in
@@ -122,7 +122,7 @@ __global__ void add_layernorm_vec_kernel(float* __restrict__ resid, const TD* __
         const int i = threadIdx.x + c * blockDim.x;
         if (i < nvec) {
             wv[c] = ln_load4(w + 4 * i);
-            bv[c] = ln_load4(b + 4 * i);
+            bv[c] = b ? ln_load4(b + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
     const int src = rows ? rows[m] : m;
@@ -145,7 +145,8 @@ __global__ void add_layernorm_vec_kernel(float* __restrict__ resid, const TD* __
             for (int c = 0; c < CHUNKS; ++c) {
                 const int i = threadIdx.x + c * blockDim.x;
                 if (i < nvec) {
-                    const float4 a = ln_load4(dw + 4 * i), o = ln_load4(db + 4 * i);
+                    const float4 a = ln_load4(dw + 4 * i);
+                    const float4 o = db ? ln_load4(db + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
                     v[4 * c] = (v[4 * c] - mean) / sd * a.x + o.x;
                     v[4 * c + 1] = (v[4 * c + 1] - mean) / sd * a.y + o.y;
                     v[4 * c + 2] = (v[4 * c + 2] - mean) / sd * a.z + o.z;
@@ -225,7 +226,7 @@ extern "C" int rv_add_layernorm(float* resid, const void* delta, int delta_dtype
     if (n_rows < 0 || hidden <= 0) RV_FAIL("add_layernorm: bad sizes");
     if (!resid && !delta) RV_FAIL("add_layernorm: neither a stream nor rows to normalise");
     if (!resid && (rows || dw)) RV_FAIL("add_layernorm: without a stream it takes plain rows, all of them");
-    if ((dw == nullptr) != (db == nullptr) || (dw && !delta))
+    if ((db && !dw) || (dw && !delta))
         RV_FAIL("add_layernorm: incomplete arguments for the norm of the added rows");
     cudaStream_t s = (cudaStream_t)stream;
 #define RV_LN(TD, TO) \

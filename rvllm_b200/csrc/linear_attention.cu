@@ -3,8 +3,10 @@
 //     S <- diag(a_t) S + k_t v_t^T;   o_t = S^T q_t
 //     y = o / sqrt(mean(o^2) + eps) * w * gate(g)          the mean over all heads or per head
 //
-// The decay a_t is a constant per head (log_decay [H]) or made by the token for every key channel,
-// log a = logsigmoid(z + bias) / tau.  q, k and v may pass silu; q is multiplied by q_scale.
+// The decay a_t is a constant per head (log_decay [H]), or made by the token for every key channel,
+// log a = logsigmoid(z + bias) / tau, or made by the token for every head (state_space.cuh, whose
+// keys and queries are shared by groups of heads and whose keys are weighed by a step size).  q, k
+// and v may pass silu; q is multiplied by q_scale.
 //
 // rows [N, stride] of the compute type: q [H d] | k [H d] | v [H dv] | g [H dv]; z [N, H d] float32.
 // A request's record: [H][d][dv] float32.  Everything after the projections is float32, but that an
@@ -49,6 +51,24 @@
 #define LA_SCAN_THREADS 64
 #define LA_NG 8             // groups a chunk
 
+// how decays are made
+#define LA_CONST 0          // a constant per head
+#define LA_CHANNEL 1        // by the token, per key channel
+#define LA_TOKEN 2          // by the token, per head
+
+// Where a token's row holds q, k and v, and how many heads share a query and key head.
+struct LaRows {
+    int q, k, v, share;
+};
+// LA_TOKEN, for tokens of portions: B [n, H], the sum of the log decays of the chunk's tokens up to
+// and with this one (float64: differences of sums that large decays have made large stay exact
+// enough), and the keys' weights w [n, H].
+struct LaToken {
+    const double* B;
+    const float* w;
+};
+__device__ __forceinline__ float la_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+
 __device__ __forceinline__ float la_logsigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float la_silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 // a projection as the recurrence reads it
@@ -88,9 +108,12 @@ __device__ __forceinline__ bool la_find(const int* q_start, const int* state_slo
 
 // ---- single tokens ---------------------------------------------------------------------
 // V = 4: 16-byte accesses to the state and sixteen lanes across a tile's 64 columns; V = 1: 64.
-template <typename T, int V>
+// LA_TOKEN: z [n, z_stride] holds the step sizes' pre-activations per head, bias [H] is theirs,
+// log_decay [H] the rates' logarithms (state_space.cuh).
+template <typename T, int V, bool TOKEN>
 __global__ void __launch_bounds__(128) la_token_kernel(
-    const T* __restrict__ rows, int stride, const float* __restrict__ z, const float* __restrict__ log_decay,
+    const T* __restrict__ rows, int stride, const LaRows lr, const float* __restrict__ z, int z_stride,
+    const float* __restrict__ log_decay,
     const float* __restrict__ bias, float tau, const int* __restrict__ q_start,
     const int* __restrict__ state_slot, float* __restrict__ state, float* __restrict__ num, int H,
     int d, int dv, int act, float q_scale) {
@@ -107,10 +130,16 @@ __global__ void __launch_bounds__(128) la_token_kernel(
     rv_pdl_wait();
     if (slot < 0) return;
     const T* row = rows + (size_t)t * stride;
-    const float ad = log_decay ? expf(log_decay[h]) : 0.f;
+    float ad = log_decay ? expf(log_decay[h]) : 0.f, wk = 1.f;
+    if (TOKEN) {
+        wk = la_softplus(z[(size_t)t * z_stride + h] + bias[h]);
+        ad = expf(-ad * wk);
+    }
+    const int kh = h / lr.share;
     for (int i = threadIdx.x; i < d; i += 128) {
-        qs[i] = la_in(row + h * d + i, act);
-        ks[i] = la_in(row + (H + h) * d + i, act);
+        qs[i] = la_in(row + lr.q + kh * d + i, act);
+        const float k = la_in(row + lr.k + kh * d + i, act);
+        ks[i] = TOKEN ? k * wk : k;
         as[i] = log_decay ? ad : expf(la_logsigmoid(z[(size_t)t * H * d + h * d + i] + bias[h * d + i]) / tau);
     }
     const int cl = threadIdx.x % LANES, rg = threadIdx.x / LANES;
@@ -119,7 +148,7 @@ __global__ void __launch_bounds__(128) la_token_kernel(
 #pragma unroll
     for (int e = 0; e < V; ++e) {
         o[e] = 0.f;
-        v[e] = col + e < dv ? la_in(row + 2 * H * d + h * dv + col + e, act) : 0.f;
+        v[e] = col + e < dv ? la_in(row + lr.v + h * dv + col + e, act) : 0.f;
     }
     __syncthreads();
     float* S = state + ((size_t)slot * H + h) * d * dv;
@@ -159,12 +188,14 @@ __global__ void __launch_bounds__(128) la_token_kernel(
 }
 
 // ---- portions: every chunk's own contribution to the state ----------------------------------
-template <typename T, bool CHANNEL>
+template <typename T, int MODE>
 __global__ void __launch_bounds__(256) la_state_kernel(
-    const T* __restrict__ rows, int stride, const float* __restrict__ zr, const float* __restrict__ log_decay,
+    const T* __restrict__ rows, int stride, const LaRows lr, const LaToken tk, const float* __restrict__ zr,
+    const float* __restrict__ log_decay,
     const float* __restrict__ bias, float tau, const int* __restrict__ q_start,
     const int* __restrict__ state_slot, int first_req, int n_reqs, float* __restrict__ kv,
     float* __restrict__ dec, int H, int d, int dv, int act) {
+    constexpr bool CHANNEL = MODE == LA_CHANNEL, TOKEN = MODE == LA_TOKEN;
     rv_pdl_launch_dependents();
     extern __shared__ __align__(16) float sm[];
     float* ks = sm;                                              // [64 tokens][LD]: channels
@@ -191,16 +222,22 @@ __global__ void __launch_bounds__(256) la_state_kernel(
     const int x = tid & 63, y = tid >> 6;
     const int dn = min(LA_T, d - d0), vn = min(LA_T, dv - v0);
     const T* base = rows + (size_t)t0 * stride;
-    const float ld = CHANNEL ? 0.f : log_decay[h];
+    const float ld = MODE != LA_CONST ? 0.f : log_decay[h];
     const float bz = CHANNEL && x < dn ? bias[h * d + d0 + x] : 0.f;
+    const int kh = h / lr.share;
+    const double last = TOKEN ? tk.B[(size_t)(t0 + L - 1) * H + h] : 0.;
     // four values of one column at a time are requested before any is worked on
 #pragma unroll 4
     for (int j = y; j < LA_C; j += 4) {
         const T* row = base + (size_t)j * stride;
         const bool tj = j < L;
-        float k = tj && x < dn ? la_in(row + (H + h) * d + d0 + x, act) : 0.f;
-        const float v = tj && x < vn ? la_in(row + 2 * H * d + h * dv + v0 + x, act) : 0.f;
-        if (!CHANNEL) k *= expf(ld * (float)(L - 1 - min(j, L - 1)));
+        float k = tj && x < dn ? la_in(row + lr.k + kh * d + d0 + x, act) : 0.f;
+        const float v = tj && x < vn ? la_in(row + lr.v + h * dv + v0 + x, act) : 0.f;
+        if (MODE == LA_CONST) k *= expf(ld * (float)(L - 1 - min(j, L - 1)));
+        if (TOKEN) {
+            const size_t at_j = (size_t)(t0 + min(j, L - 1)) * H + h;
+            k *= expf((float)(last - tk.B[at_j])) * tk.w[at_j];
+        }
         ks[j * LA_LD + x] = k;
         vs[j * LA_LD + x] = v;
         if (CHANNEL) {
@@ -260,11 +297,12 @@ __global__ void __launch_bounds__(256) la_state_kernel(
 }
 
 // ---- portions: the states between the chunks ---------------------------------------------------
-template <bool CHANNEL, int V>
+template <int MODE, int V>
 __global__ void __launch_bounds__(LA_SCAN_THREADS) la_scan_kernel(
     const float* __restrict__ log_decay, const int* __restrict__ q_start,
     const int* __restrict__ state_slot, int first_req, float* __restrict__ kv,
     const float* __restrict__ dec, float* __restrict__ state, int H, int d, int dv) {
+    constexpr bool CHANNEL = MODE == LA_CHANNEL, MADE = MODE != LA_CONST;
     rv_pdl_launch_dependents();
     const int h = blockIdx.y, r = first_req + blockIdx.z;
     const int slot = state_slot[r];
@@ -279,16 +317,17 @@ __global__ void __launch_bounds__(LA_SCAN_THREADS) la_scan_kernel(
     }
     __syncthreads();
     const int last_len = q_start[r + 1] - q_start[r] - (n - 1) * LA_C;
-    const float ld = CHANNEL ? 0.f : log_decay[h];
+    const float ld = MADE ? 0.f : log_decay[h];
     rv_pdl_wait();
     const long long el = ((long long)blockIdx.x * LA_SCAN_THREADS + threadIdx.x) * V;
     if (n == 0 || el >= (long long)d * dv) return;
     const int ch = (int)(el / dv);
     float* rec = state + ((size_t)slot * H + h) * d * dv + el;
     float* p = kv + ((size_t)first_item * H + h) * d * dv + el;
-    const float* dp = CHANNEL ? dec + ((size_t)first_item * H + h) * d + ch : nullptr;
-    const size_t step = (size_t)H * d * dv, dstep = (size_t)H * d;
-    const float full = CHANNEL ? 0.f : expf(ld * (float)LA_C), rest = CHANNEL ? 0.f : expf(ld * (float)last_len);
+    const float* dp = CHANNEL ? dec + ((size_t)first_item * H + h) * d + ch
+                              : MADE ? dec + (size_t)first_item * H + h : nullptr;
+    const size_t step = (size_t)H * d * dv, dstep = CHANNEL ? (size_t)H * d : (size_t)H;
+    const float full = MADE ? 0.f : expf(ld * (float)LA_C), rest = MADE ? 0.f : expf(ld * (float)last_len);
     float S[V];
 #pragma unroll
     for (int e = 0; e < V; ++e) S[e] = 0.f;
@@ -311,7 +350,7 @@ __global__ void __launch_bounds__(LA_SCAN_THREADS) la_scan_kernel(
             } else {
                 in[u][0] = *s;
             }
-            a[u] = CHANNEL ? dp[(size_t)(c0 + u) * dstep] : (c0 + u == n - 1 ? rest : full);
+            a[u] = MADE ? dp[(size_t)(c0 + u) * dstep] : (c0 + u == n - 1 ? rest : full);
         }
 #pragma unroll
         for (int u = 0; u < U; ++u) {
@@ -331,14 +370,18 @@ __global__ void __launch_bounds__(LA_SCAN_THREADS) la_scan_kernel(
 // A thread's share of a 64 x 64 product is rows 4 ty .. + 3 by columns 4 tx .. + 3; a warp's eight
 // rows are one group.  Operands lie with the summed index first ([c][64 tokens] and so on), so that
 // a thread reads four of its rows and four of its columns with one access each.
-template <typename T, bool CHANNEL>
+template <typename T, int MODE>
 __global__ void __launch_bounds__(256) la_out_kernel(
-    const T* __restrict__ rows, int stride, const float* __restrict__ zr, const float* __restrict__ log_decay,
+    const T* __restrict__ rows, int stride, const LaRows lr, const LaToken tk, const float* __restrict__ zr,
+    const float* __restrict__ log_decay,
     const float* __restrict__ bias, float tau, const int* __restrict__ q_start,
     const int* __restrict__ state_slot, int first_req, int n_reqs, const float* __restrict__ kv,
     float* __restrict__ num, int H, int d, int dv, int act, float q_scale) {
+    constexpr bool CHANNEL = MODE == LA_CHANNEL, TOKEN = MODE == LA_TOKEN;
     rv_pdl_launch_dependents();
     extern __shared__ __align__(16) float sm[];
+    __shared__ double bt[TOKEN ? LA_C : 1];         // TOKEN: B and the keys' weights
+    __shared__ float wt[TOKEN ? LA_C : 1];
     constexpr int SL = LA_DK * LA_LD;
     float* qt = sm;                                 // [DK][LD]: q e^(B_i - B before its group)
     float* kt = qt + SL;                            // [DK][LD]: k e^(B at its group's end - B_j)
@@ -369,13 +412,19 @@ __global__ void __launch_bounds__(256) la_out_kernel(
     const float* Sg = kv + ((size_t)item * H + h) * d * dv;
     const int vn = min(LA_T, dv - v0);
     const int ty = tid >> 4, tx = tid & 15;
-    const float ld = CHANNEL ? 0.f : log_decay[h];
+    const float ld = MODE != LA_CONST ? 0.f : log_decay[h];
+    const int kh = h / lr.share;
+    if (TOKEN && tid < LA_C) {
+        const size_t at_j = (size_t)(t0 + min(tid, L - 1)) * H + h;
+        bt[tid] = tk.B[at_j];
+        wt[tid] = tid < L ? tk.w[at_j] : 0.f;
+    }
     // values [64 tokens][64 columns]
     {
         const int x = tid & 63, y = tid >> 6;
 #pragma unroll 4
         for (int j = y; j < LA_C; j += 4)
-            vs[j * LA_LD + x] = j < L && x < vn ? la_in(base + (size_t)j * stride + 2 * H * d + h * dv + v0 + x, act) : 0.f;
+            vs[j * LA_LD + x] = j < L && x < vn ? la_in(base + (size_t)j * stride + lr.v + h * dv + v0 + x, act) : 0.f;
     }
     float p[4][4], o[4][4];
 #pragma unroll
@@ -408,9 +457,9 @@ __global__ void __launch_bounds__(256) la_out_kernel(
             for (int u = warp; u < (LA_C / 4) * (LA_DK / 8); u += 8) {
                 const int j = (u >> 2) * 4 + tl, c = (u & 3) * 8 + cl;
                 const bool in = j < L && c < cn;
-                const T* row = base + (size_t)j * stride + h * d + c0 + c;
-                const float q = in ? la_in(row, act) : 0.f;
-                const float k = in ? la_in(row + (size_t)H * d, act) : 0.f;
+                const T* row = base + (size_t)j * stride + kh * d + c0 + c;
+                const float q = in ? la_in(row + lr.q, act) : 0.f;
+                const float k = in ? la_in(row + lr.k, act) : 0.f;
                 if (CHANNEL) {
                     qr[c * LA_LD + j] = q;
                     kr[c * LA_LD + j] = k;
@@ -503,7 +552,8 @@ __global__ void __launch_bounds__(256) la_out_kernel(
     for (int i = 0; i < 4; ++i) {
         const int ri = 4 * ty + i;
         float row_f = 1.f;
-        if (!CHANNEL) row_f = expf(ld * (float)(ri + 1));
+        if (MODE == LA_CONST) row_f = expf(ld * (float)(ri + 1));
+        if (TOKEN) row_f = expf((float)bt[ri]);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int cj = 4 * tx + e;
@@ -512,7 +562,9 @@ __global__ void __launch_bounds__(256) la_out_kernel(
                 else if (J > I) ps[cj * LA_LD + ri] = 0.f;
                 else if (cj > ri) ps[cj * LA_LD + ri] = 0.f;     // inside a group: the pairs below
             } else {
-                ps[cj * LA_LD + ri] = cj <= ri ? p[i][e] * expf(ld * (float)(ri - cj)) : 0.f;
+                const float f = TOKEN ? (cj <= ri ? expf((float)(bt[ri] - bt[cj])) * wt[cj] : 0.f)
+                                      : expf(ld * (float)(ri - cj));
+                ps[cj * LA_LD + ri] = cj <= ri ? p[i][e] * f : 0.f;
                 o[i][e] *= row_f;
             }
         }
@@ -671,12 +723,14 @@ extern "C" long long rv_linear_attention_scratch(int n_tokens, int n_decode, int
 }
 
 struct LaArgs {
+    LaRows lr;
+    LaToken tk;
     float* z;
     const float *log_decay, *bias, *norm_w;
     float *state, *scratch;
     const int *token_req, *q_start, *state_slot;
     float tau, q_scale, eps;
-    int stride, n_tokens, n_decode, n_reqs, H, d, dv, act, norm_head, gate, tensor;
+    int stride, z_stride, n_tokens, n_decode, n_reqs, H, d, dv, act, norm_head, gate, tensor;
 };
 
 #define LA_SMEM(kernel, bytes)                                                                       \
@@ -691,37 +745,37 @@ struct LaArgs {
     }
 
 // The tensor-core forms exist for bfloat16 rows.
-template <bool CH>
+template <int CH>
 static int la_tensor_launch(const float* rows, const LaArgs& a, int what, dim3 grid, float* kv, float* dec,
                             float* num, cudaStream_t s) {
     (void)rows; (void)a; (void)what; (void)grid; (void)kv; (void)dec; (void)num; (void)s;
     RV_FAIL("linear_attention: float32 rows on the tensor cores");
 }
-template <bool CH>
+template <int CH>
 static int la_tensor_launch(const bf16* rows, const LaArgs& a, int what, dim3 grid, float* kv, float* dec,
                             float* num, cudaStream_t s) {
     if (what == 0) {
         const size_t smem = lm_state_smem();
         LA_SMEM(la_state_mma_kernel<CH>, smem)
-        rv_launch(la_state_mma_kernel<CH>, grid, dim3(128), smem, s, rows, a.stride, (const float*)a.z,
+        rv_launch(la_state_mma_kernel<CH>, grid, dim3(128), smem, s, rows, a.stride, a.lr, a.tk, (const float*)a.z,
                   a.log_decay, a.q_start, a.state_slot, a.n_decode, a.n_reqs, kv, dec, a.H, a.d, a.dv, a.act);
     } else {
-        const size_t smem = lm_out_smem(CH, a.d);
+        const size_t smem = lm_out_smem(CH == LA_CHANNEL, a.d);
         LA_SMEM(la_out_mma_kernel<CH>, smem)
-        rv_launch(la_out_mma_kernel<CH>, grid, dim3(128), smem, s, rows, a.stride, (const float*)a.z,
+        rv_launch(la_out_mma_kernel<CH>, grid, dim3(128), smem, s, rows, a.stride, a.lr, a.tk, (const float*)a.z,
                   a.log_decay, a.q_start, a.state_slot, a.n_decode, a.n_reqs, (const float*)kv, num, a.H, a.d, a.dv,
                   a.act, a.q_scale);
     }
     return 0;
 }
 
-template <typename T, bool CH>
+template <typename T, int CH>
 static int la_portions(const T* rows, const LaArgs& a, float* num, float* kv, float* dec, unsigned items,
                        cudaStream_t s) {
     const int tiles_d = (a.d + LA_T - 1) / LA_T, tiles_v = (a.dv + LA_T - 1) / LA_T;
     const dim3 g1(items, a.H, tiles_d * tiles_v), g3(items, a.H, tiles_v);
     if (a.tensor) {
-        if (CH) {
+        if (CH == LA_CHANNEL) {
             const int width = a.H * a.d;
             rv_launch(la_decay_kernel, dim3(items, (width + 31) / 32), dim3(256), 0, s, a.z, a.bias,
                       1.4426950408889634f / a.tau, a.q_start, a.state_slot, a.n_decode, a.n_reqs, width);
@@ -729,10 +783,10 @@ static int la_portions(const T* rows, const LaArgs& a, float* num, float* kv, fl
         }
         if (la_tensor_launch<CH>(rows, a, 0, g1, kv, dec, num, s)) return 1;
     } else {
-        const size_t smem = (size_t)((CH ? 3 : 2) * LA_C * LA_LD + 4 * 64) * sizeof(float);
+        const size_t smem = (size_t)((CH == LA_CHANNEL ? 3 : 2) * LA_C * LA_LD + 4 * 64) * sizeof(float);
         auto kernel = la_state_kernel<T, CH>;
         LA_SMEM(kernel, smem)
-        rv_launch(kernel, g1, dim3(256), smem, s, rows, a.stride, a.z, a.log_decay, a.bias, a.tau, a.q_start,
+        rv_launch(kernel, g1, dim3(256), smem, s, rows, a.stride, a.lr, a.tk, a.z, a.log_decay, a.bias, a.tau, a.q_start,
                   a.state_slot, a.n_decode, a.n_reqs, kv, dec, a.H, a.d, a.dv, a.act);
     }
     RV_CHECK_LAUNCH("linear_attention_state");
@@ -749,39 +803,44 @@ static int la_portions(const T* rows, const LaArgs& a, float* num, float* kv, fl
     if (a.tensor) {
         if (la_tensor_launch<CH>(rows, a, 1, g3, kv, dec, num, s)) return 1;
     } else {
-        const size_t smem = (size_t)((CH ? 6 : 3) * LA_DK * LA_LD + 2 * LA_C * LA_LD +
-                                     (CH ? (LA_NG + 1 + LA_NG * LA_NG) * (LA_DK + 1) : 0)) * sizeof(float);
+        const size_t smem = (size_t)((CH == LA_CHANNEL ? 6 : 3) * LA_DK * LA_LD + 2 * LA_C * LA_LD +
+                                     (CH == LA_CHANNEL ? (LA_NG + 1 + LA_NG * LA_NG) * (LA_DK + 1) : 0)) * sizeof(float);
         auto kernel = la_out_kernel<T, CH>;
         LA_SMEM(kernel, smem)
-        rv_launch(kernel, g3, dim3(256), smem, s, rows, a.stride, a.z, a.log_decay, a.bias, a.tau, a.q_start,
+        rv_launch(kernel, g3, dim3(256), smem, s, rows, a.stride, a.lr, a.tk, a.z, a.log_decay, a.bias, a.tau, a.q_start,
                   a.state_slot, a.n_decode, a.n_reqs, (const float*)kv, num, a.H, a.d, a.dv, a.act, a.q_scale);
     }
     RV_CHECK_LAUNCH("linear_attention_out");
     return 0;
 }
 
+// Requests [0, n_decode): one token each.
+template <typename T, bool TOKEN>
+static int la_tokens(const T* rows, const LaArgs& a, float* num, cudaStream_t s) {
+    const bool v4 = a.dv % 4 == 0 && ((uintptr_t)a.state & 15) == 0;
+    const size_t smem = (size_t)(3 * a.d + (v4 ? 8 : 2) * LA_T) * sizeof(float);
+    const dim3 grid((a.dv + LA_T - 1) / LA_T, a.H, a.n_decode);
+    if (v4)
+        rv_launch(la_token_kernel<T, 4, TOKEN>, grid, dim3(128), smem, s, rows, a.stride, a.lr, a.z, a.z_stride,
+                  a.log_decay, a.bias, a.tau, a.q_start, a.state_slot, a.state, num, a.H, a.d, a.dv, a.act, a.q_scale);
+    else
+        rv_launch(la_token_kernel<T, 1, TOKEN>, grid, dim3(128), smem, s, rows, a.stride, a.lr, a.z, a.z_stride,
+                  a.log_decay, a.bias, a.tau, a.q_start, a.state_slot, a.state, num, a.H, a.d, a.dv, a.act, a.q_scale);
+    RV_CHECK_LAUNCH("linear_attention_token");
+    return 0;
+}
+
 template <typename T>
 static int la_run(const T* rows, const LaArgs& a, T* out, cudaStream_t s) {
     float* num = a.scratch;
-    if (a.n_decode > 0) {
-        const bool v4 = a.dv % 4 == 0 && ((uintptr_t)a.state & 15) == 0;
-        const size_t smem = (size_t)(3 * a.d + (v4 ? 8 : 2) * LA_T) * sizeof(float);
-        const dim3 grid((a.dv + LA_T - 1) / LA_T, a.H, a.n_decode);
-        if (v4)
-            rv_launch(la_token_kernel<T, 4>, grid, dim3(128), smem, s, rows, a.stride, a.z, a.log_decay, a.bias,
-                      a.tau, a.q_start, a.state_slot, a.state, num, a.H, a.d, a.dv, a.act, a.q_scale);
-        else
-            rv_launch(la_token_kernel<T, 1>, grid, dim3(128), smem, s, rows, a.stride, a.z, a.log_decay, a.bias,
-                      a.tau, a.q_start, a.state_slot, a.state, num, a.H, a.d, a.dv, a.act, a.q_scale);
-        RV_CHECK_LAUNCH("linear_attention_token");
-    }
+    if (a.n_decode > 0 && la_tokens<T, false>(rows, a, num, s)) return 1;
     if (a.n_tokens > a.n_decode && a.n_reqs > a.n_decode) {
         const long long items = la_items(a.n_tokens - a.n_decode, a.n_reqs - a.n_decode);
         float* kv = a.scratch + (((size_t)a.n_tokens * a.H * a.dv + 3) & ~(size_t)3);
         float* dec = kv + (size_t)items * a.H * a.d * a.dv;
         if (items > 0x7fffffffLL) RV_FAIL("linear_attention: too many tokens");
-        if (a.log_decay ? la_portions<T, false>(rows, a, num, kv, dec, (unsigned)items, s)
-                        : la_portions<T, true>(rows, a, num, kv, dec, (unsigned)items, s))
+        if (a.log_decay ? la_portions<T, LA_CONST>(rows, a, num, kv, dec, (unsigned)items, s)
+                        : la_portions<T, LA_CHANNEL>(rows, a, num, kv, dec, (unsigned)items, s))
             return 1;
     }
     const int g_off = 2 * a.H * a.d + a.H * a.dv;
@@ -834,9 +893,11 @@ extern "C" int rv_linear_attention(const void* rows, int dtype, int stride, floa
     if ((uintptr_t)scratch & 15) RV_FAIL("linear_attention: the scratch must be 16-byte aligned");
     tensor = tensor && dtype == RV_DTYPE_BF16 && d % 16 == 0 && dv % 16 == 0 && d <= 128 && stride % 8 == 0 &&
              (((uintptr_t)rows | (uintptr_t)z) & 15) == 0;
-    const LaArgs a = {z, log_decay, bias, norm_w, state, scratch, token_req, q_start, state_slot, tau, q_scale, eps,
-                      stride, n_tokens, n_decode, n_reqs, H, d, dv, act, norm_head, gate, tensor};
+    const LaArgs a = {{0, H * d, 2 * H * d, 1}, {nullptr, nullptr}, z, log_decay, bias, norm_w, state, scratch, token_req, q_start, state_slot, tau, q_scale, eps,
+                      stride, H * d, n_tokens, n_decode, n_reqs, H, d, dv, act, norm_head, gate, tensor};
     RV_DISPATCH_DTYPE(dtype, "linear_attention",
                       return la_run<T>((const T*)rows, a, (T*)out, (cudaStream_t)stream));
     return 0;
 }
+
+#include "state_space.cuh"

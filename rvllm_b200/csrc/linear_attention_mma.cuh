@@ -97,12 +97,13 @@ __global__ void __launch_bounds__(256) la_decay_kernel(float* __restrict__ z, co
 }
 
 // KV = sum_j (k_j e^(B_L - B_j)) v_j^T for 64 channels by 64 columns: a warp has 16 channels.
-template <bool CHANNEL>
+template <int MODE>
 __global__ void __launch_bounds__(128) la_state_mma_kernel(
-    const bf16* __restrict__ rows, int stride, const float* __restrict__ zb,
+    const bf16* __restrict__ rows, int stride, const LaRows lr, const LaToken tk, const float* __restrict__ zb,
     const float* __restrict__ log_decay,
     const int* __restrict__ q_start, const int* __restrict__ state_slot, int first_req, int n_reqs,
     float* __restrict__ kv, float* __restrict__ dec, int H, int d, int dv, int act) {
+    constexpr bool CHANNEL = MODE == LA_CHANNEL, TOKEN = MODE == LA_TOKEN;
     rv_pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char smraw[];
     bf16* ks = (bf16*)smraw;                            // [3][64 tokens][LM_LD]
@@ -118,7 +119,9 @@ __global__ void __launch_bounds__(128) la_state_mma_kernel(
     if (t0 < 0) return;
     const int dn = min(LA_T, d - d0), vn = min(LA_T, dv - v0);
     const bf16* base = rows + (size_t)t0 * stride;
-    const float ld = CHANNEL ? 0.f : log_decay[h];
+    const float ld = MODE != LA_CONST ? 0.f : log_decay[h];
+    const int kh = h / lr.share;
+    const double last = TOKEN ? tk.B[(size_t)(t0 + L - 1) * H + h] : 0.;
     // eight columns a thread: 8 chunks a row, 16 rows a round, 4 rounds
     const int ch = tid & 7, jr = tid >> 3;
     uint4 kreg[4], vreg[4];
@@ -126,8 +129,8 @@ __global__ void __launch_bounds__(128) la_state_mma_kernel(
     for (int u = 0; u < 4; ++u) {
         const int j = jr + 16 * u;
         const bf16* row = base + (size_t)j * stride;
-        kreg[u] = lm_in8(row + (H + h) * d + d0 + 8 * ch, j < L && 8 * ch < dn, act);
-        vreg[u] = lm_in8(row + 2 * H * d + h * dv + v0 + 8 * ch, j < L && 8 * ch < vn, act);
+        kreg[u] = lm_in8(row + lr.k + kh * d + d0 + 8 * ch, j < L && 8 * ch < dn, act);
+        vreg[u] = lm_in8(row + lr.v + h * dv + v0 + 8 * ch, j < L && 8 * ch < vn, act);
     }
     float bl[8];                                        // CHANNEL: B of the chunk's last token
     if (CHANNEL) {
@@ -146,7 +149,11 @@ __global__ void __launch_bounds__(128) la_state_mma_kernel(
         const unsigned in[4] = {kreg[u].x, kreg[u].y, kreg[u].z, kreg[u].w};
         unsigned o[3][4];
         float f = 0.f, bj[8];
-        if (!CHANNEL) f = expf(ld * (float)(L - 1 - min(j, L - 1)));
+        if (MODE == LA_CONST) f = expf(ld * (float)(L - 1 - min(j, L - 1)));
+        if (TOKEN) {
+            const size_t at_j = (size_t)(t0 + min(j, L - 1)) * H + h;
+            f = expf((float)(last - tk.B[at_j])) * tk.w[at_j];
+        }
         if (CHANNEL) {
             const float* p = zb + (size_t)(t0 + min(j, L - 1)) * H * d + h * d + d0 + 8 * ch;
 #pragma unroll
@@ -205,12 +212,13 @@ __global__ void __launch_bounds__(128) la_state_mma_kernel(
 // (B in powers of two here: zb is what la_decay left.)
 // o = (scores, masked) V + (q e^(B_i)) S for the chunk's 64 tokens by 64 columns: a warp has 16
 // tokens.  CHANNEL: B is kept whole (bs), q e^(B_i) is formed in fragments, k e^(-B_j) in shared memory.
-template <bool CHANNEL>
+template <int MODE>
 __global__ void __launch_bounds__(128) la_out_mma_kernel(
-    const bf16* __restrict__ rows, int stride, const float* __restrict__ zb,
+    const bf16* __restrict__ rows, int stride, const LaRows lr, const LaToken tk, const float* __restrict__ zb,
     const float* __restrict__ log_decay,
     const int* __restrict__ q_start, const int* __restrict__ state_slot, int first_req, int n_reqs,
     const float* __restrict__ kv, float* __restrict__ num, int H, int d, int dv, int act, float q_scale) {
+    constexpr bool CHANNEL = MODE == LA_CHANNEL, TOKEN = MODE == LA_TOKEN;
     rv_pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char smraw[];
     const int LQ = d + 8, LB = d + 2;
@@ -219,15 +227,22 @@ __global__ void __launch_bounds__(128) la_out_mma_kernel(
     bf16* qs = vs + LA_C * LM_LD;                       // [64][LQ]
     bf16* ks = qs + LA_C * LQ;                          // [1 or 3][64][LQ]
     float* bs = (float*)(ks + (CHANNEL ? 3 : 1) * LA_C * LQ);   // CHANNEL: [64][LB]
-    __shared__ float pw[LA_C + 1];                      // constant decay: its powers
+    __shared__ float pw[LA_C + 1];                      // constant decay: its powers; TOKEN: weights
+    __shared__ double bt[TOKEN ? LA_C : 1];             // TOKEN: B
     __shared__ int at[2];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int item = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * LA_T;
     lm_locate(q_start, state_slot, first_req, n_reqs, item, at);
     const int t0 = at[0], L = at[1];
-    if (!CHANNEL && tid <= LA_C) pw[tid] = expf(log_decay[h] * (float)tid);
+    if (MODE == LA_CONST && tid <= LA_C) pw[tid] = expf(log_decay[h] * (float)tid);
     rv_pdl_wait();
     if (t0 < 0) return;
+    if (TOKEN && tid < LA_C) {
+        const size_t at_j = (size_t)(t0 + min(tid, L - 1)) * H + h;
+        bt[tid] = tk.B[at_j];
+        pw[tid] = tid < L ? tk.w[at_j] : 0.f;
+    }
+    const int kh = h / lr.share;
     const int vn = min(LA_T, dv - v0);
     const bf16* base = rows + (size_t)t0 * stride;
     // values, queries, keys: eight columns a thread and access
@@ -237,15 +252,15 @@ __global__ void __launch_bounds__(128) la_out_mma_kernel(
         for (int u = 0; u < 4; ++u) {
             const int j = jr + 16 * u;
             *(uint4*)(vs + j * LM_LD + 8 * ch) =
-                lm_in8(base + (size_t)j * stride + 2 * H * d + h * dv + v0 + 8 * ch, j < L && 8 * ch < vn, act);
+                lm_in8(base + (size_t)j * stride + lr.v + h * dv + v0 + 8 * ch, j < L && 8 * ch < vn, act);
         }
         const int cpr = d >> 3;                         // chunks a row
 #pragma unroll 4
         for (int n = tid; n < LA_C * cpr; n += 128) {
             const int j = n / cpr, c = (n - j * cpr) * 8;
-            const bf16* row = base + (size_t)j * stride + h * d + c;
-            *(uint4*)(qs + j * LQ + c) = lm_in8(row, j < L, act);
-            *(uint4*)(ks + j * LQ + c) = lm_in8(row + (size_t)H * d, j < L, act);
+            const bf16* row = base + (size_t)j * stride + kh * d + c;
+            *(uint4*)(qs + j * LQ + c) = lm_in8(row + lr.q, j < L, act);
+            *(uint4*)(ks + j * LQ + c) = lm_in8(row + lr.k, j < L, act);
         }
     }
     // the state before the chunk, in three parts
@@ -361,14 +376,18 @@ __global__ void __launch_bounds__(128) la_out_mma_kernel(
         }
     }
     if (!CHANNEL) {
-        const float fa = pw[row_a + 1], fb = pw[row_b + 1];
+        const float fa = TOKEN ? expf((float)bt[row_a]) : pw[row_a + 1];
+        const float fb = TOKEN ? expf((float)bt[row_b]) : pw[row_b + 1];
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
             o[i][0] *= fa; o[i][1] *= fa;
             o[i][2] *= fb; o[i][3] *= fb;
         }
     }
-    // decays between the pairs (constant ones) and the mask, then the values
+    // decays between the pairs (those of whole heads) and the mask, then the values
+    auto pair = [&](int r, int j) {
+        return TOKEN ? expf((float)(bt[r] - bt[j])) * pw[j] : pw[r - j];
+    };
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {
         if (kk > warp) continue;
@@ -377,8 +396,8 @@ __global__ void __launch_bounds__(128) la_out_mma_kernel(
         for (int e = 0; e < 4; ++e) {
             const int i = 2 * kk + (e >> 1), r = (e & 1) ? row_b : row_a, j = 8 * i + (lane & 3) * 2;
             float x = p[i][(e & 1) * 2], y = p[i][(e & 1) * 2 + 1];
-            x = j <= r ? (CHANNEL ? x : x * pw[r - j]) : 0.f;
-            y = j + 1 <= r ? (CHANNEL ? y : y * pw[r - j - 1]) : 0.f;
+            x = j <= r ? (CHANNEL ? x : x * pair(r, j)) : 0.f;
+            y = j + 1 <= r ? (CHANNEL ? y : y * pair(r, j + 1)) : 0.f;
             lm_split(x, y, a[0][e], a[1][e], a[2][e]);
         }
 #pragma unroll

@@ -24,7 +24,9 @@
 //                  max(<up_e[f], x_t>, 0)^2.
 //   moe_down       out[t, w] = sum_k weights[t, k] * <down_e(k)[w], act[t * top + k]>, the sum in
 //                  the order of k; down is [E, W, F].  `addend` [N, W], if given, is where each sum
-//                  starts (the output of an expert that every token uses).
+//                  starts (the output of an expert that every token uses).  An id of E or more (an
+//                  identity expert: the router may have more outputs than there are experts)
+//                  counts as <..> = x[t, w], the token's own value.
 // Dot products and the activation are float32; act is rounded to the storage type.
 // Plain references: tests/plain_ops.py moe_select, moe_experts.
 #include "common.cuh"
@@ -340,13 +342,15 @@ __global__ void moe_gate_up_kernel(const T* __restrict__ x, const int* __restric
 template <typename T>
 __global__ void moe_down_kernel(const T* __restrict__ act, const int* __restrict__ ids,
                                 const float* __restrict__ weights, const T* __restrict__ down,
-                                const T* __restrict__ addend, T* __restrict__ out, int top, int E,
-                                int W, int F) {
+                                const T* __restrict__ addend, const T* __restrict__ x,
+                                T* __restrict__ out, int top, int E, int W, int F) {
     rv_pdl_prologue();
     extern __shared__ float as[];                      // [top * F]
     const int t = blockIdx.x;
-    for (int i = threadIdx.x; i < top * F; i += blockDim.x)
-        as[i] = rv_load(act + (size_t)t * top * F + i);
+    for (int k = 0; k < top; ++k)
+        if ((unsigned)ids[(size_t)t * top + k] < (unsigned)E)
+            for (int i = threadIdx.x; i < F; i += blockDim.x)
+                as[k * F + i] = rv_load(act + ((size_t)t * top + k) * F + i);
     __syncthreads();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
     const int w_end = min(W, (int)(blockIdx.y + 1) * MOE_ROWS);
@@ -354,6 +358,7 @@ __global__ void moe_down_kernel(const T* __restrict__ act, const int* __restrict
         float y = addend ? rv_load(addend + (size_t)t * W + w) : 0.f;
         for (int k = 0; k < top; ++k) {
             const int e = ids[(size_t)t * top + k];
+            if (e >= E) y += weights[(size_t)t * top + k] * rv_load(x + (size_t)t * W + w);
             if (e < 0 || e >= E) continue;
             const T* row = down + ((size_t)e * W + w) * F;
             float s = 0.f;
@@ -436,8 +441,8 @@ extern "C" int rv_moe_experts_simple(const void* x, int dtype, const int* ids, c
                   dim3(128), smem1, s, (const T*)x, ids, (const T*)gate_up, (T*)act, top, E, W, F,
                   act_mode, limit, alpha);
         rv_launch(moe_down_kernel<T>, dim3(n_tokens, (W + MOE_ROWS - 1) / MOE_ROWS), dim3(128),
-                  smem2, s, (const T*)act, ids, weights, (const T*)down, (const T*)addend, (T*)out, top,
-                  E, W, F);
+                  smem2, s, (const T*)act, ids, weights, (const T*)down, (const T*)addend, (const T*)x, (T*)out,
+                  top, E, W, F);
     });
     RV_CHECK_LAUNCH("moe_experts");
     return 0;

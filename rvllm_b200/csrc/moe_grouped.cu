@@ -20,6 +20,9 @@
 //                 hold a pair, and the epilogue writes silu(gate) * up [rows, n_out / 2].
 //   moe_combine   out[t] = sum_k weights[t, k] * ys[pair_pos[t * top + k]], in the order of k.
 //
+// A pair whose id is E or more (an identity expert) takes no row: its pair_pos is -1, and the sum
+// reads x[t] itself.
+//
 // A row's sums depend on its own expert and values only, never on which other rows share its
 // tile, so a token's result does not depend on the batch.  Every wait on an mbarrier is
 // bounded (RV_WAIT_CYCLES); a wait that runs out records code 31-34 in `status`, every role
@@ -67,7 +70,7 @@ __global__ void moe_sort_kernel(const int* __restrict__ ids, int P, int E, int t
     __syncthreads();
     for (int p = threadIdx.x; p < P; p += blockDim.x) {
         const int e = ids[p];
-        int pos = 0;
+        int pos = e >= E ? -1 : 0;
         if (e >= 0 && e < E) {
             pos = off[e] + atomicAdd(&cur[e], 1);
             if (pos < rows_pad) sorted_token[pos] = p / top;
@@ -96,7 +99,8 @@ __global__ void moe_gather_kernel(const bf16* __restrict__ x, const int* __restr
 // one block per token; width a multiple of 8
 __global__ void moe_combine_kernel(const bf16* __restrict__ ys, const int* __restrict__ pair_pos,
                                    const float* __restrict__ weights, const bf16* __restrict__ addend,
-                                   bf16* __restrict__ out, int top, int W) {
+                                   const bf16* __restrict__ x, bf16* __restrict__ out, int top,
+                                   int W) {
     rv_pdl_prologue();
     const int t = blockIdx.x;
     for (int i = threadIdx.x; i < W / 8; i += blockDim.x) {
@@ -115,7 +119,8 @@ __global__ void moe_combine_kernel(const bf16* __restrict__ ys, const int* __res
         }
         for (int k = 0; k < top; ++k) {
             const float wgt = weights[(size_t)t * top + k];
-            const uint4 raw = *((const uint4*)(ys + (size_t)pair_pos[(size_t)t * top + k] * W) + i);
+            const int pos = pair_pos[(size_t)t * top + k];
+            const uint4 raw = *((const uint4*)(pos < 0 ? x + (size_t)t * W : ys + (size_t)pos * W) + i);
             const __nv_bfloat162* h = (const __nv_bfloat162*)&raw;
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
@@ -432,8 +437,8 @@ extern "C" int rv_moe_experts_grouped(const void* x, const int* ids, const float
                         max_tiles, 0, 0.f, 0.f, s))
         return 1;
     rv_launch(moe_combine_kernel, dim3(n_tokens), dim3(W / 8 < 256 ? ((W / 8 + 31) / 32) * 32 : 256), 0,
-              s, (const bf16*)ys, (const int*)pair_pos, weights, (const bf16*)addend, (bf16*)out, top,
-              W);
+              s, (const bf16*)ys, (const int*)pair_pos, weights, (const bf16*)addend, (const bf16*)x,
+              (bf16*)out, top, W);
     RV_CHECK_LAUNCH("moe_combine");
     return 0;
 }

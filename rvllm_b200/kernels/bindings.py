@@ -53,6 +53,7 @@ class CudaOps:
         self.lib.rv_gated_delta_scratch.restype = c_longlong
         self.lib.rv_mlstm_scratch.restype = c_longlong
         self.lib.rv_linear_attention_scratch.restype = c_longlong
+        self.lib.rv_state_space_scratch.restype = c_longlong
         self.lib.rv_paged_attention_pooled_scratch_bytes.restype = c_longlong
         self.lib.rv_paged_attention_mixed_scratch_bytes.restype = c_longlong
         self._scratch = {}
@@ -740,13 +741,14 @@ class CudaOps:
     def add_layernorm(self, resid, delta, weight, bias, eps, out, rows=None,
                       delta_weight=None, delta_bias=None, delta_eps=0.0):
         """out = LN(resid + d), d = delta or LN(delta; delta_weight, delta_bias, delta_eps);
-        `resid` None: out = LN(delta).  The stream is updated unless `rows` selects rows."""
+        `bias` and `delta_bias` may be None; `resid` None: out = LN(delta).  The stream is updated unless `rows` selects rows."""
         if resid is not None:
             self._need(resid, "residual stream", torch.float32)
         elif delta is None or rows is not None or delta_weight is not None:
             raise KernelError("add_layernorm: without a stream it takes rows to normalise, all of them")
         self._need(weight, "norm weight", torch.float32)
-        self._need(bias, "norm bias", torch.float32)
+        if bias is not None:
+            self._need(bias, "norm bias", torch.float32)
         self._need(out, "norm output")
         if delta is not None:
             self._need(delta, "pending sub-layer output")
@@ -754,12 +756,13 @@ class CudaOps:
                 raise KernelError("add_layernorm: the stream and the pending output differ in shape")
         if delta_weight is not None:
             self._need(delta_weight, "norm weight of the added rows", torch.float32)
+        if delta_bias is not None:
             self._need(delta_bias, "norm bias of the added rows", torch.float32)
         if rows is not None:
             self._need(rows, "row list", torch.int32)
         n, hidden = out.shape
         if (resid if resid is not None else delta).shape[1] != hidden or weight.shape[0] != hidden \
-                or bias.shape[0] != hidden:
+                or (bias is not None and bias.shape[0] != hidden):
             raise KernelError("add_layernorm: widths disagree")
         self._check(self.lib.rv_add_layernorm(
             _ptr(resid), _ptr(delta), _code(delta.dtype) if delta is not None else _F32,
@@ -847,11 +850,11 @@ class CudaOps:
             _ptr(slots), _ptr(k_cache), _ptr(v_cache), _ptr(k_blocks), _ptr(v_blocks),
             self._stream()), "rope_pool_write")
 
-    def attention_pooled_scratch_bytes(self, n_reqs, num_heads, head_dim, max_ctx_len, window,
-                                       pool) -> int:
+    def attention_pooled_scratch_bytes(self, n_reqs, num_heads, v_head_dim, max_ctx_len, window,
+                                       pool, most=0) -> int:
         return int(self.lib.rv_paged_attention_pooled_scratch_bytes(
-            c_int(n_reqs), c_int(num_heads), c_int(head_dim), c_int(max_ctx_len),
-            c_int(window or 0), c_int(pool or 0)))
+            c_int(n_reqs), c_int(num_heads), c_int(v_head_dim), c_int(max_ctx_len),
+            c_int(window or 0), c_int(pool or 0), c_int(most)))
 
     def _pooled_lib(self, head_dim: int):
         """The tensor-core pooled attention library for this head size, built at first use."""
@@ -869,9 +872,13 @@ class CudaOps:
         return lib
 
     def paged_attention_pooled(self, rows, num_heads, num_kv_heads, head_dim, k_cache, v_cache, ctx,
-                               group, pooled, scale, softcap, window, sinks, out):
+                               group, pooled, scale, softcap, window, sinks, out, v_head_dim=None,
+                               most_blocks=0):
         """Attention over the last `window` tokens (None: all) and the pooled blocks before them:
-        `pooled` = (block keys, block values, their group, tokens a block) or None.  `softcap`: scores
+        `pooled` = (block keys, block values, their group, tokens a block) or None; `most_blocks` > 0:
+        at most the first so many of them (blocks of one token whose rows are the tokens' own are
+        first tokens that stay visible).  `v_head_dim`: the size of a value head when it is not
+        `head_dim`.  `softcap`: scores
         become c tanh(score / c); `sinks` float32 [heads]: one more term in the denominator.
         Single tokens go to a split kernel and its merge, portions to one launch; bfloat16 heads
         whose size is a multiple of 16 up to 128 take the tensor cores."""
@@ -880,7 +887,8 @@ class CudaOps:
         self._need(k_cache, "key pages", rows.dtype)
         self._need(v_cache, "value pages", rows.dtype)
         H, G, d = num_heads, num_kv_heads, head_dim
-        if out.shape[1] != H * d or rows.shape[1] < H * d:
+        dv = v_head_dim or d
+        if out.shape[1] != H * dv or rows.shape[1] < H * d:
             raise KernelError("paged_attention_pooled: row widths and head sizes disagree")
         if sinks is not None:
             self._need(sinks, "sinks", torch.float32)
@@ -896,11 +904,11 @@ class CudaOps:
                 raise KernelError("paged_attention_pooled: blocks lie before a window, in pages of "
                                   "the tokens' size")
             ptable, pmax = pgroup.block_table, pgroup.max_blocks
-        mma = (self._mma_ok(rows.dtype, d) and rows.shape[1] % 8 == 0 and rows.data_ptr() % 16 == 0
-               and k_cache.data_ptr() % 16 == 0 and v_cache.data_ptr() % 16 == 0)
+        mma = (self._mma_ok(rows.dtype, d) and dv == d and rows.shape[1] % 8 == 0
+               and rows.data_ptr() % 16 == 0 and k_cache.data_ptr() % 16 == 0 and v_cache.data_ptr() % 16 == 0)
         code, nd = _code(rows.dtype), ctx.n_decode
         pages = (_ptr(k_cache), _ptr(v_cache), _ptr(group.block_table), c_int(group.max_blocks),
-                 _ptr(pk), _ptr(pv), _ptr(ptable), c_int(pmax), c_int(pool),
+                 _ptr(pk), _ptr(pv), _ptr(ptable), c_int(pmax), c_int(pool), c_int(most_blocks),
                  c_float(softcap or 0.0))
         heads = (c_int(H), c_int(G))
         win = c_int(window or 0)
@@ -915,7 +923,8 @@ class CudaOps:
                 raise KernelError(f"{what}: {msg}")
 
         if nd > 0:
-            need = self.attention_pooled_scratch_bytes(nd, H, d, ctx.max_ctx_len, window, pool)
+            need = self.attention_pooled_scratch_bytes(nd, H, dv, ctx.max_ctx_len, window, pool,
+                                                       most_blocks)
             scratch = self._scratch_buffer(need, rows.device)
             if lib is not None and self.decode_attention == "mma":
                 check_mma(getattr(lib, f"rv_paged_attention_pooled_decode_mma_{tag}")(
@@ -925,14 +934,15 @@ class CudaOps:
                     "paged_attention_pooled_decode")
                 self._check(self.lib.rv_paged_attention_pooled_merge(
                     _ptr(scratch), _ptr(ctx.ctx_lens), _ptr(out), code, c_int(nd),
-                    c_int(ctx.max_ctx_len), c_int(H), c_int(d), win, c_int(pool), _ptr(sinks),
-                    self._stream()), "paged_attention_pooled_merge")
+                    c_int(ctx.max_ctx_len), c_int(H), c_int(dv), win, c_int(pool),
+                    c_int(most_blocks), _ptr(sinks), self._stream()),
+                    "paged_attention_pooled_merge")
             else:
                 self._check(self.lib.rv_paged_attention_pooled_decode(
                     _ptr(rows), code, c_int(rows.shape[1]), *pages, _ptr(ctx.ctx_lens), _ptr(out),
                     _ptr(scratch), c_longlong(scratch.numel()), c_int(nd), c_int(ctx.max_ctx_len),
-                    *heads, c_int(d), c_int(group.page_size), c_float(scale), win, _ptr(sinks),
-                    self._stream()), "paged_attention_pooled_decode")
+                    *heads, c_int(d), c_int(group.page_size), c_float(scale), win, c_int(dv),
+                    _ptr(sinks), self._stream()), "paged_attention_pooled_decode")
                 self.launches += 1
         if ctx.n_tokens > nd and lib is not None and self.prefill_attention != "simt":
             check_mma(getattr(lib, f"rv_paged_attention_pooled_prefill_{tag}")(
@@ -945,7 +955,7 @@ class CudaOps:
                 _ptr(rows), code, c_int(rows.shape[1]), *pages, _ptr(ctx.q_start),
                 _ptr(ctx.ctx_lens), _ptr(ctx.token_req), _ptr(out), c_int(nd),
                 c_int(ctx.n_tokens - nd), *heads, c_int(d), c_int(group.page_size), c_float(scale),
-                win, _ptr(sinks), self._stream()), "paged_attention_pooled")
+                win, c_int(dv), _ptr(sinks), self._stream()), "paged_attention_pooled")
 
     # ---- attention with mixed heads ------------------------------------------------------
 
@@ -1137,7 +1147,15 @@ class CudaOps:
         x = rows.as_strided((heads, n, size), (size, rows.stride(0), 1),
                             rows.storage_offset() + offset)
         y = out.as_strided((heads, n, b), (b, out.stride(0), 1), out.storage_offset())
-        torch.bmm(x, w, out=y)
+        el = w.element_size()
+        if (size * el) % 16 == 0 and (b * el) % 16 == 0:
+            torch.bmm(x, w, out=y)
+        else:
+            # The batched product takes its vector width from the matrices' starts and row strides;
+            # heads that begin between two 16-byte boundaries inside aligned rows must not reach
+            # it.  One product per head shows the library every head's own address.
+            for h in range(heads):
+                y[h].copy_(torch.mm(x[h], w[h]))
         self.launches += 1
         if gate_rows is not None:
             self.sigmoid_gate(out, gate_rows, gate_off)
@@ -1190,8 +1208,9 @@ class CudaOps:
             self._choice_bias(choice_bias, experts), self._stream()), "moe_route")
 
     def moe_experts(self, x, ids, weights, gate_up, down, out, activation="swiglu", limit=0.0,
-                    alpha=1.0, addend=None):
+                    alpha=1.0, addend=None, identity=0):
         """out[t] = sum_k weights[t, k] * down[e](act(gate[e] x_t, up[e] x_t)), e = ids[t, k];
+        an id among the `identity` ones after the last expert's adds weights[t, k] * x_t;
         gate_up [E, 2F, W] (gate and up rows alternating), down [E, W, F].  `activation`
         "swiglu": silu(gate) * up; "glu_clamp": g = min(gate, limit), u = clamp(up, -limit,
         limit), g * sigmoid(alpha g) * (u + 1); "relu2": experts without a gate, `gate_up` is
@@ -1216,7 +1235,7 @@ class CudaOps:
                    and (self.moe_mode == "grouped" or n * top >= self.moe_grouped_min))
         if grouped:
             # the token tile follows the rows an expert gets on average
-            avg = n * top / experts
+            avg = n * top / (experts + identity)
             tn = 16 if avg <= 8 else 32 if avg <= 24 else 64 if avg <= 48 else 128
             need = int(self.lib.rv_moe_grouped_scratch_bytes(
                 c_int(n), c_int(top), c_int(experts), c_int(width), c_int(ffn), c_int(tn)))
@@ -1274,11 +1293,12 @@ class CudaOps:
     def qkv_full_norm_rope_write(self, rows, bias, num_heads, num_kv_heads, head_dim, v_head_dim,
                                  q_weight, k_weight, eps, freq, rot_dims, positions, slot_mapping,
                                  q_out, k_cache, v_cache, v_first_in=None, v_first_out=None,
-                                 lam=None):
+                                 lam=None, pairs=True, amplitude=1.0):
         """`rows` float32 [N, (heads + kv) * head_dim + kv * v_head_dim] (+ `bias`): q and k are
         normalised over their whole projection (weights [heads * head_dim], [kv * head_dim]),
         the pairs (2i, 2i + 1) of each head's first `rot_dims` dimensions turn by position *
-        freq[i]; v <- (1 - lam) v + lam v_first_in when given (`lam` a float32 scalar tensor);
+        freq[i] (`pairs` false: dimension i turns with i + rot_dims/2), cosine and sine times
+        `amplitude`; v <- (1 - lam) v + lam v_first_in when given (`lam` a float32 scalar tensor);
         `v_first_out` receives this layer's own values.  q -> `q_out`, k and v -> the cache."""
         self._need(rows, "q|k|v rows", torch.float32)
         self._need(q_out, "query rows", k_cache.dtype)
@@ -1295,7 +1315,8 @@ class CudaOps:
             c_int(rot_dims), _ptr(positions), _ptr(slot_mapping), _ptr(q_out), _ptr(k_cache),
             _ptr(v_cache), _code(k_cache.dtype), _ptr(v_first_in), _ptr(v_first_out), _ptr(lam),
             c_int(rows.shape[0]), c_int(num_heads), c_int(num_kv_heads), c_int(head_dim),
-            c_int(v_head_dim), self._stream()), "qkv_full_norm_rope_write")
+            c_int(v_head_dim), c_int(1 if pairs else 0), c_float(amplitude), self._stream()),
+            "qkv_full_norm_rope_write")
 
     # ---- gated delta rule ------------------------------------------------------------------
 
@@ -1304,11 +1325,14 @@ class CudaOps:
         return (taps - 1) * (2 * kv_heads * dim + heads * vdim) + heads * dim * vdim
 
     def gated_delta(self, proj, lowrank, filt, a_log, dt_bias, norm_w, state, ctx, out, heads,
-                    kv_heads, dim, vdim, taps, unit_eps, eps):
-        """The gated delta rule with a decay per key channel over the step's tokens; see
-        csrc/gated_delta.cu for the layout of `proj`, `lowrank` and the record."""
-        for t, what in ((proj, "projection rows"), (lowrank, "decay and gate rows"),
-                        (filt, "convolution filters"), (a_log, "decay rates"),
+                    kv_heads, dim, vdim, taps, unit_eps, eps, head_decay=False, gate="sigmoid"):
+        """The gated delta rule over the step's tokens, with a decay per key channel or, with
+        `head_decay`, per value head; see csrc/gated_delta.cu for the layout of `proj`, `lowrank`
+        (which may be columns of wider rows) and the record."""
+        self._need(lowrank, "decay and gate rows", torch.float32, contiguous=False)
+        if lowrank.stride(1) != 1:
+            raise KernelError("gated_delta: the decay and gate rows must be dense along a row")
+        for t, what in ((proj, "projection rows"), (filt, "convolution filters"), (a_log, "decay rates"),
                         (dt_bias, "decay bias"), (norm_w, "output norm weight"),
                         (state, "state records")):
             self._need(t, what, torch.float32)
@@ -1317,17 +1341,22 @@ class CudaOps:
         if state.shape[1] != rec or out.shape[1] != heads * vdim:
             raise KernelError("gated_delta: the record or the output has another size")
         n = proj.shape[0]
+        decays = heads if head_decay else heads * dim
+        if lowrank.shape[0] != n or lowrank.shape[1] < decays + heads * vdim or \
+                dt_bias.numel() != decays:
+            raise KernelError("gated_delta: the decay and gate rows have another size")
         need = self.lib.rv_gated_delta_scratch(c_int(n), c_int(heads), c_int(kv_heads), c_int(dim),
                                                c_int(vdim))
         if need < 0:
             raise KernelError(f"gated_delta: key heads of {dim} are not supported")
         scratch = torch.empty((need,), dtype=torch.float32, device=proj.device)
         self._check(self.lib.rv_gated_delta(
-            _ptr(proj), c_int(proj.shape[1]), _ptr(lowrank), c_int(lowrank.shape[1]), _ptr(filt),
+            _ptr(proj), c_int(proj.shape[1]), _ptr(lowrank), c_int(lowrank.stride(0)), _ptr(filt),
             _ptr(a_log), _ptr(dt_bias), _ptr(norm_w), _ptr(state), _ptr(ctx.token_req),
             _ptr(ctx.q_start), _ptr(ctx.state_slot), _ptr(scratch), _ptr(out), _code(out.dtype),
             c_int(n), c_int(ctx.n_reqs), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim),
-            c_int(taps), c_float(unit_eps), c_float(eps), self._stream()), "gated_delta")
+            c_int(taps), c_float(unit_eps), c_float(eps), c_int(1 if head_decay else 0),
+            c_int({"sigmoid": 0, "silu": 1}[gate]), self._stream()), "gated_delta")
         self.launches += 3
 
     # ---- clamped gated activation ----------------------------------------------------------
@@ -1370,10 +1399,11 @@ class CudaOps:
     # ---- latent rows with a query latent and a turned key part ------------------------------
 
     def latent_prepare(self, rows, q_off, q_rank, q_weight, cq, kv_off, rank, rot, kv_weight, eps,
-                       freq, positions, slot_mapping, cache):
+                       freq, positions, slot_mapping, cache, pairs=False, amplitude=1.0):
         """Columns [q_off, +q_rank) of `rows` RMS-normed into `cq` (q_rank 0: none); columns
         [kv_off, +rank) RMS-normed and the `rot` columns after them turned by the position, both
-        into the token's page slot [rank + rot]."""
+        into the token's page slot [rank + rot] (`pairs`: dimension 2i turns with 2i + 1, else i
+        with i + rot/2; cosine and sine times `amplitude`)."""
         self._need(rows, "latent rows")
         self._need(kv_weight, "latent norm weight", torch.float32)
         self._need(cache, "latent pages", rows.dtype)
@@ -1392,11 +1422,13 @@ class CudaOps:
             _ptr(rows), _code(rows.dtype), c_int(rows.shape[1]), c_int(rows.shape[0]), c_int(q_off),
             c_int(q_rank), _ptr(q_weight), _ptr(cq), c_int(kv_off), c_int(rank), c_int(rot),
             _ptr(kv_weight), c_float(eps), _ptr(freq), _ptr(positions), _ptr(slot_mapping),
-            _ptr(cache), self._stream()), "latent_prepare")
+            _ptr(cache), c_int(1 if pairs else 0), c_float(amplitude), self._stream()),
+            "latent_prepare")
 
-    def rope_heads(self, x, heads, size, off, rot, freq, positions):
+    def rope_heads(self, x, heads, size, off, rot, freq, positions, pairs=False, amplitude=1.0):
         """In every head of x [N, heads * size] the `rot` values from `off` on turn by the
-        token's position (dimension i with i + rot/2, angle position * freq[i])."""
+        token's position (dimension i with i + rot/2, or with `pairs` 2i with 2i + 1, angle
+        position * freq[i], cosine and sine times `amplitude`)."""
         if not rot:
             return
         self._need(x, "rows to turn")
@@ -1405,7 +1437,8 @@ class CudaOps:
             raise KernelError("rope_heads: sizes disagree")
         self._check(self.lib.rv_rope_heads(
             _ptr(x), _code(x.dtype), c_int(x.shape[1]), c_int(x.shape[0]), c_int(heads), c_int(size),
-            c_int(off), c_int(rot), _ptr(freq), _ptr(positions), self._stream()), "rope_heads")
+            c_int(off), c_int(rot), _ptr(freq), _ptr(positions), c_int(1 if pairs else 0),
+            c_float(amplitude), self._stream()), "rope_heads")
 
     def head_gate(self, x, heads, size, rows, gate_off):
         """x[n, h, :] <- x[n, h, :] * sigmoid(rows[n, gate_off + h])."""
@@ -1482,6 +1515,44 @@ class CudaOps:
             c_int(1 if self.linear_attention_mode == "tensor" else 0), self._stream()),
             "linear_attention")
         self.launches += (ctx.n_decode > 0) + 3 * (n > ctx.n_decode)
+
+    # ---- state space -----------------------------------------------------------------------------
+
+    def state_space(self, proj, filt, conv_bias, dt_bias, a_log, skip, norm_w, conv_state, state,
+                    ctx, out, heads, vdim, d_state, groups, taps, norm_groups, eps):
+        """A selective state space with one decay per token and head over the step's tokens; see
+        csrc/state_space.cuh for the layout of `proj`.  `conv_state` [slots, taps-1, channels] (None
+        with one tap), `state` [slots, heads * d_state * vdim]."""
+        for t, what in ((proj, "projection rows"), (filt, "convolution filters"),
+                        (conv_bias, "convolution bias"), (dt_bias, "step bias"),
+                        (a_log, "decay rates"), (skip, "skip weights"),
+                        (norm_w, "output norm weight"), (conv_state, "convolution records"),
+                        (state, "state records")):
+            if t is not None:
+                self._need(t, what, torch.float32)
+        self._need(out, "mixer output")
+        H, dv, N, G = heads, vdim, d_state, groups
+        n, inner, C = proj.shape[0], heads * vdim, heads * vdim + 2 * groups * d_state
+        if proj.shape[1] < inner + C + H or state.shape[1] != H * N * dv or out.shape != (n, inner) \
+                or filt.shape != (C, taps) or conv_bias.shape != (C,) or norm_w.shape != (inner,):
+            raise KernelError("state_space: the rows, the record or the weights have another size")
+        if any(t.shape != (H,) for t in (dt_bias, a_log, skip)):
+            raise KernelError("state_space: one step bias, rate and skip weight per head")
+        if taps > 1 and (conv_state is None or conv_state.shape[1:] != (taps - 1, C)):
+            raise KernelError("state_space: the convolution's records have another size")
+        code = _code(out.dtype)
+        need = self.lib.rv_state_space_scratch(
+            c_int(n), c_int(ctx.n_decode), c_int(ctx.n_reqs), c_int(H), c_int(dv), c_int(N), c_int(G),
+            c_int(code))
+        scratch = torch.empty((need,), dtype=torch.float32, device=proj.device)
+        self._check(self.lib.rv_state_space(
+            _ptr(proj), c_int(proj.shape[1]), _ptr(filt), _ptr(conv_bias), _ptr(dt_bias), _ptr(a_log),
+            _ptr(skip), _ptr(norm_w), _ptr(conv_state), _ptr(state), _ptr(ctx.token_req),
+            _ptr(ctx.q_start), _ptr(ctx.state_slot), _ptr(scratch), _ptr(out), c_int(code), c_int(n),
+            c_int(ctx.n_decode), c_int(ctx.n_reqs), c_int(H), c_int(dv), c_int(N), c_int(G),
+            c_int(taps), c_int(norm_groups), c_float(eps),
+            c_int(1 if self.linear_attention_mode == "tensor" else 0), self._stream()), "state_space")
+        self.launches += 1 + (ctx.n_decode > 0) + 4 * (n > ctx.n_decode)
 
     def softcap(self, logits, cap):
         self._need(logits, "logits", torch.float32)

@@ -73,7 +73,12 @@ class StateSpace(Mixer):
         self.ops = ops
         self.dtype = dtype
         n = self._names(spec)
-        self.w_in = tensors[n["in"]].contiguous()
+        w_in = tensors[n["in"]]
+        fill = -w_in.shape[0] % 8                  # zero rows, so that the product's rows stay aligned
+        if fill:
+            w_in = torch.cat([w_in, torch.zeros((fill, spec.hidden), dtype=w_in.dtype,
+                                                device=w_in.device)])
+        self.w_in = w_in.contiguous()
         self.w_out = tensors[n["o"]].contiguous()
         f32 = lambda k: tensors[n[k]].to(torch.float32).contiguous()
         self.filt, self.conv_bias = f32("conv"), f32("conv.b")

@@ -730,7 +730,7 @@ class PlainOps:
                 xs = act[i, :inner].reshape(H, dv)
                 B = act[i, inner:inner + G * N].reshape(G, N).repeat_interleave(H // G, 0)
                 Cq = act[i, inner + G * N:].reshape(G, N).repeat_interleave(H // G, 0)
-                dt = torch.nn.functional.softplus(p[a + i, inner + C:] + _f(dt_bias), threshold=60.0)
+                dt = torch.nn.functional.softplus(p[a + i, inner + C:inner + C + H] + _f(dt_bias), threshold=60.0)
                 keep = torch.exp(-torch.exp(_f(a_log)) * dt)
                 S = keep[:, None, None] * S + (dt[:, None] * B)[:, :, None] * xs[:, None, :]
                 y = torch.einsum("hnv,hn->hv", S, Cq) + _f(skip)[:, None] * xs
