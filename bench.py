@@ -46,6 +46,10 @@ run twice) beside Bizenex with as many layer runs at equal sizes.
 decays, and attention over a window and pooled blocks beside a linear attention with decays by
 channel, in turn; token shift, gated experts with a shared one; a stretch of layers run twice)
 beside Mevuvik with as many layer runs at equal sizes.
+`--only dopuvik` (not part of the default run) measures Dopuvik (a state space, a latent attention
+over a window, and a grouped-query attention over a window with kept first tokens beside a gated
+delta rule; experts and identity experts) beside Mevuvik with as many layer runs at equal sizes,
+and beside Vifanex and Fekizen for their delta rule and linear attention.
 `--only retorax` (not part of the default run) measures another design, Retorax, beside LFM2
 at equal sizes (width 1024 and 2048, eight layers): a 2,048-token prompt, single tokens at
 batch 8 and 64, and the device time of every kernel of a step against its roofline.
@@ -998,6 +1002,48 @@ def fekizen_config(sz):
             "loop": {"start": 2, "stop": 4, "times": 2}, "layers": layers}
 
 
+DOPUVIK_SIZES = {
+    # parallel layers (kept-first-tokens attention and a delta rule), with state space and windowed
+    # latent layers between them in turn; eight layers, as Mevuvik's eight layer runs.  The state
+    # space is as large as its design's usual form (twice the width, heads of 64, 128 rows).  The
+    # fields Mevuvik, Vifanex and Fekizen read are here too, so that they run beside at equal sizes:
+    # Vifanex' delta rule has the same heads, Fekizen's linear attention Mevuvik's memory's.
+    "w1024": {"width": 1024, "layers": 8, "heads": 16, "kv": 4, "dim": 64, "rank": 128, "rot": 16,
+              "q_rank": 256, "window": 512, "keep": 64, "ssm_heads": 32, "ssm_vdim": 64, "ssm_state": 128,
+              "delta_heads": 8, "delta_kv": 4, "delta_dim": 128, "low_rank": 64, "taps": 4, "streams": 4,
+              "mem_heads": 8, "mem_dim": 64, "mem_vdim": 128, "pool": 16,
+              "experts": 16, "identity": 4, "top": 4, "groups": (4, 2), "ff": 1024, "vocab": 32768},
+    "w2048": {"width": 2048, "layers": 8, "heads": 32, "kv": 8, "dim": 64, "rank": 128, "rot": 16,
+              "q_rank": 512, "window": 512, "keep": 64, "ssm_heads": 64, "ssm_vdim": 64, "ssm_state": 128,
+              "delta_heads": 16, "delta_kv": 8, "delta_dim": 128, "low_rank": 64, "taps": 4, "streams": 4,
+              "mem_heads": 16, "mem_dim": 64, "mem_vdim": 128, "pool": 16,
+              "experts": 16, "identity": 4, "top": 4, "groups": (4, 2), "ff": 2048, "vocab": 32768},
+}
+
+
+def dopuvik_config(sz):
+    mlp = {"kind": "moe", "expert": {"ff": sz["ff"]},
+           "router": {"experts": sz["experts"], "identity": sz["identity"], "top": sz["top"], "scale": 2.0,
+                      "groups": {"count": sz["groups"][0], "keep": sz["groups"][1]}}}
+    ssm = {"heads": sz["ssm_heads"], "vdim": sz["ssm_vdim"], "state": sz["ssm_state"], "groups": 1,
+           "conv": sz["taps"], "norm_groups": 1}
+    latent = {"heads": sz["heads"], "dim": sz["dim"], "rot_dim": sz["rot"], "vdim": sz["dim"],
+              "kv_rank": sz["rank"] - sz["rot"], "q_rank": sz["q_rank"],
+              "scale": (sz["dim"] + sz["rot"]) ** -0.5, "mask": {"size": sz["window"]},
+              "rot": {"base": 10000.0, "dims": sz["rot"],
+                      "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+    par = {"left": {"heads": sz["heads"], "kv_heads": sz["kv"], "dim": sz["dim"], "vdim": sz["dim"],
+                    "scale": sz["dim"] ** -0.5, "mask": {"size": sz["window"], "keep_first": sz["keep"]},
+                    "rot": {"base": 10000.0, "dims": sz["dim"]}},
+           "right": {"heads": sz["delta_heads"], "kv_heads": sz["delta_kv"], "dim": sz["delta_dim"],
+                     "vdim": sz["delta_dim"], "conv": sz["taps"]},
+           "left_scale": 1.0, "right_scale": 1.0}
+    kinds = (("mamba2", ssm), ("parallel", par), ("latent_attention", latent), ("parallel", par))
+    layers = [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": mlp} for i in range(sz["layers"])]
+    return {"architecture": "Dopuvik", "vocab": sz["vocab"], "width": sz["width"], "norm": {"eps": 1e-5},
+            "embedding": {"scale": sz["width"] ** 0.5}, "logit_scale": 0.25, "layers": layers}
+
+
 def lfm2_all_attention(sz):
     """LFM2 with the same width and layer count, attention in every layer with the same head
     counts and sizes, and a SwiGLU as wide as the experts a token uses together."""
@@ -1030,7 +1076,7 @@ class OpTimer:
              "hyper_norm", "qkv_full_norm_rope_write", "gated_delta", "glu_clamp", "relu2",
              "weighted_sum", "latent_prepare", "rope_heads", "head_gate", "mlstm",
              "add_rmsnorm_shift", "normed_sum", "rope_pool_write", "paged_attention_pooled",
-             "linear_attention")
+             "linear_attention", "state_space")
 
     def __init__(self, torch, ops):
         self.torch, self.ops, self.events, self.saved = torch, ops, [], {}
@@ -1073,7 +1119,8 @@ class OpTimer:
 
 def run_designs(args, which="retorax"):
     """Retorax (`--only retorax`) or Bizenex (`--only bizenex`) beside LFM2, Mevuvik (`--only mevuvik`) or Vifanex
-    (`--only vifanex`) beside Bizenex, or Fekizen (`--only fekizen`) beside Mevuvik, at equal sizes:
+    (`--only vifanex`) beside Bizenex, Fekizen (`--only fekizen`) beside Mevuvik, or Dopuvik (`--only
+    dopuvik`) beside Mevuvik (and Vifanex and Fekizen), at equal sizes:
     prompt and single-token throughput, and the device time of every kernel of one prompt step
     and one single-token step with its share of the roofline.  One JSON line."""
     import torch
@@ -1089,7 +1136,7 @@ def run_designs(args, which="retorax"):
     sampler = ClockSampler()
     sampler.start()
     sizes = {"retorax": RETORAX_SIZES, "bizenex": BIZENEX_SIZES, "vifanex": VIFANEX_SIZES,
-             "mevuvik": MEVUVIK_SIZES, "fekizen": FEKIZEN_SIZES}[which]
+             "mevuvik": MEVUVIK_SIZES, "fekizen": FEKIZEN_SIZES, "dopuvik": DOPUVIK_SIZES}[which]
     for size_name, sz in sizes.items():
         if args.design_size not in ("all", size_name):
             continue
@@ -1098,6 +1145,9 @@ def run_designs(args, which="retorax"):
             pair = (("retorax", retorax_config(sz)), ("lfm2", lfm2_like(sz)))
         elif which == "bizenex":
             pair = (("bizenex", bizenex_config(sz)), ("lfm2", lfm2_all_attention(sz)))
+        elif which == "dopuvik":
+            pair = (("dopuvik", dopuvik_config(sz)), ("mevuvik", mevuvik_config(sz)),
+                    ("vifanex", vifanex_config(sz)), ("fekizen", fekizen_config(sz)))
         elif which == "fekizen":
             pair = (("fekizen", fekizen_config(sz)), ("mevuvik", mevuvik_config(sz)))
         elif which == "mevuvik":
@@ -1194,7 +1244,8 @@ def run_designs(args, which="retorax"):
         entry["rooflines"] = {"retorax": design_rooflines, "bizenex": bizenex_rooflines,
                               "vifanex": vifanex_rooflines,
                               "mevuvik": mevuvik_rooflines,
-                              "fekizen": fekizen_rooflines}[which](sz, entry, pk, T, CTX)
+                              "fekizen": fekizen_rooflines,
+                              "dopuvik": dopuvik_rooflines}[which](sz, entry, pk, T, CTX)
         out[size_name] = entry
     out["clocks"] = sampler.stop()
     print(json.dumps(out))
@@ -1518,6 +1569,99 @@ def fekizen_rooflines(sz, entry, pk, T, CTX):
     return out
 
 
+def dopuvik_rooflines(sz, entry, pk, T, CTX):
+    """Per kernel (Dopuvik's, and the like kernel of another design): device time of all calls in
+    the prompt step and in a single-token step of batch 64, and the time the roofline allows: bytes /
+    measured copy rate for the elementwise kernels and for single tokens, tensor FLOPs / measured
+    GEMM rate for attention and the experts' products, and for the recurrences the larger of their
+    bytes and their float32 FLOPs (5 a state element a token: decay, write, read-out; the delta rule
+    7: it reads the state once more) on the CUDA cores at their nominal rate."""
+    W, F, H, G, D, R = sz["width"], sz["ff"], sz["heads"], sz["kv"], sz["dim"], sz["rank"]
+    top, rot, Rq, win, keep = sz["top"], sz["rot"], sz["q_rank"], sz["window"], sz["keep"]
+    Hs, Vs, N = sz["ssm_heads"], sz["ssm_vdim"], sz["ssm_state"]
+    Hd, Gd, Dd, low = sz["delta_heads"], sz["delta_kv"], sz["delta_dim"], sz["low_rank"]
+    Hm, Dm, Vm = sz["mem_heads"], sz["mem_dim"], sz["mem_vdim"]
+    runs = sz["layers"]
+    half, quarter = runs // 2, runs // 4             # parallel runs; state space and latent runs
+    hbm, tens, fp32 = pk["hbm_gbs"] * 1e3, pk["bf16_tflops"] * 1e6, FP32_TFLOPS_NOMINAL * 1e6
+    pairs = T * (T + 1) // 2
+    seen = sum(min(i + 1, win) for i in range(T))
+    seen_kept = sum(min(i + 1, win) + min(keep, max(0, i - win + 1)) for i in range(T))
+    real = top * sz["experts"] / (sz["experts"] + sz["identity"])    # experts a token uses, on average
+    stream = T * W * (4 + 4 + 2 + 2)
+    ssm_cols, delta_cols = 2 * Hs * Vs + 2 * N + Hs, 2 * Gd * Dd + 2 * Hd * Dd + 2 * Hd
+    vif_cols = 2 * Gd * Dd + Hd * Dd + Hd + 2 * Hd * Dd
+    ml_cols, la_cols = 2 * Hm * Dm + 2 * Hm * Vm + 2 * Hm, 2 * Hm * Dm + 2 * Hm * Vm
+    ideal = {
+        "add_layernorm": (2 * runs + 1) * stream / hbm,
+        "mevuvik.add_rmsnorm": (2 * runs + 2) * stream / hbm,
+        "latent_prepare": quarter * T * (Rq + R) * 4 / hbm,
+        "mevuvik.latent_prepare": half * T * (Rq + R) * 4 / hbm,
+        "rope_heads": quarter * T * H * rot * 4 / hbm,
+        "mevuvik.rope_heads": half * T * H * rot * 4 / hbm,
+        "qkv_full_norm_rope_write": half * T * ((H + 2 * G) * D * 4 + (H + 2 * G) * D * 2) / hbm,
+        "vifanex.qkv_full_norm_rope_write": half * T * ((H + 2 * G) * D * 4 + (H + 2 * G) * D * 2 + G * D * 4) / hbm,
+        "paged_attention": quarter * seen * 4.0 * H * R / tens,
+        "paged_attention_pooled": half * seen_kept * 4.0 * H * D / tens,
+        "mevuvik.paged_attention": (half * pairs * 4.0 * H * R + half * pairs * 4.0 * H * D) / tens,
+        "fekizen.paged_attention_pooled": half * sum(
+            min(i + 1, win) + max(0, i - win + 1) // sz["pool"] for i in range(T)) * 4.0 * H * D / tens,
+        "weighted_sum": half * T * W * 6 / hbm,
+        "mevuvik.weighted_sum": half * T * W * 6 / hbm,
+        "moe_route": runs * T * (W * 2 + top * 8) / hbm,
+        "mevuvik.moe_route": (runs - 1) * T * (W * 2 + top * 8) / hbm,
+        "moe_experts": runs * T * real * 6.0 * F * W / tens,
+        "mevuvik.moe_experts": (runs - 1) * T * top * 4.0 * F * W / tens,
+        "fekizen.moe_experts": runs * T * top * 6.0 * F * W / tens,
+        "state_space": quarter * max(T * 5.0 * Hs * N * Vs / fp32, T * (ssm_cols * 4 + Hs * Vs * 2) / hbm),
+        "gated_delta": half * max(T * 7.0 * Hd * Dd * Dd / fp32, T * (delta_cols * 4 + Hd * Dd * 2) / hbm),
+        "vifanex.gated_delta": half * max(T * 7.0 * Hd * Dd * Dd / fp32, T * (vif_cols * 4 + Hd * Dd * 2) / hbm),
+        "mevuvik.mlstm": half * max(T * Hm * 5.0 * Dm * (Vm + 1) / fp32, T * (ml_cols * 4 + Hm * Vm * 2) / hbm),
+        "fekizen.linear_attention": max(runs * T * 5.0 * Hm * Dm * Vm / fp32, T * (
+            runs * (la_cols * 4 + Hm * Vm * 2) + half * Hm * Dm * 4) / hbm),
+    }
+    like = (("add_layernorm", "mevuvik.add_rmsnorm"), ("latent_prepare", "mevuvik.latent_prepare"),
+            ("rope_heads", "mevuvik.rope_heads"),
+            ("qkv_full_norm_rope_write", "vifanex.qkv_full_norm_rope_write"),
+            ("paged_attention", "mevuvik.paged_attention"), ("paged_attention_pooled", "mevuvik.paged_attention"),
+            ("paged_attention_pooled", "fekizen.paged_attention_pooled"),
+            ("weighted_sum", "mevuvik.weighted_sum"), ("moe_route", "mevuvik.moe_route"),
+            ("moe_experts", "mevuvik.moe_experts"), ("moe_experts", "fekizen.moe_experts"),
+            ("state_space", "mevuvik.mlstm"), ("state_space", "fekizen.linear_attention"),
+            ("gated_delta", "mevuvik.mlstm"), ("gated_delta", "vifanex.gated_delta"))
+    # single tokens at batch 64: every request's records and visible rows are read (records written)
+    B = 64
+    dec = {
+        "state_space": quarter * B * 2.0 * Hs * N * Vs * 4 / hbm,
+        "gated_delta": half * B * 2.0 * Hd * Dd * Dd * 4 / hbm,
+        "vifanex.gated_delta": half * B * 2.0 * Hd * Dd * Dd * 4 / hbm,
+        "mevuvik.mlstm": half * B * 2.0 * Hm * Dm * (Vm + 1) * 4 / hbm,
+        "fekizen.linear_attention": runs * B * 2.0 * Hm * Dm * Vm * 4 / hbm,
+        "paged_attention": quarter * B * win * R * 2 / hbm,
+        "paged_attention_pooled": half * B * (win + keep) * 2 * G * D * 2 / hbm,
+        "mevuvik.paged_attention": half * B * CTX * (R * 2 + 2 * G * D * 2) / hbm,
+        "fekizen.paged_attention_pooled": half * B * (win + (CTX - win) // sz["pool"]) * 2 * G * D * 2 / hbm,
+    }
+
+    def table(key, bound):
+        rows = {}
+        for mine, other in like:
+            design, name = other.split(".")
+            a, b = entry["dopuvik"][key].get(mine), entry[design][key].get(name)
+            if not a or mine not in bound:
+                continue
+            row = rows.setdefault(mine, {"us": a["us"], "calls": a["calls"], "roofline_us": round(bound[mine], 1),
+                                         "times_roofline": round(a["us"] / bound[mine], 2), "like": {}})
+            if b and other in bound:
+                row["like"][other] = {"us": b["us"], "calls": b["calls"], "roofline_us": round(bound[other], 1),
+                                      "times_roofline": round(b["us"] / bound[other], 2)}
+        return rows
+
+    out = table("prefill_2048_kernels_us", ideal)
+    out["decode_b64"] = table("decode_b64_kernels_us", dec)
+    return out
+
+
 def run_reference(args):
     print(json.dumps({
         "impl": "reference",
@@ -1535,14 +1679,14 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--size", default="1.2b", choices=sorted(SIZES),
                     help="layer sizes: LFM2-1.2B (the default and the headline), 700M or 350M")
-    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "kernels", "breakdown", "workload", "further", "retorax", "bizenex", "vifanex", "mevuvik", "fekizen"],
+    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "kernels", "breakdown", "workload", "further", "retorax", "bizenex", "vifanex", "mevuvik", "fekizen", "dopuvik"],
                     help="run one part only (for profiling); the JSON line then lacks the rest")
     ap.add_argument("--workloads", default="both", choices=["both", "none"] + sorted(WORKLOADS),
                     help="scheduler workloads to add to the line (default: both)")
     ap.add_argument("--workload", default="350m-mixed", choices=sorted(WORKLOADS),
                     help="with --only workload: which one")
     ap.add_argument("--design-size", default="all", choices=["all"] + sorted(set(RETORAX_SIZES) | set(VIFANEX_SIZES)),
-                    help="with --only retorax, bizenex, vifanex, mevuvik or fekizen: which of the sizes")
+                    help="with --only retorax, bizenex, vifanex, mevuvik, fekizen or dopuvik: which of the sizes")
     ap.add_argument("--kernel", default="all",
                     help="with --only kernels: attn_decode, attn_prefill, gemm, gemm:NxK, elementwise, copy_rate or all")
     ap.add_argument("--kernel-batch", type=int, default=64)
@@ -1575,6 +1719,8 @@ def main():
         return run_designs(args, "mevuvik")
     if args.only == "fekizen":
         return run_designs(args, "fekizen")
+    if args.only == "dopuvik":
+        return run_designs(args, "dopuvik")
     if args.only == "workload":
         print(json.dumps({"only": "workload", args.workload: run_workload(args.workload)}))
         return 0
