@@ -1,0 +1,840 @@
+"""Dopuvik on the GPU against the plain implementation (tests/plain_dopuvik.py): each new kernel
+alone at sizes other than any model's, with inputs made so that a fault shows; models of one
+mechanism each, with attention made sharp so that one lost key changes the result; then the
+engine under every way of cutting requests into steps, in float32 and bfloat16, with and without
+replayed launch sequences; then greedy generation through the Python entry point and its
+scheduler, and the programs a user starts."""
+import copy
+import os
+import random
+from types import SimpleNamespace
+
+import numpy as np
+import pytest
+import torch
+
+import dopuvik_tiny as dv
+import plain_dopuvik as plain
+import schedules
+
+pytestmark = pytest.mark.gpu
+BOUND = {"float32": 2e-5, "bfloat16": 3e-2}
+
+
+@pytest.fixture(scope="module")
+def ops():
+    from rvllm_b200.kernels import cuda_ops
+    return cuda_ops()
+
+
+@pytest.fixture(scope="module")
+def folders(tmp_path_factory):
+    root = str(tmp_path_factory.mktemp("do"))
+    return {n: dv.write(root, n) for n in dv.CONFIGS}
+
+
+def dev(t, dtype=None):
+    t = torch.as_tensor(np.asarray(t)) if not isinstance(t, torch.Tensor) else t
+    return t.to("cuda", dtype) if dtype is not None else t.to("cuda")
+
+
+def f32(t):
+    return dev(t, torch.float32)
+
+
+def i32(x):
+    return torch.tensor(x, dtype=torch.int32, device="cuda")
+
+
+def close(got, want, dtype, scale=None, bound=None):
+    want = torch.as_tensor(np.asarray(want), dtype=torch.float64)
+    got = got.detach().to("cpu", torch.float64).reshape(want.shape)
+    s = float(want.abs().max()) if scale is None else scale
+    err = float((got - want).abs().max()) / max(s, 1e-30)
+    assert err < max(bound or 0.0, 1e-5 if dtype == torch.float32 else 2e-2), err
+
+
+def rnd(gen, dtype, *shape, std=1.0):
+    """Random values that both sides can hold exactly."""
+    return (torch.randn(*shape, generator=gen) * std).to(dtype).double()
+
+
+def step_context(layout):
+    """Index arrays of a step: `layout` lists (tokens, state slot) per request."""
+    starts, token_req = [0], []
+    for r, (n, _) in enumerate(layout):
+        starts.append(starts[-1] + n)
+        token_req += [r] * n
+    n_decode = 0
+    while n_decode < len(layout) and layout[n_decode][0] == 1:
+        n_decode += 1
+    return SimpleNamespace(q_start=i32(starts), state_slot=i32([s for _, s in layout]),
+                           token_req=i32(token_req), n_reqs=len(layout), n_decode=n_decode,
+                           n_tokens=starts[-1]), starts
+
+
+DTYPES = [torch.float32, torch.bfloat16]
+
+
+# ---- layer norm without a bias ---------------------------------------------------------------------
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("width", [96, 50, 1024, 2600])
+def test_layer_norm_without_bias(ops, dtype, width):
+    g = torch.Generator().manual_seed(width)
+    n, eps = 9, 1e-4
+    resid, delta, w = rnd(g, torch.float32, n, width) + 3.0, rnd(g, dtype, n, width), rnd(g, torch.float32, width)
+    out = torch.empty(n, width, device="cuda", dtype=dtype)
+    r = f32(resid)
+    ops.add_layernorm(r, dev(delta, dtype), f32(w), None, eps, out)
+    x = resid.float().double() + delta
+    close(out, plain.layer_norm(x.numpy(), eps) * w.numpy(), dtype)
+    close(r, x, torch.float32)
+    # a norm of the added rows, without biases as well
+    r = f32(resid)
+    ops.add_layernorm(r, dev(delta, dtype), f32(w), None, eps, out, delta_weight=f32(w), delta_eps=eps)
+    x = resid.float().double() + torch.as_tensor(plain.layer_norm(delta.numpy(), eps)) * w
+    close(out, plain.layer_norm(x.numpy(), eps) * w.numpy(), dtype)
+
+
+# ---- biases, rotation by halves, cache write ---------------------------------------------------------
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("sizes", [(6, 2, 32, 16, 16), (3, 3, 10, 7, 6), (4, 1, 48, 48, 48), (2, 2, 15, 20, 0),
+                                   (8, 4, 64, 128, 64), (3, 1, 9, 4, 4)])
+@pytest.mark.parametrize("pairs", [False, True])
+def test_biases_and_rotation_of_a_heads_first_dimensions(ops, dtype, sizes, pairs):
+    H, G, d, vd, dims = sizes
+    if pairs and d % 2:
+        dims = 0
+    g = torch.Generator().manual_seed(d)
+    rot = dv._rot(dims, 300.0, (4.0, 64, 8.0, 1.0)) if dims else None
+    positions, slots = [0, 1, 2, 17, 3333, 5, 90], [3, 9, 0, -1, 14, 7, 1]
+    n, total = len(positions), (H + G) * d + G * vd
+    rows, bias = rnd(g, torch.float32, n, total), rnd(g, torch.float32, total)
+    freq, amp = None, 1.0
+    if dims:
+        f, amp = plain.frequencies(rot)
+        freq = f32(f)
+    q = torch.empty(n, H * d, device="cuda", dtype=dtype)
+    k = torch.full((4, 4, G, d), 9.0, device="cuda", dtype=dtype)
+    v = torch.full((4, 4, G, vd), 9.0, device="cuda", dtype=dtype)
+    ops.qkv_full_norm_rope_write(f32(rows), f32(bias), H, G, d, vd, None, None, 0.0, freq, dims,
+                                 i32(positions), i32(slots), q, k, v, pairs=pairs, amplitude=amp)
+    x = (rows + bias).numpy()
+    turn = plain.rotate_pairs if pairs else plain.rotate_halves
+    qs, ks = x[:, :H * d].reshape(n, H, d), x[:, H * d:(H + G) * d].reshape(n, G, d)
+    # (an angle of some thousands has an error of its own in float32)
+    close(q, np.stack([turn(qs[t], positions[t], rot) for t in range(n)]), dtype, bound=3e-4)
+    kp, vp = k.reshape(16, G, d), v.reshape(16, G, vd)
+    for t, s in enumerate(slots):
+        if s >= 0:
+            close(kp[s], turn(ks[t], positions[t], rot), dtype, bound=3e-4)
+            close(vp[s], x[t, (H + G) * d:].reshape(G, vd), dtype)
+    untouched = [s for s in range(16) if s not in slots]
+    assert float((kp[untouched] - 9.0).abs().max()) == 0 and float((vp[untouched] - 9.0).abs().max()) == 0
+
+
+# ---- latent rows: norms, pairwise scaled rotation ------------------------------------------------------
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("sizes", [(4, 16, 8, 32, 24), (3, 6, 2, 11, 7), (2, 64, 32, 96, 130)])
+@pytest.mark.parametrize("pairs", [False, True])
+def test_latent_rows_with_turned_parts(ops, dtype, sizes, pairs):
+    H, d, rot, rank, qr = sizes
+    g = torch.Generator().manual_seed(rank)
+    spec = dv._rot(rot, 200.0, (8.0, 32, 4.0, 0.5))
+    f, amp = plain.frequencies(spec)
+    turn = plain.rotate_pairs if pairs else plain.rotate_halves
+    positions, slots, eps = [4, 0, 250, 31], [6, 1, -1, 3], 1e-3
+    n = len(positions)
+    rows = rnd(g, dtype, n, qr + 3 + rank + rot)
+    wq, wkv = rnd(g, torch.float32, qr), rnd(g, torch.float32, rank)
+    cq = torch.empty(n, qr, device="cuda", dtype=dtype)
+    cache = torch.full((2, 4, 1, rank + rot), 9.0, device="cuda", dtype=dtype)
+    ops.latent_prepare(dev(rows, dtype), 0, qr, f32(wq), cq, qr + 3, rank, rot, f32(wkv), eps, f32(f),
+                       i32(positions), i32(slots), cache, pairs=pairs, amplitude=amp)
+    x = rows.numpy()
+    close(cq, plain.rms(x[:, :qr], eps) * wq.numpy(), dtype)
+    want = np.concatenate([plain.rms(x[:, qr + 3:qr + 3 + rank], eps) * wkv.numpy(),
+                           np.stack([turn(x[t, qr + 3 + rank:], positions[t], spec) for t in range(n)])], axis=1)
+    for t, s in enumerate(slots):
+        if s >= 0:
+            close(cache.reshape(8, -1)[s], want[t], dtype, bound=5e-5)
+    assert float((cache.reshape(8, -1)[[0, 2, 4, 5, 7]] - 9.0).abs().max()) == 0
+    q = rnd(g, dtype, n, H * (d + rot))
+    y = dev(q, dtype)
+    ops.rope_heads(y, H, d + rot, d, rot, f32(f), i32(positions), pairs=pairs, amplitude=amp)
+    w = q.numpy().reshape(n, H, d + rot).copy()
+    for t in range(n):
+        w[t, :, d:] = turn(w[t, :, d:], positions[t], spec)
+    close(y, w.reshape(n, -1), dtype, bound=5e-5)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("sizes", [(4, 36, 60), (3, 8, 13), (2, 64, 40), (1, 5, 7)])
+def test_products_per_head_of_any_size(ops, dtype, sizes):
+    """Also heads that begin between two 16-byte boundaries inside aligned rows."""
+    H, a, b = sizes
+    g = torch.Generator().manual_seed(a)
+    x, w = rnd(g, dtype, 37, 8 + H * a), rnd(g, dtype, H, a, b)
+    out = torch.empty(37, H * b, device="cuda", dtype=dtype)
+    ops.heads_product(dev(x, dtype), 8, H, a, dev(w, dtype), out)
+    want = np.einsum("nha,hab->nhb", x[:, 8:].numpy().reshape(37, H, a), w.numpy())
+    close(out, want.reshape(37, -1), dtype)
+
+
+# ---- attention over a window with kept first tokens -----------------------------------------------------
+
+class _Pages:
+    """Keys and values of requests scattered over pages in random order."""
+
+    def __init__(self, gen, dtype, lengths, G, d, vd, page, window, keep):
+        rng = random.Random(d + page)
+        self.k = [rnd(gen, dtype, n, G, d) for n in lengths]
+        self.v = [rnd(gen, dtype, n, G, vd) for n in lengths]
+        self.page, self.dtype, self.lengths, self.window, self.keep = page, dtype, lengths, window, keep
+        blocks = [-(-n // page) for n in lengths]
+        ids = rng.sample(range(sum(blocks) + 3), sum(blocks))
+        self.table = torch.full((len(lengths), max(blocks) + 1), -1, dtype=torch.int32)
+        a = 0
+        for r in range(len(lengths)):
+            self.table[r, :blocks[r]] = torch.tensor(ids[a:a + blocks[r]], dtype=torch.int32)
+            a += blocks[r]
+        self.pages = sum(blocks) + 3
+
+    def build(self, computed):
+        """Device pages as the cache manager leaves them: pages that neither a window nor the kept
+        tokens need are released (-1) and hold large values, so that reading them would show."""
+        G, d, vd = self.k[0].shape[1], self.k[0].shape[2], self.v[0].shape[2]
+        k = torch.full((self.pages, self.page, G, d), 50.0, dtype=torch.float64)
+        v = torch.full((self.pages, self.page, G, vd), 50.0, dtype=torch.float64)
+        table = self.table.clone()
+        for r, n in enumerate(self.lengths):
+            for j in range(n):
+                at = (int(self.table[r, j // self.page]), j % self.page)
+                k[at], v[at] = self.k[r][j], self.v[r][j]
+            if self.window:
+                kept = -(-self.keep // self.page)
+                for b in range(kept, max(0, computed[r] - self.window + 1) // self.page):
+                    p = int(table[r, b])
+                    k[p], v[p] = 50.0, 50.0
+                    table[r, b] = -1
+        group = SimpleNamespace(block_table=dev(table), max_blocks=table.shape[1], page_size=self.page)
+        return dev(k, self.dtype), dev(v, self.dtype), group
+
+
+def _attention_case(ops, dtype, sizes, lengths, new, page, window, keep, scale, loud=(), filling=False):
+    """`new[r]`: the last new[r] tokens of request r are this step's.  `loud`: (request, position of
+    the key, position of the query): the query is made to point at that key, so that one score
+    stands out among all (unless it is hidden).  `keep` None: a plain window through
+    `paged_attention`."""
+    H, G, d, vd = sizes
+    g = torch.Generator().manual_seed(H * d + page)
+    pages = _Pages(g, dtype, lengths, G, d, vd, page, window, keep or 0)
+    q = [rnd(g, dtype, n, H, d) for n in lengths]
+    for r, kp, qp in loud:
+        q[r][qp] = (pages.k[r][kp].repeat_interleave(H // G, dim=0) * 8.0).to(dtype).double()
+    starts = [n - m for n, m in zip(lengths, new)]
+    assert sorted(range(len(new)), key=lambda r: new[r] != 1) == list(range(len(new)))
+    k, v, group = pages.build(starts)
+    rows = torch.cat([q[r][starts[r]:].reshape(new[r], H * d) for r in range(len(new))])
+    ctx, cum = step_context([(m, 0) for m in new])
+    ctx.ctx_lens = i32(lengths)
+    outs = []
+    for longest in (max(lengths), 4 * max(lengths)):        # as replayed steps are: made for more
+        ctx.max_q_len, ctx.max_ctx_len = max(new), longest
+        out = torch.full((rows.shape[0], H * vd), float("nan"), device="cuda", dtype=dtype)
+        if keep is None:
+            ops.paged_attention(dev(rows, dtype), H, G, d, k, v, ctx, group, scale, window, out,
+                                v_head_dim=vd)
+        else:
+            ops.paged_attention_pooled(dev(rows, dtype), H, G, d, k, v, ctx, group, (k, v, group, 1), scale,
+                                       None, window, None, out, v_head_dim=vd, most_blocks=keep)
+        outs.append(out)
+    mask = {"size": window, "keep_first": keep or 0}
+    for r in range(len(new)):
+        for t in range(new[r]):
+            p = starts[r] + t
+            see = plain.visible(p, mask)
+            for h in range(H):
+                keys, vals = pages.k[r][see, h // (H // G)].numpy(), pages.v[r][see, h // (H // G)].numpy()
+                want = plain.softmax(keys @ q[r][p, h].numpy() * scale) @ vals
+                for o in outs:
+                    close(o[cum[r] + t, h * vd:(h + 1) * vd], want, dtype, scale=1.0,
+                          bound=5e-5 if dtype == torch.float32 else 3e-2)
+
+
+SHAPES = [(torch.float32, (4, 2, 32, 32)), (torch.float32, (3, 1, 10, 7)), (torch.bfloat16, (8, 2, 64, 64)),
+          (torch.bfloat16, (6, 2, 48, 48)), (torch.bfloat16, (3, 3, 10, 14)), (torch.bfloat16, (4, 2, 64, 128)),
+          (torch.bfloat16, (2, 1, 128, 128)), (torch.bfloat16, (5, 1, 128, 32)), (torch.bfloat16, (12, 1, 32, 80))]
+
+
+@pytest.mark.parametrize("dtype,sizes", SHAPES)
+@pytest.mark.parametrize("window,keep", [(20, 8), (13, 30), (5, 1), (64, 17), (40, None), (100, 64)])
+def test_window_with_kept_first_tokens_every_visible_key(ops, dtype, sizes, window, keep):
+    d = sizes[2]
+    _attention_case(ops, dtype, sizes, (150, 1, 33, 70, 129), (1, 1, 1, 70, 67), 8, window, keep, d ** -0.5)
+
+
+@pytest.mark.parametrize("dtype,sizes", [SHAPES[0], SHAPES[2], SHAPES[4], SHAPES[5]])
+@pytest.mark.parametrize("decoded", [True, False])
+def test_one_key_stands_out_at_every_edge(ops, dtype, sizes, decoded):
+    """For one query the window's oldest key and the one before it, the last kept token and the first
+    that is not, page borders: each made the one whose score stands out."""
+    window, keep, page, n = 40, 21, 16, 200
+    P = n - 1                                                # the last query
+    for e in (P, P - 1, P - window + 1, P - window, 0, keep - 1, keep, keep + 1, page, page - 1, 2 * page, 176, 175):
+        _attention_case(ops, dtype, sizes, (n,), (1,) if decoded else (70,), page, window, keep, sizes[2] ** -0.5,
+                        loud=[(0, e, P)])
+
+
+@pytest.mark.parametrize("dtype,sizes", [SHAPES[0], SHAPES[2], SHAPES[5]])
+def test_many_kept_tokens_and_windows_beyond_a_split(ops, dtype, sizes):
+    """More than 256 kept tokens and windows of more than 256: single tokens are split over both,
+    and a far key among hundreds stands out; windows that still overlap the kept tokens."""
+    for window, keep, lengths in ((30, 300, (1000, 320)), (600, 10, (1900, 603)), (257, 513, (1101, 700))):
+        loud = [(0, 5, lengths[0] - 1), (1, lengths[1] - window, lengths[1] - 1)]
+        _attention_case(ops, dtype, sizes, lengths, (1, 1), 16, window, keep, 0.2, loud=loud)
+    _attention_case(ops, dtype, sizes, (1000,), (20,), 16, 30, 300, 0.2, loud=[(0, 5, 999), (0, 299, 985)])
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("size", [144, 60, 13, 128, 192])
+def test_windows_over_one_shared_latent_head(ops, dtype, size):
+    """Many query heads on one key head whose values are its keys (an odd size and an odd count
+    of heads among them)."""
+    H = 3 if size == 13 else 8
+    g = torch.Generator().manual_seed(size)
+    lengths, new, window, page = (150, 33, 1, 129), (1, 1, 1, 67), 40, 8
+    pages = _Pages(g, dtype, lengths, 1, size, 1, page, window, 0)
+    q = [rnd(g, dtype, n, H, size) for n in lengths]
+    starts = [n - m for n, m in zip(lengths, new)]
+    k, _, group = pages.build(starts)
+    rows = torch.cat([q[r][starts[r]:].reshape(new[r], H * size) for r in range(len(new))])
+    ctx, cum = step_context([(m, 0) for m in new])
+    ctx.ctx_lens, ctx.max_q_len, ctx.max_ctx_len = i32(lengths), max(new), max(lengths)
+    out = torch.full((rows.shape[0], H * size), float("nan"), device="cuda", dtype=dtype)
+    ops.paged_attention(dev(rows, dtype), H, 1, size, k, k, ctx, group, size ** -0.5, window, out)
+    for r in range(len(new)):
+        for t in range(new[r]):
+            see = plain.visible(starts[r] + t, {"size": window})
+            keys = pages.k[r][see, 0].numpy()
+            for h in range(H):
+                want = plain.softmax(keys @ q[r][starts[r] + t, h].numpy() * size ** -0.5) @ keys
+                close(out[cum[r] + t, h * size:(h + 1) * size], want, dtype, scale=1.0,
+                      bound=5e-5 if dtype == torch.float32 else 3e-2)
+
+
+# ---- recurrences ------------------------------------------------------------------------------------------
+
+def _feed(lengths, cuts, slots, run, ref, n_state):
+    """Requests fed in portions of unequal size beside one another, with empty and filling requests;
+    `run(rows, ctx)` -> outputs.  Returns each request's outputs in order."""
+    done, got = {r: 0 for r in lengths}, {r: [] for r in lengths}
+    for step in range(max(len(c) for c in cuts.values())):
+        parts = [(r, cuts[r][step]) for r in cuts if step < len(cuts[r])]
+        parts.sort(key=lambda p: p[1] != 1)                  # single tokens first
+        single = [p for p in parts if p[1] == 1]
+        # empty requests and filling requests without a slot, as padded steps have
+        layout = single + [(None, 1)] + parts[len(single):] + [(None, 0), (None, 70)]
+        ctx, starts = step_context([(n, slots[r] if r else -1) for r, n in layout])
+        rows = np.concatenate([ref[r][done[r]:done[r] + n] if r else np.full((n, n_state), 1e3)
+                               for r, n in layout])
+        out = run(rows, ctx)
+        for (r, n), a in zip(layout, starts):
+            if r:
+                got[r].append(out[a:a + n].cpu())
+                done[r] += n
+    assert done == lengths
+    return {r: torch.cat(got[r]) for r in lengths}
+
+
+LENGTHS = {"a": 240, "b": 9, "c": 66, "d": 131}
+CUTS = {"a": [65, 2, 1, 127, 45], "b": [1] * 9, "c": [2, 64], "d": [64, 3, 64]}
+SLOTS = {"a": 5, "b": 0, "c": 2, "d": 3}
+
+
+def _delta(gen, H, G, d, dvv, taps, strong=False):
+    m = {"heads": H, "kv_heads": G, "dim": d, "vdim": dvv, "conv": taps}
+    C = 2 * G * d + H * dvv
+    t = {"filt": rnd(gen, torch.float32, C, taps, std=0.5).numpy(),
+         "A_log": rnd(gen, torch.float32, H).numpy() * (3.0 if strong else 1.0),
+         "dt_bias": rnd(gen, torch.float32, H).numpy(), "norm": 1.0 + 0.1 * rnd(gen, torch.float32, dvv).numpy()}
+    rows = {r: rnd(gen, torch.float32, n, C + 2 * H + H * dvv).numpy() for r, n in LENGTHS.items()}
+    return m, C, t, rows
+
+
+def _delta_plain(m, C, t, rows, silu_gate=True, unit=1e-6, eps=1e-5):
+    H, G, d, dvv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    T = rows.shape[0]
+    x = plain.silu(plain.causal_conv(rows[:, :C], t["filt"]))
+    q, k, v = np.split(x, [G * d, 2 * G * d], axis=1)
+    u = lambda y: y / np.sqrt((y ** 2).sum(-1, keepdims=True) + unit)
+    q = np.repeat(u(q.reshape(T, G, d)) * d ** -0.5, H // G, axis=1)
+    k = np.repeat(u(k.reshape(T, G, d)), H // G, axis=1)
+    beta = plain.sigmoid(rows[:, C:C + H])
+    g = np.exp(-np.exp(t["A_log"]) * plain.softplus(rows[:, C + H:C + 2 * H] + t["dt_bias"]))
+    o, S = plain.delta_rule(q, k, v.reshape(T, H, dvv), g, beta)
+    z = rows[:, C + 2 * H:].reshape(T, H, dvv)
+    return (plain.rms(o, eps) * t["norm"] * (plain.silu(z) if silu_gate else plain.sigmoid(z))).reshape(T, -1), S
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("sizes", [(4, 2, 24, 16, 4), (2, 2, 16, 40, 2), (3, 1, 40, 8, 1), (3, 3, 6, 5, 3),
+                                   (2, 1, 128, 64, 4), (4, 2, 64, 32, 3), (2, 2, 64, 128, 4), (1, 1, 130, 33, 2)])
+@pytest.mark.parametrize("strong", [False, True])
+def test_delta_rule_with_a_decay_per_head(ops, dtype, sizes, strong):
+    """Four requests of unequal length in portions of unequal size, one of them token by token, in
+    state slots that are not in order; decays from nearly none to nearly all."""
+    H, G, d, dvv, taps = sizes
+    gen = torch.Generator().manual_seed(d + dvv)
+    m, C, t, rows = _delta(gen, H, G, d, dvv, taps, strong)
+    rec = ops.gated_delta_record(H, G, d, dvv, taps)
+    for silu_gate in ((True, False) if not strong else (True,)):
+        state = torch.zeros(6, rec, device="cuda")
+        state[4].fill_(3.0)
+
+        def run(x, ctx):
+            proj = f32(x)
+            out = torch.empty(x.shape[0], H * dvv, device="cuda", dtype=dtype)
+            ops.gated_delta(proj, proj[:, C + H:], f32(t["filt"]), f32(t["A_log"]), f32(t["dt_bias"]),
+                            f32(t["norm"]), state, ctx, out, H, G, d, dvv, taps, 1e-6, 1e-5, head_decay=True,
+                            gate="silu" if silu_gate else "sigmoid")
+            return out
+
+        got = _feed(LENGTHS, CUTS, SLOTS, run, rows, C + 2 * H + H * dvv)
+        for r in LENGTHS:
+            want, S = _delta_plain(m, C, t, rows[r], silu_gate)
+            close(got[r], want, dtype, bound=4e-5 if dtype == torch.float32 else None)
+            rows_of = state[SLOTS[r]][(taps - 1) * C:].reshape(H, dvv, d).transpose(1, 2)
+            close(rows_of, S, torch.float32, bound=4e-5)
+            if taps > 1:
+                old = np.concatenate([np.zeros((taps - 1, C)), rows[r][:, :C]])[-(taps - 1):]
+                close(state[SLOTS[r]][:(taps - 1) * C], old.reshape(-1), torch.float32)
+        assert float((state[4] - 3.0).abs().max()) == 0 and float(state[1].abs().max()) == 0
+
+
+def _ssm(gen, H, dvv, N, G, taps, ng, spread=1.0):
+    m = dict(heads=H, vdim=dvv, state=N, groups=G, conv=taps, norm_groups=ng)
+    C = H * dvv + 2 * G * N
+    t = {"conv": rnd(gen, torch.float32, C, taps, std=0.5).numpy(), "conv.b": rnd(gen, torch.float32, C, std=0.2).numpy(),
+         "dt_bias": rnd(gen, torch.float32, H).numpy(), "A_log": spread * rnd(gen, torch.float32, H).numpy(),
+         "D": rnd(gen, torch.float32, H).numpy(), "norm": 1.0 + 0.1 * rnd(gen, torch.float32, H * dvv).numpy()}
+    return m, C, t
+
+
+def _ssm_plain(m, C, t, rows, rounded, eps=1e-5):
+    H, dvv, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+    inner, T = H * dvv, rows.shape[0]
+    x = plain.silu(plain.causal_conv(rows[:, inner:inner + C], t["conv"], t["conv.b"]))
+    if rounded:                                               # as bfloat16 rows hold them
+        x = torch.from_numpy(x).to(torch.bfloat16).double().numpy()
+    B = np.repeat(x[:, inner:inner + G * N].reshape(T, G, N), H // G, axis=1)
+    Cq = np.repeat(x[:, inner + G * N:].reshape(T, G, N), H // G, axis=1)
+    dt = plain.softplus(rows[:, inner + C:inner + C + H] + t["dt_bias"])
+    y, S = plain.ssd_scan(x[:, :inner].reshape(T, H, dvv), B, Cq, dt, np.exp(-np.exp(t["A_log"]) * dt), t["D"])
+    y = y.reshape(T, inner) * plain.silu(rows[:, :inner])
+    return plain.grouped_rms(y, m["norm_groups"], eps) * t["norm"], S
+
+
+def _ssm_run(ops, m, C, t, state, conv, dtype):
+    H, dvv, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+
+    def run(x, ctx):
+        out = torch.full((x.shape[0], H * dvv), float("nan"), device="cuda", dtype=dtype)
+        ops.state_space(f32(x), f32(t["conv"]), f32(t["conv.b"]), f32(t["dt_bias"]), f32(t["A_log"]), f32(t["D"]),
+                        f32(t["norm"]), conv, state, ctx, out, H, dvv, N, G, m["conv"], m["norm_groups"], 1e-5)
+        return out
+    return run
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("sizes", [(6, 16, 24, 2, 3, 4), (2, 40, 8, 1, 4, 1), (4, 32, 40, 4, 2, 2), (3, 5, 7, 3, 4, 5),
+                                   (2, 9, 3, 1, 1, 1), (8, 64, 128, 2, 4, 2), (3, 16, 48, 1, 5, 3), (2, 80, 256, 1, 4, 1),
+                                   (2, 64, 272, 2, 3, 1)])
+def test_state_space_kernels(ops, dtype, sizes):
+    H, dvv, N, G, taps, ng = sizes
+    gen = torch.Generator().manual_seed(N + dvv)
+    m, C, t = _ssm(gen, H, dvv, N, G, taps, ng)
+    fill = -(H * dvv + C + H) % 8                             # the rows may be wider
+    P = H * dvv + C + H + (fill if N != 40 else 0)
+    rows = {r: rnd(gen, torch.float32, n, P).numpy() for r, n in LENGTHS.items()}
+    state = torch.zeros(6, H * N * dvv, device="cuda")
+    conv = torch.zeros(6, taps - 1, C, device="cuda") if taps > 1 else None
+    state[4].fill_(3.0)
+    got = _feed(LENGTHS, CUTS, SLOTS, _ssm_run(ops, m, C, t, state, conv, dtype), rows, P)
+    for r in LENGTHS:
+        want, S = _ssm_plain(m, C, t, rows[r], dtype == torch.bfloat16)
+        close(got[r], want, dtype, bound=4e-5 if dtype == torch.float32 else None)
+        # (a value on the way between two bfloat16 numbers may round the other way)
+        close(state[SLOTS[r]], S.reshape(-1), torch.float32, bound=4e-5 if dtype == torch.float32 else 2e-3)
+        if taps > 1:
+            old = np.concatenate([np.zeros((taps - 1, C)), rows[r][:, H * dvv:H * dvv + C]])[-(taps - 1):]
+            close(conv[SLOTS[r]], old, torch.float32)
+    assert float((state[4] - 3.0).abs().max()) == 0 and float(state[1].abs().max()) == 0
+
+
+@pytest.mark.parametrize("dtype,sizes", [(torch.float32, (3, 16, 24, 1, 4, 1)), (torch.bfloat16, (3, 32, 48, 1, 4, 1)),
+                                         (torch.bfloat16, (3, 12, 20, 3, 2, 1))])
+def test_state_space_decays_from_nothing_to_one(ops, dtype, sizes):
+    """Tokens that forget everything at once between tokens that forget nothing, over many chunks,
+    whole and in other cuts: no infinity, no lost token, no digits lost to a large sum of decays."""
+    H, dvv, N, G, taps, ng = sizes
+    gen = torch.Generator().manual_seed(5)
+    m, C, t = _ssm(gen, H, dvv, N, G, taps, ng)
+    t["A_log"] = np.array([6.0, -8.0, 0.0])
+    t["dt_bias"] = np.array([-12.0, 3.0, 0.0])
+    n, inner = 400, H * dvv
+    rows = rnd(gen, torch.float32, n, inner + C + H).numpy()
+    rows[::37, inner + C:] += 30.0                            # now and then a step that clears the state
+    want, S = _ssm_plain(m, C, t, rows, dtype == torch.bfloat16)
+    for cut in ([n], [64, 1, 2, 130] * 2 + [6], [2] * 30 + [n - 60]):
+        state = torch.zeros(1, H * N * dvv, device="cuda")
+        conv = torch.zeros(1, taps - 1, C, device="cuda")
+        run, outs, at = _ssm_run(ops, m, C, t, state, conv, dtype), [], 0
+        for c in cut:
+            ctx, _ = step_context([(c, 0)])
+            outs.append(run(rows[at:at + c], ctx).cpu())
+            at += c
+        assert at == n
+        close(torch.cat(outs), want, dtype, bound=1e-4 if dtype == torch.float32 else None)
+        close(state[0], S.reshape(-1), torch.float32, bound=1e-4 if dtype == torch.float32 else 2e-3)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("which", ["state_space", "delta"])
+def test_an_early_token_among_hundreds_is_not_lost(ops, dtype, which):
+    """One early token is large and decays are near one: it is seen by the last token, in prompts,
+    portions and single tokens."""
+    gen = torch.Generator().manual_seed(6)
+    n, H, taps = 330, 2, 3
+    if which == "state_space":
+        m, C, t = _ssm(gen, H, 16, 16, 1, taps, 1)
+        t["A_log"], t["dt_bias"] = np.array([-7.0, -6.0]), np.array([-1.0, 0.0])
+        rows = rnd(gen, torch.float32, n, H * 16 + C + H).numpy()
+        rows[:, H * 16:H * 16 + C] *= 0.1
+        rows[3, H * 16:H * 16 + C] *= 200.0
+        want, _ = _ssm_plain(m, C, t, rows, dtype == torch.bfloat16)
+        other = rows.copy()
+        other[3, H * 16:H * 16 + C] = 0.0
+        assert np.abs(_ssm_plain(m, C, t, other, False)[0][-1] - want[-1]).max() > 0.1
+    else:
+        m, C, t, _ = _delta(gen, H, 1, 64, 32, taps)
+        t["A_log"], t["dt_bias"] = np.array([-7.0, -6.0]), np.array([-1.0, 0.0])
+        rows = rnd(gen, torch.float32, n, C + 2 * H + H * 32).numpy()
+        rows[:, C:C + H] = -6.0                               # tokens write little ...
+        rows[3, C:C + H] = 8.0                                # ... but this one all of its large value
+        rows[3, 2 * 64:C] *= 100.0
+        rows[-1, :64] = rows[3, 64:128]                       # and the last query points at its key
+        want, _ = _delta_plain(m, C, t, rows)
+        other = rows.copy()
+        other[3, C:C + H] = -30.0
+        assert np.abs(_delta_plain(m, C, t, other)[0][-1] - want[-1]).max() > 0.1
+    for cut in ([n], [2, 63, 65, 200], [300] + [1] * 30):
+        outs, at = [], 0
+        if which == "state_space":
+            state, conv = torch.zeros(1, H * 16 * 16, device="cuda"), torch.zeros(1, taps - 1, C, device="cuda")
+            run = _ssm_run(ops, m, C, t, state, conv, dtype)
+        else:
+            state = torch.zeros(1, ops.gated_delta_record(H, 1, 64, 32, taps), device="cuda")
+
+            def run(x, ctx):
+                proj = f32(x)
+                out = torch.empty(x.shape[0], H * 32, device="cuda", dtype=dtype)
+                ops.gated_delta(proj, proj[:, C + H:], f32(t["filt"]), f32(t["A_log"]), f32(t["dt_bias"]),
+                                f32(t["norm"]), state, ctx, out, H, 1, 64, 32, taps, 1e-6, 1e-5, head_decay=True,
+                                gate="silu")
+                return out
+        for c in cut:
+            ctx, _ = step_context([(c, 0)])
+            outs.append(run(rows[at:at + c], ctx).cpu())
+            at += c
+        close(torch.cat(outs), want, dtype, bound=1e-4 if dtype == torch.float32 else None)
+
+
+# ---- experts and identity experts --------------------------------------------------------------------
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("sizes", [(7, 3, 3, 5, 3, 64, 32, 50), (4, 0, 4, 1, 1, 48, 40, 20), (3, 5, 5, 4, 3, 50, 21, 9),
+                                   (2, 6, 2, 2, 1, 96, 24, 70), (12, 4, 4, 4, 2, 128, 64, 150), (1, 2, 3, 1, 1, 40, 16, 33)])
+def test_experts_and_identity_experts(ops, dtype, sizes):
+    """Few tokens and many (the grouped products), with corrections so negative that a masked score of
+    0 would win, and an expert left out by its group although its score is among the largest."""
+    E, I, top, groups, keep, W, F, n = sizes
+    g = torch.Generator().manual_seed(E * 10 + I)
+    x = rnd(g, torch.bfloat16, n, W)
+    t = {"router": rnd(g, torch.float32, E + I, W, std=2 * W ** -0.5).numpy(),
+         "correction": (rnd(g, torch.float32, E + I, std=0.3) - 1.5).float().double().numpy()}
+    for e in range(E):
+        for k, shape in (("gate", (F, W)), ("up", (F, W)), ("down", (W, F))):
+            t[f"e{e}.{k}"] = rnd(g, torch.bfloat16, *shape, std=shape[1] ** -0.5).numpy()
+    mlp = {"router": {"experts": E, "identity": I, "top": top, "scale": 1.7, "groups": {"count": groups, "keep": keep}}}
+    gate_up = np.stack([np.stack([t[f"e{e}.gate"], t[f"e{e}.up"]], axis=1).reshape(2 * F, W) for e in range(E)])
+    down = np.stack([t[f"e{e}.down"] for e in range(E)])
+    for m in (n, 2):
+        want = plain.moe(x[:m].numpy(), mlp, t)
+        ids = torch.empty(m, top, dtype=torch.int32, device="cuda")
+        wts = torch.empty(m, top, dtype=torch.float32, device="cuda")
+        ops.moe_route(dev(x[:m], dtype), f32(t["router"]), groups, keep, 1, 0.0, ids, wts, score="softmax",
+                      renormalize=False, route_scale=1.7, choice_bias=f32(t["correction"]))
+        for i in range(m):
+            s = plain.softmax(t["router"] @ x[i].numpy())
+            chosen = plain.choose(s + t["correction"], top, groups, keep)
+            assert ids[i].tolist() == chosen
+            assert np.allclose(wts[i].cpu().numpy(), s[chosen] * 1.7, rtol=2e-5, atol=1e-7)
+        modes = ("simple", "grouped") if dtype == torch.bfloat16 and W % 8 == 0 and F % 8 == 0 else ("auto",)
+        for mode in modes:
+            saved, ops.moe_mode = ops.moe_mode, mode
+            try:
+                out = torch.full((m, W), float("nan"), device="cuda", dtype=dtype)
+                ops.moe_experts(dev(x[:m], dtype), ids, wts, dev(gate_up, dtype), dev(down, dtype), out, identity=I)
+            finally:
+                ops.moe_mode = saved
+            close(out, want, dtype)
+    ops.check_status()
+
+
+# ---- the engine -------------------------------------------------------------------------------------
+
+_models = {}
+
+
+def engine(folder, dtype):
+    from rvllm_b200.engine import load_model
+    if (folder, dtype) not in _models:
+        _models[(folder, dtype)] = load_model(folder, dtype, "cuda")[0]
+    return _models[(folder, dtype)]
+
+
+def run_schedule(model, steps, page, slots=4, graphs=False):
+    from rvllm_b200.engine import ModelRunner, make_cache
+    cache = make_cache(model, page, schedules.tokens_held(steps, 64) // page, slots)
+    runner = ModelRunner(model, cache, model.ops, use_graphs=graphs)
+    got = schedules.replay(runner, steps)
+    model.ops.check_status()
+    assert not cache.requests and all(g.pool.in_use == 0 for g in cache.groups)
+    return got, runner
+
+
+_plain = {}
+
+
+def compare(got, folder, cfg, reqs, dtype, share=0.04):
+    """float32: every position within the bound.  bfloat16: a router score that is a close call
+    may fall the other way after rounding and change a token's experts, which is no fault; so a
+    few positions in a hundred may lie outside the bound."""
+    over, total = [], 0
+    for rid, ids in reqs.items():
+        key = (folder, tuple(ids))
+        if key not in _plain:
+            _plain[key] = dv.plain_logits(folder, None, ids, cfg=cfg)
+        ref = _plain[key]
+        scale = float(ref.abs().max())
+        for p in range(len(ids)):
+            err = float((got[(rid, p)].double() - ref[p]).abs().max()) / scale
+            total += 1
+            if not err < BOUND[dtype]:
+                over.append((rid, p, err))
+    assert len(over) <= (0 if dtype == "float32" else share * total), (len(over), total, over[:5])
+
+
+def _requests(vocab, lengths, seed):
+    rng = random.Random(seed)
+    return {f"q{i}": [rng.randrange(vocab) for _ in range(n)] for i, n in enumerate(lengths)}
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "B", "C", "D"])
+def test_every_cut_equals_plain(folders, name, dtype):
+    """Whole prompts; a prompt then its last tokens one by one; portions down to two tokens;
+    mixed batches of unequal requests on four slots, with more requests than slots, so that
+    pages and slots are used again."""
+    model = engine(folders[name], dtype)
+    cfg = dv.config(name)
+    reqs = _requests(cfg["vocab"], (130, 1, 2, 67, 200, 33, 64, 65), 3)
+    f = folders[name]
+    compare(run_schedule(model, schedules.whole(reqs), 16)[0], f, cfg, reqs, dtype)
+    compare(run_schedule(model, schedules.tail_decode(reqs, 90), 8)[0], f, cfg, reqs, dtype)
+    compare(run_schedule(model, schedules.portions(reqs), 16)[0], f, cfg, reqs, dtype)
+    compare(run_schedule(model, schedules.portions(reqs, (64, 2, 100, 3)), 4)[0], f, cfg, reqs, dtype)
+    for seed in (0, 1):
+        compare(run_schedule(model, schedules.mixed(reqs, seed), 16)[0], f, cfg, reqs, dtype)
+
+
+def _one_mechanism(tmp, which):
+    """A model of one layer whose mixer is sharp (a large scale, large projections), so that a
+    single lost or misplaced key changes the result by much more than the bound."""
+    from rvllm_b200.config import config_from_dict
+    from rvllm_b200.weights import write_random_model
+    from rvllm_b200.weights.safetensors_io import SafetensorsFile, write_streamed
+    both = dv._both(dv._left(6, 3, 32, 48, 3.0, 25, 11, dv._rot(20, 50.0)), dv._right(4, 2, 24, 40, 3), 1.0, 1.0)
+    if which == "left":
+        both["right_scale"] = 0.0
+    if which == "right":
+        both["left_scale"] = 0.0
+    layer = {"left": {"type": "parallel", "mixer": both}, "right": {"type": "parallel", "mixer": both},
+             "latent": {"type": "latent_attention",
+                        "mixer": dv._latent(4, 24, 8, 16, 40, 32, 3.0, 19, dv._rot(8, 40.0, (3.0, 40, 6.0, 0.7)))},
+             "state_space": {"type": "mamba2", "mixer": dv._ssm(4, 24, 20, 2, 4, 2)}}[which]
+    cfg = {"architecture": "Dopuvik", "vocab": 150, "width": 72, "norm": {"eps": 1e-5},
+           "embedding": {"scale": 3.0}, "logit_scale": 0.6, "layers": [dict(layer, mlp=None)]}
+    folder = write_random_model(os.path.join(tmp, which), config_from_dict(copy.deepcopy(cfg)), 7)
+    path = os.path.join(folder, "model.safetensors")
+    f = SafetensorsFile(path)
+    tensors = {n: f.tensor(n).clone() for n in f.names()}
+    del f
+    for n, t in tensors.items():                              # projections that give scores of size
+        if n.endswith((".q", ".k", ".dq", ".dkv", ".in", "embed", ".b", ".a")):
+            tensors[n] = (t.float() * 6.0).to(t.dtype)
+    write_streamed(path, [(n, tuple(t.shape), t.dtype) for n, t in tensors.items()],
+                   lambda n: tensors[n])
+    return folder, cfg
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("which", ["left", "right", "latent", "state_space"])
+def test_one_mechanism_alone_with_sharp_scores(tmp_path_factory, which, dtype):
+    """Keys far away (hundreds of positions back), at page borders and in the first tokens,
+    in prompts, in portions that begin inside a page, a window and a chunk, and in single tokens."""
+    folder, cfg = _one_mechanism(str(tmp_path_factory.mktemp("one")), which)
+    model = engine(folder, dtype)
+    reqs = _requests(cfg["vocab"], (400, 63, 17), 11)
+    ref = dv.plain_logits(folder, None, reqs["q0"], cfg=cfg)
+    assert float(ref.abs().max()) > 0.05
+    for steps, page in ((schedules.whole(reqs), 16), (schedules.tail_decode(reqs, 40), 8),
+                        (schedules.portions(reqs, (15, 2, 17, 130, 3)), 16),
+                        (schedules.mixed(reqs, 4), 4)):
+        compare(run_schedule(model, steps, page)[0], folder, cfg, reqs, dtype, share=0.05)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "D"])
+def test_replayed_steps_equal_plain(folders, name, dtype):
+    """The same with captured launch sequences: single-token steps and padded mixtures are
+    replayed from graphs; requests come and go, so slots and pages are used again."""
+    model = engine(folders[name], dtype)
+    cfg = dv.config(name)
+    reqs = _requests(cfg["vocab"], (90, 5, 41, 120, 33, 70, 18), 8)
+    for steps, page in ((schedules.tail_decode(reqs, 40), 16), (schedules.mixed(reqs, 2), 8),
+                        (schedules.mixed(reqs, 3, max_live=3, decode_tail=20), 16)):
+        got, runner = run_schedule(model, steps, page, graphs=True)
+        compare(got, folders[name], cfg, reqs, dtype)
+        assert runner.graph_steps > 0
+
+
+def test_long_decoding(folders):
+    """600 tokens one by one after a short prompt, across many pages, windows and splits."""
+    model = engine(folders["B"], "float32")
+    cfg = dv.config("B")
+    reqs = _requests(cfg["vocab"], (640,), 6)
+    got, _ = run_schedule(model, schedules.tail_decode(reqs, 620), 16, graphs=True)
+    compare(got, folders["B"], cfg, reqs, "float32")
+
+
+def test_a_batch_does_not_change_a_request(folders):
+    """A request beside others gives what it gives alone, in the same cut."""
+    model = engine(folders["A"], "float32")
+    reqs = _requests(dv.config("A")["vocab"], (70, 31, 5), 12)
+    alone, _ = run_schedule(model, schedules.whole({"q0": reqs["q0"]}), 16)
+    steps = [{"step": 0, "entries": [{"id": r, "tokens": ids, "want": list(range(len(ids)))}
+                                      for r, ids in reqs.items()], "end": list(reqs)}]
+    together, _ = run_schedule(model, steps, 16)
+    scale = max(float(alone[("q0", p)].abs().max()) for p in range(70))
+    for p in range(70):
+        assert float((alone[("q0", p)] - together[("q0", p)]).abs().max()) < 1e-5 * scale
+
+
+@pytest.mark.parametrize("name", ["A", "C"])
+def test_greedy_generation_through_the_entry_point(folders, name):
+    """Greedy tokens through `Generator` (scheduler, portions, preemption by a small pool) equal
+    the plain implementation's argmax chain."""
+    from rvllm_b200 import GenerateOptions, Generator
+    rng = random.Random(9)
+    cfg = dv.config(name)
+    new = 20
+    tensors = dv.read_tensors(folders[name])
+
+    def plain_greedy(ids):
+        """The argmax chain, or None when two logits on the way are too close to call."""
+        ids = list(ids)
+        for _ in range(new):
+            row = dv.plain_logits(folders[name], name, ids, tensors=tensors)[-1]
+            top = torch.topk(row, 2).values
+            if float(top[0] - top[1]) < 1e-3 * float(row.abs().max()):
+                return None
+            ids.append(int(row.argmax()))
+        return ids[-new:]
+
+    prompts, want = [], []
+    for n in (5, 37, 70):
+        for attempt in range(20):
+            p = [rng.randrange(cfg["vocab"]) for _ in range(n)]
+            w = plain_greedy(p)
+            if w is not None:
+                prompts.append(p)
+                want.append(w)
+                break
+    assert len(prompts) == 3
+    gen = Generator.load(folders[name], dtype="float32")
+    for opts in (GenerateOptions(max_tokens=new, block_size=16, stop_tokens=[]),
+                 GenerateOptions(max_tokens=new, block_size=8, stop_tokens=[], prefill_chunk=7,
+                                 max_batched_tokens=12),
+                 GenerateOptions(max_tokens=new, block_size=8, stop_tokens=[], num_blocks=16,
+                                 prefill_chunk=20)):
+        assert gen.complete_batch(prompts, opts) == want
+
+
+def test_command_line_and_trace_replay(folders, tmp_path):
+    """The design through the programs a user starts: `rvllm random-model` writes a folder from a
+    config.json, `rvllm cli` completes prompts of token ids, `bin/trace_run` replays steps from
+    standard input and writes logits that equal the plain implementation's."""
+    import json
+    import subprocess
+    import sys
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    cfg_path = tmp_path / "config.json"
+    cfg_path.write_text(json.dumps(dv.config("B")))
+    folder = str(tmp_path / "model")
+    r = subprocess.run([sys.executable, os.path.join(root, "bin", "rvllm"), "random-model",
+                        "--config", str(cfg_path), "--seed", "5", "--out", folder],
+                       capture_output=True, text=True, timeout=600)
+    assert r.returncode == 0, r.stderr[-2000:]
+    tensors = dv.read_tensors(folder)
+    prompt = [3, 1, 4, 1, 5, 9, 2, 6]
+    r = subprocess.run([sys.executable, os.path.join(root, "bin", "rvllm"), "cli", "--model", folder,
+                        "--dtype", "float32", "--token-ids", "--prompt", " ".join(map(str, prompt)),
+                        "--max-tokens", "5", "--block-size", "8"],
+                       capture_output=True, text=True, timeout=600)
+    assert r.returncode == 0, r.stderr[-2000:]
+    got = [int(t) for t in r.stdout.strip().splitlines()[0].split()]
+    ids = list(prompt)
+    for tok in got:                           # each token is the plain argmax at its place
+        row = dv.plain_logits(folder, "B", ids, tensors=tensors)[-1]
+        assert float(row.max() - row[tok]) < 1e-3 * float(row.abs().max())
+        ids.append(tok)
+    assert len(got) == 5
+    reqs = _requests(dv.config("B")["vocab"], (70, 33, 90, 41, 12), 4)
+    steps = schedules.mixed(reqs, seed=2)
+    vocab = dv.config("B")["vocab"]
+    for dtype in ("float32", "bfloat16"):
+        out = tmp_path / dtype
+        cmd = [sys.executable, os.path.join(root, "bin", "trace_run"), "--model", folder,
+               "--dtype", dtype, "--out", str(out), "--max-tokens",
+               str(schedules.tokens_held(steps, 64))]
+        r = subprocess.run(cmd, input="\n".join(json.dumps(s) for s in steps) + "\n",
+                           capture_output=True, text=True, timeout=900)
+        assert r.returncode == 0, r.stderr[-2000:]
+        assert [l for l in r.stdout.split("\n") if l.startswith("done")] == \
+            [f"done {s['step']}" for s in steps]
+        got, pos = {}, {k: 0 for k in reqs}
+        for s in steps:
+            arr = np.fromfile(out / f"{s['step']}.f32", dtype="<f4").reshape(-1, vocab)
+            k = 0
+            for e in s["entries"]:
+                for w in e["want"]:
+                    got[(e["id"], pos[e["id"]] + w)] = torch.from_numpy(arr[k].copy())
+                    k += 1
+                pos[e["id"]] += len(e["tokens"])
+            assert k == arr.shape[0]
+        compare(got, folder, dv.config("B"), reqs, dtype)
