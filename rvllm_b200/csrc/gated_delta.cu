@@ -48,7 +48,12 @@
 //     taps-1 of old record | this step's rows).
 // All arithmetic is float32; y is the compute type.  Plain reference: tests/plain_ops.py
 // gated_delta.
+//
+// With one decay per head, portions of bfloat16 models take the chunk form on the tensor cores where
+// sizes allow (gated_delta_chunk.cuh).  There an activated q, k or v is rounded to bfloat16, and gdr_prepare
+// does the same (`round`), so that a token is the same in a portion and alone.
 #include "common.cuh"
+#include "gated_delta_chunk.cuh"
 
 __device__ __forceinline__ float gd_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float gd_softplus(float a) { return a > 20.f ? a : log1pf(expf(a)); }
@@ -63,7 +68,7 @@ __global__ void gdr_prepare_kernel(const float* __restrict__ proj, int P,
                                    const int* __restrict__ q_start,
                                    const int* __restrict__ state_slot, float* __restrict__ prep,
                                    int PW, int H, int G, int d, int dp, int dv, int taps,
-                                   float unit_eps, int head_decay) {
+                                   float unit_eps, int head_decay, int round) {
     extern __shared__ float act[];                 // [C], then [H] decays per head
     const int n = blockIdx.x;
     const int r = token_req[n];
@@ -81,7 +86,7 @@ __global__ void gdr_prepare_kernel(const float* __restrict__ proj, int P,
                                     : conv_state[(size_t)(taps - 1 + (m - t0)) * C + c];
             acc += filt[(size_t)c * taps + j] * x;
         }
-        act[c] = acc * gd_sigmoid(acc);
+        act[c] = round ? __bfloat162float(__float2bfloat16_rn(acc / (1.f + expf(-acc)))) : acc * gd_sigmoid(acc);
     }
     if (head_decay)
         for (int h = threadIdx.x; h < H; h += blockDim.x)
@@ -553,13 +558,24 @@ static bool gd_shape(int d, int* R, int* P) {
     return false;
 }
 
-// Floats of a row of the scratch `prep`, and of the whole scratch for n tokens (prep, then
-// the raw read-outs [n, H dv]).
-extern "C" long long rv_gated_delta_scratch(int n_tokens, int H, int G, int d, int dv) {
+// Whether the portions of a step take the chunk form: where they are long enough on average that
+// chunks of 64 are not mostly filling.
+static bool gd_chunked(int n_tokens, int n_decode, int n_reqs, int H, int G, int d, int dv, int chunks) {
+    const int tokens = n_tokens - n_decode, reqs = n_reqs - n_decode;
+    return chunks && gc_sizes_ok(H, G, d, dv) && reqs > 0 && tokens >= 24LL * reqs && tokens <= 65535 * CS_TOKENS;
+}
+
+// Floats of a row of the scratch `prep`, and of the whole scratch for n tokens: the raw read-outs
+// [n, H dv], then prep, then the chunk form's.
+extern "C" long long rv_gated_delta_scratch(int n_tokens, int n_decode, int n_reqs, int H, int G, int d, int dv,
+                                            int chunks) {
     int R = 0, P = 0;
     if (!gd_shape(d, &R, &P)) return -1;
     const long long pw = (long long)(2 * G + H) * R * P + gd_pad4(H * dv) + gd_pad4(H) + gd_pad4(G);
-    return (long long)n_tokens * (pw + (long long)H * dv);
+    const long long o = ((long long)n_tokens * H * dv + 3) & ~3LL;
+    if (!gd_chunked(n_tokens, n_decode, n_reqs, H, G, d, dv, chunks)) return o + n_tokens * pw;
+    return o + n_decode * pw +
+           gc_layout(n_tokens, la_items(n_tokens - n_decode, n_reqs - n_decode), H, d, dv, 2 * G * d + H * dv).total;
 }
 
 template <int R, int P>
@@ -604,16 +620,18 @@ static void gd_launch_scan(const float* prep, int PW, float* state, long long re
 // proj [N, P] float32 (P >= C + H); lowrank [N, LW] float32 (H d, with head_decay H, of the decays'
 // pre-activations, then H dv of the output gates'; LW is the stride of its rows, which may lie
 // inside proj's); filt [C, taps]; a_log [H]; dt_bias [H d] or [H]; norm_w
-// [dv]; state [slots, record]; scratch: rv_gated_delta_scratch floats; y [N, H dv].
+// [dv]; state [slots, record]; scratch: rv_gated_delta_scratch floats, 16-byte aligned; y [N, H dv].
+// Requests [0, n_decode) bring one token each.  `chunks` (with head_decay and bfloat16 y): the others'
+// portions may take the chunk form.
 extern "C" int rv_gated_delta(const float* proj, int P, const float* lowrank, int LW,
                               const float* filt, const float* a_log, const float* dt_bias,
                               const float* norm_w, float* state, const int* token_req,
                               const int* q_start, const int* state_slot, float* scratch, void* y,
-                              int out_dtype, int n_tokens, int n_reqs, int H, int G, int d, int dv,
-                              int taps, float unit_eps, float eps, int head_decay, int silu_gate,
-                              void* stream) {
+                              int out_dtype, int n_tokens, int n_decode, int n_reqs, int H, int G, int d,
+                              int dv, int taps, float unit_eps, float eps, int head_decay, int silu_gate,
+                              int chunks, void* stream) {
     if (n_tokens == 0 || n_reqs == 0) return 0;
-    if (n_tokens < 0 || n_reqs < 0 || H < 1 || G < 1 || H % G || d < 1 || dv < 1 || taps < 1)
+    if (n_decode < 0 || n_decode > n_reqs || n_decode > n_tokens || n_tokens < 0 || n_reqs < 0 || H < 1 || G < 1 || H % G || d < 1 || dv < 1 || taps < 1)
         RV_FAIL("gated_delta: bad sizes");
     const int C = 2 * G * d + H * dv;
     const int n_decays = head_decay ? H : H * d;
@@ -627,34 +645,46 @@ extern "C" int rv_gated_delta(const float* proj, int P, const float* lowrank, in
     const long long rec = rv_gated_delta_record(H, G, d, dv, taps);
     const size_t smem1 = (size_t)(C + (head_decay ? H : 0)) * sizeof(float);
     if (smem1 > 200 * 1024) RV_FAIL("gated_delta: %d channels do not fit shared memory", C);
-    float* prep = scratch;
-    float* o = scratch + (size_t)n_tokens * PW;
+    if ((uintptr_t)scratch & 15) RV_FAIL("gated_delta: the scratch must be 16-byte aligned");
+    float* o = scratch;
+    float* prep = scratch + (((size_t)n_tokens * H * dv + 3) & ~(size_t)3);
     cudaStream_t s = (cudaStream_t)stream;
+    chunks = chunks && head_decay && out_dtype == RV_DTYPE_BF16;
+    const bool chunked = gd_chunked(n_tokens, n_decode, n_reqs, H, G, d, dv, chunks);
+    if (chunked) {
+        const GcArgs g = {proj, lowrank, a_log, dt_bias, nullptr, q_start, state_slot, P, LW, C, n_decode, n_reqs, H,
+                          G, d, dv, unit_eps, nullptr, nullptr, nullptr, nullptr, nullptr};
+        if (gc_run(g, filt, state, rec, taps, token_req, n_decode, n_tokens, prep + (size_t)n_decode * PW, o, s)) return 1;
+    }
+    // what is left to the token-by-token form: everything, or the single tokens
+    const int n_tok = chunked ? n_decode : n_tokens, n_req = chunked ? n_decode : n_reqs;
+    if (n_tok > 0) {
     if (smem1 > 48 * 1024)
         cudaFuncSetAttribute(gdr_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
-    rv_launch(gdr_prepare_kernel, dim3(n_tokens), dim3(256), smem1, s, proj, P, lowrank, LW, filt, a_log,
+    rv_launch(gdr_prepare_kernel, dim3(n_tok), dim3(256), smem1, s, proj, P, lowrank, LW, filt, a_log,
               dt_bias, (const float*)state, rec, token_req, q_start, state_slot, prep, PW, H, G, d, dp, dv,
-              taps, unit_eps, head_decay);
+              taps, unit_eps, head_decay, chunks && gc_sizes_ok(H, G, d, dv));
     RV_CHECK_LAUNCH("gated_delta prepare");
     // the staging buffers are sized for the longest portion the step can have if every request
     // brings a token; the size changes only how often the scan's blocks meet, not what they compute
-    const int longest = n_tokens - n_reqs + 1 > 1 ? n_tokens - n_reqs + 1 : 1;
+    const int longest = n_tok - n_req + 1 > 1 ? n_tok - n_req + 1 : 1;
     if (longest == 1) {
 #define GD_CASE(r_, p_)                                                                                \
     if (R == r_ && TP == p_)                                                                           \
-        gd_launch_single<r_, p_>(prep, PW, state, rec, q_start, state_slot, o, n_reqs, H, G, d, dv, taps, s);
+        gd_launch_single<r_, p_>(prep, PW, state, rec, q_start, state_slot, o, n_req, H, G, d, dv, taps, s);
         GD_CASE(8, 1) GD_CASE(8, 2) GD_CASE(8, 4) GD_CASE(8, 8) GD_CASE(8, 16) GD_CASE(8, 32) GD_CASE(16, 32)
         GD_CASE(32, 32)
 #undef GD_CASE
     } else {
 #define GD_CASE(r_, p_)                                                                                \
     if (R == r_ && TP == p_)                                                                           \
-        gd_launch_scan<r_, p_>(prep, PW, state, rec, q_start, state_slot, o, n_reqs, longest, H, G, d, dv, taps, s);
+        gd_launch_scan<r_, p_>(prep, PW, state, rec, q_start, state_slot, o, n_req, longest, H, G, d, dv, taps, s);
         GD_CASE(8, 1) GD_CASE(8, 2) GD_CASE(8, 4) GD_CASE(8, 8) GD_CASE(8, 16) GD_CASE(8, 32) GD_CASE(16, 32)
         GD_CASE(32, 32)
 #undef GD_CASE
     }
     RV_CHECK_LAUNCH("gated_delta scan");
+    }
     RV_DISPATCH_DTYPE(out_dtype, "gated_delta", {
         rv_launch(gdr_finish_kernel<T>, dim3(n_tokens + n_reqs), dim3(128), 0, s, (const float*)o, proj, P,
                   lowrank, LW, norm_w, state, rec, token_req, q_start, state_slot, (T*)y, n_tokens, H, G, d,

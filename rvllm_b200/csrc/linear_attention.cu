@@ -42,8 +42,8 @@
 // Plain reference: tests/plain_ops.py linear_attention.
 #include "common.cuh"
 #include "mma_bf16.cuh"
+#include "chunks.cuh"
 
-#define LA_C 64             // tokens a chunk
 #define LA_T 64             // columns (and rows) of a tile
 #define LA_DK 32            // key channels staged at a time in `out`
 #define LA_LD 68            // padded row of 64
@@ -67,8 +67,6 @@ struct LaToken {
     const double* B;
     const float* w;
 };
-__device__ __forceinline__ float la_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
-
 __device__ __forceinline__ float la_logsigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float la_silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 // a projection as the recurrence reads it
@@ -76,34 +74,6 @@ __device__ __forceinline__ float la_in(const float* p, int act) { return act ? *
 __device__ __forceinline__ float la_in(const bf16* p, int act) {
     const float x = __bfloat162float(*p);
     return act ? __bfloat162float(__float2bfloat16_rn(la_silu(x))) : x;
-}
-
-// Chunk `item` of the portions of requests [first_req, n_reqs): its request and its number there;
-// and how many chunks lie before the request.  Requests without a slot have none.  Whole warp.
-__device__ __forceinline__ int la_chunks(const int* q_start, const int* state_slot, int r) {
-    return state_slot[r] < 0 ? 0 : (q_start[r + 1] - q_start[r] + LA_C - 1) / LA_C;
-}
-__device__ __forceinline__ bool la_find(const int* q_start, const int* state_slot, int first_req,
-                                        int n_reqs, int item, int lane, int& r, int& before) {
-    before = 0;
-    for (int base = first_req; base < n_reqs; base += 32) {
-        const int n = base + lane < n_reqs ? la_chunks(q_start, state_slot, base + lane) : 0;
-        int incl = n;
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const int up = __shfl_up_sync(0xffffffffu, incl, o);
-            if (lane >= o) incl += up;
-        }
-        const unsigned hit = __ballot_sync(0xffffffffu, before + incl > item);
-        if (hit) {
-            const int l = __ffs(hit) - 1;
-            r = base + l;
-            before += __shfl_sync(0xffffffffu, incl - n, l);
-            return true;
-        }
-        before += __shfl_sync(0xffffffffu, incl, 31);
-    }
-    return false;
 }
 
 // ---- single tokens ---------------------------------------------------------------------
@@ -608,34 +578,6 @@ __device__ __forceinline__ float la_gate(float g, int gate) {
     return (gate ? g : 1.f) / (1.f + expf(-g));                  // 0: sigmoid, 1: silu
 }
 
-// Four neighbouring values (16- and 8-byte accesses) or one.
-template <typename T, int V>
-__device__ __forceinline__ void la_load(const T* p, float (&x)[V]) {
-    if (V == 4 && sizeof(T) == 4) {
-        const float4 f = *(const float4*)p;
-        x[0] = f.x; x[1 % V] = f.y; x[2 % V] = f.z; x[3 % V] = f.w;
-    } else if (V == 4) {
-        const uint2 u = *(const uint2*)p;
-        const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&u.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&u.y);
-        x[0] = a.x; x[1 % V] = a.y; x[2 % V] = b.x; x[3 % V] = b.y;
-    } else {
-        x[0] = rv_load(p);
-    }
-}
-template <typename T, int V>
-__device__ __forceinline__ void la_store(T* p, const float (&x)[V]) {
-    if (V == 4 && sizeof(T) == 4) {
-        *(float4*)p = make_float4(x[0], x[1 % V], x[2 % V], x[3 % V]);
-    } else if (V == 4) {
-        const __nv_bfloat162 a = __floats2bfloat162_rn(x[0], x[1 % V]), b = __floats2bfloat162_rn(x[2 % V], x[3 % V]);
-        uint2 u;
-        u.x = *(const unsigned*)&a;
-        u.y = *(const unsigned*)&b;
-        *(uint2*)p = u;
-    } else {
-        rv_store(p, x[0]);
-    }
-}
 template <typename T, int V>
 __device__ __forceinline__ void la_finish_at(const float* nm, const T* g, const float* w, T* o, int c, float inv, int gate) {
     float x[V], y[V], z[V];
@@ -710,9 +652,6 @@ __global__ void la_finish_head_kernel(const float* __restrict__ num, const T* __
 #include "linear_attention_mma.cuh"
 
 // ---------------------------------------------------------------------------------
-// The most chunks the portions of `n_tokens` tokens in `n_reqs` requests can have.
-static long long la_items(int n_tokens, int n_reqs) { return (long long)n_tokens / LA_C + n_reqs; }
-
 // Floats of scratch: num [n, H, dv]; for portions kv [items, H, d, dv] and dec [items, H, d].
 extern "C" long long rv_linear_attention_scratch(int n_tokens, int n_decode, int n_reqs, int H, int d,
                                                  int dv) {

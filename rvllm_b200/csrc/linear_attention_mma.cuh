@@ -4,20 +4,6 @@
 
 #define LM_LD 72            // padded row of 64 bfloat16 columns
 
-// The pair (x, y) as three pairs of bfloat16 whose sum it is.
-__device__ __forceinline__ void lm_split(float x, float y, unsigned& a, unsigned& b, unsigned& c) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-    const float2 hf = __bfloat1622float2(h);
-    x -= hf.x;
-    y -= hf.y;
-    const __nv_bfloat162 m = __floats2bfloat162_rn(x, y);
-    const float2 mf = __bfloat1622float2(m);
-    const __nv_bfloat162 l = __floats2bfloat162_rn(x - mf.x, y - mf.y);
-    a = *(const unsigned*)&h;
-    b = *(const unsigned*)&m;
-    c = *(const unsigned*)&l;
-}
-__device__ __forceinline__ float2 lm_pair(unsigned u) { return __bfloat1622float2(*(const __nv_bfloat162*)&u); }
 __device__ __forceinline__ unsigned lm_silu2(unsigned u) {
     const float2 f = lm_pair(u);
     const __nv_bfloat162 r = __floats2bfloat162_rn(la_silu(f.x), la_silu(f.y));
@@ -33,19 +19,6 @@ __device__ __forceinline__ uint4 lm_in8(const bf16* p, bool there, int act) {
         v.w = lm_silu2(v.w);
     }
     return v;
-}
-// Where a chunk lies: first token and token count (0: no such chunk).  Whole block.
-__device__ __forceinline__ void lm_locate(const int* q_start, const int* state_slot, int first_req,
-                                          int n_reqs, int item, int* at) {
-    if (threadIdx.x < 32) {
-        int r = -1, before = 0;
-        const bool ok = la_find(q_start, state_slot, first_req, n_reqs, item, threadIdx.x, r, before);
-        if (threadIdx.x == 0) {
-            at[0] = ok ? q_start[r] + (item - before) * LA_C : -1;
-            at[1] = ok ? min(LA_C, q_start[r + 1] - at[0]) : 0;
-        }
-    }
-    __syncthreads();
 }
 __device__ __forceinline__ float lm_exp2(float x) {
     float y;

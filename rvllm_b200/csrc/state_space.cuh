@@ -8,11 +8,8 @@
 // B and C are shared by the heads of a group.
 //
 //   proj [n, P] float32: z [H dv] | x [H dv] | B [G N] | C [G N] | t [H] | anything else
-//   ss_conv    x, B and C pass a causal convolution over time per channel (filter [C, taps], last
-//              column the current token's, bias [C]; inputs before a request's first token of the
-//              step come from its record, [taps-1][C] oldest first) and silu -> rows [n, C] of the
-//              compute type.  A thread has some channels of eight tokens, whose inputs it requests
-//              together (of one token, where they are few).
+//   conv_silu  x, B and C pass the convolution and silu -> rows [n, C] of the compute type
+//              (conv_silu.cuh; records [taps-1][C])
 //   ss_decay   dt of every token of a portion, and the sums of the log decays of its chunk's tokens
 //              up to it (float64), once per chunk and head
 //   state, scan, out / token: linear_attention.cu with LA_TOKEN
@@ -20,96 +17,7 @@
 //              the convolution's inputs move on (the last taps-1 of old record | this step's rows)
 // Plain reference: tests/plain_ops.py state_space.
 #pragma once
-
-#define SS_TOKENS 8         // tokens a thread of ss_conv takes where there are many
-
-template <int V>
-__device__ __forceinline__ void ss_load(const float* p, float (&x)[V]) {
-    if (V == 4) {
-        const float4 f = *(const float4*)p;
-        x[0] = f.x; x[1 % V] = f.y; x[2 % V] = f.z; x[3 % V] = f.w;
-    } else {
-        x[0] = *p;
-    }
-}
-
-// TAPS 0: any number, `taps`.
-template <typename T, int TAPS, int TT, int V>
-__global__ void __launch_bounds__(128) ss_conv_kernel(
-    const float* __restrict__ proj, int P, int off, const float* __restrict__ filt,
-    const float* __restrict__ bias, const float* __restrict__ conv_state,
-    const int* __restrict__ token_req, const int* __restrict__ q_start,
-    const int* __restrict__ state_slot, T* __restrict__ out, int n_tokens, int C, int taps_any) {
-    rv_pdl_launch_dependents();
-    const int taps = TAPS ? TAPS : taps_any;
-    const int c = (blockIdx.x * 128 + threadIdx.x) * V;
-    const int first = blockIdx.y * TT;
-    constexpr int KT = TAPS ? TAPS : 1;
-    float w[KT][V], b[V];
-    if (c < C) {
-#pragma unroll
-        for (int e = 0; e < V; ++e) {
-            b[e] = bias[c + e];
-            if (TAPS)
-#pragma unroll
-                for (int j = 0; j < KT; ++j) w[j][e] = filt[(size_t)(c + e) * TAPS + j];
-        }
-    }
-    rv_pdl_wait();
-    if (c >= C) return;
-    // input `m` of the request whose first token is t0 (m < t0: from its record)
-    auto input = [&](int m, int t0, int slot, float (&x)[V]) {
-        if (m >= t0) ss_load<V>(proj + (size_t)m * P + off + c, x);
-        else ss_load<V>(conv_state + ((size_t)slot * (taps - 1) + (taps - 1 + m - t0)) * C + c, x);
-    };
-    float x[TT][V];
-#pragma unroll
-    for (int i = 0; i < TT; ++i)
-        if (first + i < n_tokens) ss_load<V>(proj + (size_t)(first + i) * P + off + c, x[i]);
-    float before[KT > 1 ? KT - 1 : 1][V];                // the taps-1 inputs before the token
-    int held = -1;                                       // the request they belong to
-#pragma unroll
-    for (int i = 0; i < TT; ++i) {
-        const int t = first + i;
-        if (t >= n_tokens) break;
-        const int r = token_req[t];
-        const int slot = state_slot[r];
-        if (slot < 0) continue;
-        const int t0 = q_start[r];
-        float acc[V];
-#pragma unroll
-        for (int e = 0; e < V; ++e) acc[e] = 0.f;
-        if (TAPS) {
-            if (r != held) {
-#pragma unroll
-                for (int j = 0; j < KT - 1; ++j) input(t - (KT - 1) + j, t0, slot, before[j]);
-                held = r;
-            }
-#pragma unroll
-            for (int e = 0; e < V; ++e) {
-#pragma unroll
-                for (int j = 0; j < KT - 1; ++j) acc[e] = fmaf(w[j][e], before[j][e], acc[e]);
-                acc[e] = fmaf(w[KT - 1][e], x[i][e], acc[e]);
-#pragma unroll
-                for (int j = 0; j + 1 < KT - 1; ++j) before[j][e] = before[j + 1][e];
-                if (KT > 1) before[KT > 1 ? KT - 2 : 0][e] = x[i][e];
-            }
-        } else {
-            for (int j = 0; j < taps; ++j) {
-                float xj[V];
-                input(t - (taps - 1 - j), t0, slot, xj);
-#pragma unroll
-                for (int e = 0; e < V; ++e) acc[e] = fmaf(filt[(size_t)(c + e) * taps + j], xj[e], acc[e]);
-            }
-        }
-#pragma unroll
-        for (int e = 0; e < V; ++e) {
-            acc[e] += b[e];
-            acc[e] = acc[e] / (1.f + expf(-acc[e]));
-        }
-        la_store<T, V>(out + (size_t)t * C + c, acc);
-    }
-}
+#include "conv_silu.cuh"
 
 // A warp has eight tokens of 32 heads.
 __global__ void __launch_bounds__(256) ss_decay_kernel(
@@ -238,20 +146,6 @@ extern "C" long long rv_state_space_scratch(int n_tokens, int n_decode, int n_re
     return ss_layout(n_tokens, n_decode, n_reqs, H, dv, N, G, dtype == RV_DTYPE_BF16 ? 2 : 4).total;
 }
 
-template <typename T, int TT, int V>
-static void ss_conv_launch(const float* proj, int P, int off, const float* filt, const float* bias,
-                           const float* conv_state, const LaArgs& a, T* rows, int C, int taps, cudaStream_t s) {
-    const dim3 grid((C / V + 127) / 128, (a.n_tokens + TT - 1) / TT);
-#define SS_CONV(K)                                                                                        \
-    rv_launch(ss_conv_kernel<T, K, TT, V>, grid, dim3(128), 0, s, proj, P, off, filt, bias, conv_state,   \
-              a.token_req, a.q_start, a.state_slot, rows, a.n_tokens, C, taps)
-    if (taps == 2) SS_CONV(2);
-    else if (taps == 3) SS_CONV(3);
-    else if (taps == 4) SS_CONV(4);
-    else SS_CONV(0);
-#undef SS_CONV
-}
-
 template <typename T>
 static int ss_run(const float* proj, int P, const float* filt, const float* conv_bias, const float* D,
                   float* conv_state, LaArgs a, const SsScratch& lay, T* out, int G, int taps, int norm_groups,
@@ -259,13 +153,9 @@ static int ss_run(const float* proj, int P, const float* filt, const float* conv
     const int inner = a.H * a.dv, C = inner + 2 * G * a.d;
     float* num = a.scratch + lay.num;
     T* rows = (T*)(a.scratch + lay.rows);
-    const bool v4 = C % 4 == 0 && P % 4 == 0 && inner % 4 == 0 &&
-                    (((uintptr_t)proj | (uintptr_t)conv_state | (uintptr_t)rows) & 15) == 0;
-    const bool few = (long long)a.n_tokens * ((C + 511) / 512) < 4 * rv_sm_count();
-    if (v4 && few) ss_conv_launch<T, 1, 4>(proj, P, inner, filt, conv_bias, conv_state, a, rows, C, taps, s);
-    else if (v4) ss_conv_launch<T, SS_TOKENS, 4>(proj, P, inner, filt, conv_bias, conv_state, a, rows, C, taps, s);
-    else if (few) ss_conv_launch<T, 1, 1>(proj, P, inner, filt, conv_bias, conv_state, a, rows, C, taps, s);
-    else ss_conv_launch<T, SS_TOKENS, 1>(proj, P, inner, filt, conv_bias, conv_state, a, rows, C, taps, s);
+    const ConvSilu conv = {proj, filt, conv_bias, conv_state, (long long)(taps - 1) * C, a.token_req, a.q_start,
+                           a.state_slot, P, inner, 0, a.n_tokens, C, taps};
+    conv_silu<T>(conv, rows, s);
     RV_CHECK_LAUNCH("state_space_conv");
     if (a.n_decode > 0 && la_tokens<T, true>((const T*)rows, a, num, s)) return 1;
     if (a.n_tokens > a.n_decode && a.n_reqs > a.n_decode) {
@@ -319,7 +209,7 @@ extern "C" int rv_state_space(const float* proj, int P, const float* filt, const
     if (P < inner + C + H) RV_FAIL("state_space: rows are too short");
     const int tiles_d = (N + LA_T - 1) / LA_T, tiles_v = (dv + LA_T - 1) / LA_T;
     if (n_reqs > 65535 || H > 65535 || N > 2048 || dv > 65535 || tiles_d * tiles_v > 65535 ||
-        norm_groups > 65535 || n_tokens > 65535 * SS_TOKENS)
+        norm_groups > 65535 || n_tokens > 65535 * CS_TOKENS)
         RV_FAIL("state_space: too many tokens, requests or heads, or heads that are too large");
     if (((uintptr_t)scratch & 15) || (taps > 1 && !conv_state))
         RV_FAIL("state_space: the scratch must be 16-byte aligned, and the convolution needs its records");

@@ -99,6 +99,9 @@ class CudaOps:
         # portions of bfloat16 linear attention: "tensor" = tensor-core kernels where the sizes allow
         # (head sizes in multiples of 16, keys up to 128), "simt" = float32 arithmetic
         self.linear_attention_mode = os.environ.get("RVLLM_LINEAR_ATTENTION", "tensor")
+        # portions of bfloat16 delta rules with a decay per head: "chunks" = the chunk form on the
+        # tensor cores where the sizes allow, "tokens" = token by token
+        self.gated_delta_mode = os.environ.get("RVLLM_GATED_DELTA", "chunks")
         # float32 products must be float32: no TF32, no reduced-precision accumulation
         torch.backends.cuda.matmul.allow_tf32 = False
         torch.backends.cudnn.allow_tf32 = False
@@ -1345,8 +1348,11 @@ class CudaOps:
         if lowrank.shape[0] != n or lowrank.shape[1] < decays + heads * vdim or \
                 dt_bias.numel() != decays:
             raise KernelError("gated_delta: the decay and gate rows have another size")
-        need = self.lib.rv_gated_delta_scratch(c_int(n), c_int(heads), c_int(kv_heads), c_int(dim),
-                                               c_int(vdim))
+        chunks = int(head_decay and out.dtype == torch.bfloat16 and self.gated_delta_mode == "chunks")
+        single = ctx.n_decode if chunks else 0       # the token-by-token form takes them as any others
+        need = self.lib.rv_gated_delta_scratch(c_int(n), c_int(single), c_int(ctx.n_reqs),
+                                               c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim),
+                                               c_int(chunks))
         if need < 0:
             raise KernelError(f"gated_delta: key heads of {dim} are not supported")
         scratch = torch.empty((need,), dtype=torch.float32, device=proj.device)
@@ -1354,10 +1360,11 @@ class CudaOps:
             _ptr(proj), c_int(proj.shape[1]), _ptr(lowrank), c_int(lowrank.stride(0)), _ptr(filt),
             _ptr(a_log), _ptr(dt_bias), _ptr(norm_w), _ptr(state), _ptr(ctx.token_req),
             _ptr(ctx.q_start), _ptr(ctx.state_slot), _ptr(scratch), _ptr(out), _code(out.dtype),
-            c_int(n), c_int(ctx.n_reqs), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim),
-            c_int(taps), c_float(unit_eps), c_float(eps), c_int(1 if head_decay else 0),
-            c_int({"sigmoid": 0, "silu": 1}[gate]), self._stream()), "gated_delta")
-        self.launches += 3
+            c_int(n), c_int(single), c_int(ctx.n_reqs), c_int(heads), c_int(kv_heads),
+            c_int(dim), c_int(vdim), c_int(taps), c_float(unit_eps), c_float(eps),
+            c_int(1 if head_decay else 0), c_int({"sigmoid": 0, "silu": 1}[gate]), c_int(chunks),
+            self._stream()), "gated_delta")
+        self.launches += 3 + chunks
 
     # ---- clamped gated activation ----------------------------------------------------------
 

@@ -103,7 +103,11 @@ class GatedDelta(Mixer):
         H, G, d, dv = spec.num_heads, spec.num_kv_heads, spec.head_dim, spec.v_head_dim
         self.channels = 2 * G * d + H * dv
         if spec.decay == "head":
-            self.w_in = cat(("q", "k", "v", "b", "a", "g"))
+            w_in = cat(("q", "k", "v", "b", "a", "g"))
+            fill = -w_in.shape[0] % 8                  # zero rows, so that the product's rows stay aligned
+            if fill:
+                w_in = torch.cat([w_in, torch.zeros((fill, spec.hidden), dtype=q.dtype, device=q.device)])
+            self.w_in = w_in.contiguous()
         else:
             self.w_in = cat(("q", "k", "v", "b"))
             self.w_low = cat(("a1", "g1"))

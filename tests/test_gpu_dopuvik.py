@@ -365,10 +365,18 @@ def _delta(gen, H, G, d, dvv, taps, strong=False):
     return m, C, t, rows
 
 
-def _delta_plain(m, C, t, rows, silu_gate=True, unit=1e-6, eps=1e-5):
+def _delta_rounds(ops, dtype, m, C):
+    """Whether activated rows are bfloat16 (sizes that the chunk form takes)."""
+    return dtype == torch.bfloat16 and ops.gated_delta_mode == "chunks" and m["dim"] % 16 == 0 and \
+        m["dim"] <= 128 and m["vdim"] % 16 == 0 and C % 8 == 0
+
+
+def _delta_plain(m, C, t, rows, silu_gate=True, rounded=False, unit=1e-6, eps=1e-5):
     H, G, d, dvv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     T = rows.shape[0]
     x = plain.silu(plain.causal_conv(rows[:, :C], t["filt"]))
+    if rounded:
+        x = torch.from_numpy(x).to(torch.bfloat16).double().numpy()
     q, k, v = np.split(x, [G * d, 2 * G * d], axis=1)
     u = lambda y: y / np.sqrt((y ** 2).sum(-1, keepdims=True) + unit)
     q = np.repeat(u(q.reshape(T, G, d)) * d ** -0.5, H // G, axis=1)
@@ -382,12 +390,16 @@ def _delta_plain(m, C, t, rows, silu_gate=True, unit=1e-6, eps=1e-5):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("sizes", [(4, 2, 24, 16, 4), (2, 2, 16, 40, 2), (3, 1, 40, 8, 1), (3, 3, 6, 5, 3),
-                                   (2, 1, 128, 64, 4), (4, 2, 64, 32, 3), (2, 2, 64, 128, 4), (1, 1, 130, 33, 2)])
+                                   (2, 1, 128, 64, 4), (4, 2, 64, 32, 3), (2, 2, 64, 128, 4), (1, 1, 130, 33, 2),
+                                   (2, 1, 112, 80, 2)])
 @pytest.mark.parametrize("strong", [False, True])
-def test_delta_rule_with_a_decay_per_head(ops, dtype, sizes, strong):
+@pytest.mark.parametrize("mode", ["chunks", "tokens"])
+def test_delta_rule_with_a_decay_per_head(ops, monkeypatch, dtype, sizes, strong, mode):
     """Four requests of unequal length in portions of unequal size, one of them token by token, in
-    state slots that are not in order; decays from nearly none to nearly all."""
+    state slots that are not in order; decays from nearly none to nearly all; in chunks on the
+    tensor cores where these take the sizes, and token by token."""
     H, G, d, dvv, taps = sizes
+    monkeypatch.setattr(ops, "gated_delta_mode", mode)
     gen = torch.Generator().manual_seed(d + dvv)
     m, C, t, rows = _delta(gen, H, G, d, dvv, taps, strong)
     rec = ops.gated_delta_record(H, G, d, dvv, taps)
@@ -405,10 +417,12 @@ def test_delta_rule_with_a_decay_per_head(ops, dtype, sizes, strong):
 
         got = _feed(LENGTHS, CUTS, SLOTS, run, rows, C + 2 * H + H * dvv)
         for r in LENGTHS:
-            want, S = _delta_plain(m, C, t, rows[r], silu_gate)
+            rounded = _delta_rounds(ops, dtype, m, C)
+            want, S = _delta_plain(m, C, t, rows[r], silu_gate, rounded)
             close(got[r], want, dtype, bound=4e-5 if dtype == torch.float32 else None)
             rows_of = state[SLOTS[r]][(taps - 1) * C:].reshape(H, dvv, d).transpose(1, 2)
-            close(rows_of, S, torch.float32, bound=4e-5)
+            # (a value on the way between two bfloat16 numbers may round the other way)
+            close(rows_of, S, torch.float32, bound=2e-3 if rounded else 4e-5)
             if taps > 1:
                 old = np.concatenate([np.zeros((taps - 1, C)), rows[r][:, :C]])[-(taps - 1):]
                 close(state[SLOTS[r]][:(taps - 1) * C], old.reshape(-1), torch.float32)
@@ -527,7 +541,7 @@ def test_an_early_token_among_hundreds_is_not_lost(ops, dtype, which):
         rows[3, C:C + H] = 8.0                                # ... but this one all of its large value
         rows[3, 2 * 64:C] *= 100.0
         rows[-1, :64] = rows[3, 64:128]                       # and the last query points at its key
-        want, _ = _delta_plain(m, C, t, rows)
+        want, _ = _delta_plain(m, C, t, rows, rounded=_delta_rounds(ops, dtype, m, C))
         other = rows.copy()
         other[3, C:C + H] = -30.0
         assert np.abs(_delta_plain(m, C, t, other)[0][-1] - want[-1]).max() > 0.1
@@ -551,6 +565,35 @@ def test_an_early_token_among_hundreds_is_not_lost(ops, dtype, which):
             outs.append(run(rows[at:at + c], ctx).cpu())
             at += c
         close(torch.cat(outs), want, dtype, bound=1e-4 if dtype == torch.float32 else None)
+
+
+@pytest.mark.parametrize("sizes", [(3, 1, 64, 32, 4), (3, 3, 16, 16, 1)])
+def test_delta_rule_decays_from_nothing_to_one(ops, sizes):
+    """Heads that forget all with some tokens and nothing with others, and keys that repeat (the
+    corrections then depend on one another through the whole chunk): chunks equal the
+    token-by-token definition whatever the cut."""
+    H, G, d, dvv, taps = sizes
+    gen = torch.Generator().manual_seed(8)
+    m, C, t, _ = _delta(gen, H, G, d, dvv, taps)
+    t["A_log"], t["dt_bias"] = np.array([6.0, -8.0, 0.0]), np.array([-12.0, 3.0, 0.0])
+    n = 400
+    rows = rnd(gen, torch.float32, n, C + 2 * H + H * dvv).numpy()
+    rows[::37, C + H:C + 2 * H] += 30.0                       # now and then a token that clears the state
+    rows[100:180, G * d:2 * G * d] = rows[100, G * d:2 * G * d]            # one key, eighty times
+    rows[100:180:2, C:C + H] = 12.0                           # written whole
+    want, S = _delta_plain(m, C, t, rows, rounded=True)
+    for cut in ([n], [64, 1, 2, 130] * 2 + [6], [30] * 10 + [1] * 20 + [80]):
+        state, outs, at = torch.zeros(1, ops.gated_delta_record(H, G, d, dvv, taps), device="cuda"), [], 0
+        for c in cut:
+            ctx, _ = step_context([(c, 0)])
+            proj, out = f32(rows[at:at + c]), torch.empty(c, H * dvv, device="cuda", dtype=torch.bfloat16)
+            ops.gated_delta(proj, proj[:, C + H:], f32(t["filt"]), f32(t["A_log"]), f32(t["dt_bias"]), f32(t["norm"]),
+                            state, ctx, out, H, G, d, dvv, taps, 1e-6, 1e-5, head_decay=True, gate="silu")
+            outs.append(out.cpu())
+            at += c
+        assert at == n
+        close(torch.cat(outs), want, torch.bfloat16)
+        close(state[0][(taps - 1) * C:].reshape(H, dvv, d).transpose(1, 2), S, torch.float32, bound=2e-3)
 
 
 # ---- experts and identity experts --------------------------------------------------------------------
