@@ -42,7 +42,7 @@
 //     the same update without the lag: every thread copies its share of the token, reads its
 //     rows meanwhile, and writes them back with the write added.  Small blocks, so that many
 //     fit a multiprocessor: the step is bound by reading and writing every state once.
-//   gdr_finish  (one block per token, and one per request)
+//   gdr_finish  (a warp per token and value head; blocks that move a request's inputs on)
 //     y = o / sqrt(mean_j o^2 + eps) * norm[j] * sigmoid(gate[n, h dv + j]) (or silu), gate being
 //     the columns of lowrank behind the decays'; and the request's convolution inputs move on (the last
 //     taps-1 of old record | this step's rows).
@@ -494,27 +494,27 @@ gdr_single_kernel(const float* __restrict__ prep, int PW, float* __restrict__ st
     }
 }
 
-template <typename TO>
-__global__ void gdr_finish_kernel(const float* __restrict__ o_in, const float* __restrict__ proj,
-                                  int P, const float* __restrict__ lowrank, int LW,
-                                  const float* __restrict__ norm_w, float* __restrict__ state,
-                                  long long rec, const int* __restrict__ token_req,
-                                  const int* __restrict__ q_start,
-                                  const int* __restrict__ state_slot, TO* __restrict__ y,
-                                  int n_tokens, int H, int G, int d, int dv, int taps, float eps,
-                                  int gate_off, int silu_gate) {
+// V = 4: 16-byte accesses.  Blocks of four warps: first one warp per (token, head), then a block per
+// request and 512 channels.
+template <typename TO, int V>
+__global__ void __launch_bounds__(128) gdr_finish_kernel(
+    const float* __restrict__ o_in, const float* __restrict__ proj, int P, const float* __restrict__ lowrank, int LW,
+    const float* __restrict__ norm_w, float* __restrict__ state, long long rec, const int* __restrict__ token_req,
+    const int* __restrict__ q_start, const int* __restrict__ state_slot, TO* __restrict__ y, int n_tokens,
+    int head_blocks, int H, int G, int d, int dv, int taps, float eps, int gate_off, int silu_gate) {
     rv_pdl_launch_dependents();
     const int C = 2 * G * d + H * dv;
-    if ((int)blockIdx.x >= n_tokens) {
+    if ((int)blockIdx.x >= head_blocks) {
         // the convolutions' inputs move on: channel by channel, oldest first, so that what a
         // place receives is read from a later place before that one is overwritten
-        const int r = blockIdx.x - n_tokens;
+        const int parts = (C + 511) / 512, b = blockIdx.x - head_blocks;
+        const int r = b / parts, c_end = min(C, (b - r * parts + 1) * 512);
         const int slot = state_slot[r];
         const int t0 = q_start[r], qlen = q_start[r + 1] - t0;
         if (slot < 0 || qlen <= 0) return;
         rv_pdl_wait();
         float* record = state + (size_t)slot * rec;
-        for (int c = threadIdx.x; c < C; c += blockDim.x)
+        for (int c = (b - r * parts) * 512 + threadIdx.x; c < c_end; c += blockDim.x)
             for (int i = 0; i < taps - 1; ++i) {
                 const int idx = qlen - (taps - 1) + i;     // among this step's rows; negative: older
                 record[(size_t)i * C + c] = idx >= 0 ? proj[(size_t)(t0 + idx) * P + c]
@@ -522,21 +522,31 @@ __global__ void gdr_finish_kernel(const float* __restrict__ o_in, const float* _
             }
         return;
     }
-    const int n = blockIdx.x;
+    const long long w = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+    const int lane = threadIdx.x & 31;
+    if (w >= (long long)n_tokens * H) return;
+    const int n = (int)(w / H), h = (int)(w - (long long)n * H);
     if (state_slot[token_req[n]] < 0) return;
     rv_pdl_wait();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
-    for (int h = warp; h < H; h += nwarps) {
-        const float* o = o_in + (size_t)n * H * dv + (size_t)h * dv;
-        float ss = 0.f;
-        for (int j = lane; j < dv; j += 32) ss += o[j] * o[j];
-        ss = rv_warp_sum(ss);
-        const float inv = 1.f / sqrtf(ss / (float)dv + eps);
-        for (int j = lane; j < dv; j += 32) {
-            const float z = lowrank[(size_t)n * LW + gate_off + h * dv + j];
-            const float gate = silu_gate ? z * gd_sigmoid(z) : gd_sigmoid(z);
-            rv_store(y + (size_t)n * H * dv + h * dv + j, o[j] * inv * norm_w[j] * gate);
-        }
+    const float* o = o_in + ((size_t)n * H + h) * dv;
+    const float* z = lowrank + (size_t)n * LW + gate_off + h * dv;
+    float ss = 0.f;
+    for (int j = lane * V; j < dv; j += 32 * V) {
+        float x[V];
+        la_load<float, V>(o + j, x);
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss += x[e] * x[e];
+    }
+    ss = rv_warp_sum(ss);
+    const float inv = 1.f / sqrtf(ss / (float)dv + eps);
+    for (int j = lane * V; j < dv; j += 32 * V) {
+        float x[V], g[V], nw[V];
+        la_load<float, V>(o + j, x);
+        la_load<float, V>(z + j, g);
+        la_load<float, V>(norm_w + j, nw);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] = x[e] * inv * nw[e] * (silu_gate ? g[e] * gd_sigmoid(g[e]) : gd_sigmoid(g[e]));
+        la_store<TO, V>(y + ((size_t)n * H + h) * dv + j, x);
     }
 }
 
@@ -685,11 +695,20 @@ extern "C" int rv_gated_delta(const float* proj, int P, const float* lowrank, in
     }
     RV_CHECK_LAUNCH("gated_delta scan");
     }
+    const bool vec = dv % 4 == 0 && LW % 4 == 0 && n_decays % 4 == 0 &&
+                     (((uintptr_t)lowrank | (uintptr_t)norm_w | (uintptr_t)y) & 15) == 0;
+    const long long head_blocks = ((long long)n_tokens * H + 3) / 4;
+    const long long blocks = head_blocks + (taps > 1 ? (long long)n_reqs * ((C + 511) / 512) : 0);
+    if (blocks > 0x7fffffffLL) RV_FAIL("gated_delta: too many tokens");
+#define GD_FINISH(V_)                                                                                          \
+    rv_launch(gdr_finish_kernel<T, V_>, dim3((unsigned)blocks), dim3(128), 0, s, (const float*)o, proj, P,     \
+              lowrank, LW, norm_w, state, rec, token_req, q_start, state_slot, (T*)y, n_tokens, (int)head_blocks, \
+              H, G, d, dv, taps, eps, n_decays, silu_gate)
     RV_DISPATCH_DTYPE(out_dtype, "gated_delta", {
-        rv_launch(gdr_finish_kernel<T>, dim3(n_tokens + n_reqs), dim3(128), 0, s, (const float*)o, proj, P,
-                  lowrank, LW, norm_w, state, rec, token_req, q_start, state_slot, (T*)y, n_tokens, H, G, d,
-                  dv, taps, eps, n_decays, silu_gate);
+        if (vec) GD_FINISH(4);
+        else GD_FINISH(1);
     });
+#undef GD_FINISH
     RV_CHECK_LAUNCH("gated_delta finish");
     return 0;
 }

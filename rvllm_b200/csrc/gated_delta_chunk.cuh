@@ -18,7 +18,7 @@
 //   gdc_scan    block per (head, 16 value columns, request): over the chunks one after another, the
 //               three products with S in float32 accumulators; the state before every chunk and U go
 //               out, the last state is the record
-//   gdc_out     block per (chunk, head, 64 value columns): o
+//   gdc_out     block per (chunk, head, 32 value columns): o
 //
 // No factor is ever above 1.  Float32 operands (S, V - .., T, U, the scores) enter the bfloat16
 // products as three parts (chunks.cuh): three products with a bfloat16 operand, the six of nine that
@@ -27,7 +27,8 @@
 #pragma once
 #include "conv_silu.cuh"
 
-#define GC_T 64             // value columns of a block of gdc_out
+#define GC_THREADS 256      // threads of a block of gdc_chunk
+#define GC_T 32             // value columns of a block of gdc_out
 #define GC_COLS 16          // value columns of a block of gdc_scan
 #define GC_LT 72            // padded row of 64 bfloat16
 #define GC_SC 384           // floats of a (chunk, head)'s scalars: rho | sigma | eq | sq | sk | e^(B_L), ...
@@ -61,7 +62,7 @@ __device__ __forceinline__ float gc_norm2(const bf16* p, int d, int sub) {      
     return s;
 }
 
-__global__ void __launch_bounds__(128) gdc_chunk_kernel(const GcArgs g) {
+__global__ void __launch_bounds__(GC_THREADS) gdc_chunk_kernel(const GcArgs g) {
     rv_pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char smraw[];
     const int d = g.d, LK = d + 8;
@@ -78,13 +79,15 @@ __global__ void __launch_bounds__(128) gdc_chunk_kernel(const GcArgs g) {
     rv_pdl_wait();
     if (t0 < 0) return;
     const bf16* base = g.rows + (size_t)t0 * g.C;
-    for (int n = tid; n < 64 * (d >> 3); n += 128) {
+    for (int n = tid; n < 64 * (d >> 3); n += GC_THREADS) {
         const int j = n / (d >> 3), c = (n - j * (d >> 3)) * 8;
         *(uint4*)(ks + j * LK + c) = j < L ? *(const uint4*)(base + (size_t)j * g.C + (g.G + kh) * d + c)
                                            : make_uint4(0, 0, 0, 0);
     }
     // norms: eight lanes a token
-    for (int j = tid >> 3; j < 64; j += 16) {
+    #pragma unroll
+    for (int u = 0; u < 64 * 8 / GC_THREADS; ++u) {
+        const int j = (tid >> 3) + u * (GC_THREADS / 8);
         const bf16* row = base + (size_t)min(j, L - 1) * g.C + kh * d;
         const float nq = gc_norm2(row, d, tid & 7), nk = gc_norm2(row + g.G * d, d, tid & 7);
         if ((tid & 7) == 0) {
@@ -92,7 +95,7 @@ __global__ void __launch_bounds__(128) gdc_chunk_kernel(const GcArgs g) {
             sk[j] = j < L ? 1.f / sqrtf(nk + g.unit_eps) : 0.f;
         }
     }
-    if (warp == 0) {                                      // two tokens a lane
+    if (warp == 7) {                                      // two tokens a lane
         const float rate = expf(g.a_log[h]), bias = g.dt_bias[h];
         double l[2];
 #pragma unroll
@@ -112,35 +115,37 @@ __global__ void __launch_bounds__(128) gdc_chunk_kernel(const GcArgs g) {
         bt[2 * lane] = incl - l[1];
     }
     __syncthreads();
-    // A: a warp has 16 rows
+    // A: two warps have 16 rows, half of the columns each
     {
-        float p[8][4];
+        const int rg = warp >> 1, half = warp & 1;
+        float p[4][4];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) p[i][0] = p[i][1] = p[i][2] = p[i][3] = 0.f;
+        for (int i = 0; i < 4; ++i) p[i][0] = p[i][1] = p[i][2] = p[i][3] = 0.f;
         for (int kk = 0; kk < (d >> 4); ++kk) {
             unsigned a[4];
-            ldmatrix_x4(a, ks + (16 * warp + (lane & 15)) * LK + kk * 16 + (lane >> 4) * 8);
+            ldmatrix_x4(a, ks + (16 * rg + (lane & 15)) * LK + kk * 16 + (lane >> 4) * 8);
 #pragma unroll
-            for (int nb = 0; nb < 4; ++nb) {
-                if (nb > warp) continue;
+            for (int u = 0; u < 2; ++u) {
+                const int nb = 2 * half + u;
+                if (nb > rg) continue;
                 unsigned b[4];
                 ldmatrix_x4(b, ks + (nb * 16 + (lane & 7) + (lane >> 4) * 8) * LK + kk * 16 + ((lane >> 3) & 1) * 8);
-                mma_bf16(p[2 * nb], a, b[0], b[1]);
-                mma_bf16(p[2 * nb + 1], a, b[2], b[3]);
+                mma_bf16(p[2 * u], a, b[0], b[1]);
+                mma_bf16(p[2 * u + 1], a, b[2], b[3]);
             }
         }
 #pragma unroll
-        for (int i = 0; i < 8; ++i)
+        for (int i = 0; i < 4; ++i)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const int r = 16 * warp + (lane >> 2) + (e >> 1) * 8, j = 8 * i + (lane & 3) * 2 + (e & 1);
+                const int r = 16 * rg + (lane >> 2) + (e >> 1) * 8, j = 32 * half + 8 * i + (lane & 3) * 2 + (e & 1);
                 As[r * 65 + j] = j < r ? beta[r] * sk[r] * sk[j] * expf((float)(bt[r] - bt[j])) * p[i][e] : 0.f;
             }
     }
     __syncthreads();
     // The inverse X of I + A.  First its four diagonal blocks of 16, a warp each, two lanes a column:
     // x_i = (i = j) - sum_(j <= m < i) A_im x_m.
-    {
+    if (warp < 4) {
         const int o = 16 * warp, j = lane >> 1, half = lane & 1;
         float x[16];
 #pragma unroll
@@ -155,10 +160,9 @@ __global__ void __launch_bounds__(128) gdc_chunk_kernel(const GcArgs g) {
 #pragma unroll
         for (int i = 0; i < 16; ++i)
             if ((i & 1) == half) Xs[(o + i) * 65 + o + j] = x[i];
-        for (int n = lane; n < 16 * 64; n += 32) {        // the rest of these rows
-            const int c = n & 63;
-            if ((c >> 4) != warp) Xs[(o + (n >> 6)) * 65 + c] = 0.f;
-        }
+    } else {                                              // beside the blocks: zeros
+        for (int n = tid - 128; n < 64 * 64; n += GC_THREADS - 128)
+            if (((n >> 4) & 3) != (n >> 10)) Xs[(n >> 6) * 65 + (n & 63)] = 0.f;
     }
     __syncthreads();
     // Then pairs of blocks of 16, and the pair of 32: X_21 = -X_22 (A_21 X_11); the inner product goes
@@ -166,12 +170,12 @@ __global__ void __launch_bounds__(128) gdc_chunk_kernel(const GcArgs g) {
 #pragma unroll
     for (int w = 16; w <= 32; w <<= 1) {
         const int per = w * w, pairs = 32 / w;            // outputs of a pair; pairs
-        constexpr int MAXO = 8;                           // 32 * 32 / 128
+        constexpr int MAXO = 32 * 32 / GC_THREADS;
         float tmp[MAXO];
         for (int pass = 0; pass < 2; ++pass) {
 #pragma unroll
             for (int u = 0; u < MAXO; ++u) {
-                const int n = tid + 128 * u;
+                const int n = tid + GC_THREADS * u;
                 if (n >= pairs * per) continue;
                 const int q = n / per, e = n - q * per, i = e / w, j = e - i * w, o = 2 * q * w;
                 float s = 0.f;
@@ -188,7 +192,7 @@ __global__ void __launch_bounds__(128) gdc_chunk_kernel(const GcArgs g) {
             __syncthreads();
 #pragma unroll
             for (int u = 0; u < MAXO; ++u) {
-                const int n = tid + 128 * u;
+                const int n = tid + GC_THREADS * u;
                 if (n >= pairs * per) continue;
                 const int q = n / per, e = n - q * per, i = e / w, j = e - i * w, o = 2 * q * w;
                 if (pass == 0) As[(o + w + i) * 65 + o + j] = tmp[u];
@@ -199,7 +203,7 @@ __global__ void __launch_bounds__(128) gdc_chunk_kernel(const GcArgs g) {
     }
     const size_t ih = (size_t)item * g.H + h;
     bf16* T = g.T + ih * 3 * 64 * 64;
-    for (int n = tid; n < 64 * 32; n += 128) {
+    for (int n = tid; n < 64 * 32; n += GC_THREADS) {
         const int i = n >> 5, j = (n & 31) * 2;
         unsigned p[3];
         lm_split(Xs[i * 65 + j] * beta[j], Xs[i * 65 + j + 1] * beta[j + 1], p[0], p[1], p[2]);
@@ -219,12 +223,15 @@ __global__ void __launch_bounds__(128) gdc_chunk_kernel(const GcArgs g) {
     }
 }
 
-// S^T lies in accumulators, 16 columns by d rows: a warp has 16 rows, or 32.
+// S^T lies in accumulators, 16 columns by d = 16 UNITS rows: a warp has 16 rows, or 32.  The products of
+// the operands' three parts have accumulators of their own, so that none is a long chain.
+template <int UNITS>
 __global__ void __launch_bounds__(128) gdc_scan_kernel(const GcArgs g, float* __restrict__ state, long long rec,
                                                        int taps) {
     rv_pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char smraw[];
-    const int d = g.d, dv = g.dv, LK = d + 8;
+    constexpr int d = 16 * UNITS, LK = d + 8, NU = (UNITS + 3) / 4;
+    const int dv = g.dv;
     bf16* ss = (bf16*)smraw;                              // [3][16][LK]: the state
     bf16* rs = ss + 3 * GC_COLS * LK;                     // [3][16][GC_LT]: V - rho Y
     bf16* us = rs + 3 * GC_COLS * GC_LT;                  // [3][16][GC_LT]: sigma U
@@ -250,11 +257,12 @@ __global__ void __launch_bounds__(128) gdc_scan_kernel(const GcArgs g, float* __
     __syncthreads();
     rv_pdl_wait();
     if (n == 0) return;
-    const int cpr = d >> 3;
+    constexpr int cpr = d >> 3;
     auto load = [&](int c) {                              // chunk c's operands into buffer c & 1
         const int L = min(LA_C, qlen - c * LA_C);
         const bf16* base = g.rows + (size_t)(t0 + c * LA_C) * g.C;
         bf16* kd = kbuf + (c & 1) * 64 * LK;
+#pragma unroll
         for (int m = tid; m < 64 * cpr; m += 128) {
             const int j = m / cpr, ch = (m - j * cpr) * 8;
             cp_async_16(kd + j * LK + ch, base + (size_t)min(j, L - 1) * g.C + (g.G + kh) * d + ch, j < L);
@@ -275,15 +283,15 @@ __global__ void __launch_bounds__(128) gdc_scan_kernel(const GcArgs g, float* __
     };
     load(0);
     // the record's rows, [column][d]: this thread has columns ca and ca + 8 of its row pairs
-    const int ca = lane >> 2, units = d >> 4;
+    const int ca = lane >> 2;
     float* Sg = state + (size_t)slot * rec + (size_t)(taps - 1) * g.C + ((size_t)h * dv + c0) * d;
     const bool wide = (((uintptr_t)Sg) & 7) == 0;
-    float S[4][4];
+    float S[2 * NU][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
+    for (int i = 0; i < 2 * NU; ++i) {
         const int un = warp + 4 * (i >> 1), row = un * 16 + (i & 1) * 8 + (lane & 3) * 2;
         S[i][0] = S[i][1] = S[i][2] = S[i][3] = 0.f;
-        if (un < units) {
+        if (un < UNITS) {
             const float *p = Sg + (size_t)ca * d + row, *q = p + (size_t)8 * d;
             if (wide) {
                 const float2 a = *(const float2*)p, b = *(const float2*)q;
@@ -301,9 +309,9 @@ __global__ void __launch_bounds__(128) gdc_scan_kernel(const GcArgs g, float* __
     };
     auto put_state = [&]() {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
+        for (int i = 0; i < 2 * NU; ++i) {
             const int un = warp + 4 * (i >> 1), row = un * 16 + (i & 1) * 8 + (lane & 3) * 2;
-            if (un >= units) continue;
+            if (un >= UNITS) continue;
             split_pair(ss, LK, ca, row, S[i][0], S[i][1]);
             split_pair(ss, LK, ca + 8, row, S[i][2], S[i][3]);
         }
@@ -324,18 +332,29 @@ __global__ void __launch_bounds__(128) gdc_scan_kernel(const GcArgs g, float* __
         // the state before the chunk
         float* S0 = g.S0 + (ih * dv + c0) * d;
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
+        for (int i = 0; i < 2 * NU; ++i) {
             const int un = warp + 4 * (i >> 1), row = un * 16 + (i & 1) * 8 + (lane & 3) * 2;
-            if (un >= units) continue;
+            if (un >= UNITS) continue;
             *(float2*)(S0 + (size_t)ca * d + row) = make_float2(S[i][0], S[i][1]);
             *(float2*)(S0 + (size_t)(ca + 8) * d + row) = make_float2(S[i][2], S[i][3]);
         }
         // Y^T = S^T K^T for this warp's 16 tokens
-        float y[2][4];
+        float y3[3][2][4], y[2][4];
+        auto clear = [&]() {
 #pragma unroll
-        for (int i = 0; i < 2; ++i) y[i][0] = y[i][1] = y[i][2] = y[i][3] = 0.f;
-#pragma unroll 2
-        for (int kk = 0; kk < units; ++kk) {
+            for (int s = 0; s < 3; ++s)
+#pragma unroll
+                for (int i = 0; i < 2; ++i) y3[s][i][0] = y3[s][i][1] = y3[s][i][2] = y3[s][i][3] = 0.f;
+        };
+        auto sum = [&]() {                                // smallest first
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) y[i][e] = (y3[2][i][e] + y3[1][i][e]) + y3[0][i][e];
+        };
+        clear();
+#pragma unroll
+        for (int kk = 0; kk < UNITS; ++kk) {
             unsigned a[3][4], b[4];
 #pragma unroll
             for (int s = 0; s < 3; ++s)
@@ -343,10 +362,11 @@ __global__ void __launch_bounds__(128) gdc_scan_kernel(const GcArgs g, float* __
             ldmatrix_x4(b, ks + (16 * warp + (lane & 7) + (lane >> 4) * 8) * LK + kk * 16 + ((lane >> 3) & 1) * 8);
 #pragma unroll
             for (int s = 2; s >= 0; --s) {
-                mma_bf16(y[0], a[s], b[0], b[1]);
-                mma_bf16(y[1], a[s], b[2], b[3]);
+                mma_bf16(y3[s][0], a[s], b[0], b[1]);
+                mma_bf16(y3[s][1], a[s], b[2], b[3]);
             }
         }
+        sum();
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             const int j = 16 * warp + 8 * i + (lane & 3) * 2;
@@ -359,8 +379,7 @@ __global__ void __launch_bounds__(128) gdc_scan_kernel(const GcArgs g, float* __
         }
         __syncthreads();
         // U^T = R^T T^T
-#pragma unroll
-        for (int i = 0; i < 2; ++i) y[i][0] = y[i][1] = y[i][2] = y[i][3] = 0.f;
+        clear();
 #pragma unroll
         for (int kk = 0; kk < 4; ++kk) {
             if (kk > warp) continue;
@@ -372,13 +391,14 @@ __global__ void __launch_bounds__(128) gdc_scan_kernel(const GcArgs g, float* __
                                       ((lane >> 3) & 1) * 8);
             }
 #pragma unroll
-            for (int x = 2; x >= 0; --x)                  // smallest products first
+            for (int z = 0; z < 3; ++z)
 #pragma unroll
-                for (int z = 0; z <= x; ++z) {
-                    mma_bf16(y[0], a[z], b[x - z][0], b[x - z][1]);
-                    mma_bf16(y[1], a[z], b[x - z][2], b[x - z][3]);
+                for (int x = 2; x >= z; --x) {
+                    mma_bf16(y3[x][0], a[z], b[x - z][0], b[x - z][1]);
+                    mma_bf16(y3[x][1], a[z], b[x - z][2], b[x - z][3]);
                 }
         }
+        sum();
         float* U = g.U + (ih * dv + c0) * 64;
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -394,9 +414,12 @@ __global__ void __launch_bounds__(128) gdc_scan_kernel(const GcArgs g, float* __
         // S^T <- e^(B_L) S^T + (sigma U)^T K
         const float keep = cs[128];
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
+        for (int i = 0; i < 2 * NU; ++i)
 #pragma unroll
             for (int e = 0; e < 4; ++e) S[i][e] *= keep;
+        float low[2 * NU][4];
+#pragma unroll
+        for (int i = 0; i < 2 * NU; ++i) low[i][0] = low[i][1] = low[i][2] = low[i][3] = 0.f;
         const int nk = (L + 15) >> 4;
         for (int kk = 0; kk < nk; ++kk) {
             unsigned a[3][4];
@@ -404,26 +427,32 @@ __global__ void __launch_bounds__(128) gdc_scan_kernel(const GcArgs g, float* __
             for (int s = 0; s < 3; ++s)
                 ldmatrix_x4(a[s], us + (s * GC_COLS + (lane & 15)) * GC_LT + kk * 16 + (lane >> 4) * 8);
 #pragma unroll
-            for (int i = 0; i < 2; ++i) {
+            for (int i = 0; i < NU; ++i) {
                 const int un = warp + 4 * i;
-                if (un >= units) continue;
+                if (un >= UNITS) continue;
                 unsigned b[4];
                 ldmatrix_x4_trans(b, ks + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LK + un * 16 + (lane >> 4) * 8);
 #pragma unroll
-                for (int s = 2; s >= 0; --s) {
-                    mma_bf16(S[2 * i], a[s], b[0], b[1]);
-                    mma_bf16(S[2 * i + 1], a[s], b[2], b[3]);
+                for (int s = 2; s > 0; --s) {
+                    mma_bf16(low[2 * i], a[s], b[0], b[1]);
+                    mma_bf16(low[2 * i + 1], a[s], b[2], b[3]);
                 }
+                mma_bf16(S[2 * i], a[0], b[0], b[1]);
+                mma_bf16(S[2 * i + 1], a[0], b[2], b[3]);
             }
         }
+#pragma unroll
+        for (int i = 0; i < 2 * NU; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) S[i][e] += low[i][e];
         put_state();                                      // (every warp has read the old one)
         // the buffer that chunk c + 2 goes to is this chunk's: everyone has to be done with it
         __syncthreads();
     }
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
+    for (int i = 0; i < 2 * NU; ++i) {
         const int un = warp + 4 * (i >> 1), row = un * 16 + (i & 1) * 8 + (lane & 3) * 2;
-        if (un >= units) continue;
+        if (un >= UNITS) continue;
         float *p = Sg + (size_t)ca * d + row, *q = p + (size_t)8 * d;
         if (wide) {
             *(float2*)p = make_float2(S[i][0], S[i][1]);
@@ -438,8 +467,8 @@ __global__ void __launch_bounds__(128) gdc_out_kernel(const GcArgs g, float* __r
     rv_pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char smraw[];
     const int d = g.d, dv = g.dv, LK = d + 8;
-    bf16* ss = (bf16*)smraw;                              // [3][64 columns][LK]: the state before the chunk
-    bf16* us = ss + 3 * GC_T * LK;                        // [3][64 columns][GC_LT]: U
+    bf16* ss = (bf16*)smraw;                              // [3][GC_T columns][LK]: the state before the chunk
+    bf16* us = ss + 3 * GC_T * LK;                        // [3][GC_T columns][GC_LT]: U
     bf16* qs = us + 3 * GC_T * GC_LT;                     // [64][LK]
     bf16* ks = qs + 64 * LK;                              // [64][LK]
     __shared__ float eq[64], sq[64], sk[64];
@@ -488,11 +517,14 @@ __global__ void __launch_bounds__(128) gdc_out_kernel(const GcArgs g, float* __r
     __syncthreads();
     if (16 * warp >= L) return;
     const int row_a = 16 * warp + (lane >> 2), row_b = row_a + 8;
-    float p[8][4], o[8][4];
+    float p[8][4], o[GC_T / 8][4];
 #pragma unroll
     for (int i = 0; i < 8; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) p[i][e] = o[i][e] = 0.f;
+        for (int e = 0; e < 4; ++e) {
+            p[i][e] = 0.f;
+            if (i < GC_T / 8) o[i][e] = 0.f;
+        }
     for (int kk = 0; kk < (d >> 4); ++kk) {
         unsigned a[4];
         ldmatrix_x4(a, qs + (16 * warp + (lane & 15)) * LK + kk * 16 + (lane >> 4) * 8);
@@ -505,7 +537,7 @@ __global__ void __launch_bounds__(128) gdc_out_kernel(const GcArgs g, float* __r
             mma_bf16(p[2 * nb + 1], a, b[2], b[3]);
         }
 #pragma unroll
-        for (int nd = 0; nd < 4; ++nd) {
+        for (int nd = 0; nd < GC_T / 16; ++nd) {
             if (16 * nd >= vn) continue;
 #pragma unroll
             for (int s = 2; s >= 0; --s) {
@@ -518,7 +550,7 @@ __global__ void __launch_bounds__(128) gdc_out_kernel(const GcArgs g, float* __r
     }
     const float fa = eq[row_a], fb = eq[row_b];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < GC_T / 8; ++i) {
         o[i][0] *= fa; o[i][1] *= fa;
         o[i][2] *= fb; o[i][3] *= fb;
     }
@@ -533,7 +565,7 @@ __global__ void __launch_bounds__(128) gdc_out_kernel(const GcArgs g, float* __r
             lm_split(p[i][(e & 1) * 2] * pair(r, j), p[i][(e & 1) * 2 + 1] * pair(r, j + 1), a[0][e], a[1][e], a[2][e]);
         }
 #pragma unroll
-        for (int nd = 0; nd < 4; ++nd) {
+        for (int nd = 0; nd < GC_T / 16; ++nd) {
             if (16 * nd >= vn) continue;
             unsigned b[3][4];
 #pragma unroll
@@ -550,7 +582,7 @@ __global__ void __launch_bounds__(128) gdc_out_kernel(const GcArgs g, float* __r
     }
     float* dst = o_out + ((size_t)t0 * g.H + h) * dv + v0 + (lane & 3) * 2;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < GC_T / 8; ++i) {
         if (8 * i >= vn) continue;
         if (row_a < L) *(float2*)(dst + (size_t)row_a * g.H * dv + 8 * i) = make_float2(o[i][0], o[i][1]);
         if (row_b < L) *(float2*)(dst + (size_t)row_b * g.H * dv + 8 * i) = make_float2(o[i][2], o[i][3]);
@@ -610,13 +642,20 @@ static int gc_run(GcArgs g, const float* filt, float* state, long long rec, int 
     const int LK = g.d + 8;
     const size_t sm1 = (size_t)2 * 64 * 65 * 4 + (size_t)64 * LK * 2;
     GC_SMEM(gdc_chunk_kernel, sm1)
-    rv_launch(gdc_chunk_kernel, dim3((unsigned)items, g.H), dim3(128), sm1, s, g);
+    rv_launch(gdc_chunk_kernel, dim3((unsigned)items, g.H), dim3(GC_THREADS), sm1, s, g);
     RV_CHECK_LAUNCH("gated_delta chunk");
     const size_t sm2 = ((size_t)(3 * GC_COLS + 2 * 64) * LK + (size_t)(6 * GC_COLS + 6 * 64) * GC_LT + 2 * 64 * 24) * 2 +
                        2 * 132 * 4;
-    GC_SMEM(gdc_scan_kernel, sm2)
-    rv_launch(gdc_scan_kernel, dim3(g.H * (g.dv / GC_COLS), g.n_reqs - g.first_req), dim3(128), sm2, s, g, state, rec,
-              taps);
+    const dim3 grid2(g.H * (g.dv / GC_COLS), g.n_reqs - g.first_req);
+#define GC_SCAN(U)                                                                            \
+    case U:                                                                                   \
+        GC_SMEM(gdc_scan_kernel<U>, sm2)                                                      \
+        rv_launch(gdc_scan_kernel<U>, grid2, dim3(128), sm2, s, g, state, rec, taps);         \
+        break;
+    switch (g.d >> 4) {
+        GC_SCAN(1) GC_SCAN(2) GC_SCAN(3) GC_SCAN(4) GC_SCAN(5) GC_SCAN(6) GC_SCAN(7) GC_SCAN(8)
+    }
+#undef GC_SCAN
     RV_CHECK_LAUNCH("gated_delta scan");
     const size_t sm3 = ((size_t)(3 * GC_T + 2 * 64) * LK + (size_t)3 * GC_T * GC_LT) * 2;
     GC_SMEM(gdc_out_kernel, sm3)
