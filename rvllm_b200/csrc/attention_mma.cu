@@ -1,6 +1,9 @@
 // Paged grouped-query attention on the tensor cores for bfloat16 storage: flash-style
 // prefill, and split-KV decode, from one kernel template.  Compiled once per head size
-// (-DRV_HD=<multiple of 16, at most 128>), at the first use of a model with that size.
+// (-DRV_HD=<multiple of 16, at most 192>), at the first use of a model with that size.  -DRV_VD: the
+// size of a value head when it is another; -DRV_SAME: the values are the keys (one page tensor, as
+// latent attention has), so every tile is copied once and read twice; -DRV_TAG: the ending of
+// the exported names of such a library.
 //
 // Work layout.  The query rows of one (request, key/value head) are *packed*: row m is
 // (token m / G, query head g*G + m % G), G = heads per key/value head, so the G query
@@ -35,8 +38,22 @@
 #ifndef RV_HD
 #error "compile with -DRV_HD=<head size>"
 #endif
-#if RV_HD % 16 != 0 || RV_HD > 128 || RV_HD < 16
-#error "RV_HD must be a multiple of 16 between 16 and 128"
+#ifndef RV_VD
+#define RV_VD RV_HD
+#endif
+#ifndef RV_SAME
+#define RV_SAME 0
+#endif
+#if RV_HD % 16 != 0 || RV_HD > 192 || RV_HD < 16 || RV_VD % 16 != 0 || RV_VD > 192 || RV_VD < 16
+#error "RV_HD and RV_VD must be multiples of 16 between 16 and 192"
+#endif
+#if RV_SAME && RV_VD != RV_HD
+#error "values that are the keys have their size"
+#endif
+// the forms whose tiles a whole warp looks up row by row (see the decode kernel)
+#define RV_ROWWISE (RV_HD > 128 || RV_VD != RV_HD || RV_SAME)
+#if RV_HD == 64 && !defined(RV_POOLED) && !RV_ROWWISE
+#define RV_STREAM 1          // the library has the streaming decode kernel
 #endif
 
 #define RV_BN 64                 // keys per tile
@@ -75,9 +92,9 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], co
                                             const bf16* vt, int tile_key0, int lane, int lo_a,
                                             int hi_a, int lo_b, int hi_b, float scale_log2,
                                             float& m_a, float& m_b, float& l_a, float& l_b,
-                                            float (&o)[HD / 8][4], float cap_arg = 0.f,
+                                            float (&o)[RV_VD / 8][4], float cap_arg = 0.f,
                                             float cap_out = 0.f) {
-    constexpr int KSTEPS = HD / 16;
+    constexpr int KSTEPS = HD / 16, VD = RV_VD;
     // S = Q K^T for 16 rows x 64 keys
     float s[RV_BN / 8][4];
 #pragma unroll
@@ -153,7 +170,7 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], co
     l_a *= corr_a;
     l_b *= corr_b;
 #pragma unroll
-    for (int i = 0; i < HD / 8; ++i) {
+    for (int i = 0; i < VD / 8; ++i) {
         o[i][0] *= corr_a; o[i][1] *= corr_a;
         o[i][2] *= corr_b; o[i][3] *= corr_b;
     }
@@ -176,9 +193,9 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], co
 #pragma unroll
     for (int kk = 0; kk < RV_BN / 16; ++kk) {
 #pragma unroll
-        for (int nd = 0; nd < HD / 16; ++nd) {
+        for (int nd = 0; nd < VD / 16; ++nd) {
             unsigned b[4];
-            ldmatrix_x4_trans(b, vt + tile_offset<HD, SW>(kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8,
+            ldmatrix_x4_trans(b, vt + tile_offset<VD, SW>(kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8,
                                                           nd * 2 + (lane >> 4)));
             mma_bf16(o[2 * nd], pa[kk], b[0], b[1]);
             mma_bf16(o[2 * nd + 1], pa[kk], b[2], b[3]);
@@ -187,7 +204,7 @@ __device__ __forceinline__ void attend_tile(const unsigned (&qf)[HD / 16][4], co
 }
 
 template <int HD, int NWARPS, bool SPLIT, bool EXT = false>
-__global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_attention_mma_kernel(
+__global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 && RV_VD <= 64 ? 4 : 1) paged_attention_mma_kernel(
     const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ k_cache,
     const bf16* __restrict__ v_cache, const int* __restrict__ block_table, int max_blocks,
     const int* __restrict__ q_start, const int* __restrict__ ctx_lens, bf16* __restrict__ out,
@@ -196,13 +213,14 @@ __global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_at
     const float* __restrict__ sinks, const RvPooled pl) {
     rv_pdl_prologue();
     constexpr int BM = 16 * NWARPS;
-    constexpr int LD = HD + 8;          // padded row: conflict-free ldmatrix for HD % 16 == 0
-    constexpr int CPR = HD / 8;         // 16-byte chunks per row
+    constexpr int VD = RV_VD;
+    constexpr int LD = HD + 8, LDV = VD + 8;   // padded rows: conflict-free ldmatrix for sizes % 16 == 0
+    constexpr int CPR = HD / 8, CPV = VD / 8;  // 16-byte chunks per row
     constexpr int KSTEPS = HD / 16;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* Qs = (bf16*)smem_raw;                         // [BM][LD]
     bf16* Ks = Qs + BM * LD;                            // [2][BN][LD]
-    bf16* Vs = Ks + 2 * RV_BN * LD;                     // [2][BN][LD]
+    bf16* Vs = RV_SAME ? Ks : Ks + 2 * RV_BN * LD;      // [2][BN][LDV]
 
     const int G = num_heads / num_kv_heads;
     const int r = first_req + blockIdx.z;
@@ -242,7 +260,7 @@ __global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_at
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int page_shift = (page_size & (page_size - 1)) == 0 ? 31 - __clz(page_size) : -1;
     const int* table = block_table + (size_t)r * max_blocks;
-    const size_t kv_row = (size_t)num_kv_heads * HD;
+    const size_t kv_row = (size_t)num_kv_heads * HD, v_row = (size_t)num_kv_heads * VD;
 
     // ---- Q tile -> shared memory (packed rows), zero beyond the last row ----------------
     for (int c = tid; c < BM * CPR; c += NWARPS * 32) {
@@ -254,12 +272,12 @@ __global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_at
         cp_async_16(Qs + m * LD + ch * 8, src, valid);
     }
     // Each thread copies the same few rows of every tile: ROWS rows, one 16-byte chunk of K
-    // and of V each.  The page lookups of a tile are all issued before the first copy, so
+    // and of V each (value heads of another size: their rows and chunks on their own).  The page lookups of a tile are all issued before the first copy, so
     // they overlap instead of forming a chain of dependent loads.
     constexpr int ROWS = RV_BN * CPR / (NWARPS * 32) > 0 ? (RV_BN * CPR + NWARPS * 32 - 1) / (NWARPS * 32) : 1;
     auto load_tile = [&](int t, int stage) {
         bf16* kd = Ks + stage * RV_BN * LD;
-        bf16* vd = Vs + stage * RV_BN * LD;
+        bf16* vd = Vs + stage * RV_BN * LDV;
         const bool blocks = EXT && t < tile_first;
         const int row0 = (blocks ? t - tile_begin : t) * RV_BN, limit = blocks ? nb_hi : clen;
         const int* tab = blocks ? pl.table + (size_t)r * pl.max_blocks : table;
@@ -286,7 +304,26 @@ __global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_at
             if (c < RV_BN * CPR) {
                 const int row = c / CPR, ch = c - row * CPR;
                 cp_async_16(kd + row * LD + ch * 8, kc + off[i], valid[i]);
-                cp_async_16(vd + row * LD + ch * 8, vc + off[i], valid[i]);
+                if (VD == HD && !RV_SAME) cp_async_16(vd + row * LDV + ch * 8, vc + off[i], valid[i]);
+            }
+        }
+        if (VD != HD) {
+            constexpr int VROWS = (RV_BN * CPV + NWARPS * 32 - 1) / (NWARPS * 32);
+            int slot[VROWS];
+#pragma unroll
+            for (int i = 0; i < VROWS; ++i) {
+                const int c = tid + i * NWARPS * 32, j = row0 + c / CPV;
+                int page = -1;
+                if (c < RV_BN * CPV && j < limit)
+                    page = tab[page_shift >= 0 ? (j >> page_shift) : (j / page_size)];
+                slot[i] = page < 0 ? -1 : page * page_size + (page_shift >= 0 ? (j & (page_size - 1)) : (j % page_size));
+            }
+#pragma unroll
+            for (int i = 0; i < VROWS; ++i) {
+                const int c = tid + i * NWARPS * 32, row = c / CPV, ch = c - row * CPV;
+                if (c < RV_BN * CPV)
+                    cp_async_16(vd + row * LDV + ch * 8,
+                                vc + (slot[i] < 0 ? 0 : (size_t)slot[i] * v_row + (size_t)g * VD + ch * 8), slot[i] >= 0);
             }
         }
     };
@@ -309,9 +346,9 @@ __global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_at
     const float cap_out = EXT ? pl.cap * 1.4426950408889634f : 0.f;
     const float cap_arg = EXT && pl.cap > 0.f ? 2.f * scale_log2 / pl.cap : 0.f;
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
-    float o[HD / 8][4];
+    float o[VD / 8][4];
 #pragma unroll
-    for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    for (int i = 0; i < VD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     unsigned qf[KSTEPS][4];
     bool q_loaded = false;
 
@@ -332,7 +369,7 @@ __global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_at
                 ldmatrix_x4(qf[kk], Qs + (warp * 16 + (lane & 15)) * LD + kk * 16 + (lane >> 4) * 8);
         }
         const bf16* kt = Ks + stage * RV_BN * LD;
-        const bf16* vt = Vs + stage * RV_BN * LD;
+        const bf16* vt = Vs + stage * RV_BN * LDV;
 
         if (EXT) {
             const bool blocks = t < tile_first;
@@ -357,35 +394,35 @@ __global__ void __launch_bounds__(NWARPS * 32, EXT && HD <= 64 ? 4 : 1) paged_at
         if (ok_a) {
             const size_t slot = ((size_t)r * num_heads + g * G + row_a) * max_splits + split;
 #pragma unroll
-            for (int i = 0; i < HD / 8; ++i)
-                *(float2*)(part_o + slot * HD + i * 8 + col) = make_float2(o[i][0], o[i][1]);
+            for (int i = 0; i < VD / 8; ++i)
+                *(float2*)(part_o + slot * VD + i * 8 + col) = make_float2(o[i][0], o[i][1]);
             if ((lane & 3) == 0) part_ml[slot] = make_float2(m_a * ln2, l_a);
         }
         if (ok_b) {
             const size_t slot = ((size_t)r * num_heads + g * G + row_b) * max_splits + split;
 #pragma unroll
-            for (int i = 0; i < HD / 8; ++i)
-                *(float2*)(part_o + slot * HD + i * 8 + col) = make_float2(o[i][2], o[i][3]);
+            for (int i = 0; i < VD / 8; ++i)
+                *(float2*)(part_o + slot * VD + i * 8 + col) = make_float2(o[i][2], o[i][3]);
             if ((lane & 3) == 0) part_ml[slot] = make_float2(m_b * ln2, l_b);
         }
     } else {
         if (ok_a) {
             const int tok = row_a / G, hg = row_a - tok * G;
-            bf16* dst = out + (size_t)(qs + tok) * num_heads * HD + (size_t)(g * G + hg) * HD + col;
+            bf16* dst = out + (size_t)(qs + tok) * num_heads * VD + (size_t)(g * G + hg) * VD + col;
             // a sink: one more term exp(sink - max) in the denominator, with no value
             if (sinks) l_a += exp2f(sinks[g * G + hg] * 1.4426950408889634f - m_a);
             const float inv = 1.f / l_a;
 #pragma unroll
-            for (int i = 0; i < HD / 8; ++i)
+            for (int i = 0; i < VD / 8; ++i)
                 *(unsigned*)(dst + i * 8) = pack_bf16(o[i][0] * inv, o[i][1] * inv);
         }
         if (ok_b) {
             const int tok = row_b / G, hg = row_b - tok * G;
-            bf16* dst = out + (size_t)(qs + tok) * num_heads * HD + (size_t)(g * G + hg) * HD + col;
+            bf16* dst = out + (size_t)(qs + tok) * num_heads * VD + (size_t)(g * G + hg) * VD + col;
             if (sinks) l_b += exp2f(sinks[g * G + hg] * 1.4426950408889634f - m_b);
             const float inv = 1.f / l_b;
 #pragma unroll
-            for (int i = 0; i < HD / 8; ++i)
+            for (int i = 0; i < VD / 8; ++i)
                 *(unsigned*)(dst + i * 8) = pack_bf16(o[i][2] * inv, o[i][3] * inv);
         }
     }
@@ -403,10 +440,11 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
     int max_splits, int num_heads, int num_kv_heads, int page_size, float scale_log2, int window,
     const RvPooled pl) {
     rv_pdl_prologue();
-    constexpr int LD = HD + 8;
+    constexpr int VD = RV_VD;
+    constexpr int LD = HD + 8, LDV = VD + 8;
     constexpr int CPR = HD / 8;
     constexpr int KSTEPS = HD / 16;
-    constexpr int TILE = RV_BN * LD;                   // elements of one K or V tile
+    constexpr int TILE = RV_BN * LD, TILE_V = RV_SAME ? 0 : RV_BN * LDV;   // elements of one K and V tile
     constexpr int SPLIT = NW * RV_BN;                  // keys per block
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* Qs = (bf16*)smem_raw;                        // [16][LD]
@@ -446,9 +484,33 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
     }
     const int t = stretch * NW + warp;   // this warp's tile
     const bool active = t * RV_BN <= key_hi && t * RV_BN + RV_BN - 1 >= key_lo;
-    bf16* kt = KV + warp * 2 * TILE;
-    bf16* vt = kt + TILE;
-    if (active) {
+    bf16* kt = KV + warp * (TILE + TILE_V);
+    bf16* vt = RV_SAME ? kt : kt + TILE;
+    if (active && RV_ROWWISE) {
+        // a lane looks up two of the tile's rows; the copies take their rows' slots from it
+        int slot[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int j = t * RV_BN + lane + 32 * i;
+            int page = -1;
+            if (j < limit) page = table[page_shift >= 0 ? (j >> page_shift) : (j / page_size)];
+            slot[i] = page < 0 ? -1 : page * page_size + (page_shift >= 0 ? (j & (page_size - 1)) : (j % page_size));
+        }
+        auto copy = [&](bf16* dst, const bf16* src, int size) {
+            const int cpr = size / 8, ld = size + 8;
+            const size_t row_len = (size_t)num_kv_heads * size;
+#pragma unroll 8
+            for (int i = 0; i < 2 * cpr; ++i) {
+                const int c = lane + i * 32, row = c / cpr, ch = c - row * cpr;
+                const int a = __shfl_sync(0xffffffffu, slot[0], row & 31), b = __shfl_sync(0xffffffffu, slot[1], row & 31);
+                const int at = row < 32 ? a : b;
+                cp_async_16(dst + row * ld + ch * 8, src + (at < 0 ? 0 : (size_t)at * row_len + (size_t)g * size + ch * 8),
+                            at >= 0);
+            }
+        };
+        copy(kt, kc, HD);
+        if (!RV_SAME) copy(vt, vc, VD);
+    } else if (active) {
         constexpr int ROWS = RV_BN * CPR / 32;
         size_t off[ROWS];
         bool valid[ROWS];
@@ -481,9 +543,9 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
     const int lo_a = key_lo, lo_b = key_lo;
     const int hi_a = ok_a ? key_hi : -1, hi_b = ok_b ? key_hi : -1;
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
-    float o[HD / 8][4];
+    float o[VD / 8][4];
 #pragma unroll
-    for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    for (int i = 0; i < VD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     if (active) {
         unsigned qf[KSTEPS][4];
 #pragma unroll
@@ -500,44 +562,44 @@ __global__ void __launch_bounds__(NW * 32) paged_attention_decode_mma_kernel(
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
     __syncthreads();                                    // the tiles are no longer needed
 
-    // park every warp's rows: red[warp][row][HD + 2] float32 over the tile memory
+    // park every warp's rows: red[warp][row][VD + 2] float32 over the tile memory
     float* red = (float*)KV;
-    constexpr int RS = HD + 2;
+    constexpr int RS = VD + 2;
     const int col = (lane & 3) * 2;
     {
         float* mine_a = red + ((size_t)warp * 16 + (lane >> 2)) * RS;
         float* mine_b = mine_a + 8 * RS;
 #pragma unroll
-        for (int i = 0; i < HD / 8; ++i) {
+        for (int i = 0; i < VD / 8; ++i) {
             mine_a[i * 8 + col] = o[i][0]; mine_a[i * 8 + col + 1] = o[i][1];
             mine_b[i * 8 + col] = o[i][2]; mine_b[i * 8 + col + 1] = o[i][3];
         }
         if ((lane & 3) == 0) {
-            mine_a[HD] = m_a; mine_a[HD + 1] = l_a;
-            mine_b[HD] = m_b; mine_b[HD + 1] = l_b;
+            mine_a[VD] = m_a; mine_a[VD + 1] = l_a;
+            mine_b[VD] = m_b; mine_b[VD + 1] = l_b;
         }
     }
     __syncthreads();
     const float ln2 = 0.6931471805599453f;
-    for (int i = tid; i < rows * HD; i += NW * 32) {
-        const int m = i / HD, d = i - m * HD;
+    for (int i = tid; i < rows * VD; i += NW * 32) {
+        const int m = i / VD, d = i - m * VD;
         float M = -INFINITY;
-        for (int w = 0; w < NW; ++w) M = fmaxf(M, red[((size_t)w * 16 + m) * RS + HD]);
+        for (int w = 0; w < NW; ++w) M = fmaxf(M, red[((size_t)w * 16 + m) * RS + VD]);
         float L = 0.f, O = 0.f;
         for (int w = 0; w < NW; ++w) {
             const float* src = red + ((size_t)w * 16 + m) * RS;
-            const float f = src[HD] == -INFINITY ? 0.f : exp2f(src[HD] - M);
-            L += src[HD + 1] * f;
+            const float f = src[VD] == -INFINITY ? 0.f : exp2f(src[VD] - M);
+            L += src[VD + 1] * f;
             O += src[d] * f;
         }
         const size_t slot = ((size_t)r * num_heads + g * G + m0 + m) * max_splits + split;
-        part_o[slot * HD + d] = O;
+        part_o[slot * VD + d] = O;
         if (d == 0) part_ml[slot] = make_float2(M * ln2, L);
     }
 }
 
 
-#if RV_HD == 64 && !defined(RV_POOLED)
+#ifdef RV_STREAM
 // ---------------------------------------------------------------------------------
 // Decode as a stream (head size 64, pages of 8, 16, 32 or 64 tokens).  One persistent block
 // per SM; each of its six warps is a pipeline of its own.  A warp takes work items --
@@ -837,7 +899,11 @@ static int fail(const char* msg) {
 }
 #define RV_CAT2(a, b) a##b
 #define RV_CAT(a, b) RV_CAT2(a, b)
+#ifdef RV_TAG
+#define RV_SYM(name) RV_CAT(RV_CAT(name, _), RV_TAG)
+#else
 #define RV_SYM(name) RV_CAT(RV_CAT(name, _hd), RV_HD)
+#endif
 
 #ifndef RV_POOLED
 extern "C" const char* RV_SYM(rv_attention_mma_last_error)() { return g_error; }
@@ -845,7 +911,12 @@ extern "C" const char* RV_SYM(rv_attention_mma_last_error)() { return g_error; }
 
 template <int NWARPS>
 static size_t smem_bytes() {
-    return (size_t)(16 * NWARPS + 4 * RV_BN) * (RV_HD + 8) * sizeof(bf16);
+    return ((size_t)(16 * NWARPS + 2 * RV_BN) * (RV_HD + 8) + (RV_SAME ? 0 : 2 * RV_BN * (RV_VD + 8))) * sizeof(bf16);
+}
+// of a decode block of NW warps
+template <int NW>
+static size_t decode_smem() {
+    return ((size_t)(16 + NW * RV_BN) * (RV_HD + 8) + (RV_SAME ? 0 : NW * RV_BN * (RV_VD + 8))) * sizeof(bf16);
 }
 
 #ifdef RV_POOLED
@@ -911,14 +982,14 @@ extern "C" int RV_SYM(rv_paged_attention_pooled_decode_mma)(
     const int psplits = rv_pooled_psplits(max_ctx_len, window, pool, most, RV_SPLIT);
     const int max_splits = psplits + rv_pooled_tsplits(max_ctx_len, window, RV_SPLIT);
     const size_t slots = (size_t)n_reqs * num_heads * max_splits;
-    if ((long long)(slots * RV_HD * 4 + slots * 8) > scratch_bytes)
+    if ((long long)(slots * RV_VD * 4 + slots * 8) > scratch_bytes)
         return fail("paged_attention_pooled_decode: scratch too small");
     const int G = num_heads / num_kv_heads;
     const int tiles_per_head = (G + 15) / 16;
     if (n_reqs > 65535 || num_kv_heads * tiles_per_head > 65535 || max_splits > 65535)
         return fail("paged_attention_pooled_decode: batch too large for one launch");
     static bool configured = false;
-    const size_t smem = (size_t)(16 + 8 * RV_BN) * (RV_HD + 8) * sizeof(bf16);
+    const size_t smem = decode_smem<4>();
     if (!configured) {
         if (smem > 48 * 1024) {
             cudaError_t e = cudaFuncSetAttribute(paged_attention_decode_mma_kernel<RV_HD, 4, true>,
@@ -929,7 +1000,7 @@ extern "C" int RV_SYM(rv_paged_attention_pooled_decode_mma)(
     }
     const RvPooled pl = {pk, pv, ptable, pmax_blocks, pool, most, cap, psplits};
     float* part_o = (float*)scratch;
-    float2* part_ml = (float2*)((char*)scratch + slots * RV_HD * 4);
+    float2* part_ml = (float2*)((char*)scratch + slots * RV_VD * 4);
     rv_launch(paged_attention_decode_mma_kernel<RV_HD, 4, true>,
               dim3(num_kv_heads * tiles_per_head, max_splits, n_reqs), dim3(128), smem,
               (cudaStream_t)stream, (const bf16*)q, q_stride, (const bf16*)k_cache,
@@ -1010,15 +1081,14 @@ extern "C" int RV_SYM(rv_paged_attention_decode_mma)(
     int max_splits = (max_ctx_len + split_keys - 1) / split_keys;
     if (max_splits < 1) max_splits = 1;
     const size_t slots = (size_t)n_reqs * num_heads * max_splits;
-    if ((long long)(slots * RV_HD * 4 + slots * 8) > scratch_bytes)
+    if ((long long)(slots * RV_VD * 4 + slots * 8) > scratch_bytes)
         return fail("paged_attention_decode_mma: scratch too small");
     const int G = num_heads / num_kv_heads;
     const int tiles_per_head = (G + 15) / 16;
     if (n_reqs > 65535 || num_kv_heads * tiles_per_head > 65535)
         return fail("paged_attention_decode_mma: batch too large for one launch");
     static bool configured = false;
-    const size_t smem4 = (size_t)(16 + 8 * RV_BN) * (RV_HD + 8) * sizeof(bf16);
-    const size_t smem2 = (size_t)(16 + 4 * RV_BN) * (RV_HD + 8) * sizeof(bf16);
+    const size_t smem4 = decode_smem<4>(), smem2 = decode_smem<2>();
     if (!configured) {
         cudaError_t e = cudaSuccess;
         if (smem4 > 48 * 1024)
@@ -1033,7 +1103,7 @@ extern "C" int RV_SYM(rv_paged_attention_decode_mma)(
     if (max_splits > 65535) return fail("paged_attention_decode_mma: context too long for one launch");
     dim3 grid(num_kv_heads * tiles_per_head, max_splits, n_reqs);
     float* part_o = (float*)scratch;
-    float2* part_ml = (float2*)((char*)scratch + slots * RV_HD * 4);
+    float2* part_ml = (float2*)((char*)scratch + slots * RV_VD * 4);
     if (split_keys == 256)
         rv_launch(paged_attention_decode_mma_kernel<RV_HD, 4>, dim3(grid), dim3(128), smem4,
                   (cudaStream_t)stream, (const bf16*)q, q_stride, (const bf16*)k_cache,
@@ -1056,7 +1126,7 @@ extern "C" int RV_SYM(rv_paged_attention_decode_mma)(
 // names (128 or 256 keys: the smaller one when the larger would leave warps without work).
 // Needs head size 64 and pages of 8, 16, 32 or 64 tokens; `total_slots` = pages * page_size
 // of the cache tensors.  `status` receives code 12 when a bounded wait runs out.
-#if RV_HD == 64
+#ifdef RV_STREAM
 typedef CUresult (*RvEncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*,
                                     const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
                                     const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
@@ -1111,7 +1181,7 @@ extern "C" int RV_SYM(rv_paged_attention_decode_stream)(
     int max_splits = (max_ctx_len + split_keys - 1) / split_keys;
     if (max_splits < 1) max_splits = 1;
     const size_t slots = (size_t)n_reqs * num_heads * max_splits;
-    if ((long long)(slots * RV_HD * 4 + slots * 8) > scratch_bytes)
+    if ((long long)(slots * RV_VD * 4 + slots * 8) > scratch_bytes)
         return fail("paged_attention_decode_stream: scratch too small");
     const int G = num_heads / num_kv_heads;
     const int tiles_per_head = (G + 15) / 16;
@@ -1132,7 +1202,7 @@ extern "C" int RV_SYM(rv_paged_attention_decode_stream)(
     long long blocks = (total + RV_STREAM_WARPS - 1) / RV_STREAM_WARPS;
     if (blocks > n_sms) blocks = n_sms;
     float* part_o = (float*)scratch;
-    float2* part_ml = (float2*)((char*)scratch + slots * RV_HD * 4);
+    float2* part_ml = (float2*)((char*)scratch + slots * RV_VD * 4);
     rv_launch(paged_attention_decode_stream_kernel<RV_HD>, dim3((unsigned)blocks),
               dim3(RV_STREAM_WARPS * 32), smem, (cudaStream_t)stream, map_k, map_v,
               (const bf16*)q, q_stride, block_table, max_blocks, ctx_lens, part_o, part_ml,

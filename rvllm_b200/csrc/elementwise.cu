@@ -248,10 +248,36 @@ __global__ void weighted_sum_kernel(const T* __restrict__ a, float sa, const T* 
         rv_store(out + i, sa * rv_load(a + i) + sb * rv_load(b + i));
 }
 
+__global__ void weighted_sum_bf16x8_kernel(const __nv_bfloat16* __restrict__ a, float sa,
+                                           const __nv_bfloat16* __restrict__ b, float sb,
+                                           __nv_bfloat16* __restrict__ out, size_t total8) {
+    rv_pdl_prologue();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total8) return;
+    uint4 u = *(const uint4*)(a + i * 8);
+    const uint4 w = *(const uint4*)(b + i * 8);
+    __nv_bfloat162* p = (__nv_bfloat162*)&u;
+    const __nv_bfloat162* q = (const __nv_bfloat162*)&w;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const float2 f = __bfloat1622float2(p[j]), g = __bfloat1622float2(q[j]);
+        p[j] = __floats2bfloat162_rn(sa * f.x + sb * g.x, sa * f.y + sb * g.y);
+    }
+    *(uint4*)(out + i * 8) = u;
+}
+
 extern "C" int rv_weighted_sum(const void* a, float sa, const void* b, float sb, void* out,
                                int dtype, long long total, void* stream) {
     if (total == 0) return 0;
     if (total < 0 || !a || !b || !out) RV_FAIL("weighted_sum: bad arguments");
+    if (dtype == RV_DTYPE_BF16 && total % 8 == 0 && total / 2048 < 0x7fffffffLL &&
+        (((uintptr_t)a | (uintptr_t)b | (uintptr_t)out) & 15) == 0) {
+        const long long total8 = total / 8;
+        rv_launch(weighted_sum_bf16x8_kernel, dim3((unsigned)((total8 + 255) / 256)), dim3(256), 0, (cudaStream_t)stream,
+                  (const __nv_bfloat16*)a, sa, (const __nv_bfloat16*)b, sb, (__nv_bfloat16*)out, (size_t)total8);
+        RV_CHECK_LAUNCH("weighted_sum");
+        return 0;
+    }
     const long long want = (total + 255) / 256;
     const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
     RV_DISPATCH_DTYPE(dtype, "weighted_sum",
@@ -348,11 +374,38 @@ __global__ void add_bias_kernel(T* __restrict__ x, const float* __restrict__ bia
         rv_store(x + i, rv_load(x + i) + bias[i % width]);
 }
 
+// eight bfloat16 values a thread, 16-byte accesses; width a multiple of 8
+__global__ void add_bias_bf16x8_kernel(__nv_bfloat16* __restrict__ x, const float* __restrict__ bias, int width8,
+                                       size_t total8) {
+    rv_pdl_launch_dependents();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total8) return;
+    const float* b = bias + (size_t)(i % width8) * 8;
+    const float4 b0 = *(const float4*)b, b1 = *(const float4*)(b + 4);
+    rv_pdl_wait();
+    uint4 v = *(const uint4*)(x + i * 8);
+    __nv_bfloat162* p = (__nv_bfloat162*)&v;
+    const float add[8] = {b0.x, b0.y, b0.z, b0.w, b1.x, b1.y, b1.z, b1.w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const float2 f = __bfloat1622float2(p[j]);
+        p[j] = __floats2bfloat162_rn(f.x + add[2 * j], f.y + add[2 * j + 1]);
+    }
+    *(uint4*)(x + i * 8) = v;
+}
+
 extern "C" int rv_add_bias(void* x, int dtype, const float* bias, int n_rows, int width,
                            void* stream) {
     if (n_rows == 0) return 0;
     if (n_rows < 0 || width <= 0) RV_FAIL("add_bias: bad sizes");
     const size_t total = (size_t)n_rows * width;
+    if (dtype == RV_DTYPE_BF16 && width % 8 == 0 && (((uintptr_t)x | (uintptr_t)bias) & 15) == 0) {
+        const size_t total8 = total / 8;
+        rv_launch(add_bias_bf16x8_kernel, dim3((unsigned)((total8 + 255) / 256)), dim3(256), 0, (cudaStream_t)stream,
+                  (__nv_bfloat16*)x, bias, width / 8, total8);
+        RV_CHECK_LAUNCH("add_bias");
+        return 0;
+    }
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
     RV_DISPATCH_DTYPE(dtype, "add_bias",
                       (rv_launch(add_bias_kernel<T>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, 

@@ -90,6 +90,19 @@ __device__ __forceinline__ void moe_select_warp(float* sc, float* gs, int E, int
     __syncwarp();
     if (groups > 1) {
         const int size = E / groups;
+        if (group_top == 1 && groups <= 32) {
+            // a group's score is its largest: a lane a group, and its rank among the groups
+            float best = -INFINITY;
+            if (lane < groups)
+                for (int e = lane * size; e < (lane + 1) * size; ++e) best = fmaxf(best, sc[e]);
+            int rank = 0;
+            for (int g = 0; g < groups; ++g) {
+                const float o = __shfl_sync(0xffffffffu, best, g);
+                rank += o > best || (o == best && g < lane);
+            }
+            if (lane < groups) gs[lane] = rank < keep ? INFINITY : 0.f;
+            __syncwarp();
+        } else {
         for (int g = 0; g < groups; ++g) {
             // the sum of the group's largest scores: take them out one by one, then put them back
             float sum = 0.f, taken_v[MOE_MAX_GROUP_TOP];
@@ -135,6 +148,7 @@ __device__ __forceinline__ void moe_select_warp(float* sc, float* gs, int E, int
             __syncwarp();
             if (lane == 0 && idx < groups) gs[idx] = INFINITY;
             __syncwarp();
+        }
         }
         for (int e = lane; e < E; e += 32)
             if (gs[e / size] != INFINITY) sc[e] = -3.0e38f;      // below every score

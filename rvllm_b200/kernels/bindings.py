@@ -60,8 +60,8 @@ class CudaOps:
         self._retired = []
         self._attn_libs = {}
         self._verbose_build = verbose_build
-        # bfloat16 attention: "mma" = mma.sync tensor-core kernels (attention_mma.cu, head
-        # sizes that are multiples of 16 up to 128), "simt" = the float32-arithmetic kernels;
+        # bfloat16 attention: "mma" = mma.sync tensor-core kernels (attention_mma.cu, key and value
+        # sizes that are multiples of 16 up to 192), "simt" = the float32-arithmetic kernels;
         # prompt portions also "tcgen05" (attention_tcgen05.cu, head size 64) and "auto" =
         # tcgen05 where it applies, else mma
         self.prefill_attention = os.environ.get("RVLLM_PREFILL_ATTENTION", "auto")
@@ -458,19 +458,40 @@ class CudaOps:
         if nbytes > 0:
             self._scratch_buffer(nbytes, device)
 
-    def _attn_lib(self, head_dim: int):
-        """The tensor-core attention library for this head size, built at first use."""
-        lib = self._attn_libs.get(head_dim)
-        if lib is None:
-            path = build_variant("attention_mma.cu", {"RV_HD": head_dim}, f"attn_hd{head_dim}",
+    def _mma_lib(self, head_dim: int, v_head_dim: int, same: bool, pooled: bool):
+        """The tensor-core attention library for these head sizes, built at first use (`same`: the
+        values are the keys; `pooled`: with the kernels for a window and rows before it), and the
+        ending of its functions' names."""
+        key = ("mma", head_dim, v_head_dim, same, pooled)
+        hit = self._attn_libs.get(key)
+        if hit is None:
+            tag = f"hd{head_dim}"
+            defines = {"RV_HD": head_dim}
+            if v_head_dim != head_dim:
+                tag += f"v{v_head_dim}"
+                defines["RV_VD"] = v_head_dim
+            if same:
+                tag += "s"
+                defines["RV_SAME"] = 1
+            if len(defines) > 1:
+                defines["RV_TAG"] = tag
+            if pooled:
+                defines["RV_POOLED"] = 1
+            path = build_variant("attention_mma.cu", defines,
+                                 f"attnpool_{tag}" if pooled else f"attn_{tag}",
                                  verbose=self._verbose_build)
             try:
                 lib = ctypes.CDLL(path)
             except OSError as e:
                 raise KernelError(f"cannot load the kernel library {path}: {e}") from None
-            getattr(lib, f"rv_attention_mma_last_error_hd{head_dim}").restype = ctypes.c_char_p
-            self._attn_libs[head_dim] = lib
-        return lib
+            kind = "pooled" if pooled else "mma"
+            getattr(lib, f"rv_attention_{kind}_last_error_{tag}").restype = ctypes.c_char_p
+            hit = self._attn_libs[key] = (lib, tag)
+        return hit
+
+    def _attn_lib(self, head_dim: int):
+        """The tensor-core attention library for keys and values of this size."""
+        return self._mma_lib(head_dim, head_dim, False, False)[0]
 
     def _attn5_lib(self, head_dim: int):
         """The tcgen05 prefill attention library for this head size, built at first use."""
@@ -528,15 +549,21 @@ class CudaOps:
         # 64 float32 values, an offset and a sum (the kernel fits its parts to what it is given)
         return 6 * self._sm_count * 128 * (64 * 4 + 8)
 
-    def _check_attn(self, lib, head_dim: int, rc: int, what: str) -> None:
+    def _check_attn(self, lib, tag: str, rc: int, what: str) -> None:
         self.launches += 1
         if rc != 0:
-            msg = getattr(lib, f"rv_attention_mma_last_error_hd{head_dim}")().decode()
+            msg = getattr(lib, f"rv_attention_mma_last_error_{tag}")().decode()
             raise KernelError(f"{what}: {msg}")
 
     @staticmethod
-    def _mma_ok(dtype, head_dim: int) -> bool:
-        return dtype == torch.bfloat16 and head_dim % 16 == 0 and 16 <= head_dim <= 128
+    def _mma_ok(dtype, head_dim: int, v_head_dim=None) -> bool:
+        return dtype == torch.bfloat16 and all(d % 16 == 0 and 16 <= d <= 192
+                                               for d in (head_dim, v_head_dim or head_dim))
+
+    @staticmethod
+    def _same_rows(k_cache, v_cache, head_dim, v_head_dim) -> bool:
+        """Whether the values are the keys: one page tensor under both names."""
+        return v_head_dim == head_dim and k_cache.data_ptr() == v_cache.data_ptr()
 
     def paged_attention(self, qkv, num_heads, num_kv_heads, head_dim, k_cache, v_cache,
                         ctx, group, scale, window, out, sinks=None, v_head_dim=None):
@@ -555,10 +582,11 @@ class CudaOps:
             raise KernelError("paged_attention: output width and head sizes disagree")
         # the tensor-core kernels fetch query rows in 16-byte pieces: rows of another stride or
         # start take the float32-arithmetic kernels
-        mma = (self._mma_ok(qkv.dtype, head_dim) and qkv.shape[1] % 8 == 0
+        mma = (self._mma_ok(qkv.dtype, head_dim, vd) and qkv.shape[1] % 8 == 0
                and qkv.data_ptr() % 16 == 0)
-        if vd != head_dim or (sinks is not None and not mma):
-            # a value size of its own, or sinks where no tensor-core kernel applies: the
+        if (vd != head_dim or sinks is not None) and not (
+                mma and self.decode_attention == "mma" and self.prefill_attention != "simt"):
+            # a value size of its own or sinks where no tensor-core kernel applies: the
             # float32-arithmetic kernels
             return self._paged_attention_options(qkv, num_heads, num_kv_heads, head_dim, vd,
                                                  k_cache, v_cache, ctx, group, scale, window, out,
@@ -571,25 +599,22 @@ class CudaOps:
                 self.paged_attention_decode_mma(qkv, num_heads, num_kv_heads, head_dim, k_cache,
                                                 v_cache, group.block_table, ctx.q_start,
                                                 ctx.ctx_lens, nd, ctx.max_ctx_len,
-                                                group.page_size, scale, window, out, sinks=sinks)
-            elif sinks is not None:
-                self._paged_attention_options(qkv, num_heads, num_kv_heads, head_dim, vd, k_cache,
-                                              v_cache, ctx, group, scale, window, out, sinks,
-                                              prompts=False)
+                                                group.page_size, scale, window, out, sinks=sinks,
+                                                v_head_dim=vd)
             else:
                 self.paged_attention_decode(qkv, num_heads, num_kv_heads, head_dim, k_cache,
                                             v_cache, group.block_table, ctx.ctx_lens, nd,
                                             ctx.max_ctx_len, group.page_size, scale, window, out)
-        if (ctx.n_tokens > nd and self.prefill_attention in ("auto", "tcgen05")
+        if (ctx.n_tokens > nd and self.prefill_attention in ("auto", "tcgen05") and vd == head_dim
                 and self._tcgen05_prefill_ok(qkv, out, num_heads, num_kv_heads, head_dim,
                                              group.page_size)):
             self.paged_attention_prefill_tcgen05(qkv, num_heads, num_kv_heads, head_dim, k_cache,
                                                  v_cache, ctx, group, scale, window, out,
                                                  sinks=sinks)
         elif ctx.n_tokens > nd and mma and self.prefill_attention in ("auto", "mma", "tcgen05"):
-            lib = self._attn_lib(head_dim)
-            fn = getattr(lib, f"rv_paged_attention_prefill_mma_hd{head_dim}")
-            self._check_attn(lib, head_dim, fn(
+            lib, tag = self._mma_lib(head_dim, vd, self._same_rows(k_cache, v_cache, head_dim, vd), False)
+            fn = getattr(lib, f"rv_paged_attention_prefill_mma_{tag}")
+            self._check_attn(lib, tag, fn(
                 _ptr(qkv), c_int(qkv.shape[1]), _ptr(k_cache), _ptr(v_cache),
                 _ptr(group.block_table), c_int(group.max_blocks), _ptr(ctx.q_start),
                 _ptr(ctx.ctx_lens), _ptr(out), c_int(nd), c_int(ctx.n_reqs - nd),
@@ -652,12 +677,14 @@ class CudaOps:
 
     def paged_attention_decode_mma(self, qkv, num_heads, num_kv_heads, head_dim, k_cache, v_cache,
                                    block_table, q_start, ctx_lens, n_reqs, max_ctx_len,
-                                   page_size, scale, window, out, scratch=None, sinks=None):
+                                   page_size, scale, window, out, scratch=None, sinks=None,
+                                   v_head_dim=None):
         """Tensor-core split-KV attention (bfloat16) for requests [0, n_reqs) that bring one
         token each; the splits are combined by the merge kernel."""
-        stream = (self.decode_kernel in ("stream", "auto") and head_dim == 64
+        vd = v_head_dim or head_dim
+        lib, tag = self._mma_lib(head_dim, vd, self._same_rows(k_cache, v_cache, head_dim, vd), False)
+        stream = (self.decode_kernel in ("stream", "auto") and tag == "hd64"
                   and page_size in (8, 16, 32, 64))
-        lib = self._attn_lib(head_dim)
         if stream and self.decode_kernel == "auto":
             items = (n_reqs * -(-max_ctx_len // 256) * num_kv_heads
                      * -(-(num_heads // num_kv_heads) // 16))
@@ -669,13 +696,13 @@ class CudaOps:
         else:
             split = self.decode_split
         need = self.lib.rv_paged_attention_decode_scratch_bytes(
-            c_int(n_reqs), c_int(num_heads), c_int(head_dim), c_int(max_ctx_len * (256 // split)))
+            c_int(n_reqs), c_int(num_heads), c_int(vd), c_int(max_ctx_len * (256 // split)))
         if scratch is None:
             scratch = self._scratch_buffer(need, qkv.device)
         win = c_int(window if window else 0)
         if stream:
             fn = getattr(lib, f"rv_paged_attention_decode_stream_hd{head_dim}")
-            self._check_attn(lib, head_dim, fn(
+            self._check_attn(lib, tag, fn(
                 _ptr(qkv), c_int(qkv.shape[1]), _ptr(k_cache), _ptr(v_cache),
                 c_longlong(k_cache.shape[0] * k_cache.shape[1]), _ptr(block_table),
                 c_int(block_table.shape[1]), _ptr(ctx_lens), _ptr(scratch),
@@ -689,8 +716,8 @@ class CudaOps:
                 c_int(max_ctx_len), c_int(num_heads), c_int(head_dim), win, c_int(split),
                 _ptr(sinks), self._stream()), "paged_attention_merge")
             return
-        fn = getattr(lib, f"rv_paged_attention_decode_mma_hd{head_dim}")
-        self._check_attn(lib, head_dim, fn(
+        fn = getattr(lib, f"rv_paged_attention_decode_mma_{tag}")
+        self._check_attn(lib, tag, fn(
             _ptr(qkv), c_int(qkv.shape[1]), _ptr(k_cache), _ptr(v_cache), _ptr(block_table),
             c_int(block_table.shape[1]), _ptr(q_start), _ptr(ctx_lens), _ptr(scratch),
             c_longlong(scratch.numel() * scratch.element_size()), c_int(n_reqs),
@@ -698,7 +725,7 @@ class CudaOps:
             c_float(scale), win, c_int(split), self._stream()), "paged_attention_decode_mma")
         self._check(self.lib.rv_paged_attention_merge_ex(
             _ptr(scratch), _ptr(ctx_lens), _ptr(out), _code(out.dtype), c_int(n_reqs),
-            c_int(max_ctx_len), c_int(num_heads), c_int(head_dim), win, c_int(split),
+            c_int(max_ctx_len), c_int(num_heads), c_int(vd), win, c_int(split),
             _ptr(sinks), self._stream()), "paged_attention_merge")
 
     def paged_attention_general(self, qkv, num_heads, num_kv_heads, head_dim, k_cache, v_cache,
@@ -859,21 +886,6 @@ class CudaOps:
             c_int(n_reqs), c_int(num_heads), c_int(v_head_dim), c_int(max_ctx_len),
             c_int(window or 0), c_int(pool or 0), c_int(most)))
 
-    def _pooled_lib(self, head_dim: int):
-        """The tensor-core pooled attention library for this head size, built at first use."""
-        key = ("pooled", head_dim)
-        lib = self._attn_libs.get(key)
-        if lib is None:
-            path = build_variant("attention_mma.cu", {"RV_HD": head_dim, "RV_POOLED": 1},
-                                 f"attnpool_hd{head_dim}", verbose=self._verbose_build)
-            try:
-                lib = ctypes.CDLL(path)
-            except OSError as e:
-                raise KernelError(f"cannot load the kernel library {path}: {e}") from None
-            getattr(lib, f"rv_attention_pooled_last_error_hd{head_dim}").restype = ctypes.c_char_p
-            self._attn_libs[key] = lib
-        return lib
-
     def paged_attention_pooled(self, rows, num_heads, num_kv_heads, head_dim, k_cache, v_cache, ctx,
                                group, pooled, scale, softcap, window, sinks, out, v_head_dim=None,
                                most_blocks=0):
@@ -884,7 +896,7 @@ class CudaOps:
         `head_dim`.  `softcap`: scores
         become c tanh(score / c); `sinks` float32 [heads]: one more term in the denominator.
         Single tokens go to a split kernel and its merge, portions to one launch; bfloat16 heads
-        whose size is a multiple of 16 up to 128 take the tensor cores."""
+        whose sizes are multiples of 16 up to 192 take the tensor cores."""
         self._need(rows, "query rows")
         self._need(out, "attention output", rows.dtype)
         self._need(k_cache, "key pages", rows.dtype)
@@ -907,7 +919,7 @@ class CudaOps:
                 raise KernelError("paged_attention_pooled: blocks lie before a window, in pages of "
                                   "the tokens' size")
             ptable, pmax = pgroup.block_table, pgroup.max_blocks
-        mma = (self._mma_ok(rows.dtype, d) and dv == d and rows.shape[1] % 8 == 0
+        mma = (self._mma_ok(rows.dtype, d, dv) and rows.shape[1] % 8 == 0
                and rows.data_ptr() % 16 == 0 and k_cache.data_ptr() % 16 == 0 and v_cache.data_ptr() % 16 == 0)
         code, nd = _code(rows.dtype), ctx.n_decode
         pages = (_ptr(k_cache), _ptr(v_cache), _ptr(group.block_table), c_int(group.max_blocks),
@@ -917,7 +929,7 @@ class CudaOps:
         win = c_int(window or 0)
         lib = tag = None
         if mma and (self.decode_attention == "mma" or self.prefill_attention != "simt"):
-            lib, tag = self._pooled_lib(d), f"hd{d}"
+            lib, tag = self._mma_lib(d, dv, False, True)
 
         def check_mma(rc, what):
             self.launches += 1
