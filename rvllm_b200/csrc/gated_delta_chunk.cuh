@@ -613,7 +613,7 @@ static bool gc_sizes_ok(int H, int G, int d, int dv) {
 
 #define GC_SMEM(kernel, bytes)                                                                        \
     {                                                                                                 \
-        static size_t have = 48 * 1024;                                                               \
+        static size_t have = 40 * 1024;       /* the default 48 KB hold the static arrays too */        \
         if ((bytes) > have) {                                                                         \
             if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,             \
                                      (int)(bytes)) != cudaSuccess)                                    \

@@ -674,7 +674,7 @@ struct LaArgs {
 
 #define LA_SMEM(kernel, bytes)                                                                       \
     {                                                                                                \
-        static size_t have = 48 * 1024;                                                              \
+        static size_t have = 40 * 1024;      /* the default 48 KB hold the static arrays too */        \
         if ((bytes) > have) {                                                                        \
             if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,            \
                                      (int)(bytes)) != cudaSuccess)                                   \
